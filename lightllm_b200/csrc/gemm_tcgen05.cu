@@ -12,8 +12,9 @@
 //               epilogue functor, store.  Two accumulators (2 x BN TMEM columns) so the epilogue
 //               of tile i overlaps the main loop of tile i+1.
 // Epilogues: plain store, + bias, + residual, SiLU/GELU-gated product of interleaved
-// gate/up column blocks (the SwiGLU FFN never materialises the [T, 2I] tensor), fp32 store
-// (lm_head logits).
+// gate/up column blocks (the SwiGLU FFN never materialises the [T, 2I] tensor), fp32 store, scaled
+// (lm_head logits), squared ReLU, and the sandwich of two dynamic-tanh norms around an fp32 residual
+// stream (x += dyt1(acc); C = dyt2(x)).
 //
 // Behavioural counterpart in the reference: the cuBLAS calls behind
 // lightllm/common/quantization/no_quant.py (torch.mm / addmm), silu_and_mul_fwd and the
@@ -32,7 +33,14 @@ constexpr int GEMM_THREADS = 192;
 constexpr int SMEM_BUDGET = 224 * 1024;
 constexpr int64_t kPanelBytes = 24ll << 20;  // A panel kept hot in L2 while W streams past it
 
-enum Epi { EPI_STORE = 0, EPI_RESIDUAL = 1, EPI_GATED_SILU = 2, EPI_F32 = 3, EPI_GATED_GELU = 4 };
+enum Epi { EPI_STORE = 0, EPI_RESIDUAL = 1, EPI_GATED_SILU = 2, EPI_F32 = 3, EPI_GATED_GELU = 4, EPI_RELU2 = 5, EPI_DYT = 6 };
+
+// dyt(v) = tanh(alpha * v) * w + b; x is the fp32 residual stream [M, ldc]
+struct DytFuse {
+  float* x;
+  const float *w1, *b1, *w2, *b2;
+  float alpha1, alpha2;
+};
 
 struct GemmParams {
   void* C;
@@ -64,6 +72,8 @@ struct GemmParams {
   bf16* push[8];
   uint32_t* push_cnt[8];
   int push_world, push_rank, push_max_mb;
+  float out_scale;  // EPI_F32: factor on the stored value
+  DytFuse dyt;      // EPI_DYT
 };
 
 // Output staging of the epilogue warps: a thread owns one accumulator row, so storing straight from registers
@@ -91,6 +101,26 @@ constexpr int smem_bytes() {
 __device__ __forceinline__ float silu_f(float v) { return v / (1.f + __expf(-v)); }
 __device__ __forceinline__ float gelu_tanh_f(float v) {
   return 0.5f * v * (1.f + tanhf(0.7978845608028654f * (v + 0.044715f * v * v * v)));
+}
+__device__ __forceinline__ float relu2_f(float v) {
+  v = fmaxf(v, 0.f);
+  return v * v;
+}
+// Four columns from `col` on: x += dyt1(v), then v = dyt2(x).
+__device__ __forceinline__ void dyt_sandwich4(const DytFuse& d, int col, float4& x, float4& v) {
+  const float4 w1 = *reinterpret_cast<const float4*>(d.w1 + col), b1 = *reinterpret_cast<const float4*>(d.b1 + col);
+  const float4 w2 = *reinterpret_cast<const float4*>(d.w2 + col), b2 = *reinterpret_cast<const float4*>(d.b2 + col);
+  x.x += tanhf(d.alpha1 * v.x) * w1.x + b1.x;
+  x.y += tanhf(d.alpha1 * v.y) * w1.y + b1.y;
+  x.z += tanhf(d.alpha1 * v.z) * w1.z + b1.z;
+  x.w += tanhf(d.alpha1 * v.w) * w1.w + b1.w;
+  v.x = tanhf(d.alpha2 * x.x) * w2.x + b2.x;
+  v.y = tanhf(d.alpha2 * x.y) * w2.y + b2.y;
+  v.z = tanhf(d.alpha2 * x.z) * w2.z + b2.z;
+  v.w = tanhf(d.alpha2 * x.w) * w2.w + b2.w;
+}
+__device__ __forceinline__ uint2 pack4(const float4& v) {
+  return make_uint2(pack_bf16x2(v.x, v.y), pack_bf16x2(v.z, v.w));
 }
 
 // Tile order: groups of `GROUP` M-blocks, M fastest inside a group, so CTAs running at the same time
@@ -182,7 +212,19 @@ template <int EPI>
 __device__ __forceinline__ void epi_direct32(const GemmParams& p, const uint32_t* r, int row, bool row_ok, int col0) {
   if (!(row_ok && col0 < p.N)) return;
   const int ncols = min(32, p.N - col0);
-  if (EPI == EPI_F32) {
+  if (EPI == EPI_DYT) {  // N is a multiple of 8
+    const int64_t off = (int64_t)row * p.ldc + col0;
+#pragma unroll
+    for (int j = 0; j < 32; j += 4) {
+      if (j >= ncols) break;
+      float4 v = make_float4(__uint_as_float(r[j]), __uint_as_float(r[j + 1]), __uint_as_float(r[j + 2]),
+                             __uint_as_float(r[j + 3]));
+      float4 x = *reinterpret_cast<const float4*>(p.dyt.x + off + j);
+      dyt_sandwich4(p.dyt, col0 + j, x, v);
+      *reinterpret_cast<float4*>(p.dyt.x + off + j) = x;
+      *reinterpret_cast<uint2*>((bf16*)p.C + off + j) = pack4(v);
+    }
+  } else if (EPI == EPI_F32) {
     float* crow = (float*)p.C + (int64_t)row * p.ldc + col0;
     if (ncols == 32) {
 #pragma unroll
@@ -195,12 +237,14 @@ __device__ __forceinline__ void epi_direct32(const GemmParams& p, const uint32_t
           v.z += __bfloat162float(p.bias[col0 + j + 2]);
           v.w += __bfloat162float(p.bias[col0 + j + 3]);
         }
+        v = make_float4(v.x * p.out_scale, v.y * p.out_scale, v.z * p.out_scale, v.w * p.out_scale);
         *reinterpret_cast<float4*>(crow + j) = v;
       }
     } else {
 #pragma unroll
       for (int j = 0; j < 32; ++j)
-        if (j < ncols) crow[j] = __uint_as_float(r[j]) + (p.bias ? __bfloat162float(p.bias[col0 + j]) : 0.f);
+        if (j < ncols)
+          crow[j] = (__uint_as_float(r[j]) + (p.bias ? __bfloat162float(p.bias[col0 + j]) : 0.f)) * p.out_scale;
     }
   } else {
     bf16* crow = (bf16*)p.C + (int64_t)row * p.ldc + col0;
@@ -223,6 +267,10 @@ __device__ __forceinline__ void epi_direct32(const GemmParams& p, const uint32_t
 #pragma unroll
           for (int e = 0; e < 8; ++e) o[e] += rv[e];
         }
+        if (EPI == EPI_RELU2) {
+#pragma unroll
+          for (int e = 0; e < 8; ++e) o[e] = relu2_f(o[e]);
+        }
         if (EPI == EPI_STORE && p.push_world > 0) {
           const bf16x8 packed = pack8(o);
           const int64_t off = (int64_t)row * p.ldc + col0 + j;
@@ -240,6 +288,7 @@ __device__ __forceinline__ void epi_direct32(const GemmParams& p, const uint32_t
           float v = __uint_as_float(r[j]);
           if (p.bias) v += __bfloat162float(p.bias[col0 + j]);
           if (EPI == EPI_RESIDUAL) v += __bfloat162float(rrow[j]);
+          if (EPI == EPI_RELU2) v = relu2_f(v);
           crow[j] = __float2bfloat16(v);
         }
       }
@@ -298,6 +347,63 @@ __device__ __forceinline__ void epilogue_store(const GemmParams& p, uint32_t t_r
         __syncwarp();
       }
     }
+  } else if (EPI == EPI_DYT) {
+#pragma unroll 1
+    for (int c = 0; c < BN; c += 32) {
+      const int col0 = col_tile0 + c;
+      if (col0 >= p.N) break;
+      const bool staged = stage != nullptr && col0 + 32 <= p.N;
+      if (staged) {  // the stream's rows: whole lines into the staging block, and back below
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+          const int id = i * 32 + lane, r = id >> 3, seg = id & 7;
+          float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+          if (row_base + r < p.M)
+            v = *reinterpret_cast<const float4*>(p.dyt.x + (int64_t)(row_base + r) * p.ldc + col0 + seg * 4);
+          *reinterpret_cast<float4*>(stage + r * EPI_ROW_PITCH + seg * 16) = v;
+        }
+        __syncwarp();
+      }
+      uint32_t r[32];
+      tmem_ld_32x32(t_row + c, r);
+      tmem_wait_ld();
+      if (has_add) add_partials(r, c);
+      if (!staged) {
+        epi_direct32<EPI>(p, r, row, row_ok, col0);
+        continue;
+      }
+      uint2 hb[8];
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        float4 v = make_float4(__uint_as_float(r[4 * j]), __uint_as_float(r[4 * j + 1]), __uint_as_float(r[4 * j + 2]),
+                               __uint_as_float(r[4 * j + 3]));
+        float4 x = *reinterpret_cast<const float4*>(my + j * 16);
+        dyt_sandwich4(p.dyt, col0 + 4 * j, x, v);
+        *reinterpret_cast<float4*>(my + j * 16) = x;
+        hb[j] = pack4(v);
+      }
+      __syncwarp();
+#pragma unroll
+      for (int i = 0; i < 8; ++i) {
+        const int id = i * 32 + lane, rr = id >> 3, seg = id & 7;
+        if (row_base + rr < p.M)
+          *reinterpret_cast<float4*>(p.dyt.x + (int64_t)(row_base + rr) * p.ldc + col0 + seg * 4) =
+              *reinterpret_cast<const float4*>(stage + rr * EPI_ROW_PITCH + seg * 16);
+      }
+      __syncwarp();
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+        *reinterpret_cast<uint4*>(my + j * 16) = make_uint4(hb[2 * j].x, hb[2 * j].y, hb[2 * j + 1].x, hb[2 * j + 1].y);
+      __syncwarp();
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const int id = i * 32 + lane, rr = id >> 2, seg = id & 3;
+        if (row_base + rr < p.M)
+          *reinterpret_cast<uint4*>((bf16*)p.C + (int64_t)(row_base + rr) * p.ldc + col0 + seg * 8) =
+              *reinterpret_cast<const uint4*>(stage + rr * EPI_ROW_PITCH + seg * 16);
+      }
+      __syncwarp();
+    }
   } else if (EPI == EPI_F32) {
 #pragma unroll 1
     for (int c = 0; c < BN; c += 32) {
@@ -317,6 +423,7 @@ __device__ __forceinline__ void epilogue_store(const GemmParams& p, uint32_t t_r
             v.z += __bfloat162float(p.bias[col0 + j + 2]);
             v.w += __bfloat162float(p.bias[col0 + j + 3]);
           }
+          v = make_float4(v.x * p.out_scale, v.y * p.out_scale, v.z * p.out_scale, v.w * p.out_scale);
           *reinterpret_cast<float4*>(my + j * 4) = v;
         }
         __syncwarp();
@@ -369,6 +476,10 @@ __device__ __forceinline__ void epilogue_store(const GemmParams& p, uint32_t t_r
             unpack8(*slot, rv);
 #pragma unroll
             for (int e = 0; e < 8; ++e) o[e] += rv[e];
+          }
+          if (EPI == EPI_RELU2) {
+#pragma unroll
+            for (int e = 0; e < 8; ++e) o[e] = relu2_f(o[e]);
           }
           *slot = pack8(o);
         }
@@ -695,6 +806,10 @@ int dispatch_epi(int epi, const CUtensorMap& ta, const CUtensorMap& tb, GemmPara
       return launch_gemm<BN, EPI_F32>(ta, tb, p, st);
     case EPI_GATED_GELU:
       return launch_gemm<BN, EPI_GATED_GELU>(ta, tb, p, st);
+    case EPI_RELU2:
+      return launch_gemm<BN, EPI_RELU2>(ta, tb, p, st);
+    case EPI_DYT:
+      return launch_gemm<BN, EPI_DYT>(ta, tb, p, st);
   }
   return LLB_ERR_UNSUPPORTED;
 }
@@ -895,6 +1010,10 @@ int dispatch_pair(int epi, const CUtensorMap& ta, const CUtensorMap& tb, GemmPar
       return launch_pair<EPI_F32>(ta, tb, p, st);
     case EPI_GATED_GELU:
       return launch_pair<EPI_GATED_GELU>(ta, tb, p, st);
+    case EPI_RELU2:
+      return launch_pair<EPI_RELU2>(ta, tb, p, st);
+    case EPI_DYT:
+      return launch_pair<EPI_DYT>(ta, tb, p, st);
   }
   return LLB_ERR_UNSUPPORTED;
 }
@@ -1131,8 +1250,16 @@ gemm_bf16_skinny_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_co
           acc.w += __bfloat162float(p.bias[gcol + 3]);
         }
         if (EPI == EPI_F32) {
-          *reinterpret_cast<float4*>((float*)p.C + (int64_t)grow * p.ldc + gcol) = acc;
+          *reinterpret_cast<float4*>((float*)p.C + (int64_t)grow * p.ldc + gcol) =
+              make_float4(acc.x * p.out_scale, acc.y * p.out_scale, acc.z * p.out_scale, acc.w * p.out_scale);
+        } else if (EPI == EPI_DYT) {
+          const int64_t off = (int64_t)grow * p.ldc + gcol;
+          float4 x = *reinterpret_cast<const float4*>(p.dyt.x + off);
+          dyt_sandwich4(p.dyt, gcol, x, acc);
+          *reinterpret_cast<float4*>(p.dyt.x + off) = x;
+          *reinterpret_cast<uint2*>((bf16*)p.C + off) = pack4(acc);
         } else {
+          if (EPI == EPI_RELU2) acc = make_float4(relu2_f(acc.x), relu2_f(acc.y), relu2_f(acc.z), relu2_f(acc.w));
           if (EPI == EPI_RESIDUAL) {
             const bf162* rr = reinterpret_cast<const bf162*>(p.residual + (int64_t)grow * p.ldc + gcol);
             const float2 r0 = __bfloat1622float2(rr[0]), r1 = __bfloat1622float2(rr[1]);
@@ -1223,6 +1350,8 @@ int dispatch_skinny(int epi, int nb, int splits, int tw, const CUtensorMap& ta, 
       case EPI_STORE: return launch_skinny<1, EPI_STORE, 128>(ta, tb, p, splits, st);
       case EPI_RESIDUAL: return launch_skinny<1, EPI_RESIDUAL, 128>(ta, tb, p, splits, st);
       case EPI_F32: return launch_skinny<1, EPI_F32, 128>(ta, tb, p, splits, st);
+      case EPI_RELU2: return launch_skinny<1, EPI_RELU2, 128>(ta, tb, p, splits, st);
+      case EPI_DYT: return launch_skinny<1, EPI_DYT, 128>(ta, tb, p, splits, st);
     }
     return LLB_ERR_UNSUPPORTED;
   }
@@ -1233,6 +1362,8 @@ int dispatch_skinny(int epi, int nb, int splits, int tw, const CUtensorMap& ta, 
       case EPI_GATED_SILU: return launch_skinny<1, EPI_GATED_SILU>(ta, tb, p, splits, st);
       case EPI_GATED_GELU: return launch_skinny<1, EPI_GATED_GELU>(ta, tb, p, splits, st);
       case EPI_F32: return launch_skinny<1, EPI_F32>(ta, tb, p, splits, st);
+      case EPI_RELU2: return launch_skinny<1, EPI_RELU2>(ta, tb, p, splits, st);
+      case EPI_DYT: return launch_skinny<1, EPI_DYT>(ta, tb, p, splits, st);
     }
   } else {
     switch (epi) {
@@ -1241,6 +1372,8 @@ int dispatch_skinny(int epi, int nb, int splits, int tw, const CUtensorMap& ta, 
       case EPI_GATED_SILU: return launch_skinny<2, EPI_GATED_SILU>(ta, tb, p, 1, st);
       case EPI_GATED_GELU: return launch_skinny<2, EPI_GATED_GELU>(ta, tb, p, 1, st);
       case EPI_F32: return launch_skinny<2, EPI_F32>(ta, tb, p, 1, st);
+      case EPI_RELU2: return launch_skinny<2, EPI_RELU2>(ta, tb, p, 1, st);
+      case EPI_DYT: return launch_skinny<2, EPI_DYT>(ta, tb, p, 1, st);
     }
   }
   return LLB_ERR_UNSUPPORTED;
@@ -1886,6 +2019,11 @@ void apply_push(GemmParams& p) {
   }
   g_push.world = 0;
 }
+struct GemmFuse {
+  float out_scale = 1.f;
+  DytFuse dyt = {nullptr, nullptr, nullptr, nullptr, nullptr, 1.f, 1.f};
+};
+
 bool g_pair_auto = true;  // measured faster than one-CTA tiles for M >= 1024, K <= 8192 on B200
 
 }  // namespace
@@ -1910,22 +2048,29 @@ LLB_EXPORT int llb_gemm_set_push(void** push, void** cnt, int rank, int world, i
 // C[M,N] (ldc) = A[M,K] (lda) . W[N,K]^T (ldw)  with epilogue `epi`:
 //   0 store bf16 (+bias)          1 store bf16 of acc (+bias) + residual[M,N] (same ldc)
 //   2 SiLU-gated: W rows interleaved as [32 gate | 32 up] blocks; C is [M, N/2]
-//   3 store fp32 (+bias)          4 GELU(tanh)-gated, layout as 2
+//   3 store fp32 (+bias)          4 GELU(tanh)-gated, layout as 2          5 store bf16 of relu(acc)^2
+//   6 dynamic-tanh sandwich (llb_gemm_bf16_fused)
 // bn: 0 = choose, else 64/128/256, or 512 = the CTA-pair (cta_group::2) kernel with 256x256 tiles.  status: optional device int receiving a wait-timeout code.
 // stream_k: 0 = whole tiles per CTA, 1 = equal (tile, k-block) shares with fix-up of split tiles,
 // -1 = choose (stream-K when the tiles would fill fewer than three waves).  Stream-K needs
 // sk_partials (>= SMs * 2 * 128 * bn floats) and sk_counters (>= tiles ints, zero before first use;
 // the kernel leaves them zero); launches that share them must not overlap on the GPU.
-LLB_EXPORT int llb_gemm_bf16(const void* A, int64_t lda, const void* W, int64_t ldw, void* C, int64_t ldc,
+static int gemm_bf16(const void* A, int64_t lda, const void* W, int64_t ldw, void* C, int64_t ldc,
                              const void* residual, const void* bias, int M, int N, int K, int epi, int bn,
                              int stream_k, float* sk_partials, int64_t sk_partials_floats, int* sk_counters,
-                             int sk_counters_len, int* status, cudaStream_t st) {
+                             int sk_counters_len, int* status, const GemmFuse& fuse, cudaStream_t st) {
   if (M <= 0 || N <= 0) return LLB_OK;
   if (K <= 0 || (K % 8) != 0) return LLB_ERR_UNSUPPORTED;
   if ((epi == EPI_GATED_SILU || epi == EPI_GATED_GELU) && (N % 64) != 0) return LLB_ERR_UNSUPPORTED;
   if (epi != EPI_F32 && (((uintptr_t)C & 15) || (ldc % 8))) return LLB_ERR_BAD_ARG;
   if (epi == EPI_F32 && (((uintptr_t)C & 15) || (ldc % 4))) return LLB_ERR_BAD_ARG;
   if (epi == EPI_RESIDUAL && (residual == nullptr || ((uintptr_t)residual & 15))) return LLB_ERR_BAD_ARG;
+  if (epi == EPI_DYT) {
+    const DytFuse& d = fuse.dyt;
+    if ((N % 8) || bias != nullptr || d.x == nullptr || d.w1 == nullptr || d.b1 == nullptr || d.w2 == nullptr ||
+        d.b2 == nullptr || (((uintptr_t)d.x | (uintptr_t)d.w1 | (uintptr_t)d.b1 | (uintptr_t)d.w2 | (uintptr_t)d.b2) & 15))
+      return LLB_ERR_BAD_ARG;
+  }
   const int kblocks = cdiv(K, BK);
   if (stream_k != 0) {
     int sk_bn = bn ? bn : (N >= 256 ? 256 : (N >= 128 ? 128 : 64));
@@ -1964,6 +2109,8 @@ LLB_EXPORT int llb_gemm_bf16(const void* A, int64_t lda, const void* W, int64_t 
     GemmParams p;
     memset(&p, 0, sizeof(p));
     apply_push(p);
+    p.out_scale = fuse.out_scale;
+    p.dyt = fuse.dyt;
     if (p.push_world > 0 && (epi != EPI_STORE || (N % 32))) return LLB_ERR_UNSUPPORTED;
     p.C = C;
     p.residual = (const bf16*)residual;
@@ -2000,6 +2147,8 @@ LLB_EXPORT int llb_gemm_bf16(const void* A, int64_t lda, const void* W, int64_t 
     GemmParams p;
     memset(&p, 0, sizeof(p));
     apply_push(p);
+    p.out_scale = fuse.out_scale;
+    p.dyt = fuse.dyt;
     if (p.push_world > 0 && (epi != EPI_STORE || (N % 32))) return LLB_ERR_UNSUPPORTED;
     p.C = C;
     p.residual = (const bf16*)residual;
@@ -2052,6 +2201,8 @@ LLB_EXPORT int llb_gemm_bf16(const void* A, int64_t lda, const void* W, int64_t 
     memset(&p, 0, sizeof(p));
     p.w_tiled_kb = w_tiled ? K / 64 : 0;
     apply_push(p);
+    p.out_scale = fuse.out_scale;
+    p.dyt = fuse.dyt;
     if (p.push_world > 0 && (epi != EPI_STORE || (N % 32))) return LLB_ERR_UNSUPPORTED;
     p.C = C;
     p.residual = (const bf16*)residual;
@@ -2083,6 +2234,8 @@ LLB_EXPORT int llb_gemm_bf16(const void* A, int64_t lda, const void* W, int64_t 
   p.w_tiled_kb = w_swz ? K / 64 : 0;
   p.w_swz = w_swz ? (const bf16*)W : nullptr;
   apply_push(p);
+  p.out_scale = fuse.out_scale;
+  p.dyt = fuse.dyt;
   if (p.push_world > 0 && (epi != EPI_STORE || (N % 32) || stream_k)) return LLB_ERR_UNSUPPORTED;
   p.C = C;
   p.residual = (const bf16*)residual;
@@ -2113,6 +2266,26 @@ LLB_EXPORT int llb_gemm_bf16(const void* A, int64_t lda, const void* W, int64_t 
   return LLB_ERR_UNSUPPORTED;
 }
 
+LLB_EXPORT int llb_gemm_bf16(const void* A, int64_t lda, const void* W, int64_t ldw, void* C, int64_t ldc,
+                             const void* residual, const void* bias, int M, int N, int K, int epi, int bn,
+                             int stream_k, float* sk_partials, int64_t sk_partials_floats, int* sk_counters,
+                             int sk_counters_len, int* status, cudaStream_t st) {
+  return gemm_bf16(A, lda, W, ldw, C, ldc, residual, bias, M, N, K, epi, bn, stream_k, sk_partials, sk_partials_floats,
+                   sk_counters, sk_counters_len, status, GemmFuse{}, st);
+}
+
+// The epilogues with parameters: out_scale multiplies fp32 output (epi 3); for epi 6 (bf16 C, same pitch for x)
+//   x += tanh(alpha1 * acc) * w1 + b1;  C = tanh(alpha2 * x) * w2 + b2        x fp32 [M, ldc], vectors fp32 [N]
+LLB_EXPORT int llb_gemm_bf16_fused(const void* A, int64_t lda, const void* W, int64_t ldw, void* C, int64_t ldc,
+                                   const void* bias, int M, int N, int K, int epi, int bn, float out_scale, float* x,
+                                   const float* w1, const float* b1, float alpha1, const float* w2, const float* b2,
+                                   float alpha2, int* status, cudaStream_t st) {
+  GemmFuse fuse;
+  fuse.out_scale = out_scale;
+  fuse.dyt = DytFuse{x, w1, b1, w2, b2, alpha1, alpha2};
+  return gemm_bf16(A, lda, W, ldw, C, ldc, nullptr, bias, M, N, K, epi, bn, 0, nullptr, 0, nullptr, 0, status, fuse, st);
+}
+
 // Grouped GEMM for MoE experts.  A [M_pad, K] holds the routed tokens sorted by expert, every expert's
 // rows padded to a multiple of 128; W [E * N, K] stacks the expert weights; mblock_expert[M_pad / 128]
 // (device) names the expert of each 128-row block, -1 for blocks beyond the routed rows (skipped).
@@ -2122,7 +2295,7 @@ LLB_EXPORT int llb_gemm_bf16_grouped(const void* A, int64_t lda, const void* W, 
                                      int* status, cudaStream_t st) {
   if (M_pad <= 0 || N <= 0 || E <= 0) return LLB_OK;
   if (K <= 0 || (K % 8) != 0 || (M_pad % BM) != 0) return LLB_ERR_UNSUPPORTED;
-  if (epi == EPI_RESIDUAL) return LLB_ERR_UNSUPPORTED;
+  if (epi == EPI_RESIDUAL || epi == EPI_DYT) return LLB_ERR_UNSUPPORTED;
   if (bn == 0) bn = (N % 256 == 0) ? 256 : ((N % 128 == 0) ? 128 : 64);
   if (N % bn != 0) return LLB_ERR_UNSUPPORTED;
   if (((uintptr_t)C & 15) || (ldc % 8)) return LLB_ERR_BAD_ARG;
@@ -2133,6 +2306,7 @@ LLB_EXPORT int llb_gemm_bf16_grouped(const void* A, int64_t lda, const void* W, 
   if (rc) return rc;
   GemmParams p;
   memset(&p, 0, sizeof(p));
+  p.out_scale = 1.f;
   p.C = C;
   p.residual = nullptr;
   p.bias = nullptr;
@@ -2178,6 +2352,7 @@ LLB_EXPORT int llb_gemm_bf16_batched(const void* A, int64_t a_row_stride, int64_
   if (rc) return rc;
   GemmParams p;
   memset(&p, 0, sizeof(p));
+  p.out_scale = 1.f;
   p.C = C;
   p.residual = nullptr;
   p.bias = nullptr;

@@ -1,0 +1,509 @@
+// Latent attention without a rotary part, over a paged pool of latents, with an optional sliding window.
+//
+// Pool row of a token: the RMS-normalised latent c (`rank` values, zero-padded to the row pitch), one "head" shared by
+// all query heads.  The query of a head is taken into the latent space with the key up-projection (q_lat = q . W_uk),
+// scores are q_lat . c, the value read is the same c, and the value up-projection follows the attention.
+// Position i sees j with 0 <= i - j < window (window 0: no lower bound).  Scores, weights and their sums are fp32.
+//
+//   latent_norm_scatter    RMSNorm of new latents, written to their pool slots
+//   latent_gather          latents of a range of positions of every request, back to back (for the expanded prefill form)
+//   latent_attn_generic    any rank <= 1024, fp32 or bf16; one CTA per (query token, head), warps stride over the keys
+//   latent_attn_mma        bf16, rank <= 512: one CTA per (query token, 16 heads, share of the keys).  The 16 query rows
+//                          live in registers as MMA fragments; 64-key tiles of the pool are gathered through the slot
+//                          table into a three-stage shared-memory ring and used for both products.  The weights enter
+//                          P . c as a sum of two bf16 values (high and low part), so that they keep fp32-like
+//                          precision.  With more than one share per query the partial results are merged by
+//   latent_attn_merge
+#include "common.cuh"
+
+using namespace llb;
+LLB_DEBUG_BOUNDS_STORAGE(latent_attn)
+
+namespace {
+
+constexpr float kLog2e = 1.4426950408889634f;
+
+__device__ __forceinline__ float to_f(float v) { return v; }
+__device__ __forceinline__ float to_f(bf16 v) { return __bfloat162float(v); }
+__device__ __forceinline__ void from_f(float* p, float v) { *p = v; }
+__device__ __forceinline__ void from_f(bf16* p, float v) { *p = __float2bfloat16(v); }
+
+// One warp per token.
+template <typename T>
+__global__ void __launch_bounds__(128)
+latent_norm_scatter_kernel(const T* __restrict__ src, int64_t src_stride, T* __restrict__ pool, int row_elems,
+                           const float* __restrict__ w, const int* __restrict__ slot, int Tn, int rank, float eps) {
+  const int t = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (t >= Tn) return;
+  const T* s = src + (int64_t)t * src_stride;
+  T* d = pool + (int64_t)LLB_CHECK_SLOT(slot[t]) * row_elems;
+  float ss = 0.f;
+  for (int i = lane; i < rank; i += 32) {
+    const float v = to_f(s[i]);
+    ss += v * v;
+  }
+  ss = warp_sum(ss);
+  const float r = 1.f / sqrtf(ss / (float)rank + eps);
+  for (int i = lane; i < row_elems; i += 32) from_f(d + i, i < rank ? to_f(s[i]) * r * w[i] : 0.f);
+}
+
+// out row cu_kv[b] + i = latent of position kv_start[b] + i of request b.  One warp per row, 16-byte pieces.
+__global__ void __launch_bounds__(256)
+latent_gather_kernel(const uint4* __restrict__ pool, int row_vec, const int* __restrict__ req_to_token,
+                     int64_t r2t_stride, const int* __restrict__ b_req_idx, const int* __restrict__ cu_kv,
+                     const int* __restrict__ kv_start, uint4* __restrict__ out, int B) {
+  const int rows = cu_kv[B];
+  const int lane = threadIdx.x & 31;
+  for (int r = blockIdx.x * 8 + (threadIdx.x >> 5); r < rows; r += gridDim.x * 8) {
+    int lo = 0, hi = B - 1;
+    while (lo < hi) {
+      const int mid = (lo + hi + 1) >> 1;
+      if (cu_kv[mid] <= r) lo = mid; else hi = mid - 1;
+    }
+    const int pos = kv_start[lo] + r - cu_kv[lo];
+    const int sl = LLB_CHECK_SLOT(req_to_token[(int64_t)LLB_CHECK_REQ(b_req_idx[lo]) * r2t_stride + LLB_CHECK_POS(pos)]);
+    for (int v = lane; v < row_vec; v += 32) out[(int64_t)r * row_vec + v] = pool[(int64_t)sl * row_vec + v];
+  }
+}
+
+// ---------------------------------------------------------------------------------------------- any rank, any type
+constexpr int GW = 8;  // warps
+
+template <typename T, int EPL>
+__global__ void __launch_bounds__(GW * 32)
+latent_attn_generic_kernel(const T* __restrict__ q_lat, const T* __restrict__ pool, int row_elems,
+                           const int* __restrict__ req_to_token, int64_t r2t_stride, const int* __restrict__ b_req_idx,
+                           const int* __restrict__ pos, const int* __restrict__ batch_of, T* __restrict__ out, int H,
+                           int rank, float scale, int window) {
+  extern __shared__ float sm[];  // [GW][rank] partial outputs, then [GW] maxima, [GW] sums
+  const int t = blockIdx.x, h = blockIdx.y;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int b = batch_of ? batch_of[t] : t;
+  const int p = pos[t];
+  const int* slots = req_to_token + (int64_t)LLB_CHECK_REQ(b_req_idx[b]) * r2t_stride;
+  float q[EPL], acc[EPL];
+#pragma unroll
+  for (int e = 0; e < EPL; ++e) {
+    const int d = lane + e * 32;
+    q[e] = d < rank ? to_f(q_lat[((int64_t)t * H + h) * rank + d]) * scale : 0.f;
+    acc[e] = 0.f;
+  }
+  float m = -INFINITY, l = 0.f;
+  const int j0 = window > 0 ? max(0, p - window + 1) : 0;
+  for (int j = j0 + warp; j <= p; j += GW) {
+    const T* c = pool + (int64_t)LLB_CHECK_SLOT(slots[j]) * row_elems;
+    float cv[EPL];
+    float s = 0.f;
+#pragma unroll
+    for (int e = 0; e < EPL; ++e) {
+      const int d = lane + e * 32;
+      cv[e] = d < rank ? to_f(c[d]) : 0.f;
+      s += q[e] * cv[e];
+    }
+    s = warp_sum(s);
+    const float mn = fmaxf(m, s);
+    const float corr = expf(m - mn), w = expf(s - mn);
+    l = l * corr + w;
+#pragma unroll
+    for (int e = 0; e < EPL; ++e) acc[e] = acc[e] * corr + w * cv[e];
+    m = mn;
+  }
+  float* s_m = sm + GW * rank;
+  float* s_l = s_m + GW;
+  if (lane == 0) {
+    s_m[warp] = m;
+    s_l[warp] = l;
+  }
+#pragma unroll
+  for (int e = 0; e < EPL; ++e) {
+    const int d = lane + e * 32;
+    if (d < rank) sm[warp * rank + d] = acc[e];
+  }
+  __syncthreads();
+  float M = -INFINITY;
+#pragma unroll
+  for (int w = 0; w < GW; ++w) M = fmaxf(M, s_m[w]);
+  float L = 0.f, c[GW];
+#pragma unroll
+  for (int w = 0; w < GW; ++w) {
+    c[w] = s_m[w] == -INFINITY ? 0.f : expf(s_m[w] - M);
+    L += s_l[w] * c[w];
+  }
+  const float inv = 1.f / L;
+  for (int d = threadIdx.x; d < rank; d += blockDim.x) {
+    float o = 0.f;
+#pragma unroll
+    for (int w = 0; w < GW; ++w) o += sm[w * rank + d] * c[w];
+    from_f(out + ((int64_t)t * H + h) * rank + d, o * inv);
+  }
+}
+
+template <typename T>
+int launch_generic(const void* q_lat, const void* pool, int row_elems, const int* r2t, int64_t r2t_stride,
+                   const int* b_req_idx, const int* pos, const int* batch_of, void* out, int T_n, int H, int rank,
+                   float scale, int window, cudaStream_t st) {
+  const dim3 grid(T_n, H);
+  const size_t smem = (size_t)(GW * rank + 2 * GW) * sizeof(float);
+#define LLB_GENERIC(EPL)                                                                                              \
+  latent_attn_generic_kernel<T, EPL><<<grid, GW * 32, smem, st>>>((const T*)q_lat, (const T*)pool, row_elems, r2t,    \
+                                                                  r2t_stride, b_req_idx, pos, batch_of, (T*)out, H,   \
+                                                                  rank, scale, window)
+  if (rank <= 128)
+    LLB_GENERIC(4);
+  else if (rank <= 512)
+    LLB_GENERIC(16);
+  else
+    LLB_GENERIC(32);
+#undef LLB_GENERIC
+  LLB_LAUNCH_CHECK();
+  return LLB_OK;
+}
+
+// ---------------------------------------------------------------------------------------------- tensor cores, bf16
+constexpr int KT = 64;       // keys per tile
+constexpr int STAGES = 3;
+constexpr int S_PITCH = KT + 8;  // floats per score row in shared memory
+
+template <int LAT>
+constexpr int mma_smem() {
+  return STAGES * KT * LAT * 2 + 16 * S_PITCH * 4 + 2 * KT * 4;
+}
+
+// byte offset of 16-byte chunk `ch` of key `row` inside a tile
+template <int LAT>
+__device__ __forceinline__ uint32_t tile_off(int row, int ch) {
+  return (uint32_t)(row * (LAT * 2) + ((ch ^ (row & 7)) << 4));
+}
+
+// LAT: rank rounded up to 128, 256, 384 or 512 (tile columns beyond the row pitch are zero-filled).
+// Partial results (splits > 1): part_o [split][token][head][rank] unnormalised, part_ml [split][token][head] (max, sum).
+template <int LAT>
+__global__ void __launch_bounds__(256, 1)
+latent_attn_mma_kernel(const bf16* __restrict__ q_lat, const bf16* __restrict__ pool, int row_elems,
+                       const int* __restrict__ req_to_token, int64_t r2t_stride, const int* __restrict__ b_req_idx,
+                       const int* __restrict__ pos, const int* __restrict__ batch_of, bf16* __restrict__ out,
+                       float* __restrict__ part_o, float2* __restrict__ part_ml, int Tn, int H, int rank,
+                       float scale_log2, int window) {
+  extern __shared__ __align__(128) uint8_t smem[];
+  constexpr int CH = LAT / 8;            // 16-byte chunks per tile row
+  constexpr int KSTEPS = LAT / 16;
+  constexpr int N2 = LAT / 128;          // pairs of 8-column output blocks per warp
+  const uint32_t kv_base = smem_u32(smem);
+  float* s_sm = reinterpret_cast<float*>(smem + STAGES * KT * LAT * 2);
+  int* slot_sm = reinterpret_cast<int*>(s_sm + 16 * S_PITCH);
+
+  const int t = blockIdx.x, head0 = blockIdx.y * 16;
+  const int split = blockIdx.z, splits = gridDim.z;
+  const int b = batch_of ? batch_of[t] : t;
+  const int p = pos[t];
+  const int* slots = req_to_token + (int64_t)LLB_CHECK_REQ(b_req_idx[b]) * r2t_stride;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int g = lane >> 2, tig = lane & 3;
+  const int row_ch = row_elems >> 3;
+
+  const int k_begin = window > 0 ? max(0, p - window + 1) : 0;
+  const int k_end = p + 1;
+  const int all_tiles = (k_end - k_begin + KT - 1) / KT;
+  const int tile0 = (int)((int64_t)split * all_tiles / splits), tile1 = (int)((int64_t)(split + 1) * all_tiles / splits);
+  const int n_tiles = tile1 - tile0;
+  const int key0 = k_begin + tile0 * KT;
+
+  // slots of tile `i` -> slot_sm[i & 1] (-1 beyond the last visible key)
+  auto fetch_slot = [&](int i) {
+    const int kp = key0 + i * KT + (int)threadIdx.x;
+    return (i < n_tiles && kp < k_end) ? LLB_CHECK_SLOT(slots[LLB_CHECK_POS(kp)]) : -1;
+  };
+  auto issue = [&](int i) {
+    if (i < n_tiles) {
+      const uint32_t sb = kv_base + (uint32_t)(i % STAGES) * (KT * LAT * 2);
+      const int* sl_sm = slot_sm + (i & 1) * KT;
+#pragma unroll 4
+      for (int c = threadIdx.x; c < KT * CH; c += 256) {
+        const int tok = c / CH, ch = c % CH;
+        const int sl = sl_sm[tok];
+        const bool ok = sl >= 0 && ch < row_ch;
+        cp_async16(sb + tile_off<LAT>(tok, ch), pool + (ok ? (int64_t)sl * row_elems + ch * 8 : 0), ok);
+      }
+    }
+    cp_async_commit();
+  };
+
+  if (threadIdx.x < KT) {
+    slot_sm[threadIdx.x] = fetch_slot(0);
+    slot_sm[KT + threadIdx.x] = fetch_slot(1);
+  }
+  // query rows as MMA fragments
+  uint32_t qf[KSTEPS][4];
+  {
+    const bf16* q0 = q_lat + ((int64_t)t * H + head0 + g) * rank;
+    const bf16* q1 = q0 + (int64_t)8 * rank;
+    const bool ok0 = head0 + g < H, ok1 = head0 + g + 8 < H;
+#pragma unroll
+    for (int ks = 0; ks < KSTEPS; ++ks) {
+      const int d = ks * 16 + tig * 2;
+      qf[ks][0] = ok0 && d < rank ? *reinterpret_cast<const uint32_t*>(q0 + d) : 0u;
+      qf[ks][1] = ok1 && d < rank ? *reinterpret_cast<const uint32_t*>(q1 + d) : 0u;
+      qf[ks][2] = ok0 && d + 8 < rank ? *reinterpret_cast<const uint32_t*>(q0 + d + 8) : 0u;
+      qf[ks][3] = ok1 && d + 8 < rank ? *reinterpret_cast<const uint32_t*>(q1 + d + 8) : 0u;
+    }
+  }
+  __syncthreads();
+  issue(0);
+  issue(1);
+  __syncthreads();  // both slot buffers read
+  if (threadIdx.x < KT) slot_sm[threadIdx.x] = fetch_slot(2);
+
+  float o[2 * N2][4];
+#pragma unroll
+  for (int i = 0; i < 2 * N2; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
+  float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
+
+  for (int i = 0; i < n_tiles; ++i) {
+    cp_async_wait<1>();  // tile i landed (its group is the second youngest)
+    __syncthreads();     // ... for all threads; every warp is done with tile i - 1; slots of tile i + 2 are visible
+    issue(i + 2);
+    const int next_slot = threadIdx.x < KT ? fetch_slot(i + 3) : 0;
+    const uint32_t kb = kv_base + (uint32_t)(i % STAGES) * (KT * LAT * 2);
+
+    // ---- scores of this warp's 8 keys over the whole latent ----
+    float sc[4][4];
+#pragma unroll
+    for (int a = 0; a < 4; ++a) sc[a][0] = sc[a][1] = sc[a][2] = sc[a][3] = 0.f;
+#pragma unroll
+    for (int k2 = 0; k2 < KSTEPS / 2; ++k2) {
+      uint32_t b0, b1, b2, b3;
+      ldmatrix_x4(b0, b1, b2, b3, kb + tile_off<LAT>(warp * 8 + (lane & 7), k2 * 4 + (lane >> 3)));
+      mma_bf16_16816(sc[(2 * k2) & 3], qf[2 * k2][0], qf[2 * k2][1], qf[2 * k2][2], qf[2 * k2][3], b0, b1);
+      mma_bf16_16816(sc[(2 * k2 + 1) & 3], qf[2 * k2 + 1][0], qf[2 * k2 + 1][1], qf[2 * k2 + 1][2], qf[2 * k2 + 1][3],
+                     b2, b3);
+    }
+    {
+      const int col = warp * 8 + tig * 2;
+      const int kp = key0 + i * KT + col;
+      const bool v0 = kp < k_end, v1 = kp + 1 < k_end;
+      float s[4];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) s[e] = ((sc[0][e] + sc[1][e]) + (sc[2][e] + sc[3][e])) * scale_log2;
+      *reinterpret_cast<float2*>(s_sm + g * S_PITCH + col) =
+          make_float2(v0 ? s[0] : -INFINITY, v1 ? s[1] : -INFINITY);
+      *reinterpret_cast<float2*>(s_sm + (g + 8) * S_PITCH + col) =
+          make_float2(v0 ? s[2] : -INFINITY, v1 ? s[3] : -INFINITY);
+    }
+    __syncthreads();
+    if (threadIdx.x < KT) slot_sm[((i + 1) & 1) * KT + threadIdx.x] = next_slot;
+
+    // ---- softmax bookkeeping, the same in all warps ----
+    float s[KT / 8][4];
+    float mx[2] = {-INFINITY, -INFINITY};
+#pragma unroll
+    for (int j = 0; j < KT / 8; ++j) {
+      const float2 lo = *reinterpret_cast<const float2*>(s_sm + g * S_PITCH + j * 8 + tig * 2);
+      const float2 hi = *reinterpret_cast<const float2*>(s_sm + (g + 8) * S_PITCH + j * 8 + tig * 2);
+      s[j][0] = lo.x; s[j][1] = lo.y; s[j][2] = hi.x; s[j][3] = hi.y;
+      mx[0] = fmaxf(mx[0], fmaxf(lo.x, lo.y));
+      mx[1] = fmaxf(mx[1], fmaxf(hi.x, hi.y));
+    }
+    float alpha[2];
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 1));
+      mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 2));
+      const float m_new = fmaxf(m_run[r], mx[r]);  // finite: every tile has a visible key
+      alpha[r] = exp2f(m_run[r] - m_new);
+      m_run[r] = m_new;
+      float rs = 0.f;
+#pragma unroll
+      for (int j = 0; j < KT / 8; ++j) {
+        s[j][2 * r] = exp2f(s[j][2 * r] - m_new);
+        s[j][2 * r + 1] = exp2f(s[j][2 * r + 1] - m_new);
+        rs += s[j][2 * r] + s[j][2 * r + 1];
+      }
+      l_run[r] = l_run[r] * alpha[r] + rs;
+    }
+#pragma unroll
+    for (int n = 0; n < 2 * N2; ++n) {
+      o[n][0] *= alpha[0];
+      o[n][1] *= alpha[0];
+      o[n][2] *= alpha[1];
+      o[n][3] *= alpha[1];
+    }
+    // ---- o[:, this warp's columns] += P . c, P = high + low bf16 parts ----
+#pragma unroll
+    for (int kk = 0; kk < KT / 16; ++kk) {
+      uint32_t ah[4], al[4];
+#pragma unroll
+      for (int q4 = 0; q4 < 4; ++q4) {  // a0: row g, a1: row g + 8, a2 / a3: the same rows, keys + 8
+        const float x = s[2 * kk + (q4 >> 1)][(q4 & 1) * 2], y = s[2 * kk + (q4 >> 1)][(q4 & 1) * 2 + 1];
+        ah[q4] = pack_bf16x2(x, y);
+        const float xh = __uint_as_float(ah[q4] << 16), yh = __uint_as_float(ah[q4] & 0xffff0000u);
+        al[q4] = pack_bf16x2(x - xh, y - yh);
+      }
+      const int tok = kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8;
+#pragma unroll
+      for (int n = 0; n < N2; ++n) {
+        uint32_t b0, b1, b2, b3;
+        ldmatrix_x4_trans(b0, b1, b2, b3, kb + tile_off<LAT>(tok, warp * (LAT / 64) + n * 2 + (lane >> 4)));
+        mma_bf16_16816(o[2 * n], ah[0], ah[1], ah[2], ah[3], b0, b1);
+        mma_bf16_16816(o[2 * n + 1], ah[0], ah[1], ah[2], ah[3], b2, b3);
+        mma_bf16_16816(o[2 * n], al[0], al[1], al[2], al[3], b0, b1);
+        mma_bf16_16816(o[2 * n + 1], al[0], al[1], al[2], al[3], b2, b3);
+      }
+    }
+  }
+
+#pragma unroll
+  for (int r = 0; r < 2; ++r) {
+    l_run[r] += __shfl_xor_sync(0xffffffffu, l_run[r], 1);
+    l_run[r] += __shfl_xor_sync(0xffffffffu, l_run[r], 2);
+    const int h = head0 + g + 8 * r;
+    if (h >= H) continue;
+    const int64_t row = (int64_t)t * H + h;
+    const int col0 = warp * (LAT / 8) + tig * 2;
+    if (splits == 1) {
+      const float inv = 1.f / l_run[r];
+#pragma unroll
+      for (int n = 0; n < 2 * N2; ++n) {
+        const int col = col0 + n * 8;
+        if (col < rank)
+          *reinterpret_cast<bf162*>(out + row * rank + col) =
+              __floats2bfloat162_rn(o[n][2 * r] * inv, o[n][2 * r + 1] * inv);
+      }
+    } else {
+      const int64_t prow = (int64_t)split * Tn * H + row;
+#pragma unroll
+      for (int n = 0; n < 2 * N2; ++n) {
+        const int col = col0 + n * 8;
+        if (col < rank)
+          *reinterpret_cast<float2*>(part_o + prow * rank + col) = make_float2(o[n][2 * r], o[n][2 * r + 1]);
+      }
+      if (warp == 0 && tig == 0) part_ml[prow] = make_float2(m_run[r], l_run[r]);
+    }
+  }
+  cp_async_wait<0>();
+}
+
+// One warp per (token, head): merges the partial results of the shares.
+__global__ void __launch_bounds__(256)
+latent_attn_merge_kernel(const float* __restrict__ part_o, const float2* __restrict__ part_ml, bf16* __restrict__ out,
+                         int rows, int rank, int splits) {
+  const int row = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (row >= rows) return;
+  float M = -INFINITY;
+  for (int s = 0; s < splits; ++s) M = fmaxf(M, part_ml[(int64_t)s * rows + row].x);
+  float L = 0.f;
+  for (int s = 0; s < splits; ++s) {
+    const float2 ml = part_ml[(int64_t)s * rows + row];
+    if (ml.x != -INFINITY) L += ml.y * exp2f(ml.x - M);
+  }
+  const float inv = 1.f / L;
+  for (int d = lane * 2; d < rank; d += 64) {
+    float2 acc = make_float2(0.f, 0.f);
+    for (int s = 0; s < splits; ++s) {
+      const float m = part_ml[(int64_t)s * rows + row].x;
+      if (m == -INFINITY) continue;
+      const float w = exp2f(m - M);
+      const float2 v = *reinterpret_cast<const float2*>(part_o + ((int64_t)s * rows + row) * rank + d);
+      acc.x += w * v.x;
+      acc.y += w * v.y;
+    }
+    *reinterpret_cast<bf162*>(out + (int64_t)row * rank + d) = __floats2bfloat162_rn(acc.x * inv, acc.y * inv);
+  }
+}
+
+struct MmaArgs {
+  const bf16 *q_lat, *pool;
+  bf16* out;
+  const int *r2t, *b_req_idx, *pos, *batch_of;
+  float* part_o;
+  float2* part_ml;
+  int64_t r2t_stride;
+  int row_elems, T, H, rank, window, splits;
+  float scale_log2;
+};
+
+template <int LAT>
+int launch_mma(const MmaArgs& a, cudaStream_t st) {
+  static DeviceOnce configured;
+  if (!configured.done()) {
+    cudaError_t e = cudaFuncSetAttribute(latent_attn_mma_kernel<LAT>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                         mma_smem<LAT>());
+    if (e != cudaSuccess) return (int)e;
+    configured.set();
+  }
+  const dim3 grid(a.T, (a.H + 15) / 16, a.splits);
+  latent_attn_mma_kernel<LAT><<<grid, 256, mma_smem<LAT>(), st>>>(
+      a.q_lat, a.pool, a.row_elems, a.r2t, a.r2t_stride, a.b_req_idx, a.pos, a.batch_of, a.out, a.part_o, a.part_ml, a.T,
+      a.H, a.rank, a.scale_log2, a.window);
+  LLB_LAUNCH_CHECK();
+  return LLB_OK;
+}
+
+}  // namespace
+
+// dtype: 0 = fp32, 1 = bf16.  `rank` values per latent; the pool row has row_elems >= rank elements.
+LLB_EXPORT int llb_latent_norm_scatter(const void* src, int dtype, int64_t src_stride, void* pool, int row_elems,
+                                       const float* w, const int* slot, int T, int rank, float eps, cudaStream_t st) {
+  if (T <= 0) return LLB_OK;
+  if (rank <= 0 || rank > row_elems) return LLB_ERR_BAD_ARG;
+  if (dtype == 0)
+    latent_norm_scatter_kernel<float><<<cdiv(T, 4), 128, 0, st>>>((const float*)src, src_stride, (float*)pool, row_elems,
+                                                                  w, slot, T, rank, eps);
+  else
+    latent_norm_scatter_kernel<bf16><<<cdiv(T, 4), 128, 0, st>>>((const bf16*)src, src_stride, (bf16*)pool, row_elems, w,
+                                                                 slot, T, rank, eps);
+  LLB_LAUNCH_CHECK();
+  return LLB_OK;
+}
+
+LLB_EXPORT int llb_latent_gather(const void* pool, int row_bytes, const int* req_to_token, int64_t r2t_stride,
+                                 const int* b_req_idx, const int* cu_kv, const int* kv_start, void* out, int B, int rows,
+                                 cudaStream_t st) {
+  if (B <= 0 || rows <= 0) return LLB_OK;
+  if ((row_bytes & 15) || ((uintptr_t)pool & 15) || ((uintptr_t)out & 15)) return LLB_ERR_BAD_ARG;
+  const int grid = cdiv(rows, 8) < 148 * 8 ? cdiv(rows, 8) : 148 * 8;
+  latent_gather_kernel<<<grid, 256, 0, st>>>((const uint4*)pool, row_bytes / 16, req_to_token, r2t_stride, b_req_idx,
+                                             cu_kv, kv_start, (uint4*)out, B);
+  LLB_LAUNCH_CHECK();
+  return LLB_OK;
+}
+
+// q_lat, out: [T, H, row_elems] contiguous, of which `rank` = row_elems columns are used (padding columns are zero).
+// pos: position of every query token; batch_of: its request (null: token i belongs to request i).
+LLB_EXPORT int llb_latent_attn_generic(const void* q_lat, int dtype, const void* pool, int row_elems,
+                                       const int* req_to_token, int64_t r2t_stride, const int* b_req_idx, const int* pos,
+                                       const int* batch_of, void* out, int T, int H, int rank, float scale, int window,
+                                       cudaStream_t st) {
+  if (T <= 0) return LLB_OK;
+  if (rank <= 0 || rank > 1024 || rank > row_elems || H <= 0 || H > 65535) return LLB_ERR_UNSUPPORTED;
+  return dtype == 0 ? launch_generic<float>(q_lat, pool, row_elems, req_to_token, r2t_stride, b_req_idx, pos, batch_of,
+                                            out, T, H, rank, scale, window, st)
+                    : launch_generic<bf16>(q_lat, pool, row_elems, req_to_token, r2t_stride, b_req_idx, pos, batch_of,
+                                           out, T, H, rank, scale, window, st);
+}
+
+// bf16; rank a multiple of 8, at most 512.  splits > 1: part_o [splits * T * H * rank] and part_ml [splits * T * H * 2]
+// floats of scratch.
+LLB_EXPORT int llb_latent_attn_mma(const void* q_lat, const void* pool, int row_elems, const int* req_to_token,
+                                   int64_t r2t_stride, const int* b_req_idx, const int* pos, const int* batch_of,
+                                   void* out, float* part_o, float* part_ml, int T, int H, int rank, int splits,
+                                   float scale, int window, cudaStream_t st) {
+  if (T <= 0) return LLB_OK;
+  if (rank <= 0 || rank > 512 || (rank % 8) || (row_elems % 8) || rank > row_elems || H <= 0) return LLB_ERR_UNSUPPORTED;
+  if (splits < 1 || splits > 256 || (splits > 1 && (part_o == nullptr || part_ml == nullptr))) return LLB_ERR_BAD_ARG;
+  if (((uintptr_t)q_lat & 15) || ((uintptr_t)pool & 15) || ((uintptr_t)out & 3)) return LLB_ERR_BAD_ARG;
+  MmaArgs a{(const bf16*)q_lat, (const bf16*)pool, (bf16*)out, req_to_token, b_req_idx, pos, batch_of, part_o,
+            (float2*)part_ml, r2t_stride, row_elems, T, H, rank, window, splits, scale * kLog2e};
+  int rc;
+  if (rank <= 128)
+    rc = launch_mma<128>(a, st);
+  else if (rank <= 256)
+    rc = launch_mma<256>(a, st);
+  else if (rank <= 384)
+    rc = launch_mma<384>(a, st);
+  else
+    rc = launch_mma<512>(a, st);
+  if (rc || splits == 1) return rc;
+  latent_attn_merge_kernel<<<cdiv(T * H, 8), 256, 0, st>>>(part_o, (const float2*)part_ml, (bf16*)out, T * H, rank, splits);
+  LLB_LAUNCH_CHECK();
+  return LLB_OK;
+}

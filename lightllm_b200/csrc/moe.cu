@@ -188,10 +188,12 @@ grouped_topk_kernel(const T* __restrict__ logits, int64_t stride, const float* _
 // outputs: sorted_pair[M_pad] (pair index of each sorted row, -1 for padding), pair_row[T*k] (row of each pair,
 // -1 if dropped), mblock_expert[M_pad/128] (local expert id or -1), expert_rows[E_local+1] (padded offsets),
 // total_rows[1]
-__global__ void __launch_bounds__(1024)
-moe_align_kernel(const int* __restrict__ ids, int n_pairs, int e0, int E_local, int m_pad, int* __restrict__ sorted_pair,
-                 int* __restrict__ pair_row, int* __restrict__ mblock_expert, int* __restrict__ expert_off,
-                 int* __restrict__ total_rows) {
+// `id_of(p)`: expert of pair p (negative: none).
+template <typename IdOf>
+__device__ __forceinline__ void align_pairs(IdOf id_of, int n_pairs, int e0, int E_local, int m_pad,
+                                            int* __restrict__ sorted_pair, int* __restrict__ pair_row,
+                                            int* __restrict__ mblock_expert, int* __restrict__ expert_off,
+                                            int* __restrict__ total_rows) {
   extern __shared__ int sm[];
   int* cnt = sm;                 // [E_local]
   int* off = sm + E_local;       // [E_local + 1]
@@ -199,7 +201,7 @@ moe_align_kernel(const int* __restrict__ ids, int n_pairs, int e0, int E_local, 
   for (int i = threadIdx.x; i < E_local; i += blockDim.x) cnt[i] = 0;
   __syncthreads();
   for (int p = threadIdx.x; p < n_pairs; p += blockDim.x) {
-    int e = (ids[p] < 0 ? ids[p] : LLB_CHECK_EXPERT(ids[p])) - e0;
+    const int e = id_of(p) - e0;
     if (e >= 0 && e < E_local) atomicAdd(&cnt[e], 1);
   }
   __syncthreads();
@@ -233,7 +235,7 @@ moe_align_kernel(const int* __restrict__ ids, int n_pairs, int e0, int E_local, 
   }
   __syncthreads();
   for (int p = threadIdx.x; p < n_pairs; p += blockDim.x) {
-    int e = ids[p] - e0;
+    const int e = id_of(p) - e0;
     if (e >= 0 && e < E_local) {
       int r = off[e] + atomicAdd(&cur[e], 1);
       sorted_pair[r] = p;
@@ -242,6 +244,40 @@ moe_align_kernel(const int* __restrict__ ids, int n_pairs, int e0, int E_local, 
       pair_row[p] = -1;
     }
   }
+}
+
+__global__ void __launch_bounds__(1024)
+moe_align_kernel(const int* __restrict__ ids, int n_pairs, int e0, int E_local, int m_pad, int* __restrict__ sorted_pair,
+                 int* __restrict__ pair_row, int* __restrict__ mblock_expert, int* __restrict__ expert_off,
+                 int* __restrict__ total_rows) {
+  align_pairs([&](int p) { return ids[p] < 0 ? ids[p] : LLB_CHECK_EXPERT(ids[p]); }, n_pairs, e0, E_local, m_pad,
+              sorted_pair, pair_row, mblock_expert, expert_off, total_rows);
+}
+
+// Table routing: the experts of a token are a row of the layer's table [vocab, k], looked up by token id, so the
+// expert-sorted layouts of ALL layers are known before the first one runs.  One CTA per layer; its slab of `stride`
+// ints holds sorted_pair [m_pad], pair_row [T * k], mblock_expert [m_pad / 128], expert_off [E_local + 1],
+// total_rows [1], with m_pad = T * k + min(E_local, T * k) * 127 rounded up to 128.
+struct TableRoute {
+  const int* table;
+  int k, e0, E_local, pad;
+};
+__global__ void __launch_bounds__(1024)
+moe_table_align_kernel(const TableRoute* __restrict__ routes, const int64_t* __restrict__ token_ids, int64_t vocab, int T,
+                       int* __restrict__ out, int64_t stride) {
+  const TableRoute r = routes[blockIdx.x];
+  const int n = T * r.k;
+  const int m_pad = ((n + min(r.E_local, n) * 127 + 127) / 128) * 128;
+  int* sorted_pair = out + (int64_t)blockIdx.x * stride;
+  int* pair_row = sorted_pair + m_pad;
+  int* mblock = pair_row + n;
+  int* off = mblock + m_pad / 128;
+  align_pairs(
+      [&](int p) {
+        const int64_t tok = token_ids[p / r.k];
+        return tok >= 0 && tok < vocab ? r.table[tok * r.k + p % r.k] : -1;
+      },
+      n, r.e0, r.E_local, m_pad, sorted_pair, pair_row, mblock, off, off + r.E_local + 1);
 }
 
 // A_sorted[row] = x[sorted_pair[row] / k]  (zeros for padding rows)
@@ -295,6 +331,17 @@ LLB_EXPORT int llb_topk_softmax(const void* logits, int dtype, int64_t stride, i
     topk_softmax_kernel<float><<<cdiv(T, 4), 128, 0, st>>>((const float*)logits, stride, T, E, k, renorm, scale, ids, weights);
   else
     topk_softmax_kernel<bf16><<<cdiv(T, 4), 128, 0, st>>>((const bf16*)logits, stride, T, E, k, renorm, scale, ids, weights);
+  LLB_LAUNCH_CHECK();
+  return LLB_OK;
+}
+
+// routes: device array of L {table pointer, k, first local expert, number of local experts, 0}.
+LLB_EXPORT int llb_moe_table_align(const void* routes, int L, int max_experts, const int64_t* token_ids, int64_t vocab,
+                                   int T, int* out, int64_t stride, cudaStream_t st) {
+  if (T <= 0 || L <= 0) return LLB_OK;
+  const size_t smem = (3 * (size_t)max_experts + 1) * sizeof(int);
+  if (smem > 48 * 1024) return LLB_ERR_UNSUPPORTED;
+  moe_table_align_kernel<<<L, 1024, smem, st>>>((const TableRoute*)routes, token_ids, vocab, T, out, stride);
   LLB_LAUNCH_CHECK();
   return LLB_OK;
 }
