@@ -97,6 +97,35 @@ def build_kernels(force: bool = False, verbose: bool = True, debug_bounds: bool 
     return out
 
 
+def build_units(units, verbose: bool = False) -> list:
+    """One library per named csrc unit (`libllb_unit_<name>.so`), compiled side by side: what a program without the
+    whole library needs on first use.  Writers in several processes are kept apart by a lock file."""
+    import fcntl
+
+    OBJ.mkdir(parents=True, exist_ok=True)
+    headers = sorted(CSRC.glob("*.cuh")) + sorted(CSRC.glob("*.h"))
+
+    def one(unit):
+        out = LIB / f"libllb_unit_{unit}.so"
+        obj = _compile_cu(CSRC / f"{unit}.cu", headers, force=False)
+        stamp = OBJ / f"unit.{unit}.sha"
+        dig = _digest([obj])
+        if not out.exists() or not stamp.exists() or stamp.read_text() != dig:
+            r = subprocess.run([_nvcc(), "-shared", "-o", str(out), str(obj), "-Xcompiler", "-fPIC"],
+                               capture_output=True, text=True)
+            if r.returncode != 0:
+                raise RuntimeError(f"link failed:\n{r.stderr[-4000:]}")
+            stamp.write_text(dig)
+            if verbose:
+                print(f"[build] linked {out}")
+        return out
+
+    with open(OBJ / "units.lock", "w") as lock:
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        with cf.ThreadPoolExecutor(max_workers=8) as ex:
+            return list(ex.map(one, units))
+
+
 def build_runtime(force: bool = False, verbose: bool = True) -> Path:
     LIB.mkdir(parents=True, exist_ok=True)
     OBJ.mkdir(parents=True, exist_ok=True)

@@ -29,6 +29,7 @@ class ModelInput:
     b_prefill_has_output: Optional[List[bool]] = None  # chunked prefill: does this chunk end the prompt
     multimodal_params: Optional[list] = None
     return_all_logits: bool = False      # prompt_logprobs: logits for every prompt position
+    logit_rows: Optional[torch.Tensor] = None      # prefill: logits of these rows instead of each request's last
     b_mtp_index: Optional[torch.Tensor] = None
     return_hidden: bool = False          # speculative decoding: also return the final residual stream [T, hidden]
     draft_input_hidden: Optional[torch.Tensor] = None  # draft modules: hidden state of the target model per token

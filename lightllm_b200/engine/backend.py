@@ -346,7 +346,9 @@ class ModelBackend:
         return {"kind": kind, "finished": finished, "tokens": n_tok}
 
     # ---- prefill ----
-    def _run_prefill(self, items) -> int:
+    def _prefill_input(self, items):
+        """The ModelInput of one prompt pass over (request, new tokens) items, with pool slots taken for the new
+        tokens, and the pass' token ids and portion lengths."""
         reqs = [r for r, _ in items]
         B = len(reqs)
         chunks = np.array([c for _, c in items], dtype=np.int32)
@@ -360,6 +362,19 @@ class ModelBackend:
             r.slots = np.concatenate([r.slots[: r.cur_kv_len], slots_np[off:off + c]])
             off += int(c)
         pin = self.pins
+        mi = ModelInput(batch_size=B, total_token_num=int((ready + chunks).sum()), max_kv_len=int((ready + chunks).max()),
+                        is_prefill=True,
+                        b_req_idx=pin.from_numpy("p_req", np.array([r.req_idx for r in reqs], dtype=np.int32), torch.int32),
+                        b_seq_len=pin.from_numpy("p_seq", ready + chunks, torch.int32),
+                        mem_indexes=slots,
+                        input_ids=pin.from_numpy("p_ids", ids.astype(np.int64), torch.int64),
+                        b_ready_cache_len=pin.from_numpy("p_ready", ready, torch.int32),
+                        b_q_len=pin.from_numpy("p_qlen", chunks, torch.int32), max_q_len=int(chunks.max()))
+        self.stats["h2d_bytes"] += total * 8 + total * 4 + B * 16
+        return mi, ids, chunks
+
+    def _run_prefill(self, items) -> int:
+        reqs = [r for r, _ in items]
         want_all = self.args.return_all_prompt_logprobs and any(r.sampling.prompt_logprobs >= 0 for r in reqs)
         mm = None
         if any(getattr(r.shm_req, "_mm_params", None) for r in reqs):
@@ -370,16 +385,9 @@ class ModelBackend:
                     p = dict(p)
                     p["_prompt_ids"] = np.asarray(r.shm_req.shm_prompt_ids.arr[: r.shm_req.input_len])
                 mm.append(p)
-        mi = ModelInput(batch_size=B, total_token_num=int((ready + chunks).sum()), max_kv_len=int((ready + chunks).max()),
-                        is_prefill=True,
-                        b_req_idx=pin.from_numpy("p_req", np.array([r.req_idx for r in reqs], dtype=np.int32), torch.int32),
-                        b_seq_len=pin.from_numpy("p_seq", ready + chunks, torch.int32),
-                        mem_indexes=slots,
-                        input_ids=pin.from_numpy("p_ids", ids.astype(np.int64), torch.int64),
-                        b_ready_cache_len=pin.from_numpy("p_ready", ready, torch.int32),
-                        b_q_len=pin.from_numpy("p_qlen", chunks, torch.int32), max_q_len=int(chunks.max()),
-                        return_all_logits=want_all, multimodal_params=mm)
-        self.stats["h2d_bytes"] += total * 8 + total * 4 + B * 16
+        mi, ids, chunks = self._prefill_input(items)
+        mi.return_all_logits, mi.multimodal_params = want_all, mm
+        total = int(chunks.sum())
         out = self.model.forward(mi)
         has_out = np.array([r.cur_kv_len + int(c) >= r.total_len() for r, c in items], dtype=bool)
         for r, c in items:
@@ -486,7 +494,8 @@ class ModelBackend:
             live.append(not r.finish_status.is_finished())
         self._post(reqs, ids_h.numpy(), lps_h.numpy(), np.array(live, dtype=bool))
 
-    def _run_decode(self, reqs: List[InferReq], defer: bool = False) -> int:
+    def _decode_input(self, reqs: List[InferReq]) -> ModelInput:
+        """The ModelInput of one decode step (the token of every request waits in the request table on the device)."""
         B = len(reqs)
         slots = self.ctx.alloc_slots(B)
         slots_np = slots.numpy()
@@ -498,10 +507,14 @@ class ModelBackend:
             seq[i] = r.cur_kv_len
             idx[i] = r.req_idx
         pin = self.pins
-        mi = ModelInput(batch_size=B, total_token_num=int(seq.sum()), max_kv_len=int(seq.max()), is_prefill=False,
-                        b_req_idx=pin.from_numpy("d_req", idx, torch.int32),
-                        b_seq_len=pin.from_numpy("d_seq", seq, torch.int32), mem_indexes=slots)
         self.stats["h2d_bytes"] += B * 12
+        return ModelInput(batch_size=B, total_token_num=int(seq.sum()), max_kv_len=int(seq.max()), is_prefill=False,
+                          b_req_idx=pin.from_numpy("d_req", idx, torch.int32),
+                          b_seq_len=pin.from_numpy("d_seq", seq, torch.int32), mem_indexes=slots)
+
+    def _run_decode(self, reqs: List[InferReq], defer: bool = False) -> int:
+        B = len(reqs)
+        mi = self._decode_input(reqs)
         timing = self._step_timing and not defer and self.device.type == "cuda"
         if timing:   # LLB_STEP_TIMING=1: device time of the synchronous decode passes (forward + sampling)
             ev0, ev1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
@@ -540,6 +553,28 @@ class ModelBackend:
         self.stats["decode_steps"] += 1
         self.stats["decode_tokens"] += B
         return B
+
+    # ---- replay ----
+    @torch.no_grad()
+    def replay_step(self, items, wanted_rows):
+        """One pass over given tokens: items = [(request, number of new tokens)], the tokens being in the request
+        already (prompt ids or `append_token`).  Runs the pass a serving step would: a decode step when every request
+        brings one token on top of cached ones, else one prompt pass over all portions.  Returns the logits of the
+        rows `wanted_rows` of the pass (tokens counted over all items), fp32 on the device; samples nothing."""
+        reqs = [r for r, _ in items]
+        rows = torch.tensor(wanted_rows, dtype=torch.int32)
+        if all(c == 1 and r.cur_kv_len > 0 for r, c in items):
+            ids = torch.tensor([int(r.get_chunked_input_token_ids(1)[0]) for r in reqs], dtype=torch.int64)
+            idx = torch.tensor([r.req_idx for r in reqs], dtype=torch.int32)
+            ops.scatter_next_token_(self.model.req_manager.req_to_next_token_ids, ids.to(self.device), idx.to(self.device))
+            logits = self.model.forward(self._decode_input(reqs)).logits
+            return logits.index_select(0, rows.to(self.device))
+        mi, _, chunks = self._prefill_input(items)
+        mi.logit_rows = rows if len(wanted_rows) else None
+        out = self.model.forward(mi)
+        for r, c in items:
+            r.cur_kv_len += int(c)
+        return out.logits if len(wanted_rows) else out.logits[:0]
 
     # ---- sampling + post ----
     sharded_sampling = True   # subclasses that read whole logit rows in their own sampling code turn this off

@@ -40,7 +40,9 @@ def normalize_config(cfg: dict) -> dict:
     """One spelling for keys that differ between config generations: `rope_parameters` (new) is unfolded into
     `rope_theta` / `rope_scaling`, `num_local_experts` doubles as `num_experts`, multimodal wrappers expose
     their `text_config` at the top level."""
-    cfg = dict(cfg)
+    from .registry import native_config
+
+    cfg = dict(native_config(cfg))
     if isinstance(cfg.get("thinker_config"), dict) and "text_config" not in cfg:  # Qwen3-Omni: thinker / talker parts
         cfg = {**cfg, **cfg["thinker_config"], "model_type": cfg.get("model_type")}
     if "text_config" in cfg and "hidden_size" not in cfg:  # multimodal wrappers
@@ -100,6 +102,8 @@ class LayerWeights:
 
 class TransformerLM:
     model_type = "llama"
+    supports_float32 = False   # the family's GPU path also exists in fp32 (data_type "float32")
+    native_units = None        # csrc units of the family's kernels, for a checkout without built libraries (None: all)
 
     # ------------------------------------------------------------------ init
     def __init__(self, config: dict, *, weight_source: Optional[WeightSource] = None, model_dir: Optional[str] = None,
@@ -118,7 +122,8 @@ class TransformerLM:
         self.tp = TPContext(self.ps, fused=tp_fused)
         dt = data_type or config.get("torch_dtype") or config.get("dtype") or "bfloat16"
         self.dtype = _DTYPES[str(dt).replace("torch.", "")]
-        if self.device.type == "cuda" and self.dtype != torch.bfloat16:
+        if self.device.type == "cuda" and self.dtype != torch.bfloat16 and \
+                not (self.supports_float32 and self.dtype == torch.float32):
             self.dtype = torch.bfloat16  # the sm_100a kernels are bf16
         self.extra = extra
         self.tpsp_mix_mode = bool(extra.get("tpsp_mix_mode", False))  # token-sharded residual stream between layers
@@ -145,7 +150,7 @@ class TransformerLM:
             weight_source = self._wrap_source(self._open_checkpoint(model_dir)) \
                 if model_dir and self._has_weights(model_dir) else RandomSource(self.weight_shapes(), dtype=self.dtype, seed=random_seed,
                              device=str(self.device) if self.device.type == "cuda" else "cpu",
-                             fp8_names=self.fp8_weight_names())
+                             fp8_names=self.fp8_weight_names(), inits=self.weight_inits())
         self.weight_source = weight_source
         from ..engine.redundancy import RedundancyConfig
 
@@ -233,6 +238,10 @@ class TransformerLM:
     # ------------------------------------------------------------------ weights
     def fp8_weight_names(self):
         return set()
+
+    def weight_inits(self):
+        """Random initialisation of tensors that are not N(0, std): name -> fn(shape, generator, device)."""
+        return {}
 
     def weight_shapes(self) -> Dict[str, tuple]:
         """HF names -> full (unsharded) shapes; drives RandomSource and documents the checkpoint format."""
@@ -484,12 +493,12 @@ class TransformerLM:
         self._prepare_prefill_state(st)
         return st, input_ids
 
-    def _last_rows(self, h, st: InferState, all_rows: bool):
+    def _last_rows(self, h, st: InferState, all_rows: bool, rows=None):
         if all_rows:
             return h
-        B = st.batch_size
-        last_idx = (st.cu_q[1:] - 1).to(torch.int32)
-        last = torch.empty((B, self.hidden), dtype=h.dtype, device=self.device)
+        B = st.batch_size if rows is None else rows.shape[0]
+        last_idx = (st.cu_q[1:] - 1).to(torch.int32) if rows is None else rows.to(self.device, torch.int32)
+        last = torch.empty((B, h.shape[1]), dtype=h.dtype, device=self.device)
         ops.copy_rows(last, h, None, last_idx, B)
         return last
 
@@ -507,7 +516,7 @@ class TransformerLM:
         if bal is not None:
             h = bal.to_origin(h)
         hidden = h if mi.return_hidden else None
-        last = self._last_rows(h, st, mi.return_all_logits)
+        last = self._last_rows(h, st, mi.return_all_logits, mi.logit_rows)
         logits = self._lm_head(last, normed=True) if st.extra.get("normed") else self._lm_head(last)
         return ModelOutput(logits=logits, hidden=hidden)
 
@@ -539,7 +548,7 @@ class TransformerLM:
         (no family hook between the layers, no multimodal rows, no hidden states wanted back), at least two
         requests and enough tokens for the transfers to matter."""
         ce = getattr(self.tp, "ce", None)
-        if ce is None or self.tp.size == 1 or mi.batch_size < 2 or mi.multimodal_params or mi.return_hidden \
+        if ce is None or self.tp.size == 1 or mi.batch_size < 2 or mi.logit_rows is not None or mi.multimodal_params or mi.return_hidden \
                 or mi.draft_input_hidden is not None or getattr(mi, "verify_pass", False) or ce.hidden != self.hidden:
             return None
         cls = type(self)

@@ -4,6 +4,28 @@ from __future__ import annotations
 from typing import Callable, Dict, Optional
 
 _REGISTRY: Dict[str, list] = {}
+_CONFIGS: Dict[str, Callable[[dict], dict]] = {}
+
+
+def register_config(architecture: str):
+    """For designs whose config.json is not in HF spelling: the decorated function turns a config with
+    `"architecture": architecture` (and no model_type) into one with the keys the framework reads."""
+    def deco(fn):
+        _CONFIGS[architecture] = fn
+        return fn
+
+    return deco
+
+
+def native_config(config: dict) -> dict:
+    if config.get("model_type") or not isinstance(config.get("architecture"), str):
+        return config
+    from . import _load_all  # noqa: F401
+
+    fn = _CONFIGS.get(config["architecture"])
+    if fn is None:
+        raise ValueError(f"unsupported architecture {config['architecture']!r}; known: {sorted(_CONFIGS)}")
+    return fn(config)
 
 
 def register_model(*model_types: str, condition: Optional[Callable[[dict], bool]] = None, is_multimodal=False):
@@ -18,7 +40,7 @@ def register_model(*model_types: str, condition: Optional[Callable[[dict], bool]
 def get_model_class(config: dict):
     from . import _load_all  # noqa: F401  (imports every model module once)
 
-    mt = config.get("model_type")
+    mt = native_config(config).get("model_type")
     cands = _REGISTRY.get(mt)
     if not cands:
         raise ValueError(f"unsupported model_type {mt!r}; known: {sorted(_REGISTRY)}")

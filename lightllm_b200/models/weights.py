@@ -97,13 +97,14 @@ class RandomSource(WeightSource):
     are generated as e4m3 payload ~ N(0, 96) plus `*_scale_inv` ~ U(0.5, 2) * std / 96 block scales."""
 
     def __init__(self, shapes: Dict[str, tuple], dtype=torch.bfloat16, std: float = 0.02, seed: int = 0,
-                 device: str = "cpu", fp8_names: Optional[set] = None):
+                 device: str = "cpu", fp8_names: Optional[set] = None, inits: Optional[dict] = None):
         self.shapes = dict(shapes)
         self.dtype = dtype
         self.std = std
         self.seed = seed
         self.device = torch.device(device)
         self.fp8_names = fp8_names or set()
+        self.inits = inits or {}
 
     def has(self, name):
         return name in self.shapes
@@ -122,7 +123,9 @@ class RandomSource(WeightSource):
 
     def get(self, name, dim=None, start=0, end=None):
         shape = self.shapes[name]
-        if name.endswith("norm.weight") or name.endswith("layernorm.weight") or name.endswith("_norm.weight") or \
+        if name in self.inits:
+            t = self.inits[name](shape, self._gen(name), self.device)
+        elif name.endswith("norm.weight") or name.endswith("layernorm.weight") or name.endswith("_norm.weight") or \
                 name.endswith("layer_scalar") or name.endswith("router.scale") or name.endswith("per_expert_scale"):
             t = torch.ones(shape, dtype=self.dtype, device=self.device)
         elif name.endswith("_scale_inv"):

@@ -15,7 +15,8 @@ from . import kv_quant
 from . import reference as ref
 from ._native import NativeError, c_int, c_void_p, check, f32, i64, kernels, ptr, stream
 
-EPI_CODES = {"store": 0, "residual": 1, "gated_silu": 2, "f32": 3, "gated_gelu": 4}
+EPI_CODES = {"store": 0, "residual": 1, "gated_silu": 2, "f32": 3, "gated_gelu": 4, "relu2": 5, "dyt": 6}
+DTYPE_CODES = {torch.float32: 0, torch.bfloat16: 1}   # kernels that exist in both number formats
 
 import os as _os
 
@@ -219,11 +220,15 @@ def _tuned_bn(M: int, N: int, K: int, epi: str) -> int:
     return _autotuner.gemm_lookup(M, N, K, epi)
 
 
-def gemm(a, w, epi: str = "store", residual=None, bias=None, out=None, bn: int = 0, stream_k: int = 0):
-    """C = A . W^T on the tcgen05 tensor cores.  a [M, K], w [N, K] (checkpoint layout).
+def gemm(a, w, epi: str = "store", residual=None, bias=None, out=None, bn: int = 0, stream_k: int = 0,
+         out_scale: float = 1.0, x=None, dyt=None):
+    """C = A . W^T on the tcgen05 tensor cores.  a [M, K], w [N, K] (checkpoint layout).  fp32 operands run on the
+    CUDA cores in fp32 (`csrc/gemm_f32.cu`).
 
     epi: "store" | "residual" (C += residual) | "gated_silu"/"gated_gelu" (w rows interleaved with
-    `reference.interleave_gate_up`, C is [M, N/2]) | "f32" (fp32 output, e.g. logits).
+    `reference.interleave_gate_up`, C is [M, N/2]) | "f32" (fp32 output, e.g. logits, times `out_scale`) |
+    "relu2" (square of relu) | "dyt": with the fp32 residual stream x [M, N] and dyt = (post, next) `DytNorm`s,
+    x += post(A . W^T) in place and C = next(x).
     stream_k: 0 whole tiles per CTA (default: fastest on every measured shape), 1 stream-K, -1 heuristic.
     """
     if type(w).__name__ == "Fp8Weight":  # block-scaled e4m3 weight: quantise the activations, fp8 tensor cores
@@ -235,12 +240,16 @@ def gemm(a, w, epi: str = "store", residual=None, bias=None, out=None, bn: int =
 
         return int8.gemm_int8(a, w, epi, residual, bias, out)
     if not _is_cuda(a):
-        res = ref.gemm(a, w, epi, residual, bias)
+        res = ref.gemm(a, w, epi, residual, bias, out_scale=out_scale, x=x, dyt=dyt)
         if out is not None:
             out.copy_(res)
             return out
         return res
+    if a.dtype == torch.float32:
+        return gemm_f32(a, w, epi, residual, bias, out, out_scale, x, dyt)
     _req_bf16(a, w, residual, bias)
+    if epi == "dyt" or out_scale != 1.0:
+        return _gemm_fused(a, w, epi, bias, out, bn, out_scale, x, dyt)
     if _GEMM_DEBUG_TORCH:  # debugging aid only (LLB_GEMM_DEBUG_TORCH=1): bypasses the tcgen05 kernel
         res = ref.gemm(a, w, epi, residual, bias)
         if out is not None:
@@ -269,6 +278,56 @@ def gemm(a, w, epi: str = "store", residual=None, bias=None, out=None, bn: int =
                                   c_int(bn), c_int(stream_k), ptr(skp), i64(skp.numel() if skp is not None else 0),
                                   ptr(skc), c_int(skc.numel() if skc is not None else 0),
                                   ptr(gemm_status(a.device)), stream()), "gemm_bf16")
+    _count()
+    return out
+
+
+def _dyt_args(n):
+    """(w, b, alpha) of a DytNorm, or nulls."""
+    return (ptr(None), ptr(None), f32(1.0)) if n is None else (ptr(n.w), ptr(n.b), f32(n.alpha))
+
+
+def _gemm_fused(a, w, epi, bias, out, bn, out_scale, x, dyt):
+    M, K = a.shape
+    N = w.shape[0]
+    assert w.shape[1] == K and w.stride(1) == 1 and a.stride(1) == 1
+    if out is None:
+        out = torch.empty((M, N), dtype=torch.float32 if epi == "f32" else a.dtype, device=a.device)
+    post, nxt = dyt if dyt is not None else (None, None)
+    if epi == "dyt":
+        assert x.dtype == torch.float32 and x.shape == (M, N) and x.stride(0) == out.stride(0) and x.stride(1) == 1
+    check(kernels().llb_gemm_bf16_fused(ptr(a), i64(a.stride(0)), ptr(w), i64(w.stride(0)), ptr(out),
+                                        i64(out.stride(0)), ptr(bias), c_int(M), c_int(N), c_int(K),
+                                        c_int(EPI_CODES[epi]), c_int(bn), f32(out_scale), ptr(x), *_dyt_args(post),
+                                        *_dyt_args(nxt), ptr(gemm_status(a.device)), stream()), "gemm_bf16_fused")
+    _count()
+    return out
+
+
+def gemm_f32(a, w, epi="store", residual=None, bias=None, out=None, out_scale=1.0, x=None, dyt=None,
+             mblock_expert=None):
+    """fp32 GEMM, same epilogues as `gemm`.  a [M, K] and w [N, K]; or a [M, batch, K] and w [batch, N, K] (per-head
+    products, out [M, batch, N]); or grouped with w [E, N, K] and the expert of every 128-row block."""
+    grouped = mblock_expert is not None
+    batched = a.dim() == 3
+    batch = a.shape[1] if batched else 1
+    M, K = a.shape[0], a.shape[-1]
+    N = w.shape[-2]
+    assert w.dtype == torch.float32 and w.shape[-1] == K and a.stride(-1) == 1 and w.stride(-1) == 1
+    assert w.dim() == (3 if grouped or batched else 2)
+    n_out = N // 2 if epi.startswith("gated") else N
+    if out is None:
+        out = torch.empty((M, batch, n_out) if batched else (M, n_out), dtype=torch.float32, device=a.device)
+    post, nxt = dyt if dyt is not None else (None, None)
+    if epi == "residual":
+        assert residual.shape == out.shape and residual.stride(0) == out.stride(0)
+    if epi == "dyt":
+        assert x.shape == (M, N) and x.stride(0) == out.stride(0)
+    check(kernels().llb_gemm_f32(ptr(a), i64(a.stride(0)), i64(a.stride(1) if batched else 0), ptr(w),
+                                 i64(w.stride(-2)), i64(w.stride(0) if batched else 0), ptr(out), i64(out.stride(0)),
+                                 i64(out.stride(1) if batched else 0), ptr(residual), ptr(bias), ptr(x),
+                                 *_dyt_args(post), *_dyt_args(nxt), ptr(mblock_expert), c_int(M), c_int(N), c_int(K),
+                                 c_int(batch), c_int(EPI_CODES[epi]), f32(out_scale), stream()), "gemm_f32")
     _count()
     return out
 
@@ -554,3 +613,54 @@ def attention_generic(q, kv_layer, req_to_token, b_req_idx, pos, batch_of, Hq, H
                                      c_int(window), f32(softcap), ptr(alibi), ptr(sinks), stream()), "attn_generic")
     _count()
     return out
+
+
+# --------------------------------------------------------------------------------------
+class DytNorm:
+    """Dynamic-tanh norm: tanh(alpha * v) * w + b, elementwise, in fp32.  `alpha` is a host number."""
+
+    __slots__ = ("w", "b", "alpha")
+
+    def __init__(self, w: torch.Tensor, b: torch.Tensor, alpha: float):
+        self.w, self.b, self.alpha = w.float().contiguous(), b.float().contiguous(), float(alpha)
+
+
+def embedding_dyt(ids, table, norm: DytNorm):
+    """(x, h): x = the table's rows as the fp32 residual stream, h = norm(x) in the table's number format."""
+    if not _is_cuda(table):
+        x = table[ids].float()
+        return x, ref.dyt(x, norm).to(table.dtype)
+    T, W = ids.shape[0], table.shape[1]
+    x = torch.empty((T, W), dtype=torch.float32, device=table.device)
+    h = torch.empty((T, W), dtype=table.dtype, device=table.device)
+    assert ids.dtype == torch.int64 and ids.is_contiguous() and table.is_contiguous()
+    check(kernels().llb_embedding_dyt(ptr(ids), ptr(table), c_int(DTYPE_CODES[table.dtype]), i64(table.shape[0]), ptr(x),
+                                      ptr(h), c_int(T), c_int(W), *_dyt_args(norm), stream()), "embedding_dyt")
+    _count()
+    return x, h
+
+
+def dyt(x, norm: DytNorm, dtype):
+    """norm(x) of the fp32 stream x [T, W], in `dtype`."""
+    if not _is_cuda(x):
+        return ref.dyt(x, norm).to(dtype)
+    assert x.dtype == torch.float32 and x.is_contiguous()
+    h = torch.empty(x.shape, dtype=dtype, device=x.device)
+    check(kernels().llb_dyt(ptr(x), ptr(h), c_int(DTYPE_CODES[dtype]), c_int(x.shape[0]), c_int(x.shape[1]),
+                            *_dyt_args(norm), stream()), "dyt")
+    _count()
+    return h
+
+
+def add_dyt_(x, y, post: DytNorm, nxt: DytNorm, dtype):
+    """x += post(y) in place (fp32 stream); returns nxt(x) in `dtype`."""
+    if not _is_cuda(x):
+        x.add_(ref.dyt(y.float(), post))
+        return ref.dyt(x, nxt).to(dtype)
+    assert x.dtype == torch.float32 and x.is_contiguous() and y.is_contiguous() and x.shape == y.shape
+    h = torch.empty(x.shape, dtype=dtype, device=x.device)
+    check(kernels().llb_add_dyt(ptr(x), ptr(y), c_int(DTYPE_CODES[y.dtype]), ptr(h), c_int(DTYPE_CODES[dtype]),
+                                c_int(x.shape[0]), c_int(x.shape[1]), *_dyt_args(post), *_dyt_args(nxt), stream()),
+          "add_dyt")
+    _count()
+    return h

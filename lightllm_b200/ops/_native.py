@@ -1,13 +1,16 @@
 """ctypes loader for the in-tree native libraries.
 
 ``kernels()`` returns ``libllb_kernels.so`` (sm_100a CUDA kernels), ``runtime()`` returns
-``libllb_runtime.so`` (host C++: shm atomics, slot allocator, radix tree).  A missing
-library is an error on a machine with a GPU: the CUDA path never falls back silently.
+``libllb_runtime.so`` (host C++: shm atomics, slot allocator, radix tree).  The CUDA path never
+falls back silently.  In a checkout without built libraries (and unless LLB_AUTOBUILD=0) the kernels are
+compiled on first use, one library per source file, so a program compiles what it calls and no more;
+`prepare` compiles a known set side by side.  `python -m lightllm_b200.build` builds everything into one library.
 """
 from __future__ import annotations
 
 import ctypes
 import os
+import re
 from pathlib import Path
 
 import torch
@@ -38,9 +41,7 @@ def _load(name: str):
         if os.environ.get("LLB_AUTOBUILD", "1") == "1":
             from .. import build as _b
 
-            if name == "libllb_kernels.so":
-                _b.build_kernels(verbose=False)
-            else:
+            if name == "libllb_runtime.so":
                 _b.build_runtime(verbose=False)
     if not path.exists():
         raise NativeError(f"{path} is missing: run `python -m lightllm_b200.build`")
@@ -49,6 +50,45 @@ def _load(name: str):
 
 def debug_bounds_enabled() -> bool:
     return os.environ.get("LLB_DEBUG_BOUNDS", "0") == "1"
+
+
+class UnitLibraries:
+    """Stands in for libllb_kernels.so: looks an entry point up in the source that exports it and loads that unit's
+    library, compiling it if need be."""
+
+    def __init__(self):
+        from .. import build
+
+        self._build = build
+        self._unit_of = {}
+        self._libs = {}
+        pat = re.compile(r"LLB_EXPORT\s+\w+\s*\*?\s*(llb_\w+)\s*\(")
+        for src in build.CSRC.glob("*.cu"):
+            for name in pat.findall(src.read_text()):
+                self._unit_of[name] = src.stem
+
+    def prepare(self, units):
+        self._build.build_units(units)
+
+    def __getattr__(self, name):
+        if not name.startswith("llb_"):
+            raise AttributeError(name)
+        unit = self._unit_of.get(name)
+        if unit is None:
+            raise AttributeError(f"no kernel source exports {name}")
+        if unit not in self._libs:
+            self._libs[unit] = ctypes.CDLL(str(self._build.build_units([unit])[0]))
+        fn = getattr(self._libs[unit], name)
+        setattr(self, name, fn)
+        return fn
+
+
+def prepare(units=None):
+    """Compiles the named csrc units side by side when there is no built library (None: the whole library)."""
+    if units is None or have_kernels() or debug_bounds_enabled() or os.environ.get("LLB_AUTOBUILD", "1") != "1":
+        kernels()
+    else:
+        kernels().prepare(units)
 
 
 def kernels():
@@ -60,12 +100,14 @@ def kernels():
 
                 _b.build_kernels(verbose=False, debug_bounds=True)
             _kernels = _load("libllb_kernels_dbg.so")
+        elif not have_kernels() and os.environ.get("LLB_AUTOBUILD", "1") == "1":
+            _kernels = UnitLibraries()
         else:
             _kernels = _load("libllb_kernels.so")
     return _kernels
 
 
-_DEBUG_UNITS = ("ops_basic", "attention", "attention_tc", "mla", "moe")
+_DEBUG_UNITS = ("ops_basic", "attention", "attention_tc", "latent_attn", "mla", "moe")
 
 
 def set_debug_bounds(pool_slots: int = 0, req_rows: int = 0, r2t_cols: int = 0, num_experts: int = 0, status=None):

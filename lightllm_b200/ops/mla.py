@@ -17,7 +17,7 @@ import math
 
 import torch
 
-from . import _count
+from . import DTYPE_CODES, _count, gemm_f32
 from ._native import c_int, check, f32, i64, kernels, ptr, stream
 
 
@@ -74,6 +74,8 @@ def gemm_batched(a, w, out=None):
     N = w.shape[1]
     if not a.is_cuda:
         return torch.einsum("thk,hnk->thn", a.float(), w.float()).to(a.dtype)
+    if a.dtype == torch.float32:
+        return gemm_f32(a, w, out=out)
     from . import gemm_status
 
     assert a.stride(2) == 1 and w.is_contiguous()
@@ -82,5 +84,131 @@ def gemm_batched(a, w, out=None):
     check(kernels().llb_gemm_bf16_batched(ptr(a), i64(a.stride(0)), i64(a.stride(1)), ptr(w), ptr(out),
                                           i64(out.stride(0)), i64(out.stride(1)), c_int(T), c_int(N), c_int(K),
                                           c_int(h), ptr(gemm_status(a.device)), stream()), "gemm_batched")
+    _count()
+    return out
+
+
+# ---------------------------------------------------------------------------------------------------------------------
+# Latent attention without a rotary part: any latent size, optional sliding window, bf16 or fp32.  The pool row is the
+# latent itself, zero-padded to the row pitch.  Position i sees j with 0 <= i - j < window (window 0: all earlier ones).
+#   absorbed form   scores and values in the latent space, straight from the pool (decode, short portions)
+#   expanded form   keys and values of every head are formed for the positions a prompt pass can see, then attention
+#                   per head (fewer operations per key for long prompts)
+# ---------------------------------------------------------------------------------------------------------------------
+def latent_norm_scatter_(kv_a, kv_layer, norm_w, slot, rank: int, eps: float):
+    """kv_layer[slot[t]] = RMSNorm(kv_a[t, :rank]) * norm_w (fp32), padding columns zero."""
+    row = kv_layer.shape[-1]
+    if not kv_a.is_cuda:
+        v = kv_a[:, :rank].float()
+        v = v * torch.rsqrt(v.pow(2).mean(-1, keepdim=True) + eps) * norm_w
+        flat = kv_layer.view(-1, row)
+        flat[slot.long()] = torch.nn.functional.pad(v, (0, row - rank)).to(kv_layer.dtype)
+        return
+    assert kv_a.stride(1) == 1 and kv_a.dtype == kv_layer.dtype and kv_layer.is_contiguous()
+    assert norm_w.dtype == torch.float32 and slot.dtype == torch.int32
+    check(kernels().llb_latent_norm_scatter(ptr(kv_a), c_int(DTYPE_CODES[kv_a.dtype]), i64(kv_a.stride(0)), ptr(kv_layer),
+                                            c_int(row), ptr(norm_w), ptr(slot), c_int(kv_a.shape[0]), c_int(rank),
+                                            f32(eps), stream()), "latent_norm_scatter")
+    _count()
+
+
+def ref_latent_attention(q_lat, kv_layer, req_to_token, b_req_idx, pos, batch_of, scale, window: int = 0):
+    T, H, rank = q_lat.shape
+    flat = kv_layer.view(-1, kv_layer.shape[-1])
+    out = torch.empty_like(q_lat)
+    for t in range(T):
+        b = int(batch_of[t]) if batch_of is not None else t
+        p = int(pos[t])
+        j0 = max(0, p - window + 1) if window else 0
+        c = flat[req_to_token[int(b_req_idx[b]), j0:p + 1].long(), :rank].float()
+        w = torch.softmax(q_lat[t].float() @ c.t() * scale, dim=-1)
+        out[t] = (w @ c).to(out.dtype)
+    return out
+
+
+def latent_num_splits(T: int, H: int, max_keys: int, sms: int = 148) -> int:
+    """Shares the keys of a query are cut into so that the grid fills the GPU: modelled as waves x tiles per CTA plus
+    the cost of merging."""
+    tiles = max(1, -(-max_keys // 64))
+    ctas = T * -(-H // 16)
+    best, best_cost = 1, None
+    for s in range(1, min(tiles, 64) + 1):
+        cost = -(-ctas * s // sms) * (-(-tiles // s) + 2.0) + (0.0 if s == 1 else 2.0 + 0.02 * s)
+        if best_cost is None or cost < best_cost:
+            best, best_cost = s, cost
+    return best
+
+
+def latent_attention(q_lat, kv_layer, req_to_token, b_req_idx, pos, batch_of, scale, window: int = 0, max_keys: int = 0,
+                     num_splits: int = 0, generic: bool = False):
+    """Absorbed form.  q_lat [T, H, rank] (padding columns zero), pos / batch_of: position and request of every query
+    token (batch_of None: token i belongs to request i).  Returns [T, H, rank].
+    `max_keys`: the most keys a query may see.  `generic`: the kernel without tensor cores (always used for fp32 and for
+    a rank above 512)."""
+    if not q_lat.is_cuda:
+        return ref_latent_attention(q_lat, kv_layer, req_to_token, b_req_idx, pos, batch_of, scale, window)
+    T, H, rank = q_lat.shape
+    row = kv_layer.shape[-1]
+    assert q_lat.is_contiguous() and kv_layer.is_contiguous() and q_lat.dtype == kv_layer.dtype
+    assert pos.dtype == torch.int32 and b_req_idx.dtype == torch.int32
+    out = torch.empty_like(q_lat)
+    if generic or q_lat.dtype != torch.bfloat16 or rank > 512 or rank % 8:
+        check(kernels().llb_latent_attn_generic(ptr(q_lat), c_int(DTYPE_CODES[q_lat.dtype]), ptr(kv_layer), c_int(row),
+                                                ptr(req_to_token), i64(req_to_token.stride(0)), ptr(b_req_idx), ptr(pos),
+                                                ptr(batch_of), ptr(out), c_int(T), c_int(H), c_int(rank), f32(scale),
+                                                c_int(window), stream()), "latent_attn_generic")
+        _count()
+        return out
+    splits = num_splits or latent_num_splits(T, H, max_keys or 64)
+    po = pl = None
+    if splits > 1:
+        n = splits * T * H
+        po = torch.empty(n * rank, dtype=torch.float32, device=q_lat.device)
+        pl = torch.empty(n * 2, dtype=torch.float32, device=q_lat.device)
+    check(kernels().llb_latent_attn_mma(ptr(q_lat), ptr(kv_layer), c_int(row), ptr(req_to_token),
+                                        i64(req_to_token.stride(0)), ptr(b_req_idx), ptr(pos), ptr(batch_of), ptr(out),
+                                        ptr(po), ptr(pl), c_int(T), c_int(H), c_int(rank), c_int(splits), f32(scale),
+                                        c_int(window), stream()), "latent_attn_mma")
+    _count(2 if splits > 1 else 1)
+    return out
+
+
+class KeyRange:
+    """The cached positions a prompt pass can see through a window: request b contributes positions kv_start[b] ..
+    (last new position), laid out back to back from row cu_kv[b] on."""
+
+    def __init__(self, ready, q_len, window: int, device):
+        ready, q_len = ready.to(torch.int64).cpu(), q_len.to(torch.int64).cpu()
+        start = (ready - (window - 1)).clamp_min(0) if window else torch.zeros_like(ready)
+        n = ready + q_len - start
+        cu = torch.zeros(len(n) + 1, dtype=torch.int32)
+        cu[1:] = torch.cumsum(n, 0)
+        self.window, self.rows = window, int(cu[-1])
+        self.kv_start = start.to(torch.int32).to(device, non_blocking=True)
+        self.cu_kv = cu.to(device, non_blocking=True)
+
+
+def latent_gather(kv_layer, req_to_token, b_req_idx, kr: KeyRange):
+    """[rows, row pitch]: the latents of the range, in order."""
+    row = kv_layer.shape[-1]
+    out = torch.empty((kr.rows, row), dtype=kv_layer.dtype, device=kv_layer.device)
+    check(kernels().llb_latent_gather(ptr(kv_layer), c_int(row * kv_layer.element_size()), ptr(req_to_token),
+                                      i64(req_to_token.stride(0)), ptr(b_req_idx), ptr(kr.cu_kv), ptr(kr.kv_start),
+                                      ptr(out), c_int(b_req_idx.shape[0]), c_int(kr.rows), stream()), "latent_gather")
+    _count()
+    return out
+
+
+def window_prefill(q, kv, H: int, dk: int, dv: int, cu_q, b_ready_len, kr: KeyRange, max_q_len: int, scale):
+    """Expanded form on the tcgen05 tensor cores: q [T, >= H * dk] (row stride free), kv [rows, H * dk | H * dv], head
+    sizes 64 or 128.  Returns [T, H * dv]."""
+    assert q.dtype == torch.bfloat16 and kv.dtype == torch.bfloat16 and q.stride(1) == 1 and kv.is_contiguous()
+    assert kv.shape == (kr.rows, H * (dk + dv)) and cu_q.dtype == torch.int32
+    T, B = q.shape[0], cu_q.shape[0] - 1
+    out = torch.empty((T, H * dv), dtype=q.dtype, device=q.device)
+    check(kernels().llb_window_prefill_tc(ptr(q), i64(q.stride(0)), ptr(kv), i64(kv.stride(0)), c_int(kr.rows), ptr(cu_q),
+                                          ptr(kr.cu_kv), ptr(kr.kv_start), ptr(b_ready_len), ptr(out),
+                                          i64(out.stride(0)), c_int(B), c_int(T), c_int(max_q_len), c_int(H), c_int(dk),
+                                          c_int(dv), f32(scale), c_int(kr.window), stream()), "window_prefill_tc")
     _count()
     return out

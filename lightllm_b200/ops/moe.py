@@ -8,7 +8,7 @@ from typing import Optional
 
 import torch
 
-from . import _count, gemm_status
+from . import DTYPE_CODES, _count, _dyt_args, gemm_f32, gemm_status
 from . import reference as ref
 from ._native import c_int, check, f32, i64, kernels, ptr, stream
 
@@ -165,6 +165,8 @@ def gemm_grouped(a_sorted, w_stacked, mblock_expert, n_per_expert: int, epi: str
     M_pad, K = a_sorted.shape
     E, N = w_stacked.shape[0], w_stacked.shape[1]
     assert N == n_per_expert and w_stacked.is_contiguous()
+    if a_sorted.dtype == torch.float32:
+        return gemm_f32(a_sorted, w_stacked, epi, out=out, mblock_expert=mblock_expert)
     n_out = N // 2 if epi.startswith("gated") else N
     if out is None:
         out = torch.empty((M_pad, n_out), dtype=a_sorted.dtype, device=a_sorted.device)
@@ -174,6 +176,18 @@ def gemm_grouped(a_sorted, w_stacked, mblock_expert, n_per_expert: int, epi: str
                                           stream()), "gemm_grouped")
     _count()
     return out
+
+
+def gather_rows(x, lay: MoeLayout):
+    """The rows of x in expert-sorted order (zero rows for padding)."""
+    T, H = x.shape
+    a = torch.empty((lay.m_pad, H), dtype=x.dtype, device=x.device)
+    halves = x.element_size() // 2          # the kernel counts 2-byte elements
+    check(kernels().llb_moe_gather(ptr(a), ptr(x), ptr(lay.sorted_pair), ptr(lay.total_rows), c_int(lay.k),
+                                   c_int(H * halves), i64(x.stride(0) * halves), c_int(lay.m_pad), stream()),
+          "moe_gather")
+    _count()
+    return a
 
 
 def fused_experts(x, w13, w2, ids, weights, act="silu", e0: int = 0, out=None, accumulate: bool = False,
@@ -199,10 +213,7 @@ def fused_experts(x, w13, w2, ids, weights, act="silu", e0: int = 0, out=None, a
     I = N13 // 2
     k = ids.shape[1]
     lay = moe_align(ids, E_local, e0)
-    a = torch.empty((lay.m_pad, H), dtype=x.dtype, device=x.device)
-    check(kernels().llb_moe_gather(ptr(a), ptr(x), ptr(lay.sorted_pair), ptr(lay.total_rows), c_int(k), c_int(H),
-                                   i64(x.stride(0)), c_int(lay.m_pad), stream()), "moe_gather")
-    _count()
+    a = gather_rows(x, lay)
     if fp8_w:
         # block-scaled e4m3 experts: quantise the gathered rows per token group, grouped fp8 GEMM with the SwiGLU
         # epilogue, quantise again, grouped fp8 GEMM (reference: lightllm/common/basemodel/layer_weights/
@@ -234,5 +245,82 @@ def fused_experts(x, w13, w2, ids, weights, act="silu", e0: int = 0, out=None, a
         accumulate = False
     check(kernels().llb_moe_combine(ptr(out), ptr(y), ptr(lay.pair_row), ptr(weights), c_int(T), c_int(k), c_int(H),
                                     c_int(1 if accumulate else 0), stream()), "moe_combine")
+    _count()
+    return out
+
+
+# ---------------------------------------------------------------- table routing
+class TableRouting:
+    """Experts chosen by token id: layer l sends token id t to the experts `table_l[t]` (int32 [vocab, k_l]), each
+    with the same weight.  Nothing of it depends on activations, so `layouts` sorts the tokens of a pass for all
+    layers in one launch, ahead of the first layer.
+
+    layers: (table, first local expert, number of local experts) per MoE layer; ids outside the local range belong
+    to another rank (expert parallel) and are dropped."""
+
+    def __init__(self, layers):
+        self.layers = layers
+        self.vocab = layers[0][0].shape[0]
+        dev = layers[0][0].device
+        for t, _, _ in layers:
+            assert t.dtype == torch.int32 and t.is_contiguous() and t.shape[0] == self.vocab
+        if dev.type == "cuda":
+            rows = [[t.data_ptr(), t.shape[1] | (e0 << 32), n] for t, e0, n in layers]
+            self._routes = torch.tensor(rows, dtype=torch.int64).to(dev)
+
+    def ids(self, layer: int, token_ids):
+        return self.layers[layer][0][token_ids]
+
+    def layouts(self, token_ids):
+        """One MoeLayout per layer (CPU tensors: the expert ids [T, k])."""
+        if not token_ids.is_cuda:
+            return [self.ids(i, token_ids) for i in range(len(self.layers))]
+        T, L = token_ids.shape[0], len(self.layers)
+        assert token_ids.dtype == torch.int64 and token_ids.is_contiguous()
+        parts = []
+        for t, _, n in self.layers:
+            k = t.shape[1]
+            m = max_padded_rows(T, k, n)
+            parts.append((m, T * k, m // 128, n + 1, 1))
+        stride = (max(sum(p) for p in parts) + 3) // 4 * 4
+        buf = torch.empty((L, stride), dtype=torch.int32, device=token_ids.device)
+        check(kernels().llb_moe_table_align(ptr(self._routes), c_int(L), c_int(max(n for _, _, n in self.layers)),
+                                            ptr(token_ids), i64(self.vocab), c_int(T), ptr(buf), i64(stride), stream()),
+              "moe_table_align")
+        _count()
+        out = []
+        for i, p in enumerate(parts):
+            lay = MoeLayout()
+            lay.m_pad, lay.k = p[0], self.layers[i][0].shape[1]
+            lay.sorted_pair, lay.pair_row, lay.mblock_expert, lay.expert_off, lay.total_rows = \
+                torch.split(buf[i, :sum(p)], p)
+            out.append(lay)
+        return out
+
+
+def uniform_experts_dyt_(h, lay, w13, w2, act, shared, gate_w, x, post, nxt, e0: int = 0):
+    """Experts of equal weight 1 / k plus a shared expert's output `shared` [T, H] (or None) scaled by
+    sigmoid(h . gate_w), inside a sandwich of dynamic-tanh norms: x += post(sum) in place, returns nxt(x).
+    x None: returns the fp32 sum instead (a tensor-parallel reduction follows)."""
+    if not h.is_cuda:
+        k = lay.shape[1]
+        w = torch.full(lay.shape, 1.0 / k)
+        y = ref_fused_experts(h, w13, w2, lay, w, act, e0).float()
+        if shared is not None:
+            g = torch.sigmoid(h.float() @ gate_w) if gate_w is not None else torch.ones(h.shape[0])
+            y = y + g[:, None] * shared.float()
+        if x is None:
+            return y
+        x.add_(ref.dyt(y, post))
+        return ref.dyt(x, nxt).to(h.dtype)
+    T, H = h.shape
+    a = gather_rows(h, lay)
+    g = gemm_grouped(a, w13, lay.mblock_expert, w13.shape[1], epi="gated_" + act)
+    y = gemm_grouped(g, w2, lay.mblock_expert, H)
+    out = torch.empty((T, H), dtype=torch.float32 if x is None else h.dtype, device=h.device)
+    check(kernels().llb_moe_combine_dyt(ptr(y), c_int(DTYPE_CODES[h.dtype]), ptr(lay.pair_row), c_int(lay.k),
+                                        f32(1.0 / lay.k), ptr(shared), ptr(h), ptr(gate_w), ptr(x),
+                                        ptr(None if x is None else out), ptr(out if x is None else None), c_int(T),
+                                        c_int(H), *_dyt_args(post), *_dyt_args(nxt), stream()), "moe_combine_dyt")
     _count()
     return out

@@ -56,7 +56,12 @@ def gated_act_interleaved(y, act="silu", block=GATE_UP_BLOCK):
     return (_act(v[:, :, 0, :], act) * v[:, :, 1, :]).reshape(T, N // 2).to(y.dtype)
 
 
-def gemm(a, w, epi="store", residual=None, bias=None, out_dtype=None):
+def dyt(x, norm):
+    """Dynamic tanh of an fp32 tensor (`ops.DytNorm`)."""
+    return torch.tanh(norm.alpha * x) * norm.w + norm.b
+
+
+def gemm(a, w, epi="store", residual=None, bias=None, out_dtype=None, out_scale=1.0, x=None, dyt=None):
     """C = A . W^T with the epilogues of the tcgen05 GEMM. `w` is [N, K]."""
     acc = a.float() @ w.float().t()
     if bias is not None:
@@ -66,7 +71,13 @@ def gemm(a, w, epi="store", residual=None, bias=None, out_dtype=None):
     if epi == "residual":
         return (acc + residual.float()).to(out_dtype or a.dtype)
     if epi == "f32":
-        return acc
+        return acc * out_scale if out_scale != 1.0 else acc
+    if epi == "relu2":
+        return torch.relu(acc).square().to(out_dtype or a.dtype)
+    if epi == "dyt":
+        post, nxt = dyt
+        x.add_(torch.tanh(post.alpha * acc) * post.w + post.b)
+        return (torch.tanh(nxt.alpha * x) * nxt.w + nxt.b).to(out_dtype or a.dtype)
     if epi in ("gated_silu", "gated_gelu"):
         return gated_act_interleaved(acc, "silu" if epi == "gated_silu" else "gelu").to(out_dtype or a.dtype)
     raise ValueError(epi)

@@ -11,6 +11,10 @@ from typing import List, Optional
 def get_config_json(model_dir: str) -> dict:
     with open(os.path.join(model_dir, "config.json")) as f:
         cfg = json.load(f)
+    if "architecture" in cfg and not cfg.get("model_type"):   # not in HF spelling
+        from ..models.registry import native_config
+
+        cfg = native_config(cfg)
     return cfg
 
 
