@@ -46,18 +46,6 @@ __device__ __forceinline__ uint32_t tile_off(int r, int ch) {
   return (uint32_t)((ch >> 3) * BLOCK_BYTES + r * 128 + (((ch & 7) ^ (r & 7)) << 4));
 }
 
-// shared-memory descriptor for an MN-major operand block (rows = K index, 128 bytes of MN elements per row,
-// 128-byte swizzle): groups of 8 rows are 1024 bytes apart.  Both offset fields carry that stride: the MN extent
-// of one instruction (64 elements) fits the swizzle width, so no second stride is ever applied.
-__device__ __forceinline__ uint64_t umma_smem_desc_sw128_mn(uint32_t smem_addr) {
-  uint64_t d = (uint64_t)((smem_addr >> 4) & 0x3FFF);
-  d |= (uint64_t)(1024 >> 4) << 16;
-  d |= (uint64_t)(1024 >> 4) << 32;
-  d |= (uint64_t)1 << 46;
-  d |= (uint64_t)2 << 61;
-  return d;
-}
-
 __device__ __forceinline__ float ex2_fast(float x) {  // 2^x, one MUFU instruction (x = -inf gives 0)
   float y;
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));

@@ -140,6 +140,17 @@ __device__ __forceinline__ uint64_t umma_smem_desc_sw128(uint32_t smem_addr) {
   d |= (uint64_t)2 << 61;            // SWIZZLE_128B
   return d;
 }
+// Shared-memory descriptor for an MN-major operand block (rows = K index, 128 bytes of MN elements per row,
+// 128-byte swizzle): groups of 8 rows are 1024 bytes apart.  Both offset fields carry that stride: the MN extent
+// of one instruction (64 elements) fits the swizzle width, so no second stride is ever applied.
+__device__ __forceinline__ uint64_t umma_smem_desc_sw128_mn(uint32_t smem_addr) {
+  uint64_t d = (uint64_t)((smem_addr >> 4) & 0x3FFF);
+  d |= (uint64_t)(1024 >> 4) << 16;
+  d |= (uint64_t)(1024 >> 4) << 32;
+  d |= (uint64_t)1 << 46;
+  d |= (uint64_t)2 << 61;
+  return d;
+}
 // Instruction descriptor: D fp32, A/B of `fmt` (kind::f16: 0 = fp16, 1 = bf16; kind::f8f6f4: 0 = e4m3, 1 = e5m2),
 // both operands K-major, dense.
 __host__ __device__ constexpr uint32_t umma_idesc(int M, int N, int fmt) {
