@@ -89,6 +89,7 @@ class LayerSpec:
 class TaduzenLM(TransformerLM):
     model_type = "taduzen"
     supports_float32 = True
+    stream_tap = None          # fn(layer, stream): sees the residual stream after every layer (tests)
     native_units = ("dyt", "gemm_f32", "gemm_tcgen05", "latent_attn", "moe", "ops_basic", "sampling",
                     "window_prefill_tc")
 
@@ -295,7 +296,7 @@ class TaduzenLM(TransformerLM):
     def _layers_forward(self, x, st: InferState):
         """x: the fp32 residual stream.  Returns the final norm's output."""
         h = st.extra.pop("first_normed")
-        tap = st.extra.get("stream_tap")
+        tap = self.stream_tap
         n = len(self.layers)
         for i, lw in enumerate(self.layers):
             after = self.layers[i + 1].norm1 if i + 1 < n else self.final_norm
