@@ -96,6 +96,11 @@ def parse():
     ap.add_argument("--rate", type=float, default=8.0, help="config 3: Poisson arrival rate, requests per second")
     ap.add_argument("--in-range", default="128,4096", help="config 3: uniform prompt length range")
     ap.add_argument("--out-range", default="64,1024", help="config 3: uniform output length range")
+    ap.add_argument("--design", default=None, choices=["taduzen"],
+                    help="instead of the serving workload: prefill and decode passes of this model design beside the "
+                         "closest other model at equal sizes")
+    ap.add_argument("--design-size", default=None, choices=["small", "base", "wide"], help="one size only (default: all)")
+    ap.add_argument("--design-kernels", action="store_true", help="also time the kernels of both models")
     ap.add_argument("--layers", type=int, default=None,
                     help="development aid: build only this many layers (the result line says so and is not a "
                          "measurement of the named configuration)")
@@ -364,6 +369,10 @@ def serving_config(args, world):
 
 def main():
     args = parse()
+    if args.design:
+        from lightllm_b200.benchmark import design_bench
+
+        return design_bench.run(args)
     if args.impl == "reference":
         reference_arm(args)
         return

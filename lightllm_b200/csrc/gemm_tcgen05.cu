@@ -2345,10 +2345,17 @@ LLB_EXPORT int llb_gemm_bf16_batched(const void* A, int64_t a_row_stride, int64_
   int bn = N >= 256 && N % 256 == 0 ? 256 : (N % 128 == 0 ? 128 : 64);
   if ((int64_t)cdiv(M, BM) * cdiv(N, bn) * batch < sm_count() && bn > 64) bn = bn / 2;
   CUtensorMap ta, tb;
-  int rc = make_tmap_3d(&ta, A, 2, (uint64_t)batch, (uint64_t)M, (uint64_t)K, (uint64_t)a_row_stride,
-                        (uint64_t)a_batch_stride, BM, BK);
-  if (rc) return rc;
-  rc = make_tmap_3d(&tb, W, 2, (uint64_t)batch, (uint64_t)N, (uint64_t)K, (uint64_t)K, (uint64_t)N * K, (uint32_t)bn, BK);
+  int rc;
+  if (batch == 1) {  // the kernel reads a single matrix through 2-D maps
+    rc = make_tmap_2d(&ta, A, 2, (uint64_t)M, (uint64_t)K, (uint64_t)a_row_stride, BM, BK);
+    if (rc) return rc;
+    rc = make_tmap_2d(&tb, W, 2, (uint64_t)N, (uint64_t)K, (uint64_t)K, (uint32_t)bn, BK);
+  } else {
+    rc = make_tmap_3d(&ta, A, 2, (uint64_t)batch, (uint64_t)M, (uint64_t)K, (uint64_t)a_row_stride,
+                      (uint64_t)a_batch_stride, BM, BK);
+    if (rc) return rc;
+    rc = make_tmap_3d(&tb, W, 2, (uint64_t)batch, (uint64_t)N, (uint64_t)K, (uint64_t)K, (uint64_t)N * K, (uint32_t)bn, BK);
+  }
   if (rc) return rc;
   GemmParams p;
   memset(&p, 0, sizeof(p));

@@ -30,7 +30,8 @@ def test_mla_rope_kv_scatter(dev):
     assert (pool.float() - pool_ref.float()).abs().max().item() < 5e-2
 
 
-@pytest.mark.parametrize("T,h,N,K", [(5, 16, 512, 128), (300, 16, 512, 128), (64, 128, 128, 512), (257, 4, 128, 512)])
+@pytest.mark.parametrize("T,h,N,K", [(5, 16, 512, 128), (300, 16, 512, 128), (64, 128, 128, 512), (257, 4, 128, 512),
+                                       (1, 1, 80, 192), (200, 1, 512, 128)])
 def test_gemm_batched(dev, T, h, N, K):
     torch.manual_seed(1)
     wide = (torch.randn(T, h, K + 64, device=dev) * 0.5).to(BF)
