@@ -114,8 +114,8 @@ def kernels(size: str, T: int = 8192, B: int = 64, ctx: int = 4096):
     w13, w2 = rnd(E, 2 * ff, W), rnd(E, W, ff)
     tables = torch.rand(VOCAB, E, device=dev).topk(k, -1)[1].to(torch.int32)
     routing = moe.TableRouting([(tables, 0, E)])
+    four = moe.TableRouting([(tables, 0, E)] * 4)
     gate = torch.ones(W, device=dev)
-    rw = rnd(E, W)
     for t in (T, B):
         h, x, sh, res = rnd(t, W), rnd(t, W, dtype=torch.float32), rnd(t, W), rnd(t, W)
         tok = torch.randint(0, VOCAB, (t,), device=dev)
@@ -126,15 +126,13 @@ def kernels(size: str, T: int = 8192, B: int = 64, ctx: int = 4096):
         wts = torch.full((t, k), 1.0 / k, device=dev)
         idl = tables[tok].contiguous()
 
-        def like_route():
-            moe.moe_align(moe.topk_softmax(ops.gemm(h, rw, epi="f32"), k, False)[0], E)
-
         def like_experts():
             out = sh.clone()
             moe.fused_experts(h, w13, w2, idl, wts, out=out, accumulate=True)
             ops.add_rmsnorm_(res, out, nw, 1e-5)
 
-        pair(f"routing + layout, {t} rows", (lambda: routing.layouts(tok), t * k * 8, 0), (like_route, t * (k * 8 + W * 2), 0))
+        pair(f"expert-sorted layouts of 4 layers, {t} rows", (lambda: four.layouts(tok), 4 * t * k * 12, 0),
+             (lambda: [moe.moe_align(idl, E) for _ in range(4)], 4 * t * k * 12, 0))
         pair(f"experts + norms, {t} rows",
              (lambda: moe.uniform_experts_dyt_(h, lay, w13, w2, "silu", sh, gate, x, n1, n1), byt + t * W * 14, fl),
              (like_experts, byt + t * W * 10, fl))

@@ -175,6 +175,18 @@ __device__ __forceinline__ float warp_max(float v) {
   return v;
 }
 
+// tanh in fp32 without a branch, for row passes and epilogues whose result is stored in bf16: the Taylor series
+// x - x^3/3 + 2x^5/15 - 17x^7/315 + 62x^9/2835 for |x| < 1/4 (the next term is below 1e-8 of the value), else
+// 1 - 2 / (1 + e^2x).  Error below 3e-7.
+__device__ __forceinline__ float tanh_fast(float x) {
+  const float e = __expf(2.f * x);
+  const float big = 1.f - __fdividef(2.f, 1.f + e);
+  const float x2 = x * x;
+  const float s = fmaf(x2, fmaf(x2, fmaf(x2, 62.f / 2835.f, -17.f / 315.f), 2.f / 15.f), -1.f / 3.f);
+  const float small = fmaf(x * x2, s, x);
+  return fabsf(x) < 0.25f ? small : big;
+}
+
 // Block-wide sum; `red` is a shared array of >= 33 floats. All threads get the result.
 __device__ __forceinline__ float block_sum(float v, float* red) {
   int lane = threadIdx.x & 31, w = threadIdx.x >> 5, nw = (blockDim.x + 31) >> 5;

@@ -35,12 +35,17 @@ struct Dyt {
   float alpha;
 };
 
+__device__ __forceinline__ float tanh_for(float x, const float*) { return tanhf(x); }
+__device__ __forceinline__ float tanh_for(float x, const bf16*) { return tanh_fast(x); }
+
+// TH: the number format the pass writes
+template <typename TH>
 __device__ __forceinline__ void dyt8(const Dyt& n, int col, const float* in, float* out) {
   float w[8], b[8];
   ld8(n.w + col, w);
   ld8(n.b + col, b);
 #pragma unroll
-  for (int i = 0; i < 8; ++i) out[i] = tanhf(n.alpha * in[i]) * w[i] + b[i];
+  for (int i = 0; i < 8; ++i) out[i] = tanh_for(n.alpha * in[i], (const TH*)nullptr) * w[i] + b[i];
 }
 
 template <typename TE, typename TH>
@@ -54,7 +59,7 @@ __global__ void __launch_bounds__(256) embedding_dyt_kernel(const int64_t* __res
     float v[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f}, o[8];
     if (id >= 0 && id < rows) ld8(table + id * W + c, v);
     st8(x + (int64_t)t * W + c, v);
-    dyt8(n, c, v, o);
+    dyt8<TH>(n, c, v, o);
     st8(h + (int64_t)t * W + c, o);
   }
 }
@@ -65,7 +70,7 @@ __global__ void __launch_bounds__(256) dyt_kernel(const float* __restrict__ x, T
   for (int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; i < n_vec; i += (int64_t)gridDim.x * blockDim.x) {
     float v[8], o[8];
     ld8(x + i * 8, v);
-    dyt8(n, (int)(i % wv) * 8, v, o);
+    dyt8<TH>(n, (int)(i % wv) * 8, v, o);
     st8(h + i * 8, o);
   }
 }
@@ -77,12 +82,12 @@ __global__ void __launch_bounds__(256) add_dyt_kernel(float* __restrict__ x, con
     const int c = (int)(i % wv) * 8;
     float v[8], a[8], o[8];
     ld8(y + i * 8, v);
-    dyt8(post, c, v, a);
+    dyt8<TH>(post, c, v, a);
     ld8(x + i * 8, v);
 #pragma unroll
     for (int e = 0; e < 8; ++e) v[e] += a[e];
     st8(x + i * 8, v);
-    dyt8(next, c, v, o);
+    dyt8<TH>(next, c, v, o);
     st8(h + i * 8, o);
   }
 }
@@ -130,12 +135,12 @@ moe_combine_dyt_kernel(const T* __restrict__ y, const int* __restrict__ pair_row
       continue;
     }
     float a[8], v[8], o[8];
-    dyt8(post, c, acc, a);
+    dyt8<T>(post, c, acc, a);
     ld8(x + row + c, v);
 #pragma unroll
     for (int e = 0; e < 8; ++e) v[e] += a[e];
     st8(x + row + c, v);
-    dyt8(next, c, v, o);
+    dyt8<T>(next, c, v, o);
     st8(h_out + row + c, o);
   }
 }

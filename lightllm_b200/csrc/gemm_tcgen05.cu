@@ -110,14 +110,14 @@ __device__ __forceinline__ float relu2_f(float v) {
 __device__ __forceinline__ void dyt_sandwich4(const DytFuse& d, int col, float4& x, float4& v) {
   const float4 w1 = *reinterpret_cast<const float4*>(d.w1 + col), b1 = *reinterpret_cast<const float4*>(d.b1 + col);
   const float4 w2 = *reinterpret_cast<const float4*>(d.w2 + col), b2 = *reinterpret_cast<const float4*>(d.b2 + col);
-  x.x += tanhf(d.alpha1 * v.x) * w1.x + b1.x;
-  x.y += tanhf(d.alpha1 * v.y) * w1.y + b1.y;
-  x.z += tanhf(d.alpha1 * v.z) * w1.z + b1.z;
-  x.w += tanhf(d.alpha1 * v.w) * w1.w + b1.w;
-  v.x = tanhf(d.alpha2 * x.x) * w2.x + b2.x;
-  v.y = tanhf(d.alpha2 * x.y) * w2.y + b2.y;
-  v.z = tanhf(d.alpha2 * x.z) * w2.z + b2.z;
-  v.w = tanhf(d.alpha2 * x.w) * w2.w + b2.w;
+  x.x += tanh_fast(d.alpha1 * v.x) * w1.x + b1.x;
+  x.y += tanh_fast(d.alpha1 * v.y) * w1.y + b1.y;
+  x.z += tanh_fast(d.alpha1 * v.z) * w1.z + b1.z;
+  x.w += tanh_fast(d.alpha1 * v.w) * w1.w + b1.w;
+  v.x = tanh_fast(d.alpha2 * x.x) * w2.x + b2.x;
+  v.y = tanh_fast(d.alpha2 * x.y) * w2.y + b2.y;
+  v.z = tanh_fast(d.alpha2 * x.z) * w2.z + b2.z;
+  v.w = tanh_fast(d.alpha2 * x.w) * w2.w + b2.w;
 }
 __device__ __forceinline__ uint2 pack4(const float4& v) {
   return make_uint2(pack_bf16x2(v.x, v.y), pack_bf16x2(v.z, v.w));
@@ -348,20 +348,30 @@ __device__ __forceinline__ void epilogue_store(const GemmParams& p, uint32_t t_r
       }
     }
   } else if (EPI == EPI_DYT) {
+    // the stream's rows come as whole lines, one step of 32 columns ahead of their use, and go through the staging block
+    float4 nx[8];
+    auto fetch_x = [&](int col0) {
+#pragma unroll
+      for (int i = 0; i < 8; ++i) {
+        const int id = i * 32 + lane, r = id >> 3, seg = id & 7;
+        nx[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (row_base + r < p.M && col0 + 32 <= p.N)
+          nx[i] = *reinterpret_cast<const float4*>(p.dyt.x + (int64_t)(row_base + r) * p.ldc + col0 + seg * 4);
+      }
+    };
+    if (stage != nullptr) fetch_x(col_tile0);
 #pragma unroll 1
     for (int c = 0; c < BN; c += 32) {
       const int col0 = col_tile0 + c;
       if (col0 >= p.N) break;
       const bool staged = stage != nullptr && col0 + 32 <= p.N;
-      if (staged) {  // the stream's rows: whole lines into the staging block, and back below
+      if (staged) {
 #pragma unroll
         for (int i = 0; i < 8; ++i) {
-          const int id = i * 32 + lane, r = id >> 3, seg = id & 7;
-          float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-          if (row_base + r < p.M)
-            v = *reinterpret_cast<const float4*>(p.dyt.x + (int64_t)(row_base + r) * p.ldc + col0 + seg * 4);
-          *reinterpret_cast<float4*>(stage + r * EPI_ROW_PITCH + seg * 16) = v;
+          const int id = i * 32 + lane;
+          *reinterpret_cast<float4*>(stage + (id >> 3) * EPI_ROW_PITCH + (id & 7) * 16) = nx[i];
         }
+        if (c + 32 < BN) fetch_x(col0 + 32);
         __syncwarp();
       }
       uint32_t r[32];

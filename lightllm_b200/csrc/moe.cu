@@ -200,9 +200,18 @@ __device__ __forceinline__ void align_pairs(IdOf id_of, int n_pairs, int e0, int
   int* cur = sm + 2 * E_local + 1;  // [E_local]
   for (int i = threadIdx.x; i < E_local; i += blockDim.x) cnt[i] = 0;
   __syncthreads();
-  for (int p = threadIdx.x; p < n_pairs; p += blockDim.x) {
-    const int e = id_of(p) - e0;
-    if (e >= 0 && e < E_local) atomicAdd(&cnt[e], 1);
+  // eight look-ups in flight per thread: they are latency-bound
+  constexpr int U = 8;
+  for (int p0 = threadIdx.x; p0 < n_pairs; p0 += U * blockDim.x) {
+    int e[U];
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int p = p0 + u * blockDim.x;
+      e[u] = p < n_pairs ? id_of(p) - e0 : -1;
+    }
+#pragma unroll
+    for (int u = 0; u < U; ++u)
+      if (e[u] >= 0 && e[u] < E_local) atomicAdd(&cnt[e[u]], 1);
   }
   __syncthreads();
   if (threadIdx.x == 0) {
@@ -234,14 +243,23 @@ __device__ __forceinline__ void align_pairs(IdOf id_of, int n_pairs, int e0, int
     mblock_expert[b] = e;
   }
   __syncthreads();
-  for (int p = threadIdx.x; p < n_pairs; p += blockDim.x) {
-    const int e = id_of(p) - e0;
-    if (e >= 0 && e < E_local) {
-      int r = off[e] + atomicAdd(&cur[e], 1);
-      sorted_pair[r] = p;
+  for (int p0 = threadIdx.x; p0 < n_pairs; p0 += U * blockDim.x) {
+    int e[U];
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int p = p0 + u * blockDim.x;
+      e[u] = p < n_pairs ? id_of(p) - e0 : -1;
+    }
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int p = p0 + u * blockDim.x;
+      if (p >= n_pairs) break;
+      int r = -1;
+      if (e[u] >= 0 && e[u] < E_local) {
+        r = off[e[u]] + atomicAdd(&cur[e[u]], 1);
+        sorted_pair[r] = p;
+      }
       pair_row[p] = r;
-    } else {
-      pair_row[p] = -1;
     }
   }
 }

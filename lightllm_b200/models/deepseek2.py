@@ -218,6 +218,10 @@ class DeepseekV2LM(TransformerLM):
         st.b_ready_cache_len = b_seq_len - 1
         return st
 
+    def _prepare_decode_state(self, st):
+        # inside a decode graph the lengths must come from the replay's own inputs: cached tokens = own position
+        st.b_ready_cache_len = st.seq_pos
+
     def _attention_block(self, i, lw, h, st):
         T = h.shape[0]
         hq, nope, rope, kvl = self.hq, self.nope, self.rope_d, self.kv_lora

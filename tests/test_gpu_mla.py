@@ -160,3 +160,27 @@ def test_deepseek_v32_sparse_attention_gpu_matches_cpu(dev):
     assert d.mean().item() < 0.02 * scale, (d.mean().item(), scale)
     assert d.max().item() < 0.5 * scale, (d.max().item(), scale)
     assert d[:64].max().item() < 0.08 * scale + 0.05     # the first index_topk positions select everything
+
+
+def test_decode_graph_sees_the_whole_context(dev):
+    """Logits of decode steps replayed as CUDA graphs equal those of eager steps, with contexts that grow after capture."""
+    from lightllm_b200.engine.trace import TraceReplayer
+    from lightllm_b200.engine.llm import LLM
+    from lightllm_b200.parallel.dist import ParallelState
+
+    cfg = dict(model_type="deepseek_v2", hidden_size=256, num_hidden_layers=2, vocab_size=512, num_attention_heads=4,
+               num_key_value_heads=4, q_lora_rank=None, kv_lora_rank=512, qk_nope_head_dim=64, qk_rope_head_dim=64,
+               v_head_dim=64, intermediate_size=512, first_k_dense_replace=2, rms_norm_eps=1e-5, rope_theta=1e4)
+    toks = torch.randint(0, 512, (60,), generator=torch.Generator().manual_seed(1)).tolist()
+    outs = []
+    for eager in (False, True):
+        llm = LLM(config=cfg, max_total_token_num=256, running_max_req_size=2, max_req_total_len=128,
+                  disable_dynamic_prompt_cache=True, disable_cudagraph=eager, pstate=ParallelState(device=dev))
+        rep = TraceReplayer(llm)
+        rep.step([("a", toks[:50], [])])
+        outs.append(torch.cat([torch.from_numpy(rep.step([("a", [t], [0])])) for t in toks[50:]]))
+    assert (outs[0] - outs[1]).abs().max() < 1e-3 * outs[1].abs().max()
+    llm = LLM(config=cfg, max_total_token_num=256, running_max_req_size=2, max_req_total_len=128,
+              disable_dynamic_prompt_cache=True, pstate=ParallelState(device=dev))
+    whole = torch.from_numpy(TraceReplayer(llm).step([("a", toks, list(range(50, 60)))]))
+    assert (outs[0] - whole).norm() < 3e-2 * whole.norm()
