@@ -703,6 +703,10 @@ class TransformerLM:
         h = self._layers_forward(h, st)
         return self._lm_head(h, normed=True) if st.extra.get("normed") else self._lm_head(h)
 
+    def _graph_decode_splits(self, bucket: int) -> int:
+        """Shares the decode attention of a captured step cuts every context into."""
+        return ops.gqa_decode_num_splits(bucket, self.hq, max(self.hkv, 1), self.graph_max_len_in_batch)
+
     def _capture_decode_graph(self, bucket: int) -> dict:
         dev = self.device
         # the launch shapes of the expert-parallel exchange are frozen into the graph: use the decode bound, also
@@ -713,7 +717,7 @@ class TransformerLM:
             "b_seq_len": torch.ones(bucket, dtype=torch.int32, device=dev),
             "mem_index": torch.full((bucket,), self.mem_manager.HOLD_TOKEN_MEMINDEX, dtype=torch.int32, device=dev),
         }
-        splits = ops.gqa_decode_num_splits(bucket, self.hq, max(self.hkv, 1), self.graph_max_len_in_batch)
+        splits = self._graph_decode_splits(bucket)
         st = self._make_decode_state(bucket, g["b_req_idx"], g["b_seq_len"], g["mem_index"],
                                      self.graph_max_len_in_batch, num_splits=splits)
         if splits > 1:

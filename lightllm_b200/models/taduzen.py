@@ -286,6 +286,9 @@ class TaduzenLM(TransformerLM):
         return InferState(is_prefill=False, batch_size=B, num_tokens=B, max_kv_len=max_kv_len, max_q_len=1,
                           b_req_idx=b_req_idx, b_seq_len=b_seq_len, mem_index=mem_index)
 
+    def _graph_decode_splits(self, bucket):
+        return 1        # per layer, from its window (ops.mla.latent_attention)
+
     def _embed(self, ids, st):
         x, st.extra["first_normed"] = ops.embedding_dyt(ids, self.embed_w, self.layers[0].norm1)
         if self.routing is not None:

@@ -63,12 +63,24 @@ class UnitLibraries:
         self._unit_of = {}
         self._libs = {}
         pat = re.compile(r"LLB_EXPORT\s+\w+\s*\*?\s*(llb_\w+)\s*\(")
-        for src in build.CSRC.glob("*.cu"):
-            for name in pat.findall(src.read_text()):
-                self._unit_of[name] = src.stem
+        text = {src.stem: src.read_text() for src in build.CSRC.glob("*.cu")}
+        for unit, body in text.items():
+            for name in pat.findall(body):
+                self._unit_of[name] = unit
+        # units whose entry points another unit calls
+        code = {u: re.sub(r"//[^\n]*", "", b) for u, b in text.items()}
+        self._needs = {u: sorted({self._unit_of[n] for n in re.findall(r"\b(llb_\w+)\s*\(", b)
+                                  if self._unit_of.get(n, u) != u}) for u, b in code.items()}
 
     def prepare(self, units):
         self._build.build_units(units)
+
+    def _load_unit(self, unit):
+        if unit not in self._libs:
+            for other in self._needs[unit]:
+                self._load_unit(other)
+            self._libs[unit] = ctypes.CDLL(str(self._build.build_units([unit])[0]), mode=ctypes.RTLD_GLOBAL)
+        return self._libs[unit]
 
     def __getattr__(self, name):
         if not name.startswith("llb_"):
@@ -76,9 +88,7 @@ class UnitLibraries:
         unit = self._unit_of.get(name)
         if unit is None:
             raise AttributeError(f"no kernel source exports {name}")
-        if unit not in self._libs:
-            self._libs[unit] = ctypes.CDLL(str(self._build.build_units([unit])[0]))
-        fn = getattr(self._libs[unit], name)
+        fn = getattr(self._load_unit(unit), name)
         setattr(self, name, fn)
         return fn
 

@@ -466,5 +466,7 @@ def test_every_kernel_entry_has_a_source():
         with open(os.path.join(ROOT, "lightllm_b200", "ops", name + ".py")) as f:
             called |= set(re.findall(r"kernels\(\)\.(llb_\w+)", f.read()))
     assert called <= set(units)
+    assert UnitLibraries()._needs["attention"] == ["attention_tc"]
+    assert not any(UnitLibraries()._needs[u] for u in TaduzenLM.native_units)
     assert {units[n] for n in ("llb_dyt", "llb_gemm_f32", "llb_gemm_bf16_fused", "llb_latent_attn_mma", "llb_moe_table_align",
                                "llb_window_prefill_tc", "llb_decode_prologue", "llb_sample")} <= set(TaduzenLM.native_units)
