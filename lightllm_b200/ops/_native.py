@@ -62,7 +62,7 @@ class UnitLibraries:
         self._build = build
         self._unit_of = {}
         self._libs = {}
-        pat = re.compile(r"LLB_EXPORT\s+\w+\s*\*?\s*(llb_\w+)\s*\(")
+        pat = re.compile(r"LLB_EXPORT\s+\w+\s*\*?\s*(llb_\w+)\s*\([^;{]*\)\s*\{")   # definitions only
         text = {src.stem: src.read_text() for src in build.CSRC.glob("*.cu")}
         for unit, body in text.items():
             for name in pat.findall(body):
