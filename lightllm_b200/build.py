@@ -97,9 +97,9 @@ def build_kernels(force: bool = False, verbose: bool = True, debug_bounds: bool 
     return out
 
 
-def build_units(units, verbose: bool = False) -> list:
-    """One library per named csrc unit (`libllb_unit_<name>.so`), compiled side by side: what a program without the
-    whole library needs on first use.  Writers in several processes are kept apart by a lock file."""
+def build_units(units, needs: dict, verbose: bool = False) -> list:
+    """One library per named csrc unit (`libllb_unit_<name>.so`, with the units it `needs`), compiled side by side: what
+    a program without the whole library needs on first use.  A lock file keeps several processes apart."""
     import fcntl
 
     OBJ.mkdir(parents=True, exist_ok=True)
@@ -107,11 +107,11 @@ def build_units(units, verbose: bool = False) -> list:
 
     def one(unit):
         out = LIB / f"libllb_unit_{unit}.so"
-        obj = _compile_cu(CSRC / f"{unit}.cu", headers, force=False)
+        objs = [_compile_cu(CSRC / f"{u}.cu", headers, force=False) for u in (unit, *needs.get(unit, ()))]
         stamp = OBJ / f"unit.{unit}.sha"
-        dig = _digest([obj])
+        dig = _digest(objs)
         if not out.exists() or not stamp.exists() or stamp.read_text() != dig:
-            r = subprocess.run([_nvcc(), "-shared", "-o", str(out), str(obj), "-Xcompiler", "-fPIC"],
+            r = subprocess.run([_nvcc(), "-shared", "-o", str(out), *map(str, objs), "-Xcompiler", "-fPIC"],
                                capture_output=True, text=True)
             if r.returncode != 0:
                 raise RuntimeError(f"link failed:\n{r.stderr[-4000:]}")

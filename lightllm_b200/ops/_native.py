@@ -67,19 +67,17 @@ class UnitLibraries:
         for unit, body in text.items():
             for name in pat.findall(body):
                 self._unit_of[name] = unit
-        # units whose entry points another unit calls
+        # units whose entry points a unit calls: linked into its library
         code = {u: re.sub(r"//[^\n]*", "", b) for u, b in text.items()}
         self._needs = {u: sorted({self._unit_of[n] for n in re.findall(r"\b(llb_\w+)\s*\(", b)
                                   if self._unit_of.get(n, u) != u}) for u, b in code.items()}
 
     def prepare(self, units):
-        self._build.build_units(units)
+        self._build.build_units(units, self._needs)
 
     def _load_unit(self, unit):
         if unit not in self._libs:
-            for other in self._needs[unit]:
-                self._load_unit(other)
-            self._libs[unit] = ctypes.CDLL(str(self._build.build_units([unit])[0]), mode=ctypes.RTLD_GLOBAL)
+            self._libs[unit] = ctypes.CDLL(str(self._build.build_units([unit], self._needs)[0]))
         return self._libs[unit]
 
     def __getattr__(self, name):
