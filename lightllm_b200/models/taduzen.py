@@ -54,7 +54,8 @@ def normalize_taduzen(cfg: dict) -> dict:
     layers = cfg["layers"]
     moe = [l["mlp"]["router"] for l in layers if l.get("mlp") and l["mlp"]["kind"] == "moe"]
     out = dict(cfg, model_type="taduzen", hidden_size=cfg["width"], vocab_size=cfg["vocab"],
-               num_hidden_layers=len(layers), num_attention_heads=max(l["mixer"]["heads"] for l in layers))
+               num_hidden_layers=len(layers), num_attention_heads=max(l["mixer"]["heads"] for l in layers),
+               kv_lora_rank=max(_up(l["mixer"]["kv_rank"], 16) for l in layers), qk_rope_head_dim=0)
     if moe:
         out.update(num_experts=max(r["experts"] for r in moe), num_experts_per_tok=max(r["top"] for r in moe),
                    decoder_sparse_step=1, mlp_only_layers=[i for i, l in enumerate(layers)

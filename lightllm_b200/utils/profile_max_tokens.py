@@ -17,6 +17,8 @@ import os
 import struct
 from typing import Dict, Tuple
 
+from .config_utils import get_config_json
+
 ELEM = {"F64": 8, "F32": 4, "F16": 2, "BF16": 2, "I64": 8, "I32": 4, "I16": 2, "I8": 1, "U8": 1, "BOOL": 1,
         "F8_E4M3": 1, "F8_E5M2": 1}
 DTYPE_BYTES = {"bf16": 2, "bfloat16": 2, "fp16": 2, "float16": 2, "fp32": 4, "float32": 4}
@@ -71,8 +73,7 @@ def kv_bytes_per_token(cfg: dict, tp: int, kv_elem_bytes: int = 2) -> int:
 
 def max_total_tokens(model_dir: str, tp: int = 1, mem_fraction: float = 0.9, gpu_gib: float = None,
                      data_type: str = None, kv_elem_bytes: int = 2) -> dict:
-    with open(os.path.join(model_dir, "config.json")) as f:
-        cfg = json.load(f)
+    cfg = get_config_json(model_dir)
     if gpu_gib is None:
         import torch
 

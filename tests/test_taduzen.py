@@ -470,3 +470,11 @@ def test_every_kernel_entry_has_a_source():
     assert not any(UnitLibraries()._needs[u] for u in TaduzenLM.native_units)
     assert {units[n] for n in ("llb_dyt", "llb_gemm_f32", "llb_gemm_bf16_fused", "llb_latent_attn_mma", "llb_moe_table_align",
                                "llb_window_prefill_tc", "llb_decode_prologue", "llb_sample")} <= set(TaduzenLM.native_units)
+
+
+def test_capacity_estimate(tmp_path):
+    from lightllm_b200.utils.profile_max_tokens import kv_bytes_per_token, max_total_tokens
+
+    path = write(tmp_path, MIXED, weights(MIXED))
+    assert kv_bytes_per_token(load_config(path), 1) == 5 * 112 * 2      # five layers, the widest latent padded to 112
+    assert max_total_tokens(path, gpu_gib=1)["max_total_token_num"] > 0
