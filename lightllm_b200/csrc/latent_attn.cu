@@ -166,7 +166,7 @@ constexpr int S_PITCH = KT + 8;  // floats per score row in shared memory
 
 template <int LAT>
 constexpr int mma_smem() {
-  return STAGES * KT * LAT * 2 + 16 * S_PITCH * 4 + 2 * KT * 4;
+  return STAGES * KT * LAT * 2 + 2 * 16 * S_PITCH * 4 + 2 * KT * 4;
 }
 
 // byte offset of 16-byte chunk `ch` of key `row` inside a tile
@@ -190,7 +190,7 @@ latent_attn_mma_kernel(const bf16* __restrict__ q_lat, const bf16* __restrict__ 
   constexpr int N2 = LAT / 128;          // pairs of 8-column output blocks per warp
   const uint32_t kv_base = smem_u32(smem);
   float* s_sm = reinterpret_cast<float*>(smem + STAGES * KT * LAT * 2);
-  int* slot_sm = reinterpret_cast<int*>(s_sm + 16 * S_PITCH);
+  int* slot_sm = reinterpret_cast<int*>(s_sm + 2 * 16 * S_PITCH);
 
   const int t = blockIdx.x, head0 = blockIdx.y * 16;
   const int split = blockIdx.z, splits = gridDim.z;
@@ -247,25 +247,10 @@ latent_attn_mma_kernel(const bf16* __restrict__ q_lat, const bf16* __restrict__ 
       qf[ks][3] = ok1 && d + 8 < rank ? *reinterpret_cast<const uint32_t*>(q1 + d + 8) : 0u;
     }
   }
-  __syncthreads();
-  issue(0);
-  issue(1);
-  __syncthreads();  // both slot buffers read
-  if (threadIdx.x < KT) slot_sm[threadIdx.x] = fetch_slot(2);
-
-  float o[2 * N2][4];
-#pragma unroll
-  for (int i = 0; i < 2 * N2; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
-  float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
-
-  for (int i = 0; i < n_tiles; ++i) {
-    cp_async_wait<1>();  // tile i landed (its group is the second youngest)
-    __syncthreads();     // ... for all threads; every warp is done with tile i - 1; slots of tile i + 2 are visible
-    issue(i + 2);
-    const int next_slot = threadIdx.x < KT ? fetch_slot(i + 3) : 0;
+  // scores of this warp's 8 keys of tile i over the whole latent, scaled and masked: columns (warp * 8 + tig * 2, + 1) of
+  // rows g and g + 8
+  auto scores = [&](int i, float* s) {
     const uint32_t kb = kv_base + (uint32_t)(i % STAGES) * (KT * LAT * 2);
-
-    // ---- scores of this warp's 8 keys over the whole latent ----
     float sc[4][4];
 #pragma unroll
     for (int a = 0; a < 4; ++a) sc[a][0] = sc[a][1] = sc[a][2] = sc[a][3] = 0.f;
@@ -277,28 +262,54 @@ latent_attn_mma_kernel(const bf16* __restrict__ q_lat, const bf16* __restrict__ 
       mma_bf16_16816(sc[(2 * k2 + 1) & 3], qf[2 * k2 + 1][0], qf[2 * k2 + 1][1], qf[2 * k2 + 1][2], qf[2 * k2 + 1][3],
                      b2, b3);
     }
-    {
-      const int col = warp * 8 + tig * 2;
-      const int kp = key0 + i * KT + col;
-      const bool v0 = kp < k_end, v1 = kp + 1 < k_end;
-      float s[4];
+    const int kp = key0 + i * KT + warp * 8 + tig * 2;
 #pragma unroll
-      for (int e = 0; e < 4; ++e) s[e] = ((sc[0][e] + sc[1][e]) + (sc[2][e] + sc[3][e])) * scale_log2;
-      *reinterpret_cast<float2*>(s_sm + g * S_PITCH + col) =
-          make_float2(v0 ? s[0] : -INFINITY, v1 ? s[1] : -INFINITY);
-      *reinterpret_cast<float2*>(s_sm + (g + 8) * S_PITCH + col) =
-          make_float2(v0 ? s[2] : -INFINITY, v1 ? s[3] : -INFINITY);
-    }
+    for (int e = 0; e < 4; ++e)
+      s[e] = kp + (e & 1) < k_end ? ((sc[0][e] + sc[1][e]) + (sc[2][e] + sc[3][e])) * scale_log2 : -INFINITY;
+  };
+  auto store_scores = [&](int i, const float* s) {
+    float* dst = s_sm + (i & 1) * 16 * S_PITCH + warp * 8 + tig * 2;
+    *reinterpret_cast<float2*>(dst + g * S_PITCH) = make_float2(s[0], s[1]);
+    *reinterpret_cast<float2*>(dst + (g + 8) * S_PITCH) = make_float2(s[2], s[3]);
+  };
+
+  __syncthreads();
+  issue(0);
+  issue(1);
+  __syncthreads();  // both slot buffers read
+  if (threadIdx.x < KT) slot_sm[threadIdx.x] = fetch_slot(2);
+
+  float o[2 * N2][4];
+#pragma unroll
+  for (int i = 0; i < 2 * N2; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
+  float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
+
+  if (n_tiles > 0) {
+    cp_async_wait<1>();  // tile 0 landed
     __syncthreads();
-    if (threadIdx.x < KT) slot_sm[((i + 1) & 1) * KT + threadIdx.x] = next_slot;
+    float s0[4];
+    scores(0, s0);
+    store_scores(0, s0);
+  }
+  // One barrier per tile: between two of them every warp computes the scores of tile i + 1 and the softmax and P . c of
+  // tile i, which do not depend on each other.
+  for (int i = 0; i < n_tiles; ++i) {
+    cp_async_wait<0>();  // tile i + 1 landed
+    __syncthreads();     // ... for all threads; scores of tile i and slots of tile i + 2 visible; tile i - 1 free
+    issue(i + 2);
+    const int next_slot = threadIdx.x < KT ? fetch_slot(i + 3) : 0;
+    const uint32_t kb = kv_base + (uint32_t)(i % STAGES) * (KT * LAT * 2);
+    const float* s_cur = s_sm + (i & 1) * 16 * S_PITCH;
+    float s_next[4];
+    if (i + 1 < n_tiles) scores(i + 1, s_next);
 
     // ---- softmax bookkeeping, the same in all warps ----
     float s[KT / 8][4];
     float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
     for (int j = 0; j < KT / 8; ++j) {
-      const float2 lo = *reinterpret_cast<const float2*>(s_sm + g * S_PITCH + j * 8 + tig * 2);
-      const float2 hi = *reinterpret_cast<const float2*>(s_sm + (g + 8) * S_PITCH + j * 8 + tig * 2);
+      const float2 lo = *reinterpret_cast<const float2*>(s_cur + g * S_PITCH + j * 8 + tig * 2);
+      const float2 hi = *reinterpret_cast<const float2*>(s_cur + (g + 8) * S_PITCH + j * 8 + tig * 2);
       s[j][0] = lo.x; s[j][1] = lo.y; s[j][2] = hi.x; s[j][3] = hi.y;
       mx[0] = fmaxf(mx[0], fmaxf(lo.x, lo.y));
       mx[1] = fmaxf(mx[1], fmaxf(hi.x, hi.y));
@@ -349,6 +360,8 @@ latent_attn_mma_kernel(const bf16* __restrict__ q_lat, const bf16* __restrict__ 
         mma_bf16_16816(o[2 * n + 1], al[0], al[1], al[2], al[3], b2, b3);
       }
     }
+    if (i + 1 < n_tiles) store_scores(i + 1, s_next);
+    if (threadIdx.x < KT) slot_sm[((i + 1) & 1) * KT + threadIdx.x] = next_slot;
   }
 
 #pragma unroll
