@@ -3,7 +3,8 @@
 // Pool row of a token: the RMS-normalised latent c (`rank` values, zero-padded to the row pitch), one "head" shared by
 // all query heads.  The query of a head is taken into the latent space with the key up-projection (q_lat = q . W_uk),
 // scores are q_lat . c, the value read is the same c, and the value up-projection follows the attention.
-// Position i sees j with 0 <= i - j < window (window 0: no lower bound).  Scores, weights and their sums are fp32.
+// A query sees its own position and the window - 1 positions before it (window 0: all of them).  Scores, weights and
+// their sums are fp32.
 //
 //   latent_norm_scatter    RMSNorm of new latents, written to their pool slots
 //   latent_gather          latents of a range of positions of every request, back to back (for the expanded prefill form)

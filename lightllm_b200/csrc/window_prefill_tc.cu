@@ -3,7 +3,7 @@
 // Key sizes and value sizes are 64 or 128 and may differ; every query head has its own keys and values.
 //
 //   kv [rows, H * DK | H * DV]: request b's keys are rows cu_kv[b] .., position kv_start[b] first
-//   position i sees j with 0 <= i - j < window  (window 0: all j <= i)
+//   a query sees its own position and the window - 1 before it  (window 0: all before it)
 //
 // One CTA computes 128 query rows of one (request, head), as in attention_tc.cu: per 128-key tile S = Q . K^T into one of
 // two tensor-memory buffers, softmax by eight warps (two threads per query row), P . V into a third buffer that the

@@ -1,9 +1,8 @@
 """Taduzen: latent attention without positions through a sliding window, mixture-of-experts layers whose experts are
 looked up by token id, and dynamic-tanh norms before and after every sublayer around an fp32 residual stream.
 
-    x = embed[token]
-    x <- x + norm1b(attention(norm1(x)));  x <- x + norm2b(ffn(norm2(x)))       per layer (the ffn may be absent)
-    logits = head . final_norm(x) * logit_scale
+    stream = embedding row;  per layer: stream += post1(attention(pre1(stream))), stream += post2(ffn(pre2(stream)))
+    (a layer may have no ffn);  logits = logit_scale * head . final(stream)
 
 Every layer has its own sizes (`layers` in config.json).  How it maps onto this package:
 

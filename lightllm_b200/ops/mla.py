@@ -90,7 +90,8 @@ def gemm_batched(a, w, out=None):
 
 # ---------------------------------------------------------------------------------------------------------------------
 # Latent attention without a rotary part: any latent size, optional sliding window, bf16 or fp32.  The pool row is the
-# latent itself, zero-padded to the row pitch.  Position i sees j with 0 <= i - j < window (window 0: all earlier ones).
+# latent itself, zero-padded to the row pitch.  A query sees its own position and the window - 1 before it (window 0:
+# all before it).
 #   absorbed form   scores and values in the latent space, straight from the pool (decode, short portions)
 #   expanded form   keys and values of every head are formed for the positions a prompt pass can see, then attention
 #                   per head (fewer operations per key for long prompts)

@@ -16,7 +16,8 @@ def rms(x, w, eps):
 
 
 def visible(n_query, n_key, first_query, window):
-    """[n_query, n_key] bool: the query at position first_query + i sees key j when 0 <= i' - j < window."""
+    """[n_query, n_key] bool: a query sees its own position and the window - 1 before it; the first query stands at
+    position first_query, the first key at 0."""
     i = torch.arange(first_query, first_query + n_query)[:, None]
     j = torch.arange(n_key)[None, :]
     d = i - j

@@ -4,7 +4,6 @@ tests run on a GPU in fp32 and bf16."""
 import json
 import os
 import subprocess
-import sys
 
 import pytest
 import torch
