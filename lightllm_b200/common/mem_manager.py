@@ -157,6 +157,48 @@ class MemoryManager:
             ops.copy_rows(self.kv_buffer[l], pages[l], idx, None, n)
 
 
+class LayeredKVMemoryManager(MemoryManager):
+    """Pool whose layers have rows of different sizes: layer(i) is [size + 1, rows[i]].  A layer without a cache has no
+    entry.  To the code that moves KV the manager looks like one layer whose row is a token's elements of all of them."""
+
+    def __init__(self, size: int, dtype: torch.dtype, rows, device: torch.device):
+        self.rows = [int(r) for r in rows]
+        super().__init__(size, dtype, 1, sum(self.rows), 1, device)
+
+    def kv_row_shape(self):
+        return (sum(self.rows),)
+
+    def _init_buffers(self):
+        self.kv_layers = [torch.zeros((self.size + 1, r), dtype=self.dtype, device=self.device) for r in self.rows]
+        self.kv_buffer = self.kv_layers[0] if self.kv_layers else torch.zeros((self.size + 1, 0), dtype=self.dtype,
+                                                                              device=self.device)
+
+    @staticmethod
+    def bytes_per_token(dtype, rows) -> int:
+        return sum(rows) * torch.empty((), dtype=dtype).element_size()
+
+    def layer(self, i: int) -> torch.Tensor:
+        return self.kv_layers[i]
+
+    def gather_pages(self, slots: torch.Tensor, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+        idx = slots.to(self.device, torch.long)
+        n = idx.shape[0]
+        if out is None:
+            out = torch.empty((1, n, sum(self.rows)), dtype=self.dtype, device=self.device)
+        at = 0
+        for buf, r in zip(self.kv_layers, self.rows):
+            out[0, :n, at:at + r].copy_(buf[idx])
+            at += r
+        return out
+
+    def scatter_pages(self, slots: torch.Tensor, pages: torch.Tensor) -> None:
+        idx = slots.to(self.device, torch.long)
+        at = 0
+        for buf, r in zip(self.kv_layers, self.rows):
+            buf[idx] = pages[0, : idx.shape[0], at:at + r].to(self.device)
+            at += r
+
+
 class Int8KVMemoryManager(MemoryManager):
     """GQA/MHA pool with int8 rows: every (slot, head) row is `head_dim` int8 values, an fp32 scale and padding to
     a multiple of 16 bytes (`ops/kv_quant.py`).  `layer(i)` returns an `Int8KVLayer`, which the attention ops accept

@@ -1,11 +1,11 @@
 // Paged causal attention for the layer shapes the tensor-core kernels do not cover: any head size up to
-// 256 (Gemma 256, Phi-3 96, StableLM 80 ...), sliding windows, ALiBi slopes, logit soft-capping and
-// attention sinks.  One CTA per (query token, query head); its four warps stride over the keys, each
+// 256 (Gemma 256, Phi-3 96, StableLM 80 ...; up to 512 in the form with its own value size, in bf16 or fp32),
+// sliding windows, ALiBi slopes, logit soft-capping, attention sinks and a sigmoid output gate per head.  One CTA per (query token, query head); its four warps stride over the keys, each
 // keeps an online-softmax state with the head vector spread over the lanes, and the states are merged
 // in shared memory.  Prefill and decode use the same kernel: a query is described by its position and
 // the request row it belongs to.
 //
-// KV pool row layout (one layer): [slot][2 * Hkv][D], K heads first, then V heads.
+// KV pool row layout (one layer): [slot][Hkv * D | Hkv * DV], K heads first, then V heads.
 #include "common.cuh"
 
 using namespace llb;
@@ -13,82 +13,96 @@ using namespace llb;
 constexpr int GEN_WARPS = 4;
 constexpr int GEN_MAX_EPL = 8;  // elements per lane: D <= 256
 
+namespace {
+__device__ __forceinline__ float to_f(float v) { return v; }
+__device__ __forceinline__ float to_f(bf16 v) { return __bfloat162float(v); }
+__device__ __forceinline__ void from_f(float v, float* p) { *p = v; }
+__device__ __forceinline__ void from_f(float v, bf16* p) { *p = __float2bfloat16(v); }
+__device__ __forceinline__ float exp_for(float v, const float*) { return expf(v); }
+__device__ __forceinline__ float exp_for(float v, const bf16*) { return __expf(v); }
+}  // namespace
+
+// EPL: elements per lane (sizes up to 32 * EPL).  gate [T, >= Hq] (row pitch gate_stride) or null: head h of the output
+// is multiplied by out_scale * sigmoid(gate[t, h]).
+template <typename E, int EPL>
 __global__ void __launch_bounds__(GEN_WARPS * 32)
-attn_generic_kernel(const bf16* __restrict__ q, int64_t q_stride, const bf16* __restrict__ kv,
+attn_generic_kernel(const E* __restrict__ q, int64_t q_stride, const E* __restrict__ kv,
                     const int* __restrict__ req_to_token, int64_t r2t_stride, const int* __restrict__ b_req_idx,
-                    const int* __restrict__ pos, const int* __restrict__ batch_of, bf16* __restrict__ out,
-                    int64_t out_stride, int Hq, int Hkv, int D, float sm_scale, int window, float softcap,
-                    const float* __restrict__ alibi, const float* __restrict__ sinks) {
+                    const int* __restrict__ pos, const int* __restrict__ batch_of, E* __restrict__ out,
+                    int64_t out_stride, int Hq, int Hkv, int D, int DV, float sm_scale, int window, float softcap,
+                    const float* __restrict__ alibi, const float* __restrict__ sinks, const E* __restrict__ gate,
+                    int64_t gate_stride, float out_scale) {
   const int t = blockIdx.x, h = blockIdx.y;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int b = batch_of ? batch_of[t] : t;
   const int qpos = pos[t];
   const int kvh = h / (Hq / Hkv);
   const int* slots = req_to_token + (int64_t)b_req_idx[b] * r2t_stride;
-  const int64_t row = (int64_t)2 * Hkv * D;
+  const int64_t row = (int64_t)Hkv * (D + DV);
 
-  float qv[GEN_MAX_EPL], acc[GEN_MAX_EPL];
+  float qv[EPL], acc[EPL];
 #pragma unroll
-  for (int e = 0; e < GEN_MAX_EPL; ++e) {
+  for (int e = 0; e < EPL; ++e) {
     int d = lane + e * 32;
-    qv[e] = d < D ? __bfloat162float(q[(int64_t)t * q_stride + (int64_t)h * D + d]) * sm_scale : 0.f;
+    qv[e] = d < D ? to_f(q[(int64_t)t * q_stride + (int64_t)h * D + d]) * sm_scale : 0.f;
     acc[e] = 0.f;
   }
   float m = -INFINITY, l = 0.f;
   const int j0 = (window > 0 && qpos - window + 1 > 0) ? qpos - window + 1 : 0;
   const float slope = alibi ? alibi[h] : 0.f;
   for (int j = j0 + warp; j <= qpos; j += GEN_WARPS) {
-    const bf16* kr = kv + (int64_t)slots[j] * row + (int64_t)kvh * D;
+    const E* kr = kv + (int64_t)slots[j] * row + (int64_t)kvh * D;
     float s = 0.f;
 #pragma unroll
-    for (int e = 0; e < GEN_MAX_EPL; ++e) {
+    for (int e = 0; e < EPL; ++e) {
       int d = lane + e * 32;
-      if (d < D) s += qv[e] * __bfloat162float(kr[d]);
+      if (d < D) s += qv[e] * to_f(kr[d]);
     }
     s = warp_sum(s);
     if (softcap > 0.f) s = softcap * tanhf(s / softcap);
     s += slope * (float)(j - qpos);
     const float mn = fmaxf(m, s);
-    const float corr = __expf(m - mn), p = __expf(s - mn);
+    const float corr = exp_for(m - mn, q), p = exp_for(s - mn, q);
     l = l * corr + p;
-    const bf16* vr = kr + (int64_t)Hkv * D;
+    const E* vr = kv + (int64_t)slots[j] * row + (int64_t)Hkv * D + (int64_t)kvh * DV;
 #pragma unroll
-    for (int e = 0; e < GEN_MAX_EPL; ++e) {
+    for (int e = 0; e < EPL; ++e) {
       int d = lane + e * 32;
-      if (d < D) acc[e] = acc[e] * corr + p * __bfloat162float(vr[d]);
+      if (d < DV) acc[e] = acc[e] * corr + p * to_f(vr[d]);
     }
     m = mn;
   }
   __shared__ float s_m[GEN_WARPS], s_l[GEN_WARPS];
-  __shared__ float s_acc[GEN_WARPS][GEN_MAX_EPL * 32];
+  __shared__ float s_acc[GEN_WARPS][EPL * 32];
   if (lane == 0) {
     s_m[warp] = m;
     s_l[warp] = l;
   }
 #pragma unroll
-  for (int e = 0; e < GEN_MAX_EPL; ++e) s_acc[warp][lane + e * 32] = acc[e];
+  for (int e = 0; e < EPL; ++e) s_acc[warp][lane + e * 32] = acc[e];
   __syncthreads();
   if (warp == 0) {
     float M = sinks ? sinks[h] : -INFINITY;
 #pragma unroll
     for (int w = 0; w < GEN_WARPS; ++w) M = fmaxf(M, s_m[w]);
-    float L = sinks ? __expf(sinks[h] - M) : 0.f;
-    float o[GEN_MAX_EPL];
+    float L = sinks ? exp_for(sinks[h] - M, q) : 0.f;
+    float o[EPL];
 #pragma unroll
-    for (int e = 0; e < GEN_MAX_EPL; ++e) o[e] = 0.f;
+    for (int e = 0; e < EPL; ++e) o[e] = 0.f;
 #pragma unroll
     for (int w = 0; w < GEN_WARPS; ++w) {
       if (s_m[w] == -INFINITY) continue;
-      const float c = __expf(s_m[w] - M);
+      const float c = exp_for(s_m[w] - M, q);
       L += s_l[w] * c;
 #pragma unroll
-      for (int e = 0; e < GEN_MAX_EPL; ++e) o[e] += s_acc[w][lane + e * 32] * c;
+      for (int e = 0; e < EPL; ++e) o[e] += s_acc[w][lane + e * 32] * c;
     }
-    const float inv = L > 0.f ? 1.f / L : 0.f;
+    float inv = L > 0.f ? out_scale / L : 0.f;
+    if (gate != nullptr) inv /= 1.f + exp_for(-to_f(gate[(int64_t)t * gate_stride + h]), q);
 #pragma unroll
-    for (int e = 0; e < GEN_MAX_EPL; ++e) {
+    for (int e = 0; e < EPL; ++e) {
       int d = lane + e * 32;
-      if (d < D) out[(int64_t)t * out_stride + (int64_t)h * D + d] = __float2bfloat16(o[e] * inv);
+      if (d < DV) from_f(o[e] * inv, &out[(int64_t)t * out_stride + (int64_t)h * DV + d]);
     }
   }
 }
@@ -100,9 +114,36 @@ LLB_EXPORT int llb_attn_generic(const void* q, int64_t q_stride, const void* kv_
   if (T <= 0) return LLB_OK;
   if (D <= 0 || D > 32 * GEN_MAX_EPL || Hkv <= 0 || Hq % Hkv != 0) return LLB_ERR_UNSUPPORTED;
   dim3 grid(T, Hq);
-  attn_generic_kernel<<<grid, GEN_WARPS * 32, 0, st>>>((const bf16*)q, q_stride, (const bf16*)kv_layer, req_to_token,
-                                                       r2t_stride, b_req_idx, pos, batch_of, (bf16*)out, out_stride,
-                                                       Hq, Hkv, D, sm_scale, window, softcap, alibi_slopes, sinks);
+  attn_generic_kernel<bf16, GEN_MAX_EPL><<<grid, GEN_WARPS * 32, 0, st>>>(
+      (const bf16*)q, q_stride, (const bf16*)kv_layer, req_to_token, r2t_stride, b_req_idx, pos, batch_of, (bf16*)out,
+      out_stride, Hq, Hkv, D, D, sm_scale, window, softcap, alibi_slopes, sinks, nullptr, 0, 1.f);
+  LLB_LAUNCH_CHECK();
+  return LLB_OK;
+}
+
+// The form with a value size of its own, an output gate per head, and fp32 (dt 0) beside bf16 (dt 1).
+LLB_EXPORT int llb_attn_generic_kv(const void* q, int dt, int64_t q_stride, const void* kv_layer, const int* req_to_token,
+                                   int64_t r2t_stride, const int* b_req_idx, const int* pos, const int* batch_of,
+                                   void* out, int64_t out_stride, int T, int Hq, int Hkv, int D, int DV, float sm_scale,
+                                   int window, const void* gate, int64_t gate_stride, float out_scale, cudaStream_t st) {
+  if (T <= 0) return LLB_OK;
+  if (D <= 0 || DV <= 0 || D > 512 || DV > 512 || Hkv <= 0 || Hq % Hkv != 0 || Hq > 65535) return LLB_ERR_UNSUPPORTED;
+  const dim3 grid(T, Hq);
+#define LLB_GENERIC(E, EPL)                                                                                           \
+  attn_generic_kernel<E, EPL><<<grid, GEN_WARPS * 32, 0, st>>>(                                                       \
+      (const E*)q, q_stride, (const E*)kv_layer, req_to_token, r2t_stride, b_req_idx, pos, batch_of, (E*)out,         \
+      out_stride, Hq, Hkv, D, DV, sm_scale, window, 0.f, nullptr, nullptr, (const E*)gate, gate_stride, out_scale)
+  if (D <= 128 && DV <= 128) {
+    if (dt == 0)
+      LLB_GENERIC(float, 4);
+    else
+      LLB_GENERIC(bf16, 4);
+  } else if (dt == 0) {
+    LLB_GENERIC(float, 16);
+  } else {
+    LLB_GENERIC(bf16, 16);
+  }
+#undef LLB_GENERIC
   LLB_LAUNCH_CHECK();
   return LLB_OK;
 }
@@ -155,6 +196,106 @@ LLB_EXPORT int llb_rope_kv_scatter_generic(void* qkv, void* kv_layer, const floa
     cudaFuncSetAttribute(rope_kv_scatter_generic_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   rope_kv_scatter_generic_kernel<<<T, 256, smem, st>>>((bf16*)qkv, (bf16*)kv_layer, cos_t, sin_t, pos, slot, Hq, Hkv, D,
                                                       rot_dim, qkv_stride);
+  LLB_LAUNCH_CHECK();
+  return LLB_OK;
+}
+
+// Per-head RMS norm of q and k over the first `dim` of their D elements, rotary positions on the first rot_dim, and the
+// cache write, for layers whose value size DV differs from the key size D.  qkv row: [Hq * D | Hkv * D | Hkv * DV]; q is
+// rewritten in place, K and V go to kv_layer[slot].  Sizes are multiples of 8; a group of 2^k lanes works on one head, a
+// lane on 8 elements of it at a time, and rotation partners meet in shared memory.
+template <typename E>
+__global__ void __launch_bounds__(256)
+qk_norm_rope_scatter_kernel(E* __restrict__ qkv, int64_t qkv_stride, E* __restrict__ kv_layer,
+                            const float* __restrict__ cos_t, const float* __restrict__ sin_t, const int* __restrict__ pos,
+                            const int* __restrict__ slot, const float* __restrict__ qw, const float* __restrict__ kw,
+                            float eps, int T, int Hq, int Hkv, int D, int dim, int DV, int rot_dim, int lanes) {
+  pdl_wait();
+  extern __shared__ float srow[];  // [groups][D]
+  const int gl = threadIdx.x % lanes, grp = threadIdx.x / lanes, groups = blockDim.x / lanes;
+  const int heads = Hq + 2 * Hkv;
+  const int64_t item = (int64_t)blockIdx.x * groups + grp;
+  const bool live = item < (int64_t)T * heads;
+  const int t = live ? (int)(item / heads) : 0, head = live ? (int)(item - (int64_t)t * heads) : Hq + Hkv;
+  E* row = qkv + (int64_t)t * qkv_stride;
+  const int half = rot_dim >> 1;
+  float* sh = srow + grp * D;
+  if (head >= Hq + Hkv) {  // V
+    const int g = head - Hq - Hkv;
+    const uint4* src = reinterpret_cast<const uint4*>(row + (int64_t)(Hq + Hkv) * D + (int64_t)g * DV);
+    if (live) {
+      uint4* dst = reinterpret_cast<uint4*>(kv_layer + (int64_t)slot[t] * Hkv * (D + DV) + (int64_t)Hkv * D + (int64_t)g * DV);
+      for (int v = gl; v < DV * (int)sizeof(E) / 16; v += lanes) dst[v] = src[v];
+    }
+  }
+  const bool qk = live && head < Hq + Hkv;
+  E* x = row + (int64_t)head * D;
+  const float* w = head < Hq ? qw : kw;
+  float ss = 0.f;
+  if (qk) {
+    for (int d = gl * 8; d < D; d += lanes * 8) {
+      float f[8];
+      if constexpr (sizeof(E) == 2) {
+        unpack8(*reinterpret_cast<const bf16x8*>(x + d), f);
+      } else {
+#pragma unroll
+        for (int i = 0; i < 8; ++i) f[i] = x[d + i];
+      }
+#pragma unroll
+      for (int i = 0; i < 8; ++i) {
+        sh[d + i] = f[i];
+        ss = fmaf(f[i], f[i], ss);
+      }
+    }
+  }
+  for (int o = lanes >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+  __syncwarp();
+  if (!qk) return;
+  const float inv = rsqrtf(ss / (float)dim + eps);
+  const float *cr = cos_t + (int64_t)pos[t] * half, *sr = sin_t + (int64_t)pos[t] * half;
+  E* dst = head < Hq ? x : kv_layer + (int64_t)slot[t] * Hkv * (D + DV) + (int64_t)(head - Hq) * D;
+  for (int d = gl * 8; d < D; d += lanes * 8) {
+    float o[8];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      const int e = d + i;
+      float v = sh[e] * inv * w[e];
+      if (e < half)
+        v = v * cr[e] - sh[e + half] * inv * w[e + half] * sr[e];
+      else if (e < rot_dim)
+        v = v * cr[e - half] + sh[e - half] * inv * w[e - half] * sr[e - half];
+      o[i] = v;
+    }
+    if constexpr (sizeof(E) == 2) {
+      *reinterpret_cast<bf16x8*>(dst + d) = pack8(o);
+    } else {
+#pragma unroll
+      for (int i = 0; i < 8; ++i) dst[d + i] = o[i];
+    }
+  }
+}
+
+// qw, kw: fp32 [D], zero beyond dim.  dt: 0 = fp32, 1 = bf16.
+LLB_EXPORT int llb_qk_norm_rope_scatter(void* qkv, int dt, int64_t qkv_stride, void* kv_layer, const float* cos_t,
+                                        const float* sin_t, const int* pos, const int* slot, const float* qw,
+                                        const float* kw, float eps, int T, int Hq, int Hkv, int D, int dim, int DV,
+                                        int rot_dim, cudaStream_t st) {
+  if (T <= 0) return LLB_OK;
+  if (D <= 0 || (D % 8) || DV <= 0 || (DV % 8) || D > 512 || dim <= 0 || dim > D || (rot_dim & 1) || rot_dim > dim ||
+      (qkv_stride % 8) || Hkv <= 0)
+    return LLB_ERR_UNSUPPORTED;
+  int lanes = 4;
+  while (lanes < 32 && lanes * 8 < D) lanes *= 2;
+  const int groups = 256 / lanes;
+  const int64_t blocks = cdiv64((int64_t)T * (Hq + 2 * Hkv), groups);
+  const size_t smem = (size_t)groups * D * sizeof(float);
+  if (smem > 48 * 1024 || blocks > 0x7fffffff) return LLB_ERR_UNSUPPORTED;
+  if (dt == 0)
+    launch_pdl(qk_norm_rope_scatter_kernel<float>, dim3((unsigned)blocks), dim3(256), smem, st, (float*)qkv, qkv_stride,
+               (float*)kv_layer, cos_t, sin_t, pos, slot, qw, kw, eps, T, Hq, Hkv, D, dim, DV, rot_dim, lanes);
+  else
+    launch_pdl(qk_norm_rope_scatter_kernel<bf16>, dim3((unsigned)blocks), dim3(256), smem, st, (bf16*)qkv, qkv_stride,
+               (bf16*)kv_layer, cos_t, sin_t, pos, slot, qw, kw, eps, T, Hq, Hkv, D, dim, DV, rot_dim, lanes);
   LLB_LAUNCH_CHECK();
   return LLB_OK;
 }

@@ -10,7 +10,8 @@ using namespace llb;
 
 namespace {
 
-enum Epi { F_STORE = 0, F_RESIDUAL = 1, F_GATED_SILU = 2, F_F32 = 3, F_GATED_GELU = 4, F_RELU2 = 5, F_DYT = 6 };
+enum Epi { F_STORE = 0, F_RESIDUAL = 1, F_GATED_SILU = 2, F_F32 = 3, F_GATED_GELU = 4, F_RELU2 = 5, F_DYT = 6, F_GATED_CLAMP = 7 };
+__host__ __device__ constexpr bool gated_epi(int e) { return e == F_GATED_SILU || e == F_GATED_GELU || e == F_GATED_CLAMP; }
 
 struct DytPair {
   float* x;  // residual stream, same pitch as C
@@ -29,6 +30,7 @@ struct F32Params {
   int M, N, K;
   float alpha;
   DytPair d;
+  float act_alpha, act_limit;  // F_GATED_CLAMP
 };
 
 constexpr int TM = 64, TN = 64, TK = 16;
@@ -41,7 +43,7 @@ __device__ __forceinline__ float act_gelu_tanh(float v) {
 template <int EPI>
 __global__ void __launch_bounds__(256) gemm_f32_kernel(const F32Params p) {
   __shared__ float As[TK][TM + 4], Ws[TK][TN + 4];
-  constexpr bool GATED = EPI == F_GATED_SILU || EPI == F_GATED_GELU;
+  constexpr bool GATED = gated_epi(EPI);
   __shared__ float gate_tile[GATED ? TM : 1][GATED ? TN + 1 : 1];
   const int m0 = blockIdx.y * TM, n0 = blockIdx.x * TN;
   const float* A = p.A + blockIdx.z * p.a_batch;
@@ -90,8 +92,15 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const F32Params p) {
     for (int i = threadIdx.x; i < TM * 32; i += 256) {
       const int r = i >> 5, c = i & 31;
       if (m0 + r < p.M && n0 + c < p.N) {
-        const float g = gate_tile[r][c], u = gate_tile[r][c + 32];
-        C[(int64_t)(m0 + r) * p.ldc + n0 / 2 + c] = (EPI == F_GATED_SILU ? act_silu(g) : act_gelu_tanh(g)) * u;
+        float g = gate_tile[r][c], u = gate_tile[r][c + 32], v;
+        if (EPI == F_GATED_CLAMP) {
+          g = fminf(g, p.act_limit);
+          u = fminf(fmaxf(u, -p.act_limit), p.act_limit);
+          v = g / (1.f + expf(-p.act_alpha * g)) * (u + 1.f);
+        } else {
+          v = (EPI == F_GATED_SILU ? act_silu(g) : act_gelu_tanh(g)) * u;
+        }
+        C[(int64_t)(m0 + r) * p.ldc + n0 / 2 + c] = v;
       }
     }
   } else {
@@ -139,10 +148,10 @@ LLB_EXPORT int llb_gemm_f32(const float* A, int64_t lda, int64_t a_batch, const 
                             float* C, int64_t ldc, int64_t c_batch, const float* residual, const float* bias, float* x,
                             const float* w1, const float* b1, float alpha1, const float* w2, const float* b2,
                             float alpha2, const int* mblock_expert, int M, int N, int K, int batch, int epi,
-                            float alpha, cudaStream_t st) {
+                            float alpha, float act_alpha, float act_limit, cudaStream_t st) {
   if (M <= 0 || N <= 0 || batch <= 0) return LLB_OK;
   if (K <= 0 || cdiv(M, TM) > 65535 || batch > 65535) return LLB_ERR_UNSUPPORTED;
-  if ((epi == F_GATED_SILU || epi == F_GATED_GELU) && (N % 64)) return LLB_ERR_UNSUPPORTED;
+  if (gated_epi(epi) && (N % 64)) return LLB_ERR_UNSUPPORTED;
   if (mblock_expert != nullptr && (batch != 1 || (M % 128))) return LLB_ERR_BAD_ARG;
   if (epi == F_RESIDUAL && residual == nullptr) return LLB_ERR_BAD_ARG;
   if (epi == F_DYT && (x == nullptr || w1 == nullptr || b1 == nullptr || w2 == nullptr || b2 == nullptr || batch != 1))
@@ -164,6 +173,8 @@ LLB_EXPORT int llb_gemm_f32(const float* A, int64_t lda, int64_t a_batch, const 
   p.N = N;
   p.K = K;
   p.alpha = alpha;
+  p.act_alpha = act_alpha;
+  p.act_limit = act_limit;
   p.d = DytPair{x, w1, b1, w2, b2, alpha1, alpha2};
   switch (epi) {
     case F_STORE: return launch<F_STORE>(p, batch, st);
@@ -173,6 +184,7 @@ LLB_EXPORT int llb_gemm_f32(const float* A, int64_t lda, int64_t a_batch, const 
     case F_GATED_GELU: return launch<F_GATED_GELU>(p, batch, st);
     case F_RELU2: return launch<F_RELU2>(p, batch, st);
     case F_DYT: return launch<F_DYT>(p, batch, st);
+    case F_GATED_CLAMP: return launch<F_GATED_CLAMP>(p, batch, st);
   }
   return LLB_ERR_UNSUPPORTED;
 }

@@ -33,7 +33,11 @@ constexpr int GEMM_THREADS = 192;
 constexpr int SMEM_BUDGET = 224 * 1024;
 constexpr int64_t kPanelBytes = 24ll << 20;  // A panel kept hot in L2 while W streams past it
 
-enum Epi { EPI_STORE = 0, EPI_RESIDUAL = 1, EPI_GATED_SILU = 2, EPI_F32 = 3, EPI_GATED_GELU = 4, EPI_RELU2 = 5, EPI_DYT = 6 };
+enum Epi { EPI_STORE = 0, EPI_RESIDUAL = 1, EPI_GATED_SILU = 2, EPI_F32 = 3, EPI_GATED_GELU = 4, EPI_RELU2 = 5, EPI_DYT = 6,
+           EPI_GATED_CLAMP = 7 };
+__host__ __device__ constexpr bool epi_gated(int epi) {
+  return epi == EPI_GATED_SILU || epi == EPI_GATED_GELU || epi == EPI_GATED_CLAMP;
+}
 
 // dyt(v) = tanh(alpha * v) * w + b; x is the fp32 residual stream [M, ldc]
 struct DytFuse {
@@ -74,6 +78,7 @@ struct GemmParams {
   int push_world, push_rank, push_max_mb;
   float out_scale;  // EPI_F32: factor on the stored value
   DytFuse dyt;      // EPI_DYT
+  float act_alpha, act_limit;  // EPI_GATED_CLAMP
 };
 
 // Output staging of the epilogue warps: a thread owns one accumulator row, so storing straight from registers
@@ -101,6 +106,16 @@ constexpr int smem_bytes() {
 __device__ __forceinline__ float silu_f(float v) { return v / (1.f + __expf(-v)); }
 __device__ __forceinline__ float gelu_tanh_f(float v) {
   return 0.5f * v * (1.f + tanhf(0.7978845608028654f * (v + 0.044715f * v * v * v)));
+}
+// gate and up accumulators of one column -> output of a gated epilogue
+template <int EPI>
+__device__ __forceinline__ float gated_f(const GemmParams& p, float g, float u) {
+  if (EPI == EPI_GATED_CLAMP) {
+    g = fminf(g, p.act_limit);
+    u = fminf(fmaxf(u, -p.act_limit), p.act_limit);
+    return __fdividef(g, 1.f + __expf(-p.act_alpha * g)) * (u + 1.f);
+  }
+  return (EPI == EPI_GATED_SILU ? silu_f(g) : gelu_tanh_f(g)) * u;
 }
 __device__ __forceinline__ float relu2_f(float v) {
   v = fmaxf(v, 0.f);
@@ -305,7 +320,7 @@ __device__ __forceinline__ void epilogue_store(const GemmParams& p, uint32_t t_r
   const int lane = threadIdx.x & 31;
   const int row_base = row - lane;
   uint8_t* my = stage + lane * EPI_ROW_PITCH;
-  if (EPI == EPI_GATED_SILU || EPI == EPI_GATED_GELU) {
+  if (epi_gated(EPI)) {
     // columns come as [32 gate | 32 up] pairs; output has N/2 columns
     bf16* crow = (bf16*)p.C + (int64_t)row * p.ldc;
     constexpr int STEP = (BN % 128 == 0) ? 128 : 64;
@@ -332,7 +347,7 @@ __device__ __forceinline__ void epilogue_store(const GemmParams& p, uint32_t t_r
             for (int e = 0; e < 8; ++e) {
               float gv = __uint_as_float(gr[j + e]);
               float uv = __uint_as_float(ur[j + e]);
-              o[e] = (EPI == EPI_GATED_SILU ? silu_f(gv) : gelu_tanh_f(gv)) * uv;
+              o[e] = gated_f<EPI>(p, gv, uv);
             }
             if (staged)
               *reinterpret_cast<bf16x8*>(my + sub * 64 + j * 2) = pack8(o);
@@ -816,6 +831,8 @@ int dispatch_epi(int epi, const CUtensorMap& ta, const CUtensorMap& tb, GemmPara
       return launch_gemm<BN, EPI_F32>(ta, tb, p, st);
     case EPI_GATED_GELU:
       return launch_gemm<BN, EPI_GATED_GELU>(ta, tb, p, st);
+    case EPI_GATED_CLAMP:
+      return launch_gemm<BN, EPI_GATED_CLAMP>(ta, tb, p, st);
     case EPI_RELU2:
       return launch_gemm<BN, EPI_RELU2>(ta, tb, p, st);
     case EPI_DYT:
@@ -1020,6 +1037,8 @@ int dispatch_pair(int epi, const CUtensorMap& ta, const CUtensorMap& tb, GemmPar
       return launch_pair<EPI_F32>(ta, tb, p, st);
     case EPI_GATED_GELU:
       return launch_pair<EPI_GATED_GELU>(ta, tb, p, st);
+    case EPI_GATED_CLAMP:
+      return launch_pair<EPI_GATED_CLAMP>(ta, tb, p, st);
     case EPI_RELU2:
       return launch_pair<EPI_RELU2>(ta, tb, p, st);
     case EPI_DYT:
@@ -1353,7 +1372,7 @@ int launch_skinny(const CUtensorMap& ta, const CUtensorMap& tb, const GemmParams
 // tw: 256, or 128 (nb == 1, plain epilogues only)
 int dispatch_skinny(int epi, int nb, int splits, int tw, const CUtensorMap& ta, const CUtensorMap& tb,
                     const GemmParams& p, cudaStream_t st) {
-  if (splits > 1 && (nb != 1 || epi == EPI_GATED_SILU || epi == EPI_GATED_GELU)) return LLB_ERR_UNSUPPORTED;
+  if (splits > 1 && (nb != 1 || epi_gated(epi))) return LLB_ERR_UNSUPPORTED;
   if (tw == 128) {
     if (nb != 1) return LLB_ERR_UNSUPPORTED;
     switch (epi) {
@@ -1371,6 +1390,7 @@ int dispatch_skinny(int epi, int nb, int splits, int tw, const CUtensorMap& ta, 
       case EPI_RESIDUAL: return launch_skinny<1, EPI_RESIDUAL>(ta, tb, p, splits, st);
       case EPI_GATED_SILU: return launch_skinny<1, EPI_GATED_SILU>(ta, tb, p, splits, st);
       case EPI_GATED_GELU: return launch_skinny<1, EPI_GATED_GELU>(ta, tb, p, splits, st);
+      case EPI_GATED_CLAMP: return launch_skinny<1, EPI_GATED_CLAMP>(ta, tb, p, splits, st);
       case EPI_F32: return launch_skinny<1, EPI_F32>(ta, tb, p, splits, st);
       case EPI_RELU2: return launch_skinny<1, EPI_RELU2>(ta, tb, p, splits, st);
       case EPI_DYT: return launch_skinny<1, EPI_DYT>(ta, tb, p, splits, st);
@@ -1381,6 +1401,7 @@ int dispatch_skinny(int epi, int nb, int splits, int tw, const CUtensorMap& ta, 
       case EPI_RESIDUAL: return launch_skinny<2, EPI_RESIDUAL>(ta, tb, p, 1, st);
       case EPI_GATED_SILU: return launch_skinny<2, EPI_GATED_SILU>(ta, tb, p, 1, st);
       case EPI_GATED_GELU: return launch_skinny<2, EPI_GATED_GELU>(ta, tb, p, 1, st);
+      case EPI_GATED_CLAMP: return launch_skinny<2, EPI_GATED_CLAMP>(ta, tb, p, 1, st);
       case EPI_F32: return launch_skinny<2, EPI_F32>(ta, tb, p, 1, st);
       case EPI_RELU2: return launch_skinny<2, EPI_RELU2>(ta, tb, p, 1, st);
       case EPI_DYT: return launch_skinny<2, EPI_DYT>(ta, tb, p, 1, st);
@@ -1398,7 +1419,7 @@ bool g_skinny_auto = true;
 bool g_skinny_tw128 = true;
 
 void skinny_plan(int M, int N, int K, int epi, int* nb, int* splits, bool* use_pair, int* tw) {
-  const bool gated = epi == EPI_GATED_SILU || epi == EPI_GATED_GELU;
+  const bool gated = epi_gated(epi);
   const int sms = sm_count();
   const int tiles = cdiv(N, 256), kb = cdiv(K, BK);
   *nb = 0;
@@ -1459,7 +1480,7 @@ gemm_bf16_splitk_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_co
   constexpr int STAGE_BYTES = spk_stage_bytes<MBLK>();
   constexpr uint32_t TMEM_COLS = MBLK * SPK_BN;
   constexpr uint32_t IDESC = umma_idesc(BM, SPK_BN, 1);
-  constexpr bool GATED = EPI == EPI_GATED_SILU || EPI == EPI_GATED_GELU;
+  constexpr bool GATED = epi_gated(EPI);
   constexpr int UW = GATED ? 64 : 32;     // unit width in accumulator columns
   constexpr int UPB = SPK_BN / UW;        // units per 128-row block
   constexpr int U = MBLK * UPB;
@@ -1661,7 +1682,7 @@ gemm_bf16_splitk_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_co
 #pragma unroll
                 for (int e = 0; e < 8; ++e) {
                   const float gv = __uint_as_float(r[j + e]), uv = __uint_as_float(r[32 + j + e]);
-                  o[e] = (EPI == EPI_GATED_SILU ? silu_f(gv) : gelu_tanh_f(gv)) * uv;
+                  o[e] = gated_f<EPI>(p, gv, uv);
                 }
                 *reinterpret_cast<bf16x8*>(crow + j) = pack8(o);
               }
@@ -1710,6 +1731,7 @@ int dispatch_splitk(int epi, const CUtensorMap& ta, const CUtensorMap& tb, const
     case EPI_RESIDUAL: return launch_splitk<MBLK, EPI_RESIDUAL>(ta, tb, p, splits, st);
     case EPI_GATED_SILU: return launch_splitk<MBLK, EPI_GATED_SILU>(ta, tb, p, splits, st);
     case EPI_GATED_GELU: return launch_splitk<MBLK, EPI_GATED_GELU>(ta, tb, p, splits, st);
+    case EPI_GATED_CLAMP: return launch_splitk<MBLK, EPI_GATED_CLAMP>(ta, tb, p, splits, st);
     case EPI_F32: return launch_splitk<MBLK, EPI_F32>(ta, tb, p, splits, st);
   }
   return LLB_ERR_UNSUPPORTED;
@@ -1739,7 +1761,7 @@ gemm_bf16_pairsplit_kernel(const __grid_constant__ CUtensorMap tmA, const __grid
   constexpr int STAGE_BYTES = PSK_STAGE_BYTES;
   constexpr uint32_t TMEM_COLS = PSK_TW;
   constexpr uint32_t IDESC = umma_idesc(256, PSK_TW, 1);
-  constexpr bool GATED = EPI == EPI_GATED_SILU || EPI == EPI_GATED_GELU;
+  constexpr bool GATED = epi_gated(EPI);
   constexpr int UW = GATED ? 64 : 32;
   constexpr int U = PSK_TW / UW;
 
@@ -1933,7 +1955,7 @@ gemm_bf16_pairsplit_kernel(const __grid_constant__ CUtensorMap tmA, const __grid
 #pragma unroll
                 for (int e = 0; e < 8; ++e) {
                   const float gv = __uint_as_float(r[j + e]), uv = __uint_as_float(r[32 + j + e]);
-                  o[e] = (EPI == EPI_GATED_SILU ? silu_f(gv) : gelu_tanh_f(gv)) * uv;
+                  o[e] = gated_f<EPI>(p, gv, uv);
                 }
                 *reinterpret_cast<bf16x8*>(crow + j) = pack8(o);
               }
@@ -1981,6 +2003,7 @@ int dispatch_pairsplit(int epi, const CUtensorMap& ta, const CUtensorMap& tb, co
     case EPI_RESIDUAL: return launch_pairsplit<EPI_RESIDUAL>(ta, tb, p, splits, st);
     case EPI_GATED_SILU: return launch_pairsplit<EPI_GATED_SILU>(ta, tb, p, splits, st);
     case EPI_GATED_GELU: return launch_pairsplit<EPI_GATED_GELU>(ta, tb, p, splits, st);
+    case EPI_GATED_CLAMP: return launch_pairsplit<EPI_GATED_CLAMP>(ta, tb, p, splits, st);
     case EPI_F32: return launch_pairsplit<EPI_F32>(ta, tb, p, splits, st);
   }
   return LLB_ERR_UNSUPPORTED;
@@ -1990,7 +2013,7 @@ int dispatch_pairsplit(int epi, const CUtensorMap& ta, const CUtensorMap& tb, co
 // k-block, the units of a tile must divide among the splits, and all CTAs must be resident at once.
 int pairsplit_max_splits(int M, int N, int K, int epi) {
   if ((N % 8) != 0) return 0;
-  const bool gated = epi == EPI_GATED_SILU || epi == EPI_GATED_GELU;
+  const bool gated = epi_gated(epi);
   const int units = gated ? 4 : 8;
   const int pairs = cdiv(M, 256) * cdiv(N, PSK_TW), kb = cdiv(K, BK);
   if (pairs * 2 > sm_count() || pairs * 2 > SPK_MAX_TILES) return 0;
@@ -2002,7 +2025,7 @@ int pairsplit_max_splits(int M, int N, int K, int epi) {
 // Largest usable split count for the split-K kernel (0: the shape does not fit it).
 int splitk_max_splits(int M, int N, int K, int epi) {
   if (M > 256 || (N % 8) != 0) return 0;
-  const bool gated = epi == EPI_GATED_SILU || epi == EPI_GATED_GELU;
+  const bool gated = epi_gated(epi);
   const int mblk = M > 128 ? 2 : 1;
   const int units = mblk * (gated ? 2 : 4);
   const int tiles = cdiv(N, SPK_BN), kb = cdiv(K, BK);
@@ -2032,6 +2055,7 @@ void apply_push(GemmParams& p) {
 struct GemmFuse {
   float out_scale = 1.f;
   DytFuse dyt = {nullptr, nullptr, nullptr, nullptr, nullptr, 1.f, 1.f};
+  float act_alpha = 1.f, act_limit = INFINITY;
 };
 
 bool g_pair_auto = true;  // measured faster than one-CTA tiles for M >= 1024, K <= 8192 on B200
@@ -2059,7 +2083,7 @@ LLB_EXPORT int llb_gemm_set_push(void** push, void** cnt, int rank, int world, i
 //   0 store bf16 (+bias)          1 store bf16 of acc (+bias) + residual[M,N] (same ldc)
 //   2 SiLU-gated: W rows interleaved as [32 gate | 32 up] blocks; C is [M, N/2]
 //   3 store fp32 (+bias)          4 GELU(tanh)-gated, layout as 2          5 store bf16 of relu(acc)^2
-//   6 dynamic-tanh sandwich (llb_gemm_bf16_fused)
+//   6 dynamic-tanh sandwich (llb_gemm_bf16_fused)   7 clamped gate (llb_gemm_bf16_fused), layout as 2
 // bn: 0 = choose, else 64/128/256, or 512 = the CTA-pair (cta_group::2) kernel with 256x256 tiles.  status: optional device int receiving a wait-timeout code.
 // stream_k: 0 = whole tiles per CTA, 1 = equal (tile, k-block) shares with fix-up of split tiles,
 // -1 = choose (stream-K when the tiles would fill fewer than three waves).  Stream-K needs
@@ -2071,7 +2095,7 @@ static int gemm_bf16(const void* A, int64_t lda, const void* W, int64_t ldw, voi
                              int sk_counters_len, int* status, const GemmFuse& fuse, cudaStream_t st) {
   if (M <= 0 || N <= 0) return LLB_OK;
   if (K <= 0 || (K % 8) != 0) return LLB_ERR_UNSUPPORTED;
-  if ((epi == EPI_GATED_SILU || epi == EPI_GATED_GELU) && (N % 64) != 0) return LLB_ERR_UNSUPPORTED;
+  if ((epi_gated(epi)) && (N % 64) != 0) return LLB_ERR_UNSUPPORTED;
   if (epi != EPI_F32 && (((uintptr_t)C & 15) || (ldc % 8))) return LLB_ERR_BAD_ARG;
   if (epi == EPI_F32 && (((uintptr_t)C & 15) || (ldc % 4))) return LLB_ERR_BAD_ARG;
   if (epi == EPI_RESIDUAL && (residual == nullptr || ((uintptr_t)residual & 15))) return LLB_ERR_BAD_ARG;
@@ -2121,6 +2145,8 @@ static int gemm_bf16(const void* A, int64_t lda, const void* W, int64_t ldw, voi
     apply_push(p);
     p.out_scale = fuse.out_scale;
     p.dyt = fuse.dyt;
+    p.act_alpha = fuse.act_alpha;
+    p.act_limit = fuse.act_limit;
     if (p.push_world > 0 && (epi != EPI_STORE || (N % 32))) return LLB_ERR_UNSUPPORTED;
     p.C = C;
     p.residual = (const bf16*)residual;
@@ -2159,6 +2185,8 @@ static int gemm_bf16(const void* A, int64_t lda, const void* W, int64_t ldw, voi
     apply_push(p);
     p.out_scale = fuse.out_scale;
     p.dyt = fuse.dyt;
+    p.act_alpha = fuse.act_alpha;
+    p.act_limit = fuse.act_limit;
     if (p.push_world > 0 && (epi != EPI_STORE || (N % 32))) return LLB_ERR_UNSUPPORTED;
     p.C = C;
     p.residual = (const bf16*)residual;
@@ -2213,6 +2241,8 @@ static int gemm_bf16(const void* A, int64_t lda, const void* W, int64_t ldw, voi
     apply_push(p);
     p.out_scale = fuse.out_scale;
     p.dyt = fuse.dyt;
+    p.act_alpha = fuse.act_alpha;
+    p.act_limit = fuse.act_limit;
     if (p.push_world > 0 && (epi != EPI_STORE || (N % 32))) return LLB_ERR_UNSUPPORTED;
     p.C = C;
     p.residual = (const bf16*)residual;
@@ -2246,6 +2276,8 @@ static int gemm_bf16(const void* A, int64_t lda, const void* W, int64_t ldw, voi
   apply_push(p);
   p.out_scale = fuse.out_scale;
   p.dyt = fuse.dyt;
+  p.act_alpha = fuse.act_alpha;
+  p.act_limit = fuse.act_limit;
   if (p.push_world > 0 && (epi != EPI_STORE || (N % 32) || stream_k)) return LLB_ERR_UNSUPPORTED;
   p.C = C;
   p.residual = (const bf16*)residual;
@@ -2286,11 +2318,15 @@ LLB_EXPORT int llb_gemm_bf16(const void* A, int64_t lda, const void* W, int64_t 
 
 // The epilogues with parameters: out_scale multiplies fp32 output (epi 3); for epi 6 (bf16 C, same pitch for x)
 //   x += tanh(alpha1 * acc) * w1 + b1;  C = tanh(alpha2 * x) * w2 + b2        x fp32 [M, ldc], vectors fp32 [N]
+// for epi 7 with g, u the gate and up columns:
+//   g = min(g, act_limit); u = clamp(u, -act_limit, act_limit); C = (u + 1) * g * sigmoid(act_alpha * g)
 LLB_EXPORT int llb_gemm_bf16_fused(const void* A, int64_t lda, const void* W, int64_t ldw, void* C, int64_t ldc,
                                    const void* bias, int M, int N, int K, int epi, int bn, float out_scale, float* x,
                                    const float* w1, const float* b1, float alpha1, const float* w2, const float* b2,
-                                   float alpha2, int* status, cudaStream_t st) {
+                                   float alpha2, float act_alpha, float act_limit, int* status, cudaStream_t st) {
   GemmFuse fuse;
+  fuse.act_alpha = act_alpha;
+  fuse.act_limit = act_limit;
   fuse.out_scale = out_scale;
   fuse.dyt = DytFuse{x, w1, b1, w2, b2, alpha1, alpha2};
   return gemm_bf16(A, lda, W, ldw, C, ldc, nullptr, bias, M, N, K, epi, bn, 0, nullptr, 0, nullptr, 0, status, fuse, st);
@@ -2302,7 +2338,7 @@ LLB_EXPORT int llb_gemm_bf16_fused(const void* A, int64_t lda, const void* W, in
 // C [M_pad, N] (or [M_pad, N/2] for the gated epilogues).  N must be a multiple of the tile width.
 LLB_EXPORT int llb_gemm_bf16_grouped(const void* A, int64_t lda, const void* W, int64_t ldw, void* C, int64_t ldc,
                                      const int* mblock_expert, int M_pad, int N, int K, int E, int epi, int bn,
-                                     int* status, cudaStream_t st) {
+                                     float act_alpha, float act_limit, int* status, cudaStream_t st) {
   if (M_pad <= 0 || N <= 0 || E <= 0) return LLB_OK;
   if (K <= 0 || (K % 8) != 0 || (M_pad % BM) != 0) return LLB_ERR_UNSUPPORTED;
   if (epi == EPI_RESIDUAL || epi == EPI_DYT) return LLB_ERR_UNSUPPORTED;
@@ -2317,6 +2353,8 @@ LLB_EXPORT int llb_gemm_bf16_grouped(const void* A, int64_t lda, const void* W, 
   GemmParams p;
   memset(&p, 0, sizeof(p));
   p.out_scale = 1.f;
+  p.act_alpha = act_alpha;
+  p.act_limit = act_limit;
   p.C = C;
   p.residual = nullptr;
   p.bias = nullptr;

@@ -31,20 +31,9 @@ from ..ops import moe as moe_ops
 from ..ops import reference as ref
 from .base import LayerWeights, TransformerLM
 from .registry import register_config, register_model
-from .weights import tp_range
-
-
-def _up(n: int, m: int) -> int:
-    return -(-n // m) * m
-
-
-def _pad(t: torch.Tensor, *sizes: int) -> torch.Tensor:
-    """Zero-pads t to `sizes`."""
-    if tuple(t.shape) == sizes:
-        return t
-    out = torch.zeros(sizes, dtype=t.dtype, device=t.device)
-    out[tuple(slice(0, n) for n in t.shape)] = t
-    return out
+from .weights import get_shaped, tp_range
+from .weights import pad_zeros as _pad
+from .weights import round_up as _up
 
 
 @register_config("Taduzen")
@@ -182,31 +171,25 @@ class TaduzenLM(TransformerLM):
                 out[name] = table(self.specs[int(name[1:].split(".")[0])].experts)
         return out
 
-    def _get(self, src, name, *shape):
-        """A checkpoint tensor, whose shape must be the one config.json implies."""
-        if tuple(src.shape(name)) != shape:
-            raise ValueError(f"tensor {name}: shape {tuple(src.shape(name))}, config.json says {shape}")
-        return src.get(name)
-
     def _load_norm(self, src, name) -> ops.DytNorm:
         W, P = self.hidden, self.hidden_p
-        return ops.DytNorm(_pad(self._get(src, name, W).float(), P).to(self.device),
-                           _pad(self._get(src, name + ".b", W).float(), P).to(self.device),
-                           float(self._get(src, name + ".alpha").float()))
+        return ops.DytNorm(_pad(get_shaped(src, name, W).float(), P).to(self.device),
+                           _pad(get_shaped(src, name + ".b", W).float(), P).to(self.device),
+                           float(get_shaped(src, name + ".alpha").float()))
 
     def _load_gated(self, src, p, ff, i0, i1):
         """(gate | up interleaved [2I, width], down [width, I]) of the columns i0 .. i1 of a feed-forward, padded."""
         W, P, I = self.hidden, self.hidden_p, _up(i1 - i0, 64)
-        g, u = (_pad(self._get(src, p + n, ff, W)[i0:i1], I, P) for n in ("gate", "up"))
-        return ref.interleave_gate_up(g, u), _pad(self._get(src, p + "down", W, ff)[:, i0:i1], P, I)
+        g, u = (_pad(get_shaped(src, p + n, ff, W)[i0:i1], I, P) for n in ("gate", "up"))
+        return ref.interleave_gate_up(g, u), _pad(get_shaped(src, p + "down", W, ff)[:, i0:i1], P, I)
 
     def _load_weights(self, src):
         tp, r = self.tp.size, self.tp.rank
         W, P = self.hidden, self.hidden_p
-        self.embed_w = self._dev(_pad(self._get(src, "embed", self.vocab, W), self.vocab, P))
+        self.embed_w = self._dev(_pad(get_shaped(src, "embed", self.vocab, W), self.vocab, P))
         self.embed_range = (0, self.vocab)
         v0, v1 = tp_range(self.vocab, r, tp)
-        self.lm_head_w = self._dev(_pad(self._get(src, "head", self.vocab, W)[v0:v1], _up(v1 - v0, 8), P))
+        self.lm_head_w = self._dev(_pad(get_shaped(src, "head", self.vocab, W)[v0:v1], _up(v1 - v0, 8), P))
         self.final_norm = self._load_norm(src, "final.norm")
         self.final_norm_w = None
         self.layers, tables = [], []
@@ -221,8 +204,8 @@ class TaduzenLM(TransformerLM):
             if l.kind == "dense":
                 i0, i1 = tp_range(l.ff, r, tp)
                 I = _up(i1 - i0, 64)
-                lw.up_w = self._dev(_pad(self._get(src, p + "mlp.up", l.ff, W)[i0:i1], I, P))
-                lw.down_w = self._dev(_pad(self._get(src, p + "mlp.down", W, l.ff)[:, i0:i1], P, I))
+                lw.up_w = self._dev(_pad(get_shaped(src, p + "mlp.up", l.ff, W)[i0:i1], I, P))
+                lw.down_w = self._dev(_pad(get_shaped(src, p + "mlp.down", W, l.ff)[:, i0:i1], P, I))
             elif l.kind == "moe":
                 tables.append(self._load_moe(lw, src, p + "mlp.", l))
                 lw.moe_index = len(tables) - 1
@@ -233,16 +216,16 @@ class TaduzenLM(TransformerLM):
         W, P = self.hidden, self.hidden_p
         h0, h1 = tp_range(l.heads, self.tp.rank, self.tp.size)
         n = lw.heads = h1 - h0
-        q = self._get(src, m + "q", l.heads * l.dim, W).view(l.heads, l.dim, W)[h0:h1]
-        dkv = self._get(src, m + "dkv", l.rank, W)
+        q = get_shaped(src, m + "q", l.heads * l.dim, W).view(l.heads, l.dim, W)[h0:h1]
+        dkv = get_shaped(src, m + "dkv", l.rank, W)
         lw.qkv_w = self._dev(torch.cat([_pad(q, n, l.dp, P).view(n * l.dp, P), _pad(dkv, l.rp, P)]))
-        lw.kv_norm = self._dev(self._get(src, m + "dkv.norm", l.rank), torch.float32)
-        uk = _pad(self._get(src, m + "uk", l.heads * l.dim, l.rank).view(l.heads, l.dim, l.rank)[h0:h1], n, l.dp, l.rp)
-        uv = _pad(self._get(src, m + "uv", l.heads * l.vdim, l.rank).view(l.heads, l.vdim, l.rank)[h0:h1], n, l.vp, l.rp)
+        lw.kv_norm = self._dev(get_shaped(src, m + "dkv.norm", l.rank), torch.float32)
+        uk = _pad(get_shaped(src, m + "uk", l.heads * l.dim, l.rank).view(l.heads, l.dim, l.rank)[h0:h1], n, l.dp, l.rp)
+        uv = _pad(get_shaped(src, m + "uv", l.heads * l.vdim, l.rank).view(l.heads, l.vdim, l.rank)[h0:h1], n, l.vp, l.rp)
         lw.w_uk_t = self._dev(uk.transpose(1, 2))                                     # [heads, rank, dim]: q -> q_lat
         lw.w_ukv = self._dev(torch.cat([uk.reshape(n * l.dp, l.rp), uv.reshape(n * l.vp, l.rp)]))  # latent -> k | v
         lw.w_uv = lw.w_ukv[n * l.dp:].view(n, l.vp, l.rp)                             # o_lat -> o
-        o = self._get(src, m + "o", W, l.heads * l.vdim).view(W, l.heads, l.vdim)[:, h0:h1]
+        o = get_shaped(src, m + "o", W, l.heads * l.vdim).view(W, l.heads, l.vdim)[:, h0:h1]
         lw.o_w = self._dev(_pad(o, P, n, l.vp).view(P, n * l.vp))
 
     def _load_moe(self, lw, src, p, l: LayerSpec):
@@ -262,9 +245,9 @@ class TaduzenLM(TransformerLM):
             s0, s1 = tp_range(l.shared_ff, r, tp)
             a, b = self._load_gated(src, p + "shared.", l.shared_ff, s0, s1)
             lw.shared_gate_up_w, lw.shared_down_w = self._dev(a), self._dev(b)
-            sg = self._get(src, p + "shared.sg", 1, self.hidden).float().view(-1)
+            sg = get_shaped(src, p + "shared.sg", 1, self.hidden).float().view(-1)
             lw.shared_gate_w = self._dev(_pad(sg, self.hidden_p), torch.float32)
-        table = self._get(src, p + "table", self.vocab, l.top).to(torch.int32)
+        table = get_shaped(src, p + "table", self.vocab, l.top).to(torch.int32)
         if int(table.min()) < 0 or int(table.max()) >= l.experts:
             raise ValueError(f"{p}table names an expert outside 0 .. {l.experts - 1}")
         return table.to(self.device).contiguous(), e0, e1 - e0

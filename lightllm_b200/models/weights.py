@@ -144,6 +144,26 @@ class RandomSource(WeightSource):
         return t
 
 
+def round_up(n: int, m: int) -> int:
+    return -(-n // m) * m
+
+
+def pad_zeros(t: torch.Tensor, *sizes: int) -> torch.Tensor:
+    """t in a tensor of `sizes`, zero beyond it (zero rows and columns add nothing to a matrix product)."""
+    if tuple(t.shape) == sizes:
+        return t
+    out = torch.zeros(sizes, dtype=t.dtype, device=t.device)
+    out[tuple(slice(0, n) for n in t.shape)] = t
+    return out
+
+
+def get_shaped(src: WeightSource, name: str, *shape: int) -> torch.Tensor:
+    """A checkpoint tensor, whose shape must be the one config.json implies."""
+    if tuple(src.shape(name)) != shape:
+        raise ValueError(f"tensor {name}: shape {tuple(src.shape(name))}, config.json says {shape}")
+    return src.get(name)
+
+
 def tp_range(total: int, tp_rank: int, tp_size: int):
     """Even split [start, end) of `total` items for a rank (total must divide)."""
     assert total % tp_size == 0, f"{total} not divisible by tp {tp_size}"

@@ -15,7 +15,8 @@ from . import kv_quant
 from . import reference as ref
 from ._native import NativeError, c_int, c_void_p, check, f32, i64, kernels, ptr, stream
 
-EPI_CODES = {"store": 0, "residual": 1, "gated_silu": 2, "f32": 3, "gated_gelu": 4, "relu2": 5, "dyt": 6}
+EPI_CODES = {"store": 0, "residual": 1, "gated_silu": 2, "f32": 3, "gated_gelu": 4, "relu2": 5, "dyt": 6,
+             "gated_clamp": 7}
 DTYPE_CODES = {torch.float32: 0, torch.bfloat16: 1}   # kernels that exist in both number formats
 
 import os as _os
@@ -221,14 +222,15 @@ def _tuned_bn(M: int, N: int, K: int, epi: str) -> int:
 
 
 def gemm(a, w, epi: str = "store", residual=None, bias=None, out=None, bn: int = 0, stream_k: int = 0,
-         out_scale: float = 1.0, x=None, dyt=None):
+         out_scale: float = 1.0, x=None, dyt=None, clamp=None):
     """C = A . W^T on the tcgen05 tensor cores.  a [M, K], w [N, K] (checkpoint layout).  fp32 operands run on the
     CUDA cores in fp32 (`csrc/gemm_f32.cu`).
 
     epi: "store" | "residual" (C += residual) | "gated_silu"/"gated_gelu" (w rows interleaved with
     `reference.interleave_gate_up`, C is [M, N/2]) | "f32" (fp32 output, e.g. logits, times `out_scale`) |
     "relu2" (square of relu) | "dyt": with the fp32 residual stream x [M, N] and dyt = (post, next) `DytNorm`s,
-    x += post(A . W^T) in place and C = next(x).
+    x += post(A . W^T) in place and C = next(x) | "gated_clamp": interleaved as the other gated forms, with
+    clamp = (alpha, limit): g = min(g, limit), u = clamp(u, -limit, limit), C = (u + 1) g sigmoid(alpha g).
     stream_k: 0 whole tiles per CTA (default: fastest on every measured shape), 1 stream-K, -1 heuristic.
     """
     if type(w).__name__ == "Fp8Weight":  # block-scaled e4m3 weight: quantise the activations, fp8 tensor cores
@@ -240,16 +242,16 @@ def gemm(a, w, epi: str = "store", residual=None, bias=None, out=None, bn: int =
 
         return int8.gemm_int8(a, w, epi, residual, bias, out)
     if not _is_cuda(a):
-        res = ref.gemm(a, w, epi, residual, bias, out_scale=out_scale, x=x, dyt=dyt)
+        res = ref.gemm(a, w, epi, residual, bias, out_scale=out_scale, x=x, dyt=dyt, clamp=clamp)
         if out is not None:
             out.copy_(res)
             return out
         return res
     if a.dtype == torch.float32:
-        return gemm_f32(a, w, epi, residual, bias, out, out_scale, x, dyt)
+        return gemm_f32(a, w, epi, residual, bias, out, out_scale, x, dyt, clamp=clamp)
     _req_bf16(a, w, residual, bias)
-    if epi == "dyt" or out_scale != 1.0:
-        return _gemm_fused(a, w, epi, bias, out, bn, out_scale, x, dyt)
+    if epi in ("dyt", "gated_clamp") or out_scale != 1.0:
+        return _gemm_fused(a, w, epi, bias, out, bn, out_scale, x, dyt, clamp)
     if _GEMM_DEBUG_TORCH:  # debugging aid only (LLB_GEMM_DEBUG_TORCH=1): bypasses the tcgen05 kernel
         res = ref.gemm(a, w, epi, residual, bias)
         if out is not None:
@@ -287,25 +289,32 @@ def _dyt_args(n):
     return (ptr(None), ptr(None), f32(1.0)) if n is None else (ptr(n.w), ptr(n.b), f32(n.alpha))
 
 
-def _gemm_fused(a, w, epi, bias, out, bn, out_scale, x, dyt):
+def _clamp_args(clamp):
+    alpha, limit = clamp if clamp is not None else (1.0, float("inf"))
+    return f32(alpha), f32(limit)
+
+
+def _gemm_fused(a, w, epi, bias, out, bn, out_scale, x, dyt, clamp=None):
     M, K = a.shape
     N = w.shape[0]
     assert w.shape[1] == K and w.stride(1) == 1 and a.stride(1) == 1
     if out is None:
-        out = torch.empty((M, N), dtype=torch.float32 if epi == "f32" else a.dtype, device=a.device)
+        out = torch.empty((M, N // 2 if epi.startswith("gated") else N),
+                          dtype=torch.float32 if epi == "f32" else a.dtype, device=a.device)
     post, nxt = dyt if dyt is not None else (None, None)
     if epi == "dyt":
         assert x.dtype == torch.float32 and x.shape == (M, N) and x.stride(0) == out.stride(0) and x.stride(1) == 1
     check(kernels().llb_gemm_bf16_fused(ptr(a), i64(a.stride(0)), ptr(w), i64(w.stride(0)), ptr(out),
                                         i64(out.stride(0)), ptr(bias), c_int(M), c_int(N), c_int(K),
                                         c_int(EPI_CODES[epi]), c_int(bn), f32(out_scale), ptr(x), *_dyt_args(post),
-                                        *_dyt_args(nxt), ptr(gemm_status(a.device)), stream()), "gemm_bf16_fused")
+                                        *_dyt_args(nxt), *_clamp_args(clamp), ptr(gemm_status(a.device)), stream()),
+          "gemm_bf16_fused")
     _count()
     return out
 
 
 def gemm_f32(a, w, epi="store", residual=None, bias=None, out=None, out_scale=1.0, x=None, dyt=None,
-             mblock_expert=None):
+             mblock_expert=None, clamp=None):
     """fp32 GEMM, same epilogues as `gemm`.  a [M, K] and w [N, K]; or a [M, batch, K] and w [batch, N, K] (per-head
     products, out [M, batch, N]); or grouped with w [E, N, K] and the expert of every 128-row block."""
     grouped = mblock_expert is not None
@@ -327,7 +336,8 @@ def gemm_f32(a, w, epi="store", residual=None, bias=None, out=None, out_scale=1.
                                  i64(w.stride(-2)), i64(w.stride(0) if batched else 0), ptr(out), i64(out.stride(0)),
                                  i64(out.stride(1) if batched else 0), ptr(residual), ptr(bias), ptr(x),
                                  *_dyt_args(post), *_dyt_args(nxt), ptr(mblock_expert), c_int(M), c_int(N), c_int(K),
-                                 c_int(batch), c_int(EPI_CODES[epi]), f32(out_scale), stream()), "gemm_f32")
+                                 c_int(batch), c_int(EPI_CODES[epi]), f32(out_scale), *_clamp_args(clamp), stream()),
+          "gemm_f32")
     _count()
     return out
 
@@ -664,3 +674,90 @@ def add_dyt_(x, y, post: DytNorm, nxt: DytNorm, dtype):
           "add_dyt")
     _count()
     return h
+
+
+# --------------------------------------------------------------------------------------
+class BigramTable:
+    """Second embedding table, looked up by the pair (previous token, token): row (prev * mul_prev + token * mul_cur) mod
+    buckets of `table` [buckets + 1, W], the last row for a sequence's first token.  `slot_token` (int32, one entry per
+    pool slot) keeps the token id behind every cached position, so the previous token of a later pass is found through the
+    request table like its keys."""
+
+    def __init__(self, table: torch.Tensor, buckets: int, mul_prev: int, mul_cur: int):
+        assert table.shape[0] == buckets + 1
+        self.table, self.buckets, self.mul_prev, self.mul_cur = table, int(buckets), int(mul_prev), int(mul_cur)
+        self.slot_token = None
+
+
+def embedding_pair(ids, table, bigram, req_to_token, b_req_idx, pos, batch_of, mem_index):
+    """(x, h): x = the table's rows (+ the bigram table's) as the fp32 residual stream, h = x in the table's format.
+    batch_of None: row t is the one token of request t."""
+    if not _is_cuda(table):
+        x = table[ids].float()
+        if bigram is not None:
+            x = x + ref.bigram_rows(ids, bigram, req_to_token, b_req_idx, pos, batch_of, mem_index).float()
+        return x, x.to(table.dtype)
+    T, W = ids.shape[0], table.shape[1]
+    x = torch.empty((T, W), dtype=torch.float32, device=table.device)
+    h = torch.empty((T, W), dtype=table.dtype, device=table.device)
+    assert ids.dtype == torch.int64 and ids.is_contiguous() and table.is_contiguous()
+    g = bigram
+    check(kernels().llb_embedding_pair(ptr(ids), ptr(table), c_int(DTYPE_CODES[table.dtype]), i64(table.shape[0]),
+                                       ptr(g.table if g else None), i64(g.buckets if g else 1),
+                                       i64(g.mul_prev if g else 0), i64(g.mul_cur if g else 0),
+                                       ptr(g.slot_token if g else None), ptr(mem_index), ptr(pos), ptr(batch_of),
+                                       ptr(b_req_idx), ptr(req_to_token), i64(req_to_token.stride(0)), ptr(x), ptr(h),
+                                       c_int(T), c_int(W), stream()), "embedding_pair")
+    _count()
+    return x, h
+
+
+def add_rms_(x, y, w, width: int, eps: float, dtype, next_w=None):
+    """x += rms(y) * w in place (fp32 stream, the mean taken over the first `width` columns); returns x, or
+    rms(x) * next_w, in `dtype`."""
+    if not _is_cuda(x):
+        return ref.add_rms_(x, y, w, width, eps, dtype, next_w)
+    assert x.dtype == torch.float32 and x.is_contiguous() and y.is_contiguous() and x.shape == y.shape
+    h = torch.empty(x.shape, dtype=dtype, device=x.device)
+    check(kernels().llb_add_rms(ptr(y), c_int(DTYPE_CODES[y.dtype]), ptr(x), ptr(h), c_int(DTYPE_CODES[dtype]), ptr(w),
+                                ptr(next_w), c_int(x.shape[0]), c_int(width), c_int(x.shape[1]), f32(eps), stream()),
+          "add_rms")
+    _count()
+    return h
+
+
+def qk_norm_rope_scatter_(qkv, kv_layer, cos, sin, pos, slot, q_w, k_w, eps, Hq, Hkv, D, dim, DV, rot_dim):
+    """Rows [Hq * D | Hkv * D | Hkv * DV] of qkv: RMS norm of every q and k head over its first `dim` elements (weights
+    q_w, k_w fp32 [D]), rotation of the first rot_dim, q in place, K and V to kv_layer[slot] ([slots, Hkv * (D + DV)])."""
+    if not _is_cuda(qkv):
+        return ref.qk_norm_rope_scatter_(qkv, kv_layer, cos, sin, pos, slot, q_w, k_w, eps, Hq, Hkv, D, dim, DV, rot_dim)
+    assert qkv.stride(1) == 1 and kv_layer.is_contiguous() and qkv.dtype == kv_layer.dtype
+    check(kernels().llb_qk_norm_rope_scatter(ptr(qkv), c_int(DTYPE_CODES[qkv.dtype]), i64(qkv.stride(0)), ptr(kv_layer),
+                                             ptr(cos), ptr(sin), ptr(pos), ptr(slot), ptr(q_w), ptr(k_w), f32(eps),
+                                             c_int(qkv.shape[0]), c_int(Hq), c_int(Hkv), c_int(D), c_int(dim), c_int(DV),
+                                             c_int(rot_dim), stream()), "qk_norm_rope_scatter")
+    _count()
+    return qkv
+
+
+def window_attention(q, kv_layer, req_to_token, st, Hq, Hkv, D, DV, sm_scale, window, gate=None, out_scale=1.0, out=None):
+    """Causal paged attention with key size D and value size DV through a sliding window (0: none) for the pass `st`
+    (InferState).  q [T, >= Hq * D]; gate [T, Hq] (or None): head h is multiplied by sigmoid(gate[:, h]); all heads by
+    out_scale.  Returns out [T, Hq * DV]."""
+    T = q.shape[0]
+    if out is None:
+        out = torch.empty((T, Hq * DV), dtype=q.dtype, device=q.device)
+    if not _is_cuda(q):
+        return ref.window_attention(q, kv_layer, req_to_token, st.b_req_idx, st.seq_pos,
+                                    st.batch_of_token if st.is_prefill else None, Hq, Hkv, D, DV, sm_scale, window, gate,
+                                    out_scale, out)
+    assert q.stride(1) == 1 and kv_layer.is_contiguous() and out.stride(1) == 1
+    gs = 0 if gate is None else gate.stride(0)
+    check(kernels().llb_attn_generic_kv(ptr(q), c_int(DTYPE_CODES[q.dtype]), i64(q.stride(0)), ptr(kv_layer),
+                                        ptr(req_to_token), i64(req_to_token.stride(0)), ptr(st.b_req_idx),
+                                        ptr(st.seq_pos), ptr(st.batch_of_token if st.is_prefill else None), ptr(out),
+                                        i64(out.stride(0)), c_int(T), c_int(Hq), c_int(Hkv), c_int(D), c_int(DV),
+                                        f32(sm_scale), c_int(window), ptr(gate), i64(gs), f32(out_scale), stream()),
+          "attn_generic_kv")
+    _count()
+    return out

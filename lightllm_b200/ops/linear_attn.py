@@ -1,4 +1,6 @@
-"""Gated DeltaNet linear attention (Qwen3-Next / Qwen3.5 hybrid layers) on torch ops.
+"""Linear attention with matrix states.  First the Gated DeltaNet (Qwen3-Next / Qwen3.5 hybrid layers) on torch ops, with
+its decode kernels; at the end of the file `DecayedState`: gated linear attention with a decay per key channel, and the
+matrix memory of xLSTM (mLSTM), on the kernels of `csrc/recurrent.cu`.
 
 Per head the layer keeps a matrix state S [dk, dv] and updates it token by token:
 
@@ -146,3 +148,138 @@ def rmsnorm_gated(x: torch.Tensor, z: torch.Tensor, w: torch.Tensor, eps: float)
     xf = x.float()
     y = xf * torch.rsqrt(xf.pow(2).mean(-1, keepdim=True) + eps)
     return (w.float() * y * F.silu(z.float())).to(z.dtype)
+
+
+# ---------------------------------------------------------------- states with decays (GLA, mLSTM)
+CHUNK = 64
+
+
+class ChunkPlan:
+    """The 64-token chunks of a prompt pass: first token row and length of every chunk, chunks of every request."""
+
+    def __init__(self, q_len: torch.Tensor, device):
+        q_len = q_len.to(torch.int64)
+        n = (q_len + CHUNK - 1) // CHUNK
+        zero = torch.zeros(1, dtype=torch.int64)
+        cu_q, cu_c = torch.cat([zero, q_len.cumsum(0)]), torch.cat([zero, n.cumsum(0)])
+        self.count = int(cu_c[-1])
+        b = torch.repeat_interleave(torch.arange(len(q_len)), n)
+        off = (torch.arange(self.count) - cu_c[b]) * CHUNK
+        tok0, length = cu_q[b] + off, (q_len[b] - off).clamp_max(CHUNK)
+        host = torch.cat([tok0, length, cu_c]).to(torch.int32)
+        dev = host.to(device, non_blocking=True)
+        self.tok0, self.len, self.cu_chunk = torch.split(dev, [self.count, self.count, len(q_len) + 1])
+
+
+class DecayedState:
+    """One layer's recurrence S_t = diag(a_t) S_(t-1) + b_t k_t v_t^T, o_t = dim^(-1/2) S_t^T q_t over per-request states,
+    with its output step: RMS norm of every head over its values, times a weight, times silu(g) or sigmoid(g).
+
+    kind "gla":    a = sigmoid(z)^(1 / tau) per key channel, z = a2 (a1 h) + bias; b = 1; silu(g).
+    kind "mlstm":  log gates i = cap tanh(zi / cap), f = logsigmoid(cap tanh(zf / cap)) per head, a running maximum m (0 at
+                   the start) that keeps the exponentials in range, a normaliser n; sigmoid(g).
+
+    dk, dv: padded head sizes (multiples of 16), dim, vdim: the true ones.  weight: fp32 [dv] or [H * dv]."""
+
+    def __init__(self, kind: str, H: int, dk: int, dv: int, dim: int, vdim: int, eps: float, weight: torch.Tensor,
+                 tau: float = 1.0, a2=None, a2_bias=None, cap: float = 1.0, out_scale: float = 1.0):
+        assert kind in ("gla", "mlstm") and dk % 16 == 0 and dv % 16 == 0
+        self.kind, self.H, self.dk, self.dv, self.dim, self.vdim = kind, H, dk, dv, dim, vdim
+        self.eps, self.tau, self.cap, self.out_scale = float(eps), float(tau), float(cap), float(out_scale)
+        self.weight, self.a2, self.a2_bias = weight, a2, a2_bias
+        assert weight.dtype == torch.float32 and weight.numel() in (dv, H * dv)
+        self.w_stride = 0 if weight.numel() == dv else dv
+        self.rank = 0 if a2 is None else a2.shape[1]
+
+    @staticmethod
+    def state_elems(kind: str, H: int, dk: int, dv: int) -> int:
+        return H * dk * dv + (H * (dk + 1) if kind == "mlstm" else 0)
+
+    @staticmethod
+    def chunked_sizes(dk: int, dv: int, rank: int) -> bool:
+        return dk <= 256 and dv <= 512 and rank <= 128
+
+    def __call__(self, q, k, v, g, state, st, a1=None, zi=None, zf=None, out=None, plan=None, token_by_token=False):
+        """q, k [T, H * dk], v, g [T, H * dv] (columns of one matrix, or with its row pitch); a1 [T, rank] likewise; zi, zf
+        fp32 [T, H] with one row pitch; state [slots, elems].  Prompt passes in bf16 run chunked (`plan`), everything else
+        token by token."""
+        T = q.shape[0]
+        if out is None:
+            out = torch.empty((T, self.H * self.dv), dtype=q.dtype, device=q.device)
+        first = st.b_ready_cache_len if st.is_prefill else st.seq_pos
+        if not q.is_cuda:
+            return self._torch(q, k, v, g, state, st, a1, zi, zf, out)
+        from . import DTYPE_CODES, _count
+        from ._native import c_int, check, f32, i64, kernels, ptr, stream
+
+        ld = q.stride(0)
+        assert all(t.stride(0) == ld and t.stride(1) == 1 for t in (q, k, v, g)) and state.stride(1) == 1
+        assert a1 is None or a1.stride(0) == ld
+        ldz = 0 if zi is None else zi.stride(0)
+        kind = 0 if self.kind == "gla" else 1
+        common = (ptr(q), ptr(k), ptr(v), ptr(g), i64(ld), ptr(a1), ptr(self.a2), ptr(self.a2_bias), c_int(self.rank),
+                  f32(1.0 / self.tau), ptr(zi), ptr(zf), i64(ldz), f32(self.cap), ptr(state), i64(state.stride(0)),
+                  ptr(self.weight), c_int(self.w_stride), f32(self.eps), ptr(out), i64(out.stride(0)), f32(self.out_scale),
+                  ptr(st.b_req_idx))
+        sizes = (c_int(st.batch_size), c_int(self.H), c_int(self.dk), c_int(self.dv), c_int(self.dim), c_int(self.vdim),
+                 stream())
+        chunked = st.is_prefill and q.dtype == torch.bfloat16 and not token_by_token and \
+            self.chunked_sizes(self.dk, self.dv, self.rank)
+        if not chunked:
+            check(kernels().llb_recurrent_scan(c_int(kind), c_int(DTYPE_CODES[q.dtype]), *common,
+                                               ptr(st.cu_q if st.is_prefill else None), ptr(first), *sizes),
+                  "recurrent_scan")
+            _count()
+            return out
+        n, dev = plan.count, q.device
+        decay = torch.empty(T * self.H * (self.dk if kind == 0 else 3), dtype=torch.float32, device=dev)
+        m_prev = n_prev = None
+        if kind == 1:
+            m_prev = torch.empty(n * self.H, dtype=torch.float32, device=dev)
+            n_prev = torch.empty(n * self.H * self.dk, dtype=torch.float32, device=dev)
+        planes = torch.empty((2, n * self.H * self.dk * self.dv), dtype=torch.bfloat16, device=dev)
+        check(kernels().llb_recurrent_chunks(c_int(kind), *common, ptr(first), ptr(plan.tok0), ptr(plan.len),
+                                             ptr(plan.cu_chunk), ptr(decay), ptr(m_prev), ptr(n_prev), ptr(planes[0]),
+                                             ptr(planes[1]), c_int(T), c_int(n), *sizes), "recurrent_chunks")
+        _count(3)
+        return out
+
+    def _torch(self, q, k, v, g, state, st, a1, zi, zf, out):
+        """Token by token on torch ops (CPU tensors)."""
+        H, dk, dv = self.H, self.dk, self.dv
+        T = q.shape[0]
+        qf, kf = q.float().view(T, H, dk) * self.dim ** -0.5, k.float().view(T, H, dk)
+        vf, gf = v.float().view(T, H, dv), g.float().view(T, H, dv)
+        if self.kind == "gla":
+            z = a1.float() @ self.a2.float().t() + self.a2_bias
+            decay = torch.exp(F.logsigmoid(z) / self.tau).view(T, H, dk)
+        else:
+            li = self.cap * torch.tanh(zi / self.cap)
+            lf = F.logsigmoid(self.cap * torch.tanh(zf / self.cap))
+        ends = st.cu_q.tolist() if st.is_prefill else list(range(T + 1))
+        first = (st.b_ready_cache_len if st.is_prefill else st.seq_pos).tolist()
+        weight = self.weight.view(-1, dv)
+        o = torch.empty(T, H, dv)
+        for b, r in enumerate(st.b_req_idx.tolist()):
+            row = state[r]
+            if first[b] == 0:
+                row.zero_()
+            S = row[: H * dk * dv].view(H, dk, dv)
+            n, m = (row[H * dk * dv: H * dk * (dv + 1)].view(H, dk), row[H * dk * (dv + 1):]) \
+                if self.kind == "mlstm" else (None, None)
+            for t in range(ends[b], ends[b + 1]):
+                if self.kind == "gla":
+                    S.mul_(decay[t].unsqueeze(-1)).add_(kf[t].unsqueeze(-1) * vf[t].unsqueeze(1))
+                    o[t] = torch.einsum("hdv,hd->hv", S, qf[t])
+                    continue
+                m1 = torch.maximum(lf[t] + m, li[t])
+                a, kb = torch.exp(lf[t] + m - m1)[:, None], torch.exp(li[t] - m1)[:, None] * kf[t]
+                S.mul_(a.unsqueeze(-1)).add_(kb.unsqueeze(-1) * vf[t].unsqueeze(1))
+                n.mul_(a).add_(kb)
+                m.copy_(m1)
+                den = torch.maximum((n * qf[t]).sum(-1).abs(), torch.exp(-m)) + 1e-6
+                o[t] = torch.einsum("hdv,hd->hv", S, qf[t]) / den[:, None]
+        o = o * torch.rsqrt(o.square().sum(-1, keepdim=True) / self.vdim + self.eps) * weight * self.out_scale
+        gate = torch.sigmoid(gf) * (gf if self.kind == "gla" else 1.0)
+        out.copy_((o * gate).view(T, H * dv))
+        return out

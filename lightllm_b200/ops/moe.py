@@ -8,7 +8,7 @@ from typing import Optional
 
 import torch
 
-from . import DTYPE_CODES, _count, _dyt_args, gemm_f32, gemm_status
+from . import DTYPE_CODES, _clamp_args, _count, _dyt_args, gemm_f32, gemm_status
 from . import reference as ref
 from ._native import c_int, check, f32, i64, kernels, ptr, stream
 
@@ -40,15 +40,11 @@ def ref_grouped_topk(logits, bias, k, n_group, topk_group, use_sigmoid=True, ren
     return ids.to(torch.int32), (w * scale).float()
 
 
-def _swiglu_oai(h, alpha=1.702, limit=7.0):
-    """h [.., 2I] with gate / up interleaved in 32-column blocks (GPT-OSS clamped SwiGLU)."""
-    n = h.shape[-1] // 64
-    hv = h.reshape(*h.shape[:-1], n, 2, 32)
-    g, u = hv[..., 0, :].clamp(max=limit), hv[..., 1, :].clamp(min=-limit, max=limit)
-    return ((u + 1) * g * torch.sigmoid(alpha * g)).reshape(*h.shape[:-1], n * 32)
+SWIGLU_OAI = (1.702, 7.0)    # (alpha, limit) of the clamped gate of GPT-OSS
 
 
-def ref_fused_experts(x, w13, w2, ids, weights, act="silu", e0=0, interleaved=True, b13=None, b2=None):
+def ref_fused_experts(x, w13, w2, ids, weights, act="silu", e0=0, interleaved=True, b13=None, b2=None,
+                      clamp=SWIGLU_OAI):
     """x [T,H]; w13 [E_local, 2I, H] (gate/up interleaved in 32-row blocks when `interleaved`), w2 [E_local, H, I];
     experts outside [e0, e0+E_local) contribute nothing (expert parallel shard)."""
     T, H = x.shape
@@ -64,7 +60,7 @@ def ref_fused_experts(x, w13, w2, ids, weights, act="silu", e0=0, interleaved=Tr
         if b13 is not None:
             h = h.to(x.dtype).float() + b13[e].float()
         if act == "swiglu_oai":
-            a = _swiglu_oai(h)
+            a = ref.gated_clamp_interleaved(h, *clamp)
         elif interleaved:
             a = ref.gated_act_interleaved(h, act).float()
         else:
@@ -158,7 +154,8 @@ def count_remap(ids, table, counter=None):
     return out
 
 
-def gemm_grouped(a_sorted, w_stacked, mblock_expert, n_per_expert: int, epi: str = "store", out=None, bn: int = 0):
+def gemm_grouped(a_sorted, w_stacked, mblock_expert, n_per_expert: int, epi: str = "store", out=None, bn: int = 0,
+                 clamp=None):
     """a_sorted [M_pad, K] bf16, w_stacked [E, N, K] bf16 -> [M_pad, N] (or [M_pad, N/2] gated)."""
     from . import EPI_CODES
 
@@ -166,14 +163,14 @@ def gemm_grouped(a_sorted, w_stacked, mblock_expert, n_per_expert: int, epi: str
     E, N = w_stacked.shape[0], w_stacked.shape[1]
     assert N == n_per_expert and w_stacked.is_contiguous()
     if a_sorted.dtype == torch.float32:
-        return gemm_f32(a_sorted, w_stacked, epi, out=out, mblock_expert=mblock_expert)
+        return gemm_f32(a_sorted, w_stacked, epi, out=out, mblock_expert=mblock_expert, clamp=clamp)
     n_out = N // 2 if epi.startswith("gated") else N
     if out is None:
         out = torch.empty((M_pad, n_out), dtype=a_sorted.dtype, device=a_sorted.device)
     check(kernels().llb_gemm_bf16_grouped(ptr(a_sorted), i64(a_sorted.stride(0)), ptr(w_stacked), i64(K), ptr(out),
                                           i64(out.stride(0)), ptr(mblock_expert), c_int(M_pad), c_int(N), c_int(K),
-                                          c_int(E), c_int(EPI_CODES[epi]), c_int(bn), ptr(gemm_status(a_sorted.device)),
-                                          stream()), "gemm_grouped")
+                                          c_int(E), c_int(EPI_CODES[epi]), c_int(bn), *_clamp_args(clamp),
+                                          ptr(gemm_status(a_sorted.device)), stream()), "gemm_grouped")
     _count()
     return out
 
@@ -191,7 +188,7 @@ def gather_rows(x, lay: MoeLayout):
 
 
 def fused_experts(x, w13, w2, ids, weights, act="silu", e0: int = 0, out=None, accumulate: bool = False,
-                  b13=None, b2=None):
+                  b13=None, b2=None, clamp=SWIGLU_OAI):
     """Routed expert FFN:  out[t] (+)= sum_k w[t,k] * down_e( act(gate_e(x_t)) * up_e(x_t) ),  e = ids[t,k].
 
     w13 [E_local, 2I, H] with gate/up rows interleaved in 32-row blocks, w2 [E_local, H, I].  On CUDA: align
@@ -200,7 +197,7 @@ def fused_experts(x, w13, w2, ids, weights, act="silu", e0: int = 0, out=None, a
     if not x.is_cuda:
         if fp8_w:  # CPU: same arithmetic with the de-quantised weights
             w13, w2 = w13.dequant().to(x.dtype), w2.dequant().to(x.dtype)
-        r = ref_fused_experts(x, w13, w2, ids, weights, act, e0, b13=b13, b2=b2)
+        r = ref_fused_experts(x, w13, w2, ids, weights, act, e0, b13=b13, b2=b2, clamp=clamp)
         if out is not None:
             if accumulate:
                 out.add_(r)
@@ -227,12 +224,14 @@ def fused_experts(x, w13, w2, ids, weights, act="silu", e0: int = 0, out=None, a
         y = fp8.gemm_fp8_quantized(hq, hsc, w2.w, "store", mblock_expert=lay.mblock_expert, n_per_expert=H)
     elif b13 is None and act in ("silu", "gelu"):
         h = gemm_grouped(a, w13, lay.mblock_expert, N13, epi="gated_" + act)
-    else:  # biased experts / clamped SwiGLU: plain grouped GEMM, then bias + activation in one pass
+    elif b13 is None and act == "swiglu_oai":
+        h = gemm_grouped(a, w13, lay.mblock_expert, N13, epi="gated_clamp", clamp=clamp)
+    else:  # biased experts: plain grouped GEMM, then bias + activation in one pass
         h13 = gemm_grouped(a, w13, lay.mblock_expert, N13, epi="store")
         h = torch.empty((lay.m_pad, I), dtype=x.dtype, device=x.device)
         kind = {"silu": 0, "gelu": 1, "swiglu_oai": 2}[act]
         check(kernels().llb_moe_bias_act(ptr(h13), ptr(b13), ptr(lay.mblock_expert), ptr(h), c_int(lay.m_pad), c_int(I),
-                                         c_int(kind), f32(1.702), f32(7.0), stream()), "moe_bias_act")
+                                         c_int(kind), f32(clamp[0]), f32(clamp[1]), stream()), "moe_bias_act")
         _count()
     if not fp8_w:
         y = gemm_grouped(h, w2, lay.mblock_expert, H, epi="store")
@@ -322,5 +321,30 @@ def uniform_experts_dyt_(h, lay, w13, w2, act, shared, gate_w, x, post, nxt, e0:
                                         f32(1.0 / lay.k), ptr(shared), ptr(h), ptr(gate_w), ptr(x),
                                         ptr(None if x is None else out), ptr(out if x is None else None), c_int(T),
                                         c_int(H), *_dyt_args(post), *_dyt_args(nxt), stream()), "moe_combine_dyt")
+    _count()
+    return out
+
+
+def routed_experts_rms_(h, ids, weights, w13, w2, clamp, shared, x, w, width, eps, next_w=None, e0: int = 0):
+    """Routed experts with the clamped gate plus a shared expert's output `shared` [T, H] (or None), inside an output norm:
+    x += rms(sum) * w in place, returns x (or rms(x) * next_w) in h's format (`ops.add_rms_`).  x None: returns the fp32 sum
+    instead (a tensor-parallel reduction follows)."""
+    from . import add_rms_
+
+    if not h.is_cuda:
+        y = ref_fused_experts(h, w13, w2, ids, weights, "swiglu_oai", e0, clamp=clamp).float()
+        if shared is not None:
+            y = y + shared.float()
+        return y if x is None else add_rms_(x, y, w, width, eps, h.dtype, next_w)
+    T, H = h.shape
+    lay = moe_align(ids, w13.shape[0], e0)
+    a = gather_rows(h, lay)
+    g = gemm_grouped(a, w13, lay.mblock_expert, w13.shape[1], epi="gated_clamp", clamp=clamp)
+    y = gemm_grouped(g, w2, lay.mblock_expert, H)
+    out = torch.empty((T, H), dtype=torch.float32 if x is None else h.dtype, device=h.device)
+    check(kernels().llb_moe_combine_rms(ptr(y), c_int(DTYPE_CODES[h.dtype]), ptr(lay.pair_row), ptr(weights), c_int(lay.k),
+                                        ptr(shared), ptr(x), ptr(None if x is None else out), c_int(DTYPE_CODES[h.dtype]),
+                                        ptr(out if x is None else None), ptr(w), ptr(next_w), c_int(T), c_int(width),
+                                        c_int(H), f32(eps), stream()), "moe_combine_rms")
     _count()
     return out

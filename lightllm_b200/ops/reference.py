@@ -49,6 +49,13 @@ def interleave_gate_up(w_gate, w_up, block=GATE_UP_BLOCK):
     return torch.cat([g, u], dim=-3).reshape(*lead, 2 * I, K).contiguous()
 
 
+def gated_clamp_interleaved(y, alpha, limit, block=GATE_UP_BLOCK):
+    """Clamped gate of y [.., 2I] with interleaved columns: (clamp(u) + 1) g sigmoid(alpha g), g = min(g, limit)."""
+    v = y.float().reshape(*y.shape[:-1], -1, 2, block)
+    g, u = v[..., 0, :].clamp(max=limit), v[..., 1, :].clamp(-limit, limit)
+    return ((u + 1) * g * torch.sigmoid(alpha * g)).reshape(*y.shape[:-1], y.shape[-1] // 2).to(y.dtype)
+
+
 def gated_act_interleaved(y, act="silu", block=GATE_UP_BLOCK):
     """y [T, 2I] produced with interleaved weights -> [T, I]."""
     T, N = y.shape
@@ -61,7 +68,8 @@ def dyt(x, norm):
     return torch.tanh(norm.alpha * x) * norm.w + norm.b
 
 
-def gemm(a, w, epi="store", residual=None, bias=None, out_dtype=None, out_scale=1.0, x=None, dyt=None):
+def gemm(a, w, epi="store", residual=None, bias=None, out_dtype=None, out_scale=1.0, x=None, dyt=None,
+         clamp=None):
     """C = A . W^T with the epilogues of the tcgen05 GEMM. `w` is [N, K]."""
     acc = a.float() @ w.float().t()
     if bias is not None:
@@ -78,6 +86,8 @@ def gemm(a, w, epi="store", residual=None, bias=None, out_dtype=None, out_scale=
         post, nxt = dyt
         x.add_(torch.tanh(post.alpha * acc) * post.w + post.b)
         return (torch.tanh(nxt.alpha * x) * nxt.w + nxt.b).to(out_dtype or a.dtype)
+    if epi == "gated_clamp":
+        return gated_clamp_interleaved(acc, *clamp).to(out_dtype or a.dtype)
     if epi in ("gated_silu", "gated_gelu"):
         return gated_act_interleaved(acc, "silu" if epi == "gated_silu" else "gelu").to(out_dtype or a.dtype)
     raise ValueError(epi)
@@ -397,4 +407,63 @@ def attention_generic(q, kv_layer, req_to_token, b_req_idx, pos, batch_of, Hq, H
         else:
             pr = torch.softmax(s, dim=-1)
         out[t] = torch.einsum("hl,lhd->hd", pr, v).to(q.dtype)
+    return out
+
+
+def bigram_rows(ids, bigram, req_to_token, b_req_idx, pos, batch_of, mem_index):
+    """Rows of a `BigramTable` for the tokens of a pass; records the pass's tokens in `bigram.slot_token`."""
+    T = ids.shape[0]
+    b = batch_of.long() if batch_of is not None else torch.arange(T, device=ids.device)
+    p = pos.long()
+    cached = bigram.slot_token[req_to_token[b_req_idx.long()[b], (p - 1).clamp_min(0)].long()].long()
+    before = torch.cat([ids[:1], ids[:-1]])
+    inside = torch.cat([torch.zeros(1, dtype=torch.bool, device=ids.device), b[1:] == b[:-1]])
+    prev = torch.where(inside, before, cached)
+    rows = (prev * bigram.mul_prev + ids * bigram.mul_cur) % bigram.buckets
+    rows = torch.where(p == 0, torch.full_like(rows, bigram.buckets), rows)
+    bigram.slot_token[mem_index.long()] = ids.to(torch.int32)
+    return bigram.table[rows]
+
+
+def _rms_over(v, width, eps):
+    return v * torch.rsqrt(v.square().sum(-1, keepdim=True) / width + eps)
+
+
+def add_rms_(x, y, w, width, eps, dtype, next_w=None):
+    x.add_(_rms_over(y.float(), width, eps) * w)
+    return (x if next_w is None else _rms_over(x, width, eps) * next_w).to(dtype)
+
+
+def qk_norm_rope_scatter_(qkv, kv_layer, cos, sin, pos, slot, q_w, k_w, eps, Hq, Hkv, D, dim, DV, rot_dim):
+    T, half = qkv.shape[0], rot_dim // 2
+    nq, nk = Hq * D, Hkv * D
+    c, s = cos[pos.long()].unsqueeze(1), sin[pos.long()].unsqueeze(1)
+
+    def turn(x, w):
+        x = _rms_over(x.float(), dim, eps) * w
+        u, v = x[..., :half], x[..., half:2 * half]
+        return torch.cat([u * c - v * s, v * c + u * s, x[..., 2 * half:]], -1).reshape(T, -1).to(qkv.dtype)
+
+    q = turn(qkv[:, :nq].reshape(T, Hq, D), q_w)
+    kv_layer[slot.long(), :nk] = turn(qkv[:, nq:nq + nk].reshape(T, Hkv, D), k_w)
+    kv_layer[slot.long(), nk:] = qkv[:, nq + nk:nq + nk + Hkv * DV]
+    qkv[:, :nq] = q
+    return qkv
+
+
+def window_attention(q, kv_layer, req_to_token, b_req_idx, pos, batch_of, Hq, Hkv, D, DV, sm_scale, window, gate, out_scale,
+                     out):
+    G = Hq // Hkv
+    for t in range(q.shape[0]):
+        b = int(batch_of[t]) if batch_of is not None else t
+        p = int(pos[t])
+        j0 = max(0, p - window + 1) if window > 0 else 0
+        rows = kv_layer[req_to_token[int(b_req_idx[b]), j0:p + 1].long()].float()
+        k = rows[:, : Hkv * D].view(-1, Hkv, D).repeat_interleave(G, dim=1)
+        v = rows[:, Hkv * D:].reshape(-1, Hkv, DV).repeat_interleave(G, dim=1)
+        pr = torch.softmax(torch.einsum("hd,lhd->hl", q[t, : Hq * D].view(Hq, D).float(), k) * sm_scale, dim=-1)
+        o = torch.einsum("hl,lhd->hd", pr, v) * out_scale
+        if gate is not None:
+            o = o * torch.sigmoid(gate[t].float())[:, None]
+        out[t] = o.reshape(-1).to(out.dtype)
     return out

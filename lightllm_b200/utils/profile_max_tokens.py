@@ -62,6 +62,8 @@ def kv_bytes_per_token(cfg: dict, tp: int, kv_elem_bytes: int = 2) -> int:
         L = sum(1 for t in c["layer_types"][:L] if t != "linear_attention")
     elif c.get("full_attention_interval") and c.get("linear_num_key_heads"):
         L = L // int(c["full_attention_interval"])
+    if c.get("kv_elems_per_token"):  # layers with rows of different sizes: stated by the family's configuration
+        return int(c["kv_elems_per_token"]) * kv_elem_bytes // max(tp, 1)
     if c.get("kv_lora_rank"):  # MLA: one latent row per token and layer, replicated on every rank
         return L * (int(c["kv_lora_rank"]) + int(c.get("qk_rope_head_dim", 64))) * kv_elem_bytes
     hq = int(c.get("num_attention_heads") or c.get("n_head"))
