@@ -37,18 +37,29 @@ constexpr float kLn2 = 0.6931471805599453f;
 // ---------------------------------------------------------------------------------------
 // decode
 // ---------------------------------------------------------------------------------------
-template <int D, int STAGES>
+// DK, DV: key and value size; pool row [Hkv * DK | Hkv * DV].  window: only the last `window` positions are seen (0: all).
+// SPLIT_P: the weights enter P . V as the sum of two bf16 values (high and low part).  gate (or null): head h of request b
+// is multiplied by out_scale * sigmoid(gate[b, h]) when the result is final.
+struct HeadGate {
+  const bf16* gate;
+  int64_t stride;
+  float scale;
+  __device__ __forceinline__ float factor(int b, int h) const {
+    return gate == nullptr ? scale : scale / (1.f + __expf(-__bfloat162float(gate[b * stride + h])));
+  }
+};
+
+template <int DK, int DV, int STAGES, bool SPLIT_P>
 __global__ void __launch_bounds__(128)
 gqa_decode_kernel(const bf16* __restrict__ q, int64_t q_stride, const bf16* __restrict__ kv_layer,
                   const int* __restrict__ req_to_token, int64_t r2t_stride, const int* __restrict__ b_req_idx,
                   const int* __restrict__ b_seq_len, bf16* __restrict__ out, int64_t out_stride,
                   float* __restrict__ part_o, float* __restrict__ part_lse, int Hq, int Hkv, int num_splits,
-                  float scale_log2) {
+                  float scale_log2, int window, const HeadGate gate) {
   pdl_wait();
-  constexpr int CH = D / 8;            // 16-byte chunks per row
-  constexpr int ROW_BYTES = D * 2;
-  constexpr int TILE_BYTES = 16 * ROW_BYTES;           // 16 tokens
-  constexpr int STAGE_BYTES = 2 * TILE_BYTES;          // K + V
+  constexpr int CH = DK / 8, CHV = DV / 8;             // 16-byte chunks per row
+  constexpr int TILE_BYTES = 16 * DK * 2;              // 16 tokens' keys
+  constexpr int STAGE_BYTES = TILE_BYTES + 16 * DV * 2;  // K + V
   constexpr int WARP_BYTES = STAGES * STAGE_BYTES;
   extern __shared__ __align__(128) uint8_t smem[];
   uint8_t* q_smem = smem;                                // 16 x D bf16
@@ -67,9 +78,10 @@ gqa_decode_kernel(const bf16* __restrict__ q, int64_t q_stride, const bf16* __re
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int g = lane >> 2, tig = lane & 3;
 
-  const int tiles_total = (L + 15) >> 4;
+  const int lo = window > 0 ? max(0, L - window) : 0;
+  const int tiles_total = (L - lo + 15) >> 4;
   const int tiles_per_split = (tiles_total + num_splits - 1) / num_splits;
-  const int s0 = split * tiles_per_split * 16;
+  const int s0 = lo + split * tiles_per_split * 16;
   const int e0 = min(L, s0 + tiles_per_split * 16);
 
   if (s0 >= e0) {  // empty split: tell the merge kernel to ignore it
@@ -77,8 +89,8 @@ gqa_decode_kernel(const bf16* __restrict__ q, int64_t q_stride, const bf16* __re
       for (int r = threadIdx.x; r < nrows; r += blockDim.x)
         part_lse[((int64_t)b * Hq + head0 + r) * num_splits + split] = -INFINITY;
     } else {
-      for (int i = threadIdx.x; i < nrows * D; i += blockDim.x)
-        out[(int64_t)b * out_stride + (int64_t)(head0 + i / D) * D + (i % D)] = __float2bfloat16(0.f);
+      for (int i = threadIdx.x; i < nrows * DV; i += blockDim.x)
+        out[(int64_t)b * out_stride + (int64_t)(head0 + i / DV) * DV + (i % DV)] = __float2bfloat16(0.f);
     }
     return;
   }
@@ -87,17 +99,17 @@ gqa_decode_kernel(const bf16* __restrict__ q, int64_t q_stride, const bf16* __re
   for (int c = threadIdx.x; c < 16 * CH; c += blockDim.x) {
     int r = c / CH, ch = c % CH;
     uint4 v = make_uint4(0, 0, 0, 0);
-    if (r < nrows) v = *reinterpret_cast<const uint4*>(q + (int64_t)b * q_stride + (int64_t)(head0 + r) * D + ch * 8);
-    *reinterpret_cast<uint4*>(q_smem + swz<D>(r, ch)) = v;
+    if (r < nrows) v = *reinterpret_cast<const uint4*>(q + (int64_t)b * q_stride + (int64_t)(head0 + r) * DK + ch * 8);
+    *reinterpret_cast<uint4*>(q_smem + swz<DK>(r, ch)) = v;
   }
   __syncthreads();
-  uint32_t qa[D / 16][4];
+  uint32_t qa[DK / 16][4];
   {
     const uint32_t qb = smem_u32(q_smem);
     const int row = (lane & 7) + ((lane >> 3) & 1) * 8;
 #pragma unroll
-    for (int ks = 0; ks < D / 16; ++ks)
-      ldmatrix_x4(qa[ks][0], qa[ks][1], qa[ks][2], qa[ks][3], qb + swz<D>(row, ks * 2 + (lane >> 4)));
+    for (int ks = 0; ks < DK / 16; ++ks)
+      ldmatrix_x4(qa[ks][0], qa[ks][1], qa[ks][2], qa[ks][3], qb + swz<DK>(row, ks * 2 + (lane >> 4)));
   }
 
   const int ntiles = (e0 - s0 + 15) >> 4;
@@ -128,17 +140,28 @@ gqa_decode_kernel(const bf16* __restrict__ q, int64_t q_stride, const bf16* __re
         int tok = c / CH, ch = c % CH;
         int sl = __shfl_sync(0xffffffffu, slot, tok);
         bool ok = sl >= 0;
-        const bf16* src = kv_layer + ((int64_t)(ok ? sl : 0) * (2 * Hkv) + kvh) * D + ch * 8;
-        cp_async16(sb + swz<D>(tok, ch), src, ok);
-        cp_async16(sb + TILE_BYTES + swz<D>(tok, ch), src + (int64_t)Hkv * D, ok);
+        const bf16* src = kv_layer + (int64_t)(ok ? sl : 0) * Hkv * (DK + DV) + kvh * DK + ch * 8;
+        cp_async16(sb + swz<DK>(tok, ch), src, ok);
+        if (DK == DV) cp_async16(sb + TILE_BYTES + swz<DV>(tok, ch), src + (int64_t)Hkv * DK, ok);
+      }
+      if (DK != DV) {
+#pragma unroll
+        for (int j = 0; j < (16 * CHV) / 32; ++j) {
+          int c = lane + 32 * j;
+          int tok = c / CHV, ch = c % CHV;
+          int sl = __shfl_sync(0xffffffffu, slot, tok);
+          bool ok = sl >= 0;
+          const bf16* src = kv_layer + (int64_t)(ok ? sl : 0) * Hkv * (DK + DV) + (int64_t)Hkv * DK + kvh * DV + ch * 8;
+          cp_async16(sb + TILE_BYTES + swz<DV>(tok, ch), src, ok);
+        }
       }
     }
     cp_async_commit();
   };
 
-  float o[D / 8][4];
+  float o[DV / 8][4];
 #pragma unroll
-  for (int i = 0; i < D / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
+  for (int i = 0; i < DV / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
   float m_run[2] = {-INFINITY, -INFINITY};
   float l_run[2] = {0.f, 0.f};
 
@@ -159,9 +182,9 @@ gqa_decode_kernel(const bf16* __restrict__ q, int64_t q_stride, const bf16* __re
     {
       const int tok = (lane & 7) + (lane >> 4) * 8;
 #pragma unroll
-      for (int ks = 0; ks < D / 16; ++ks) {
+      for (int ks = 0; ks < DK / 16; ++ks) {
         uint32_t b0, b1, b2, b3;
-        ldmatrix_x4(b0, b1, b2, b3, kb + swz<D>(tok, ks * 2 + ((lane >> 3) & 1)));
+        ldmatrix_x4(b0, b1, b2, b3, kb + swz<DK>(tok, ks * 2 + ((lane >> 3) & 1)));
         mma_bf16_16816(s[0], qa[ks][0], qa[ks][1], qa[ks][2], qa[ks][3], b0, b1);
         mma_bf16_16816(s[1], qa[ks][0], qa[ks][1], qa[ks][2], qa[ks][3], b2, b3);
       }
@@ -197,7 +220,7 @@ gqa_decode_kernel(const bf16* __restrict__ q, int64_t q_stride, const bf16* __re
       l_run[r] = l_run[r] * alpha[r] + rs;
     }
 #pragma unroll
-    for (int nt = 0; nt < D / 8; ++nt) {
+    for (int nt = 0; nt < DV / 8; ++nt) {
       o[nt][0] *= alpha[0];
       o[nt][1] *= alpha[0];
       o[nt][2] *= alpha[1];
@@ -205,14 +228,26 @@ gqa_decode_kernel(const bf16* __restrict__ q, int64_t q_stride, const bf16* __re
     }
     const uint32_t a0 = pack_bf16x2(s[0][0], s[0][1]), a1 = pack_bf16x2(s[0][2], s[0][3]);
     const uint32_t a2 = pack_bf16x2(s[1][0], s[1][1]), a3 = pack_bf16x2(s[1][2], s[1][3]);
+    uint32_t low[4];
+    if (SPLIT_P) {
+      const uint32_t hi[4] = {a0, a1, a2, a3};
+#pragma unroll
+      for (int e = 0; e < 4; ++e)
+        low[e] = pack_bf16x2(s[e >> 1][2 * (e & 1)] - __uint_as_float(hi[e] << 16),
+                             s[e >> 1][2 * (e & 1) + 1] - __uint_as_float(hi[e] & 0xffff0000u));
+    }
     {
       const int tok = (lane & 7) + ((lane >> 3) & 1) * 8;
 #pragma unroll
-      for (int n2 = 0; n2 < D / 16; ++n2) {
+      for (int n2 = 0; n2 < DV / 16; ++n2) {
         uint32_t b0, b1, b2, b3;
-        ldmatrix_x4_trans(b0, b1, b2, b3, vb + swz<D>(tok, n2 * 2 + (lane >> 4)));
+        ldmatrix_x4_trans(b0, b1, b2, b3, vb + swz<DV>(tok, n2 * 2 + (lane >> 4)));
         mma_bf16_16816(o[2 * n2], a0, a1, a2, a3, b0, b1);
         mma_bf16_16816(o[2 * n2 + 1], a0, a1, a2, a3, b2, b3);
+        if (SPLIT_P) {
+          mma_bf16_16816(o[2 * n2], low[0], low[1], low[2], low[3], b0, b1);
+          mma_bf16_16816(o[2 * n2 + 1], low[0], low[1], low[2], low[3], b2, b3);
+        }
       }
     }
     __syncwarp();
@@ -226,14 +261,14 @@ gqa_decode_kernel(const bf16* __restrict__ q, int64_t q_stride, const bf16* __re
     l_run[r] += __shfl_xor_sync(0xffffffffu, l_run[r], 1);
     l_run[r] += __shfl_xor_sync(0xffffffffu, l_run[r], 2);
   }
-  static_assert(WARP_BYTES >= 16 * D * 4 + 128, "ring too small for the merge buffer");
-  float* wo = reinterpret_cast<float*>(warp_smem);          // [16][D]
-  float* wml = reinterpret_cast<float*>(warp_smem + 16 * D * 4);  // m[16], l[16]
+  static_assert(WARP_BYTES >= 16 * DV * 4 + 128, "ring too small for the merge buffer");
+  float* wo = reinterpret_cast<float*>(warp_smem);          // [16][DV]
+  float* wml = reinterpret_cast<float*>(warp_smem + 16 * DV * 4);  // m[16], l[16]
 #pragma unroll
-  for (int nt = 0; nt < D / 8; ++nt) {
+  for (int nt = 0; nt < DV / 8; ++nt) {
     int d = nt * 8 + tig * 2;
-    *reinterpret_cast<float2*>(wo + g * D + d) = make_float2(o[nt][0], o[nt][1]);
-    *reinterpret_cast<float2*>(wo + (g + 8) * D + d) = make_float2(o[nt][2], o[nt][3]);
+    *reinterpret_cast<float2*>(wo + g * DV + d) = make_float2(o[nt][0], o[nt][1]);
+    *reinterpret_cast<float2*>(wo + (g + 8) * DV + d) = make_float2(o[nt][2], o[nt][3]);
   }
   if (tig == 0) {
     wml[g] = m_run[0];
@@ -243,29 +278,29 @@ gqa_decode_kernel(const bf16* __restrict__ q, int64_t q_stride, const bf16* __re
   }
   __syncthreads();
   const uint8_t* ring0 = smem + TILE_BYTES;
-  for (int idx = threadIdx.x; idx < nrows * D; idx += blockDim.x) {
-    int r = idx / D, d = idx % D;
+  for (int idx = threadIdx.x; idx < nrows * DV; idx += blockDim.x) {
+    int r = idx / DV, d = idx % DV;
     float M = -INFINITY;
 #pragma unroll
-    for (int w = 0; w < 4; ++w) M = fmaxf(M, reinterpret_cast<const float*>(ring0 + w * WARP_BYTES + 16 * D * 4)[r]);
+    for (int w = 0; w < 4; ++w) M = fmaxf(M, reinterpret_cast<const float*>(ring0 + w * WARP_BYTES + 16 * DV * 4)[r]);
     float num = 0.f, den = 0.f;
     if (M != -INFINITY) {
 #pragma unroll
       for (int w = 0; w < 4; ++w) {
         const float* po = reinterpret_cast<const float*>(ring0 + w * WARP_BYTES);
-        const float* pml = reinterpret_cast<const float*>(ring0 + w * WARP_BYTES + 16 * D * 4);
+        const float* pml = reinterpret_cast<const float*>(ring0 + w * WARP_BYTES + 16 * DV * 4);
         float sc = exp2f(pml[r] - M);
-        num += sc * po[r * D + d];
+        num += sc * po[r * DV + d];
         den += sc * pml[16 + r];
       }
     }
     float val = den > 0.f ? num / den : 0.f;
     int head = head0 + r;
     if (num_splits == 1) {
-      out[(int64_t)b * out_stride + (int64_t)head * D + d] = __float2bfloat16(val);
+      out[(int64_t)b * out_stride + (int64_t)head * DV + d] = __float2bfloat16(val * gate.factor(b, head));
     } else {
       int64_t pi = ((int64_t)b * Hq + head) * num_splits + split;
-      part_o[pi * D + d] = val;
+      part_o[pi * DV + d] = val;
       if (d == 0) part_lse[pi] = den > 0.f ? (M + log2f(den)) * kLn2 : -INFINITY;
     }
   }
@@ -274,7 +309,7 @@ gqa_decode_kernel(const bf16* __restrict__ q, int64_t q_stride, const bf16* __re
 template <int D>
 __global__ void __launch_bounds__(D)
 decode_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_lse, bf16* __restrict__ out,
-                    int64_t out_stride, int Hq, int num_splits) {
+                    int64_t out_stride, int Hq, int num_splits, const HeadGate gate) {
   pdl_wait();
   const int bh = blockIdx.x;
   const int b = bh / Hq, h = bh % Hq;
@@ -291,7 +326,7 @@ decode_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ 
       den += w;
     }
   }
-  out[(int64_t)b * out_stride + (int64_t)h * D + d] = __float2bfloat16(den > 0.f ? num / den : 0.f);
+  out[(int64_t)b * out_stride + (int64_t)h * D + d] = __float2bfloat16(den > 0.f ? num / den * gate.factor(b, h) : 0.f);
 }
 
 // ---------------------------------------------------------------------------------------
@@ -470,9 +505,13 @@ gqa_prefill_kernel(const bf16* __restrict__ q, int64_t q_stride, const bf16* __r
 }
 
 constexpr int kDecodeStages = 3;
-template <int D>
+template <int DK, int DV>
+constexpr int decode_stages() {  // large rows: fewer stages, so that two CTAs stay on an SM where they can
+  return DK + DV <= 256 ? kDecodeStages : 2;
+}
+template <int DK, int DV>
 constexpr int decode_smem_bytes() {
-  return 16 * D * 2 + 4 * kDecodeStages * 2 * 16 * D * 2;
+  return 16 * DK * 2 + 4 * decode_stages<DK, DV>() * 16 * (DK + DV) * 2;
 }
 template <int D>
 constexpr int prefill_smem_bytes() {
@@ -502,6 +541,32 @@ LLB_EXPORT int llb_gqa_decode_num_splits(int B, int Hq, int Hkv, int max_seq_len
   return s;
 }
 
+template <int DK, int DV, bool SPLIT_P>
+static int launch_decode(const void* q, int64_t q_stride, const void* kv_layer, const int* req_to_token, int64_t r2t_stride,
+                         const int* b_req_idx, const int* b_seq_len, void* out, int64_t out_stride, float* part_o,
+                         float* part_lse, int B, int Hq, int Hkv, int num_splits, float sm_scale, int window,
+                         const HeadGate& gate, cudaStream_t st) {
+  constexpr int STAGES = decode_stages<DK, DV>();
+  const int G = Hq / Hkv;
+  const dim3 grid(num_splits, Hkv * ((G + 15) / 16), B);
+  static DeviceOnce configured;
+  if (!configured.done()) {
+    int rc = set_smem(gqa_decode_kernel<DK, DV, STAGES, SPLIT_P>, decode_smem_bytes<DK, DV>());
+    if (rc) return rc;
+    configured.set();
+  }
+  launch_pdl(gqa_decode_kernel<DK, DV, STAGES, SPLIT_P>, grid, dim3(128), decode_smem_bytes<DK, DV>(), st, (const bf16*)q,
+             q_stride, (const bf16*)kv_layer, req_to_token, r2t_stride, b_req_idx, b_seq_len, (bf16*)out, out_stride, part_o,
+             part_lse, Hq, Hkv, num_splits, sm_scale * kLog2e, window, gate);
+  LLB_LAUNCH_CHECK();
+  if (num_splits > 1) {
+    launch_pdl(decode_merge_kernel<DV>, dim3(B * Hq), dim3(DV), 0, st, (const float*)part_o, (const float*)part_lse,
+               (bf16*)out, out_stride, Hq, num_splits, gate);
+    LLB_LAUNCH_CHECK();
+  }
+  return LLB_OK;
+}
+
 // q [B, Hq, D] (row stride q_stride elements), out [B, Hq, D] (row stride out_stride).
 // part_o: fp32 [B, Hq, num_splits, D], part_lse: fp32 [B, Hq, num_splits]; only touched when num_splits > 1.
 LLB_EXPORT int llb_gqa_decode(const void* q, int64_t q_stride, const void* kv_layer, const int* req_to_token,
@@ -511,35 +576,40 @@ LLB_EXPORT int llb_gqa_decode(const void* q, int64_t q_stride, const void* kv_la
   if (B <= 0) return LLB_OK;
   if (Hkv <= 0 || Hq % Hkv != 0 || num_splits < 1) return LLB_ERR_BAD_ARG;
   if (num_splits > 1 && (part_o == nullptr || part_lse == nullptr)) return LLB_ERR_BAD_ARG;
-  const int G = Hq / Hkv;
-  dim3 grid(num_splits, Hkv * ((G + 15) / 16), B);
-  const float sl2 = sm_scale * kLog2e;
-#define LAUNCH_DECODE(DD)                                                                                         \
-  {                                                                                                               \
-    static DeviceOnce configured;                                                                                    \
-    if (!configured.done()) {                                                                                            \
-      int rc = set_smem(gqa_decode_kernel<DD, kDecodeStages>, decode_smem_bytes<DD>());                           \
-      if (rc) return rc;                                                                                          \
-      configured.set();                                                                                            \
-    }                                                                                                             \
-    launch_pdl(gqa_decode_kernel<DD, kDecodeStages>, grid, dim3(128), decode_smem_bytes<DD>(), st, (const bf16*)q, \
-               q_stride, (const bf16*)kv_layer, req_to_token, r2t_stride, b_req_idx, b_seq_len, (bf16*)out,       \
-               out_stride, part_o, part_lse, Hq, Hkv, num_splits, sl2);                                           \
-    LLB_LAUNCH_CHECK();                                                                                           \
-    if (num_splits > 1) {                                                                                         \
-      launch_pdl(decode_merge_kernel<DD>, dim3(B * Hq), dim3(DD), 0, st, (const float*)part_o,                    \
-                 (const float*)part_lse, (bf16*)out, out_stride, Hq, num_splits);                                 \
-      LLB_LAUNCH_CHECK();                                                                                         \
-    }                                                                                                             \
-  }
+  const HeadGate none{nullptr, 0, 1.f};
   if (D == 128)
-    LAUNCH_DECODE(128)
-  else if (D == 64)
-    LAUNCH_DECODE(64)
-  else
-    return LLB_ERR_UNSUPPORTED;
-#undef LAUNCH_DECODE
-  return LLB_OK;
+    return launch_decode<128, 128, false>(q, q_stride, kv_layer, req_to_token, r2t_stride, b_req_idx, b_seq_len, out,
+                                          out_stride, part_o, part_lse, B, Hq, Hkv, num_splits, sm_scale, 0, none, st);
+  if (D == 64)
+    return launch_decode<64, 64, false>(q, q_stride, kv_layer, req_to_token, r2t_stride, b_req_idx, b_seq_len, out,
+                                        out_stride, part_o, part_lse, B, Hq, Hkv, num_splits, sm_scale, 0, none, st);
+  return LLB_ERR_UNSUPPORTED;
+}
+
+// The windowed form: key size dk and value size dv (64, 128, 192 or 256), pool rows [Hkv * dk | Hkv * dv], window (0: none),
+// gate [B, >= Hq] (or null): head h of the output times out_scale * sigmoid(gate).  part_o: fp32 [B, Hq, num_splits, dv].
+LLB_EXPORT int llb_window_gqa_decode(const void* q, int64_t q_stride, const void* kv_layer, const int* req_to_token,
+                                     int64_t r2t_stride, const int* b_req_idx, const int* b_seq_len, void* out,
+                                     int64_t out_stride, float* part_o, float* part_lse, int B, int Hq, int Hkv, int dk,
+                                     int dv, int num_splits, float sm_scale, int window, const void* gate,
+                                     int64_t gate_stride, float out_scale, cudaStream_t st) {
+  if (B <= 0) return LLB_OK;
+  if (Hkv <= 0 || Hq % Hkv != 0 || num_splits < 1 || window < 0 || (q_stride % 8) || ((uintptr_t)q & 15)) return LLB_ERR_BAD_ARG;
+  if (num_splits > 1 && (part_o == nullptr || part_lse == nullptr)) return LLB_ERR_BAD_ARG;
+  const HeadGate g{(const bf16*)gate, gate_stride, out_scale};
+#define LLB_WINDOW_DECODE(DK, DV)                                                                                        \
+  if (dk == DK && dv == DV)                                                                                              \
+    return launch_decode<DK, DV, true>(q, q_stride, kv_layer, req_to_token, r2t_stride, b_req_idx, b_seq_len, out,       \
+                                       out_stride, part_o, part_lse, B, Hq, Hkv, num_splits, sm_scale, window, g, st);
+#define LLB_WINDOW_DECODE_V(DK)                                                                                          \
+  LLB_WINDOW_DECODE(DK, 64) LLB_WINDOW_DECODE(DK, 128) LLB_WINDOW_DECODE(DK, 192) LLB_WINDOW_DECODE(DK, 256)
+  LLB_WINDOW_DECODE_V(64)
+  LLB_WINDOW_DECODE_V(128)
+  LLB_WINDOW_DECODE_V(192)
+  LLB_WINDOW_DECODE_V(256)
+#undef LLB_WINDOW_DECODE_V
+#undef LLB_WINDOW_DECODE
+  return LLB_ERR_UNSUPPORTED;
 }
 
 // tcgen05 kernel for head size 128 (attention_tc.cu); LLB_ATTN_TC=0 keeps the mma.sync kernel below
