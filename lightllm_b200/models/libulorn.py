@@ -346,6 +346,13 @@ class LibulornLM(RecurrentStateMixin, TransformerLM):
             self.bigram.slot_token = torch.zeros(self.mem_manager.size + 1, dtype=torch.int32, device=self.device)
 
     # ------------------------------------------------------------------ forward
+    def _make_decode_state(self, B, b_req_idx, b_seq_len, mem_index, max_kv_len, num_splits=None):
+        return InferState(is_prefill=False, batch_size=B, num_tokens=B, max_kv_len=max_kv_len, max_q_len=1,
+                          b_req_idx=b_req_idx, b_seq_len=b_seq_len, mem_index=mem_index)
+
+    def _graph_decode_splits(self, bucket):
+        return 1        # per layer, from its window (ops.window_attention)
+
     def _embed(self, ids, st):
         x, st.extra["stream_h"] = ops.embedding_pair(ids, self.embed_w, self.bigram, self.req_manager.req_to_token_indexs,
                                                      st.b_req_idx, st.seq_pos,

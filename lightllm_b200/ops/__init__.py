@@ -740,6 +740,9 @@ def qk_norm_rope_scatter_(qkv, kv_layer, cos, sin, pos, slot, q_w, k_w, eps, Hq,
     return qkv
 
 
+_WINDOW_SIZES = (64, 128, 192, 256)   # head sizes of the tensor-core kernels
+
+
 def window_attention(q, kv_layer, req_to_token, st, Hq, Hkv, D, DV, sm_scale, window, gate=None, out_scale=1.0, out=None):
     """Causal paged attention with key size D and value size DV through a sliding window (0: none) for the pass `st`
     (InferState).  q [T, >= Hq * D]; gate [T, Hq] (or None): head h is multiplied by sigmoid(gate[:, h]); all heads by
@@ -753,11 +756,33 @@ def window_attention(q, kv_layer, req_to_token, st, Hq, Hkv, D, DV, sm_scale, wi
                                     out_scale, out)
     assert q.stride(1) == 1 and kv_layer.is_contiguous() and out.stride(1) == 1
     gs = 0 if gate is None else gate.stride(0)
+    tail = (f32(sm_scale), c_int(window), ptr(gate), i64(gs), f32(out_scale), stream())
+    if q.dtype == torch.bfloat16 and D in _WINDOW_SIZES and DV % 64 == 0:
+        common = (ptr(q), i64(q.stride(0)), ptr(kv_layer), ptr(req_to_token), i64(req_to_token.stride(0)),
+                  ptr(st.b_req_idx))
+        if st.is_prefill:
+            check(kernels().llb_window_gqa_prefill_tc(*common, ptr(st.cu_q), ptr(st.b_ready_cache_len), ptr(out),
+                                                      i64(out.stride(0)), c_int(st.batch_size), c_int(st.max_q_len),
+                                                      c_int(Hq), c_int(Hkv), c_int(D), c_int(DV), *tail),
+                  "window_gqa_prefill_tc")
+            _count()
+            return out
+        if DV in _WINDOW_SIZES:
+            keys = min(window, st.max_kv_len) if window > 0 else st.max_kv_len
+            n = gqa_decode_num_splits(T, Hq, Hkv, max(keys, 1))
+            po = pl = None
+            if n > 1:
+                po = torch.empty(T * Hq * n * DV, dtype=torch.float32, device=q.device)
+                pl = torch.empty(T * Hq * n, dtype=torch.float32, device=q.device)
+            check(kernels().llb_window_gqa_decode(*common, ptr(st.b_seq_len), ptr(out), i64(out.stride(0)), ptr(po), ptr(pl),
+                                                  c_int(T), c_int(Hq), c_int(Hkv), c_int(D), c_int(DV), c_int(n), *tail),
+                  "window_gqa_decode")
+            _count(2 if n > 1 else 1)
+            return out
     check(kernels().llb_attn_generic_kv(ptr(q), c_int(DTYPE_CODES[q.dtype]), i64(q.stride(0)), ptr(kv_layer),
                                         ptr(req_to_token), i64(req_to_token.stride(0)), ptr(st.b_req_idx),
                                         ptr(st.seq_pos), ptr(st.batch_of_token if st.is_prefill else None), ptr(out),
-                                        i64(out.stride(0)), c_int(T), c_int(Hq), c_int(Hkv), c_int(D), c_int(DV),
-                                        f32(sm_scale), c_int(window), ptr(gate), i64(gs), f32(out_scale), stream()),
+                                        i64(out.stride(0)), c_int(T), c_int(Hq), c_int(Hkv), c_int(D), c_int(DV), *tail),
           "attn_generic_kv")
     _count()
     return out

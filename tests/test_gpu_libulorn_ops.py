@@ -8,6 +8,7 @@ from lightllm_b200 import ops
 from lightllm_b200.common.infer_state import InferState
 from lightllm_b200.ops import moe
 from lightllm_b200.ops import reference as ref
+from lightllm_b200.ops._native import kernels
 from lightllm_b200.ops.linear_attn import ChunkPlan, DecayedState
 
 pytestmark = pytest.mark.gpu
@@ -143,13 +144,13 @@ def test_chunked_recurrence_any_decay(dev, tau, zscale, shift):
 
 
 @pytest.mark.parametrize("kind", ["gla", "mlstm"])
-@pytest.mark.parametrize("dtype,tol", [(BF, 4e-3), (F32, 3e-6)])
+@pytest.mark.parametrize("dtype,tol", [(BF, 4e-3), (F32, 8e-6)])
 @pytest.mark.parametrize("H,dim,vdim", SHAPES + [(1, 300, 600)])
 def test_recurrence_token_by_token(dev, kind, dtype, tol, H, dim, vdim):
     out, state = recurrence_case(dev, kind, dtype, [1] * 7, [0, 1, 2, 3, 64, 65, 0], H, dim, vdim, decode=True)
-    assert out < tol and state < 3e-6, ("decode", out, state)
+    assert out < tol and state < 5e-6, ("decode", out, state)
     out, state = recurrence_case(dev, kind, dtype, [1, 9, 30], [0, 3, 0], H, dim, vdim, scan=True)
-    assert out < tol and state < 3e-6, ("prompt", out, state)
+    assert out < tol and state < 5e-6, ("prompt", out, state)
 
 
 def test_chunked_and_token_by_token_agree_over_a_long_prompt(dev):
@@ -208,6 +209,7 @@ def attention_case(dev, dtype, new, ready, Hq, Hkv, D, DV, window, seed=0, decod
     ops.window_attention(qw[:, : Hq * D], pool.to(dev), r2t, st, Hq, Hkv, D, DV, scale, window,
                          gw[:, :Hq] if gated else None, 1.3 if gated else 1.0, wide[:, 8:])
     torch.cuda.synchronize()
+    assert kernels().llb_attn_tc_status() == 0
     assert (wide[:, :8] == 3).all()
     return rel(wide[:, 8:], want.reshape(T, -1))
 
