@@ -261,3 +261,314 @@ def test_add_rms_operator():
     h = ops.add_rms_(x, y, w, 12, 0.1, torch.float32, nw)
     torch.testing.assert_close(x.double(), want, atol=1e-6, rtol=1e-5)
     torch.testing.assert_close(h.double()[:, :12], plain.rms(want[:, :12], 0.1) * nw[:12], atol=1e-6, rtol=1e-5)
+
+
+# ------------------------------------------------------------------------------------------------ the engine
+@target
+def test_stream_after_every_layer(mixed_model, tgt):
+    path, t = mixed_model
+    toks, want, got = tokens(60, 7), [], []
+    plain.forward(t, MIXED, toks, streams=want)
+    rep = replayer(path, tgt)
+    rep.llm.model.stream_tap = lambda i, x: got.append(x[:, : MIXED["width"]].double().cpu())
+    rep.step([("a", toks, [])])
+    assert len(got) == len(want)
+    for i, (g, w) in enumerate(zip(got, want)):
+        close(g, w, tgt, f"layer {i}")
+
+
+@target
+def test_prompt_decode_and_portions(mixed_model, tgt):
+    path, t = mixed_model
+    toks = tokens(139, 2)
+    want = plain.forward(t, MIXED, toks)
+    rep = replayer(path, tgt)
+    for portions in ([139], [1], [2], [9, 10], [37, 36, 1], [64], [65, 63, 1], [100, 3, 1]):
+        close(run_portions(rep, f"p{portions}", toks, portions), want, tgt, portions)
+    assert rep.backend.ctx.get_can_alloc_token_num() == 512
+
+
+@target
+def test_first_tokens(mixed_model, tgt):
+    path, t = mixed_model
+    rep = replayer(path, tgt)
+    for n in (1, 2, 3, 5):
+        toks = tokens(n, 40 + n)
+        close(run_portions(rep, f"w{n}", toks, [n]), plain.forward(t, MIXED, toks), tgt)
+        close(run_portions(rep, f"s{n}", toks, [1]), plain.forward(t, MIXED, toks), tgt)
+
+
+@target
+def test_unequal_batches_and_reused_slots(mixed_model, tgt):
+    """Four live requests in one step, portions beside single tokens, in a pool they fill: requests end and their cache
+    and state slots are used again by others, and requests rest for some steps."""
+    path, t = mixed_model
+    lens = {"a": 90, "b": 33, "c": 150, "d": 7, "e": 70, "f": 41, "g": 128}
+    toks = {k: tokens(n, 60 + i) for i, (k, n) in enumerate(lens.items())}
+    want = {k: plain.forward(t, MIXED, v) for k, v in toks.items()}
+    rep = replayer(path, tgt, pool=320)
+    g = torch.Generator().manual_seed(5)
+    at, waiting, live, seen = {k: 0 for k in lens}, list(lens), [], {k: [] for k in lens}
+    while waiting or live:
+        room = 320 - sum(lens[k] for k in live)
+        while waiting and len(live) < 4 and lens[waiting[0]] <= room:
+            room -= lens[waiting[0]]
+            live.append(waiting.pop(0))
+        entries = []
+        for k in live:
+            n = (1, 1, 2, 17, 40, 0)[int(torch.randint(0, 6, (), generator=g))]
+            n = min(n, lens[k] - at[k])
+            if n:
+                entries.append((k, toks[k][at[k]:at[k] + n], range(n)))
+        if not entries:
+            continue
+        ends = [k for k, new, _ in entries if at[k] + len(new) == lens[k]]
+        out, off = torch.from_numpy(rep.step(entries, ends)), 0
+        for k, new, _ in entries:
+            seen[k].append(out[off:off + len(new)])
+            off, at[k] = off + len(new), at[k] + len(new)
+        live = [k for k in live if k not in ends]
+    for k in lens:
+        close(torch.cat(seen[k]), want[k], tgt, k)
+    assert rep.backend.ctx.get_can_alloc_token_num() == 320
+
+
+@target
+@pytest.mark.parametrize("window", [1, 2, 31, 64, 65, 129])
+def test_window_edges(tmp_path, tgt, window):
+    """One windowed attention layer alone (the recurrent side and the bigram embedding weigh nothing): position p depends on
+    exactly the tokens p - window + 1 .. p.  The scores are kept small, so that every visible key has a share."""
+    cfg = config([parallel(attention(2, 1, 24, 40, window, 0.01, 16), gla(1, 16, 16, 2.0), None, 1.0, 0.0)])
+    t = weights(cfg, window)
+    t["bigram"] = torch.zeros_like(t["bigram"])
+    rep = replayer(write(tmp_path, cfg, t), tgt)
+    n = window + 35
+    base = tokens(n, 3)
+    p = n - 1
+    for portions in ([n], [n - 5, 2, 3], [30, n - 31, 1]):
+        first = run_portions(rep, "base", base, portions)
+        close(first, plain.forward(t, cfg, base), tgt, portions)
+        for d, inside in ((window - 1, True), (window, False), (window + 1, False)):
+            best = 0.0
+            for delta in (1, 40):       # some other tokens there
+                other = list(base)
+                other[p - d] = (other[p - d] + delta) % VOCAB
+                got = run_portions(rep, "other", other, portions)
+                close(got[p:], plain.forward(t, cfg, other)[p:], tgt, (portions, d))
+                best = max(best, float((got[p] - first[p]).abs().max()))
+            assert (best > 1e-4) == inside, (portions, d, best)
+
+
+@target
+def test_one_key_that_stands_out(tmp_path, tgt):
+    """A single key takes nearly all the weight of a far query, first just inside, then just outside the window, in a prompt
+    and in decoding."""
+    H, dim, W, window = 2, 16, 80, 100
+    cfg = config([parallel(attention(H, 1, dim, 32, window, 60.0 / dim, 4), gla(1, 16, 16, 2.0), None, 1.0, 0.0)])
+    t = weights(cfg, 11)
+    t["bigram"] = torch.zeros_like(t["bigram"])
+    beacon, asker = 5, 6
+    e = t["embed"].float()
+    g = torch.Generator().manual_seed(2)
+    q, k = torch.randn(H * dim, W, generator=g) * 0.02, torch.randn(dim, W, generator=g) / W ** 0.5
+    for h in range(H):                      # dimension 9 is not rotated
+        q[h * dim + 9] += e[asker] / e[asker].square().sum() * 30
+    k[9] += e[beacon] / e[beacon].square().sum() * 30
+    t["l0.mix.left.q"], t["l0.mix.left.k"] = q.to(torch.bfloat16), k.to(torch.bfloat16)
+    rep = replayer(write(tmp_path, cfg, t), tgt)
+    # fillers whose keys do not point along dimension 9 by themselves
+    filler = [x for x in tokens(2000, 9) if x not in (beacon, asker) and
+              plain.rms(k.double() @ e[x].double(), 1e-4)[9] < 1.0][:150]
+    assert len(filler) == 150
+    results = []
+    for d in (window - 1, window):
+        toks = list(filler)
+        toks[149], toks[149 - d] = asker, beacon
+        want = plain.forward(t, cfg, toks)
+        for portions in ([150], [149, 1], [120, 2]):
+            got = run_portions(rep, "x", toks, portions)
+            close(got, want, tgt, (d, portions))
+        results.append(got[149])
+    assert (results[0] - results[1]).abs().max() > 0.05
+
+
+@target
+@pytest.mark.parametrize("kind", ["mlstm", "gla"])
+def test_state_remembers_far_tokens(tmp_path, tgt, kind):
+    """Slow decays: the first tokens still show after hundreds of others, over every chunk border, and a changed one is seen."""
+    if kind == "mlstm":
+        cfg = config([mlstm(2, 24, 40, 12.0, None)])
+        t = weights(cfg, 3)
+        t["l0.mix.f.b"] = torch.full((2,), 9.0).to(torch.bfloat16)
+        t["l0.mix.f"] = t["l0.mix.f"] * 0.1
+    else:
+        cfg = config([parallel(attention(1, 1, 8, 8, 3, 0.3, 4), gla(2, 24, 40, 60.0), None, 0.5, 1.5)])
+        t = weights(cfg, 4)
+        t["l0.mix.right.a2.b"] = t["l0.mix.right.a2.b"] + 4
+    rep = replayer(write(tmp_path, cfg, t), tgt)
+    n = 270
+    base = tokens(n, 3)
+    other = list(base)
+    other[1] = (other[1] + 31) % VOCAB
+    for portions in ([n], [64, 2, 63], [n - 60, 1]):
+        a, b = run_portions(rep, "a", base, portions), run_portions(rep, "b", other, portions)
+        close(a, plain.forward(t, cfg, base), tgt, portions)
+        close(b, plain.forward(t, cfg, other), tgt, portions)
+        assert (a[n - 1] - b[n - 1]).abs().max() > (2e-2 if tgt[1] == "bfloat16" else 2e-3)
+
+
+@target
+def test_long_decoding_and_greedy_generation(mixed_model, tgt):
+    """Greedy generation through the engine's own scheduler: every produced token is the arg-max of the plain restatement up
+    to rounding, far beyond the windows; a second run starts from snapshots of the recurrent state."""
+    path, t = mixed_model
+    llm = LLM(model_dir=path, data_type=tgt[1], max_total_token_num=2000, running_max_req_size=4, max_req_total_len=400,
+              chunked_prefill_size=48, batch_max_tokens=96, state_snapshot_slots=24, linear_att_hash_page_size=32,
+              pstate=pstate(tgt))
+    prompts = [tokens(n, 80 + n) for n in (1, 30, 111)]
+    outs = llm.generate(prompts, {"max_new_tokens": 120, "do_sample": False})
+    again = llm.generate(prompts, {"max_new_tokens": 120, "do_sample": False})
+    for p, o, o2 in zip(prompts, outs, again):
+        assert len(o["token_ids"]) == 120
+        for out in (o, o2):
+            lg = plain.forward(t, MIXED, p + out["token_ids"])[len(p) - 1:-1]
+            chosen = lg.gather(1, torch.tensor(out["token_ids"])[:, None])[:, 0]
+            gap = lg.max(-1)[0] - chosen
+            if tgt[1] == "bfloat16":
+                assert (gap > 0.2).float().mean() < 0.1
+            else:
+                assert gap.max() < 1e-3
+    assert again[2]["prompt_cache_len"] > 0 and llm.backend.state_cache.stats["hits"] > 0
+    llm.close()
+
+
+@target
+def test_random_weights_and_sampling(tgt):
+    """A model without a checkpoint (benchmarks), sampled generation."""
+    llm = LLM(config=MIXED, data_type=tgt[1], max_total_token_num=600, running_max_req_size=3, max_req_total_len=200,
+              pstate=pstate(tgt))
+    outs = llm.generate([tokens(20, 1), tokens(3, 2)], {"max_new_tokens": 8, "do_sample": True, "temperature": 0.9,
+                                                        "top_k": 20, "seed": 3})
+    assert all(len(o["token_ids"]) == 8 and max(o["token_ids"]) < VOCAB for o in outs)
+    llm.close()
+
+
+def test_recurrent_layers_only(tmp_path):
+    """Without attention the pool has no rows, only slots."""
+    cfg = config([mlstm(2, 8, 8, 5.0, experts(3, 2, 16, 1.0)), mlstm(1, 24, 16, 3.0, None)])
+    t = weights(cfg, 2)
+    rep = replayer(write(tmp_path, cfg, t), ("cpu", "float32"), pool=128)
+    toks = tokens(100, 1)
+    close(run_portions(rep, "a", toks, [50, 49, 1]), plain.forward(t, cfg, toks), ("cpu", "float32"))
+    pages = rep.llm.model.mem_manager.gather_pages(torch.arange(3, dtype=torch.int32))
+    assert pages.shape == (1, 3, 0)
+
+
+def test_pages_carry_every_layer(mixed_model):
+    mm = replayer(mixed_model[0], ("cpu", "float32")).llm.model.mem_manager
+    for i, buf in enumerate(mm.kv_layers):
+        buf.normal_(generator=torch.Generator().manual_seed(i))
+    src, dst = torch.tensor([3, 9], dtype=torch.int32), torch.tensor([20, 1], dtype=torch.int32)
+    mm.scatter_pages(dst, mm.gather_pages(src))
+    for buf in mm.kv_layers:
+        assert torch.equal(buf[dst.long()], buf[src.long()])
+
+
+def test_returned_routed_experts(tmp_path):
+    cfg = config([mlstm(2, 16, 16, 5.0, experts(6, 2, 32, 1.0)), mlstm(2, 16, 16, 5.0, None),
+                  mlstm(2, 16, 16, 5.0, experts(5, 2, 32, 1.0, (8, 1.0)))])
+    t = weights(cfg, 4)
+    llm = LLM(model_dir=write(tmp_path, cfg, t), data_type="float32", max_total_token_num=200, running_max_req_size=2,
+              max_req_total_len=64, enable_return_routed_experts=True)
+    seen = []
+    route, p = plain.route, tokens(11, 5)
+    o = llm.generate([p], {"max_new_tokens": 4, "do_sample": False})[0]
+    try:
+        plain.route = lambda *a: seen.append(route(*a)[0]) or route(*a)
+        plain.forward(t, cfg, p + o["token_ids"][:-1])
+    finally:
+        plain.route = route
+    for j in range(2):
+        got = torch.as_tensor(o["routed_experts"][:, j].astype("int64"))
+        assert torch.equal(got.sort(-1)[0], seen[j].sort(-1)[0])
+
+
+def test_config_reaches_the_server_side(tmp_path):
+    from lightllm_b200.server.tokenizer import get_tokenizer
+    from lightllm_b200.utils import config_utils
+    from lightllm_b200.utils.profile_max_tokens import kv_bytes_per_token, max_total_tokens
+
+    path = write(tmp_path, MIXED, weights(MIXED))
+    cfg = load_config(path)
+    assert cfg["model_type"] == "libulorn" and cfg["hidden_size"] == 80 and cfg["num_hidden_layers"] == 5
+    assert config_utils.get_vocab_size(path) == VOCAB and config_utils.get_dtype(path) == "bfloat16"
+    assert get_tokenizer(path, vocab_size=VOCAB).encode("3 4 5") == [3, 4, 5]
+    assert get_model_class(cfg).__name__ == "LibulornLM"
+    assert kv_bytes_per_token(cfg, 1) == 2 * (2 * (64 + 128) + (192 + 64) + 4 * 128)
+    assert max_total_tokens(path, gpu_gib=1)["max_total_token_num"] > 0
+
+
+def _bad(tmp_path, match, cfg=None, change=None, **kw):
+    t = weights(MIXED)
+    if change:
+        change(t)
+    path = write(tmp_path, cfg or MIXED, t)
+    with pytest.raises(ValueError, match=match):
+        LLM(model_dir=path, max_total_token_num=64, max_req_total_len=64, data_type="float32", **kw)
+
+
+def test_wrong_checkpoints_are_refused(tmp_path):
+    def shape(t):
+        t["l1.mix.right.v"] = t["l1.mix.right.v"][:-1].contiguous()
+
+    _bad(tmp_path, "l1.mix.right.v: shape", change=shape)
+    for where, what in ((("layers", 1, "type"), "unknown mixer"), (("layers", 0, "mlp", "kind"), "unknown feed-forward")):
+        other = json.loads(json.dumps(MIXED))
+        at = other
+        for k in where[:-1]:
+            at = at[k]
+        at[where[-1]] = "something"
+        _bad(tmp_path, what, cfg=other)
+    _bad(tmp_path, "bf16 or fp32 only", quant_type="fp8w8a8-b128")
+    _bad(tmp_path, "no quantised form", kv_type="int8kv")
+
+
+def test_trace_run_program(tmp_path, mixed_model):
+    import numpy as np
+
+    path, t = mixed_model
+    a, b = tokens(70, 1), tokens(9, 2)
+    lines = [{"step": 0, "entries": [{"id": "a", "tokens": a[:50], "want": [0, 49]}], "end": []},
+             {"step": 1, "entries": [{"id": "b", "tokens": b[:8], "want": []}, {"id": "a", "tokens": a[50:51], "want": []}],
+              "end": []},
+             {"step": 2, "entries": [{"id": "a", "tokens": a[51:], "want": [18]}, {"id": "b", "tokens": b[8:], "want": [0]}],
+              "end": ["a", "b"]}]
+    r = subprocess.run([os.path.join(ROOT, "bin", "trace_run"), "--model", path, "--out", str(tmp_path), "--device", "cpu",
+                        "--dtype", "float32", "--max-tokens", "128"], input="".join(json.dumps(x) + "\n" for x in lines),
+                       capture_output=True, text=True, timeout=240)
+    assert r.returncode == 0, r.stderr[-2000:]
+    assert [x for x in r.stdout.splitlines() if x.startswith("done")] == ["done 0", "done 1", "done 2"]
+    wa, wb = plain.forward(t, MIXED, a), plain.forward(t, MIXED, b)
+    got = {i: torch.from_numpy(np.fromfile(tmp_path / f"{i}.f32", dtype="<f4").reshape(-1, VOCAB)) for i in (0, 2)}
+    close(got[0], wa[[0, 49]], ("cpu", "float32"))
+    close(got[2], torch.stack([wa[69], wb[8]]), ("cpu", "float32"))
+    assert not (tmp_path / "1.f32").exists()
+
+
+def test_every_kernel_entry_has_a_source():
+    """The units the family names for a checkout without built libraries cover what its operators call."""
+    import re
+
+    from lightllm_b200.models.libulorn import LibulornLM
+    from lightllm_b200.ops._native import UnitLibraries
+
+    units = UnitLibraries()._unit_of
+    called = set()
+    for name in ("__init__", "linear_attn", "moe"):
+        with open(os.path.join(ROOT, "lightllm_b200", "ops", name + ".py")) as f:
+            called |= set(re.findall(r"kernels\(\)\.(llb_\w+)", f.read()))
+    assert called <= set(units)
+    assert {units[n] for n in ("llb_embedding_pair", "llb_add_rms", "llb_moe_combine_rms", "llb_recurrent_scan",
+                               "llb_recurrent_chunks", "llb_qk_norm_rope_scatter", "llb_window_gqa_prefill_tc",
+                               "llb_window_gqa_decode", "llb_attn_generic_kv", "llb_gemm_f32", "llb_gemm_bf16_fused",
+                               "llb_topk_softmax", "llb_decode_prologue", "llb_sample")} <= set(LibulornLM.native_units)
