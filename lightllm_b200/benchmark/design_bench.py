@@ -1,7 +1,8 @@
-"""Prefill and decode throughput of the Taduzen family beside the framework's closest model (DeepSeek-V2: latent
-attention, routed and shared experts) at equal sizes, and the kernels of both with their roofline fractions.
+"""Prefill and decode throughput of a model design beside the framework's closest model at equal sizes, and the kernels
+of both with their roofline fractions.  Taduzen: DeepSeek-V2 (latent attention, routed and shared experts); Libulorn:
+Qwen3-Next (`design_libulorn.py`).
 
-    python bench.py --design taduzen [--design-size small|base|wide] [--design-kernels]
+    python bench.py --design taduzen|libulorn [--design-size small|base|wide] [--design-kernels]
 
 Random weights, random tokens, bf16.  Whole passes through the models' own forward (decode as CUDA graph), timed with CUDA
 events after three warm-up passes; a pass reads far more weight bytes than L2 holds.  Kernels: median of 10 samples with L2
@@ -88,10 +89,22 @@ PREFILL = [(4, 0, 2048), (1, 0, 8192), (8, 4096, 512)]      # requests, cached t
 DECODE = [(16, 4096), (64, 4096), (256, 1024)]              # requests, context
 
 
-def passes(size: str, steps: int):
-    z = SIZES[size]
+def _design(name):
+    """(sizes, configuration, closest model's name and configuration, kernels)"""
+    if name == "taduzen":
+        from .design_kernels import kernels
+
+        return SIZES, taduzen_config, "deepseek_v2", deepseek_config, kernels
+    from . import design_libulorn as d
+
+    return d.SIZES, d.config, "qwen3_next", d.closest_config, d.kernels
+
+
+def passes(design: str, size: str, steps: int):
+    sizes, config, closest, closest_config, _ = _design(design)
+    z = sizes[size]
     res = {}
-    for name, cfg in (("taduzen", taduzen_config(z)), ("deepseek_v2", deepseek_config(z))):
+    for name, cfg in ((design, config(z)), (closest, closest_config(z))):
         tokens = max(max(b * (r + n) for b, r, n in PREFILL), max(b * (c + 1) for b, c in DECODE)) + 64
         model = _model(cfg, tokens, 8192, 256)
         for b, ready, new in PREFILL:
@@ -104,22 +117,20 @@ def passes(size: str, steps: int):
         del model
         torch.cuda.empty_cache()
     for (name, what), (ms, n) in res.items():
-        if name != "taduzen":
+        if name != design:
             continue
-        other = res["deepseek_v2", what][0]
-        print(json.dumps({"design": "taduzen", "size": size, "pass": what, "ms": round(ms, 3),
-                          "tokens_per_s": round(n / ms * 1e3), "deepseek_v2_ms": round(other, 3),
-                          "deepseek_v2_tokens_per_s": round(n / other * 1e3), "speedup": round(other / ms, 2),
+        other = res[closest, what][0]
+        print(json.dumps({"design": design, "size": size, "pass": what, "ms": round(ms, 3),
+                          "tokens_per_s": round(n / ms * 1e3), f"{closest}_ms": round(other, 3),
+                          f"{closest}_tokens_per_s": round(n / other * 1e3), "speedup": round(other / ms, 2),
                           "layers": LAYERS, "dtype": "bf16", "data": "synthetic"}), flush=True)
 
 
 def run(args):
-    sizes = [args.design_size] if args.design_size else list(SIZES)
-    for s in sizes:
-        passes(s, args.steps)
+    sizes, *_, kernels = _design(args.design)
+    for s in [args.design_size] if args.design_size else list(sizes):
+        passes(args.design, s, args.steps)
         if args.design_kernels:
-            from .design_kernels import kernels
-
             kernels(s)
 
 
