@@ -202,76 +202,97 @@ LLB_EXPORT int llb_rope_kv_scatter_generic(void* qkv, void* kv_layer, const floa
 
 // Per-head RMS norm of q and k over the first `dim` of their D elements, rotary positions on the first rot_dim, and the
 // cache write, for layers whose value size DV differs from the key size D.  qkv row: [Hq * D | Hkv * D | Hkv * DV]; q is
-// rewritten in place, K and V go to kv_layer[slot].  Sizes are multiples of 8; a group of 2^k lanes works on one head, a
-// lane on 8 elements of it at a time, and rotation partners meet in shared memory.
-template <typename E>
+// rewritten in place, K and V go to kv_layer[slot].  Sizes are multiples of 8; a group of 2^k lanes works on one head, a lane
+// on 8 elements of it (NIT times, 8 * lanes apart); rotation partners meet in shared memory.
+__device__ __forceinline__ void load8(const bf16* p, float* f) { unpack8(*reinterpret_cast<const bf16x8*>(p), f); }
+__device__ __forceinline__ void load8(const float* p, float* f) {
+  const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
+  f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w;
+  f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
+}
+__device__ __forceinline__ void store8(bf16* p, const float* f) { *reinterpret_cast<bf16x8*>(p) = pack8(f); }
+__device__ __forceinline__ void store8(float* p, const float* f) {
+  reinterpret_cast<float4*>(p)[0] = make_float4(f[0], f[1], f[2], f[3]);
+  reinterpret_cast<float4*>(p)[1] = make_float4(f[4], f[5], f[6], f[7]);
+}
+
+template <typename E, int NIT>
 __global__ void __launch_bounds__(256)
 qk_norm_rope_scatter_kernel(E* __restrict__ qkv, int64_t qkv_stride, E* __restrict__ kv_layer,
                             const float* __restrict__ cos_t, const float* __restrict__ sin_t, const int* __restrict__ pos,
                             const int* __restrict__ slot, const float* __restrict__ qw, const float* __restrict__ kw,
-                            float eps, int T, int Hq, int Hkv, int D, int dim, int DV, int rot_dim, int lanes) {
+                            float eps, unsigned items, int Hq, int Hkv, int D, int dim, int DV, int rot_dim, int lanes_log2) {
   pdl_wait();
-  extern __shared__ float srow[];  // [groups][D]
-  const int gl = threadIdx.x % lanes, grp = threadIdx.x / lanes, groups = blockDim.x / lanes;
-  const int heads = Hq + 2 * Hkv;
-  const int64_t item = (int64_t)blockIdx.x * groups + grp;
-  const bool live = item < (int64_t)T * heads;
-  const int t = live ? (int)(item / heads) : 0, head = live ? (int)(item - (int64_t)t * heads) : Hq + Hkv;
+  extern __shared__ float srow[];  // [groups][rot_dim]
+  const int lanes = 1 << lanes_log2;
+  const int gl = threadIdx.x & (lanes - 1), grp = threadIdx.x >> lanes_log2;
+  const unsigned heads = Hq + 2 * Hkv;
+  const unsigned item = blockIdx.x * (256u >> lanes_log2) + grp;
+  const bool live = item < items;
+  const unsigned t = live ? item / heads : 0;
+  const int head = live ? (int)(item - t * heads) : Hq + Hkv;
   E* row = qkv + (int64_t)t * qkv_stride;
   const int half = rot_dim >> 1;
-  float* sh = srow + grp * D;
-  if (head >= Hq + Hkv) {  // V
-    const int g = head - Hq - Hkv;
-    const uint4* src = reinterpret_cast<const uint4*>(row + (int64_t)(Hq + Hkv) * D + (int64_t)g * DV);
-    if (live) {
-      uint4* dst = reinterpret_cast<uint4*>(kv_layer + (int64_t)slot[t] * Hkv * (D + DV) + (int64_t)Hkv * D + (int64_t)g * DV);
-      for (int v = gl; v < DV * (int)sizeof(E) / 16; v += lanes) dst[v] = src[v];
-    }
-  }
+  float* sh = srow + grp * rot_dim;
   const bool qk = live && head < Hq + Hkv;
   E* x = row + (int64_t)head * D;
-  const float* w = head < Hq ? qw : kw;
+  E* kv_row = kv_layer + (int64_t)slot[t] * Hkv * (D + DV);
+  if (live && !qk) {  // V
+    const int g = head - Hq - Hkv;
+    const uint4* src = reinterpret_cast<const uint4*>(row + (int64_t)(Hq + Hkv) * D + (int64_t)g * DV);
+    uint4* dst = reinterpret_cast<uint4*>(kv_row + (int64_t)Hkv * D + (int64_t)g * DV);
+    for (int v = gl; v < DV * (int)sizeof(E) / 16; v += lanes) dst[v] = src[v];
+  }
+  float f[NIT][8];
   float ss = 0.f;
   if (qk) {
-    for (int d = gl * 8; d < D; d += lanes * 8) {
-      float f[8];
-      if constexpr (sizeof(E) == 2) {
-        unpack8(*reinterpret_cast<const bf16x8*>(x + d), f);
-      } else {
 #pragma unroll
-        for (int i = 0; i < 8; ++i) f[i] = x[d + i];
-      }
+    for (int n = 0; n < NIT; ++n) {
+      const int d = (gl + n * lanes) * 8;
+      if (d >= D) continue;
+      load8(x + d, f[n]);
 #pragma unroll
-      for (int i = 0; i < 8; ++i) {
-        sh[d + i] = f[i];
-        ss = fmaf(f[i], f[i], ss);
-      }
+      for (int i = 0; i < 8; ++i) ss = fmaf(f[n][i], f[n][i], ss);
     }
   }
   for (int o = lanes >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+  const float inv = rsqrtf(ss / (float)dim + eps);
+  const float* w = head < Hq ? qw : kw;
+  if (qk) {
+#pragma unroll
+    for (int n = 0; n < NIT; ++n) {
+      const int d = (gl + n * lanes) * 8;
+      if (d >= D) continue;
+      float wv[8];
+      load8(w + d, wv);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) f[n][i] *= inv * wv[i];
+      if (d < rot_dim) {
+#pragma unroll
+        for (int i = 0; i < 8; ++i)
+          if (d + i < rot_dim) sh[d + i] = f[n][i];
+      }
+    }
+  }
   __syncwarp();
   if (!qk) return;
-  const float inv = rsqrtf(ss / (float)dim + eps);
   const float *cr = cos_t + (int64_t)pos[t] * half, *sr = sin_t + (int64_t)pos[t] * half;
-  E* dst = head < Hq ? x : kv_layer + (int64_t)slot[t] * Hkv * (D + DV) + (int64_t)(head - Hq) * D;
-  for (int d = gl * 8; d < D; d += lanes * 8) {
-    float o[8];
+  E* dst = head < Hq ? x : kv_row + (int64_t)(head - Hq) * D;
 #pragma unroll
-    for (int i = 0; i < 8; ++i) {
-      const int e = d + i;
-      float v = sh[e] * inv * w[e];
-      if (e < half)
-        v = v * cr[e] - sh[e + half] * inv * w[e + half] * sr[e];
-      else if (e < rot_dim)
-        v = v * cr[e - half] + sh[e - half] * inv * w[e - half] * sr[e - half];
-      o[i] = v;
-    }
-    if constexpr (sizeof(E) == 2) {
-      *reinterpret_cast<bf16x8*>(dst + d) = pack8(o);
-    } else {
+  for (int n = 0; n < NIT; ++n) {
+    const int d = (gl + n * lanes) * 8;
+    if (d >= D) continue;
+    if (d < rot_dim) {
 #pragma unroll
-      for (int i = 0; i < 8; ++i) dst[d + i] = o[i];
+      for (int i = 0; i < 8; ++i) {
+        const int e = d + i;
+        if (e < half)
+          f[n][i] = f[n][i] * cr[e] - sh[e + half] * sr[e];
+        else if (e < rot_dim)
+          f[n][i] = f[n][i] * cr[e - half] + sh[e - half] * sr[e - half];
+      }
     }
+    store8(dst + d, f[n]);
   }
 }
 
@@ -284,18 +305,27 @@ LLB_EXPORT int llb_qk_norm_rope_scatter(void* qkv, int dt, int64_t qkv_stride, v
   if (D <= 0 || (D % 8) || DV <= 0 || (DV % 8) || D > 512 || dim <= 0 || dim > D || (rot_dim & 1) || rot_dim > dim ||
       (qkv_stride % 8) || Hkv <= 0)
     return LLB_ERR_UNSUPPORTED;
-  int lanes = 4;
-  while (lanes < 32 && lanes * 8 < D) lanes *= 2;
-  const int groups = 256 / lanes;
-  const int64_t blocks = cdiv64((int64_t)T * (Hq + 2 * Hkv), groups);
-  const size_t smem = (size_t)groups * D * sizeof(float);
-  if (smem > 48 * 1024 || blocks > 0x7fffffff) return LLB_ERR_UNSUPPORTED;
-  if (dt == 0)
-    launch_pdl(qk_norm_rope_scatter_kernel<float>, dim3((unsigned)blocks), dim3(256), smem, st, (float*)qkv, qkv_stride,
-               (float*)kv_layer, cos_t, sin_t, pos, slot, qw, kw, eps, T, Hq, Hkv, D, dim, DV, rot_dim, lanes);
-  else
-    launch_pdl(qk_norm_rope_scatter_kernel<bf16>, dim3((unsigned)blocks), dim3(256), smem, st, (bf16*)qkv, qkv_stride,
-               (bf16*)kv_layer, cos_t, sin_t, pos, slot, qw, kw, eps, T, Hq, Hkv, D, dim, DV, rot_dim, lanes);
+  int lg = 2;
+  while (lg < 5 && (8 << lg) < D) ++lg;
+  const int64_t items = (int64_t)T * (Hq + 2 * Hkv);
+  const int groups = 256 >> lg;
+  const size_t smem = (size_t)groups * rot_dim * sizeof(float);
+  if (smem > 48 * 1024 || items > 0x7fffff00) return LLB_ERR_UNSUPPORTED;
+  const dim3 grid((unsigned)cdiv64(items, groups));
+#define LLB_QK(E, NIT)                                                                                                    \
+  launch_pdl(qk_norm_rope_scatter_kernel<E, NIT>, grid, dim3(256), smem, st, (E*)qkv, qkv_stride, (E*)kv_layer, cos_t,  \
+             sin_t, pos, slot, qw, kw, eps, (unsigned)items, Hq, Hkv, D, dim, DV, rot_dim, lg)
+  if (D <= 256) {
+    if (dt == 0)
+      LLB_QK(float, 1);
+    else
+      LLB_QK(bf16, 1);
+  } else if (dt == 0) {
+    LLB_QK(float, 2);
+  } else {
+    LLB_QK(bf16, 2);
+  }
+#undef LLB_QK
   LLB_LAUNCH_CHECK();
   return LLB_OK;
 }

@@ -13,8 +13,9 @@
 //                  same four columns of every 256 / (dv / 4)-th state row, which it reads and writes once per token.
 // chunked form     prompts in bf16, 64 tokens at a time on tensor cores:
 //   *_prep         decays summed within every chunk (GLA: per channel, with the low-rank product; mLSTM: F, m, i)
-//   chunk_state    a CTA carries a 64 x 64 tile of one state through the request's chunks in registers and leaves the
-//                  state before every chunk as the sum of two bf16 planes
+//   chunk_local    what every chunk adds to the state, decayed to the chunk's end: K'^T V, all chunks side by side
+//   chunk_scan     the recurrence over chunks, elementwise; leaves the state before every chunk as the sum of two bf16
+//                  planes and the last one in the request's row
 //   chunk_output   per (chunk, head): pairs inside the chunk plus the state before it, then the output step
 // Decay factors are only formed between positions where they are at most 1 (or in a range checked to be small), so nothing
 // overflows however strong the decay; fp32 quantities enter tensor-core products as two bf16 planes (high and low part).
@@ -172,7 +173,10 @@ __global__ void __launch_bounds__(256) recurrent_scan_kernel(const Mix p) {
 struct Chunks {
   const int *tok0, *len, *cu_chunk;
   float* decay;            // GLA: [T, H * dk] log decays summed from the chunk's start; mLSTM: F, i, m [3][T, H]
+  float* total;            // decay over the whole chunk: GLA [chunks, H, dk], mLSTM [chunks, H]
   float *m_prev, *n_prev;  // mLSTM: [chunks, H], [chunks, H, dk] before the chunk
+  float* s_loc;            // [chunks, H, dk, dv] what the chunk adds
+  float* n_loc;            // mLSTM: [chunks, H, dk]
   bf16 *s_hi, *s_lo;       // [chunks, H, dk, dv] state before the chunk
   int T;
 };
@@ -215,6 +219,7 @@ __global__ void __launch_bounds__(256) gla_prep_kernel(const Mix p, const Chunks
       // log1p through log: the argument is in (1, 2], the absolute error stays below 1e-7
       sum += (fminf(z[t], 0.f) - __logf(1.f + __expf(-fabsf(z[t])))) * p.inv_tau;
       if (t < len) dst[(int64_t)t * p.H * p.dk] = sum;
+      if (t == len - 1) c.total[((int64_t)ch * p.H + h) * p.dk + d] = __expf(sum);
     }
   }
 }
@@ -263,7 +268,10 @@ __global__ void __launch_bounds__(512) mlstm_prep_kernel(const Mix p, const Chun
       m_end = fmaxf(sF[w] + m_end, sM[w]);  // chunks past the end: (0, -inf)
     }
     m_run = m_end;
-    if (lane == 0 && ch < c1) c.m_prev[(int64_t)ch * p.H + h] = mp;
+    if (lane == 0 && ch < c1) {
+      c.m_prev[(int64_t)ch * p.H + h] = mp;
+      c.total[(int64_t)ch * p.H + h] = __expf(sF[warp] + mp - fmaxf(sF[warp] + mp, sM[warp]));
+    }
 #pragma unroll
     for (int u = 0; u < 2; ++u) {
       Mx = fmaxf(Mx + f[u], in[u]);
@@ -298,147 +306,178 @@ __device__ __forceinline__ void split2(float a, float b, uint32_t& hi, uint32_t&
   lo = pack_bf16x2(a - __uint_as_float(hi << 16), b - __uint_as_float(hi & 0xffff0000u));
 }
 
-struct StateSmem {
-  bf16 k[2][C * TP], v[2][C * TP], kh[C * TP], kl[C * TP];
-  float b[2][C][64];
-  float decay[64], wt[C], npart[2][64];
+struct LocalSmem {
+  bf16 k[C * TP], kh[C * TP], kl[C * TP], v[2][C * TP];
+  float b[C][64];
+  float wt[C];
 };
 
-template <int MODE>
-__global__ void __launch_bounds__(128) chunk_state_kernel(const Mix p, const Chunks c) {
+// NV: 64-column value tiles per CTA (a warp works on 16 key channels x 64 values)
+template <int MODE, int NV>
+__global__ void __launch_bounds__(128 * NV) chunk_local_kernel(const Mix p, const Chunks c) {
   pdl_wait();
+  constexpr int THREADS = 128 * NV;
   extern __shared__ __align__(16) uint8_t raw[];
-  StateSmem& s = *reinterpret_cast<StateSmem*>(raw);
-  const int vt = (p.dv + 63) / 64;
-  const int d0 = (blockIdx.x / vt) * 64, v0 = (blockIdx.x % vt) * 64;
-  const int h = blockIdx.y, b = blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int c0 = c.cu_chunk[b], c1 = c.cu_chunk[b + 1];
-  if (c0 >= c1) return;
-  const int g = lane >> 2, tig = lane & 3;
-  float* row = p.state + (int64_t)p.req[b] * p.state_row;
-  float* S = row + (int64_t)h * p.dk * p.dv;
-  float* n_st = row + (int64_t)p.H * p.dk * p.dv + (int64_t)h * p.dk;
-  const bool fresh = p.first_pos[b] == 0;
-  const bool own_n = MODE == MLSTM && v0 == 0 && tid < 64 && d0 + tid < p.dk;
-  float acc[8][4], n_run = 0.f;
-#pragma unroll
-  for (int j = 0; j < 8; ++j)
-#pragma unroll
-    for (int r = 0; r < 2; ++r) {
-      const int d = d0 + warp * 16 + g + r * 8, v = v0 + j * 8 + tig * 2;
-      float2 x = make_float2(0.f, 0.f);
-      if (!fresh && d < p.dk && v < p.dv) x = *reinterpret_cast<const float2*>(S + (int64_t)d * p.dv + v);
-      acc[j][2 * r] = x.x;
-      acc[j][2 * r + 1] = x.y;
+  LocalSmem& s = *reinterpret_cast<LocalSmem*>(raw);
+  const int vt = (p.dv + 64 * NV - 1) / (64 * NV);
+  const int d0 = (blockIdx.z / vt) * 64, v0 = (blockIdx.z % vt) * 64 * NV;
+  const int ch = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int g = lane >> 2, tig = lane & 3, wr = warp & 3, wv = warp >> 2;
+  const int t0 = c.tok0[ch], len = c.len[ch];
+  load_tile<THREADS>(s.k, (const bf16*)p.k + (int64_t)t0 * p.ld + h * p.dk, p.ld, C, len, d0, p.dk);
+  if (MODE == GLA) {
+    const float* src = c.decay + (int64_t)t0 * p.H * p.dk + h * p.dk;
+    for (int i = tid; i < C * 16; i += THREADS) {
+      const int r = i >> 4, x = (i & 15) * 4;
+      const bool ok = r < len && d0 + x < p.dk;
+      cp_async16(smem_u32(&s.b[r][x]), ok ? src + (int64_t)r * p.H * p.dk + d0 + x : src, ok);
     }
-  if (own_n && !fresh) n_run = n_st[d0 + tid];
-  auto issue = [&](int ch) {
-    if (ch < c1) {
-      const int st = (ch - c0) & 1, t0 = c.tok0[ch], len = c.len[ch];
-      load_tile<128>(s.k[st], (const bf16*)p.k + (int64_t)t0 * p.ld + h * p.dk, p.ld, C, len, d0, p.dk);
-      load_tile<128>(s.v[st], (const bf16*)p.v + (int64_t)t0 * p.ld + h * p.dv, p.ld, C, len, v0, p.dv);
+  }
+  cp_async_commit();
+#pragma unroll
+  for (int j = 0; j < NV; ++j)
+    load_tile<THREADS>(s.v[j], (const bf16*)p.v + (int64_t)t0 * p.ld + h * p.dv, p.ld, C, len, v0 + j * 64, p.dv);
+  cp_async_commit();
+  if (MODE == MLSTM && tid < C) {
+    const float *F = c.decay, *I = F + (int64_t)c.T * p.H, *M = I + (int64_t)c.T * p.H;
+    const int64_t oe = (int64_t)(t0 + len - 1) * p.H + h, o = (int64_t)(t0 + tid) * p.H + h;
+    s.wt[tid] = tid < len ? __expf(F[oe] - F[o] + I[o] - M[oe]) : 0.f;
+  }
+  cp_async_wait<1>();
+  __syncthreads();
+  {  // keys times their decay to the chunk's end, as two planes: two channels per thread
+    const int d = (tid & 31) * 2, part = tid >> 5;
+    constexpr int TOK = C / (THREADS / 32);
+    float2 be = make_float2(0.f, 0.f);
+    if (MODE == GLA) be = *reinterpret_cast<const float2*>(&s.b[len - 1][d]);
+    float2 ns = make_float2(0.f, 0.f);
+#pragma unroll 8
+    for (int t = part * TOK; t < part * TOK + TOK; ++t) {
+      const uint32_t kk = *reinterpret_cast<const uint32_t*>(s.k + t * TP + d);
+      float x = __uint_as_float(kk << 16), y = __uint_as_float(kk & 0xffff0000u);
       if (MODE == GLA) {
-        const float* src = c.decay + (int64_t)t0 * p.H * p.dk + h * p.dk;
-        for (int i = tid; i < C * 16; i += 128) {
-          const int r = i >> 4, x = (i & 15) * 4;
-          const bool ok = r < len && d0 + x < p.dk;
-          cp_async16(smem_u32(&s.b[st][r][x]), ok ? src + (int64_t)r * p.H * p.dk + d0 + x : src, ok);
-        }
-      }
-    }
-    cp_async_commit();
-  };
-  issue(c0);
-  for (int ch = c0; ch < c1; ++ch) {
-    issue(ch + 1);
-    const int st = (ch - c0) & 1, t0 = c.tok0[ch], len = c.len[ch];
-    float decay = 1.f;
-    if (MODE == MLSTM) {
-      const float *F = c.decay, *I = F + (int64_t)c.T * p.H, *M = I + (int64_t)c.T * p.H;
-      const int64_t oe = (int64_t)(t0 + len - 1) * p.H + h;
-      const float Fe = F[oe], Me = M[oe];
-      decay = __expf(Fe + c.m_prev[(int64_t)ch * p.H + h] - Me);
-      if (tid < C) {
-        const int64_t o = (int64_t)(t0 + tid) * p.H + h;
-        s.wt[tid] = tid < len ? __expf(Fe - F[o] + I[o] - Me) : 0.f;
-      }
-      if (own_n) c.n_prev[((int64_t)ch * p.H + h) * p.dk + d0 + tid] = n_run;
-    }
-    // the state before this chunk
-    const int64_t base = ((int64_t)ch * p.H + h) * p.dk * p.dv;
-#pragma unroll
-    for (int j = 0; j < 8; ++j)
-#pragma unroll
-      for (int r = 0; r < 2; ++r) {
-        const int d = d0 + warp * 16 + g + r * 8, v = v0 + j * 8 + tig * 2;
-        if (d < p.dk && v < p.dv) {
-          uint32_t hi, lo;
-          split2(acc[j][2 * r], acc[j][2 * r + 1], hi, lo);
-          *reinterpret_cast<uint32_t*>(c.s_hi + base + (int64_t)d * p.dv + v) = hi;
-          *reinterpret_cast<uint32_t*>(c.s_lo + base + (int64_t)d * p.dv + v) = lo;
-        }
-      }
-    cp_async_wait<1>();
-    __syncthreads();
-    {  // keys times their decay to the chunk's end, as two planes
-      const int d = tid & 63, hf = tid >> 6;
-      const float be = MODE == GLA ? s.b[st][len - 1][d] : 0.f;
-      float ns = 0.f;
-#pragma unroll 4
-      for (int t = hf * 32; t < hf * 32 + 32; ++t) {
-        const float w = MODE == GLA ? __expf(be - s.b[st][t][d]) : s.wt[t];
-        const float x = __bfloat162float(s.k[st][t * TP + d]) * w;
-        const bf16 hi = __float2bfloat16(x);
-        s.kh[t * TP + d] = hi;
-        s.kl[t * TP + d] = __float2bfloat16(x - __bfloat162float(hi));
-        ns += x;
-      }
-      if (MODE == GLA) {
-        if (hf == 0) s.decay[d] = __expf(be);
+        const float2 bb = *reinterpret_cast<const float2*>(&s.b[t][d]);
+        x *= __expf(be.x - bb.x);
+        y *= __expf(be.y - bb.y);
       } else {
-        s.npart[hf][d] = ns;
+        x *= s.wt[t];
+        y *= s.wt[t];
+        ns.x += x;
+        ns.y += y;
       }
+      uint32_t hi, lo;
+      split2(x, y, hi, lo);
+      *reinterpret_cast<uint32_t*>(s.kh + t * TP + d) = hi;
+      *reinterpret_cast<uint32_t*>(s.kl + t * TP + d) = lo;
     }
-    __syncthreads();
-    if (own_n) n_run = decay * n_run + s.npart[0][tid] + s.npart[1][tid];
-    const float e0 = MODE == GLA ? s.decay[warp * 16 + g] : decay, e1 = MODE == GLA ? s.decay[warp * 16 + g + 8] : decay;
-#pragma unroll
-    for (int j = 0; j < 8; ++j) {
-      acc[j][0] *= e0;
-      acc[j][1] *= e0;
-      acc[j][2] *= e1;
-      acc[j][3] *= e1;
+    if (MODE == MLSTM && v0 == 0) {  // sums over the tokens through the (now idle) decay tile, in a fixed order
+      s.b[part][d] = ns.x;
+      s.b[part][d + 1] = ns.y;
     }
-#pragma unroll
-    for (int ks = 0; ks < C / 16; ++ks) {
-      if (ks * 16 >= len) break;
-      uint32_t ah[4], al[4];
-      const int at = ks * 16 + (lane >> 4) * 8 + (lane & 7), ad = warp * 16 + ((lane >> 3) & 1) * 8;
-      ldmatrix_x4_trans(ah[0], ah[1], ah[2], ah[3], smem_u32(s.kh + at * TP + ad));
-      ldmatrix_x4_trans(al[0], al[1], al[2], al[3], smem_u32(s.kl + at * TP + ad));
-      const int bt = ks * 16 + (lane & 7) + ((lane >> 3) & 1) * 8;
-#pragma unroll
-      for (int n2 = 0; n2 < 4; ++n2) {
-        uint32_t b0, b1, b2, b3;
-        ldmatrix_x4_trans(b0, b1, b2, b3, smem_u32(s.v[st] + bt * TP + n2 * 16 + (lane >> 4) * 8));
-        mma_bf16_16816(acc[2 * n2], ah[0], ah[1], ah[2], ah[3], b0, b1);
-        mma_bf16_16816(acc[2 * n2 + 1], ah[0], ah[1], ah[2], ah[3], b2, b3);
-        mma_bf16_16816(acc[2 * n2], al[0], al[1], al[2], al[3], b0, b1);
-        mma_bf16_16816(acc[2 * n2 + 1], al[0], al[1], al[2], al[3], b2, b3);
-      }
-    }
-    __syncthreads();
   }
   cp_async_wait<0>();
+  __syncthreads();
+  if (MODE == MLSTM && v0 == 0 && tid < 64 && d0 + tid < p.dk) {
+    float n = 0.f;
+#pragma unroll
+    for (int i = 0; i < THREADS / 32; ++i) n += s.b[i][tid];
+    c.n_loc[((int64_t)ch * p.H + h) * p.dk + d0 + tid] = n;
+  }
+  float acc[8][4] = {};
+#pragma unroll
+  for (int ks = 0; ks < C / 16; ++ks) {
+    if (ks * 16 >= len) break;
+    uint32_t ah[4], al[4];
+    const int at = ks * 16 + (lane >> 4) * 8 + (lane & 7), ad = wr * 16 + ((lane >> 3) & 1) * 8;
+    ldmatrix_x4_trans(ah[0], ah[1], ah[2], ah[3], smem_u32(s.kh + at * TP + ad));
+    ldmatrix_x4_trans(al[0], al[1], al[2], al[3], smem_u32(s.kl + at * TP + ad));
+    const int bt = ks * 16 + (lane & 7) + ((lane >> 3) & 1) * 8;
+#pragma unroll
+    for (int n2 = 0; n2 < 4; ++n2) {
+      uint32_t b0, b1, b2, b3;
+      ldmatrix_x4_trans(b0, b1, b2, b3, smem_u32(s.v[wv] + bt * TP + n2 * 16 + (lane >> 4) * 8));
+      mma_bf16_16816(acc[2 * n2], ah[0], ah[1], ah[2], ah[3], b0, b1);
+      mma_bf16_16816(acc[2 * n2 + 1], ah[0], ah[1], ah[2], ah[3], b2, b3);
+      mma_bf16_16816(acc[2 * n2], al[0], al[1], al[2], al[3], b0, b1);
+      mma_bf16_16816(acc[2 * n2 + 1], al[0], al[1], al[2], al[3], b2, b3);
+    }
+  }
+  float* dst = c.s_loc + ((int64_t)ch * p.H + h) * p.dk * p.dv;
 #pragma unroll
   for (int j = 0; j < 8; ++j)
 #pragma unroll
     for (int r = 0; r < 2; ++r) {
-      const int d = d0 + warp * 16 + g + r * 8, v = v0 + j * 8 + tig * 2;
+      const int d = d0 + wr * 16 + g + r * 8, v = v0 + wv * 64 + j * 8 + tig * 2;
       if (d < p.dk && v < p.dv)
-        *reinterpret_cast<float2*>(S + (int64_t)d * p.dv + v) = make_float2(acc[j][2 * r], acc[j][2 * r + 1]);
+        *reinterpret_cast<float2*>(dst + (int64_t)d * p.dv + v) = make_float2(acc[j][2 * r], acc[j][2 * r + 1]);
     }
-  if (own_n) n_st[d0 + tid] = n_run;
+}
+
+// A thread carries four neighbouring values of one state row through the request's chunks.
+template <int MODE>
+__global__ void __launch_bounds__(256) chunk_scan_kernel(const Mix p, const Chunks c) {
+  pdl_wait();
+  constexpr int U = 8;  // chunks in flight
+  const int h = blockIdx.y, b = blockIdx.z;
+  const int c0 = c.cu_chunk[b], c1 = c.cu_chunk[b + 1];
+  if (c0 >= c1) return;
+  const int n4 = p.dk * p.dv / 4;
+  const int i = blockIdx.x * 256 + threadIdx.x;
+  float* row = p.state + (int64_t)p.req[b] * p.state_row;
+  const bool fresh = p.first_pos[b] == 0;
+  auto decay = [&](int ch, int d) {
+    return MODE == GLA ? c.total[((int64_t)ch * p.H + h) * p.dk + d] : c.total[(int64_t)ch * p.H + h];
+  };
+  if (i < n4) {
+    const int d = i / (p.dv / 4);
+    float4* S = reinterpret_cast<float4*>(row + (int64_t)h * p.dk * p.dv) + i;
+    float4 x = fresh ? make_float4(0.f, 0.f, 0.f, 0.f) : *S;
+    for (int cb = c0; cb < c1; cb += U) {
+      float4 a[U];
+      float e[U];
+#pragma unroll
+      for (int u = 0; u < U; ++u) {
+        if (cb + u < c1) {
+          a[u] = reinterpret_cast<const float4*>(c.s_loc + ((int64_t)(cb + u) * p.H + h) * p.dk * p.dv)[i];
+          e[u] = decay(cb + u, d);
+        }
+      }
+#pragma unroll
+      for (int u = 0; u < U; ++u) {
+        if (cb + u < c1) {
+          uint2 hi, lo;
+          split2(x.x, x.y, hi.x, lo.x);
+          split2(x.z, x.w, hi.y, lo.y);
+          const int64_t o = ((int64_t)(cb + u) * p.H + h) * n4 + i;
+          reinterpret_cast<uint2*>(c.s_hi)[o] = hi;
+          reinterpret_cast<uint2*>(c.s_lo)[o] = lo;
+          x = make_float4(fmaf(e[u], x.x, a[u].x), fmaf(e[u], x.y, a[u].y), fmaf(e[u], x.z, a[u].z), fmaf(e[u], x.w, a[u].w));
+        }
+      }
+    }
+    *S = x;
+  }
+  if (MODE == MLSTM && blockIdx.x == 0) {
+    float* n_st = row + (int64_t)p.H * p.dk * p.dv + (int64_t)h * p.dk;
+    for (int d = threadIdx.x; d < p.dk; d += 256) {
+      float n = fresh ? 0.f : n_st[d];
+      for (int cb = c0; cb < c1; cb += U) {
+        float a[U], e[U];
+#pragma unroll
+        for (int u = 0; u < U; ++u) {
+          if (cb + u < c1) a[u] = c.n_loc[((int64_t)(cb + u) * p.H + h) * p.dk + d], e[u] = decay(cb + u, d);
+        }
+#pragma unroll
+        for (int u = 0; u < U; ++u) {
+          if (cb + u < c1) {
+            c.n_prev[((int64_t)(cb + u) * p.H + h) * p.dk + d] = n;
+            n = fmaf(e[u], n, a[u]);
+          }
+        }
+      }
+      n_st[d] = n;
+    }
+  }
 }
 
 // shared memory of chunk_output, in bytes, for key size dk
@@ -785,10 +824,20 @@ int launch_chunks(const Mix& p, const Chunks& c, int B, int n_chunks, cudaStream
     launch_pdl(mlstm_prep_kernel, dim3(p.H, B), dim3(512), 0, st, p, c);
   }
   LLB_LAUNCH_CHECK();
-  static DeviceOnce once;
-  int rc = opt_in(chunk_state_kernel<MODE>, (int)sizeof(StateSmem), once);
-  if (rc) return rc;
-  launch_pdl(chunk_state_kernel<MODE>, dim3(cdiv(p.dk, 64) * cdiv(p.dv, 64), p.H, B), dim3(128), sizeof(StateSmem), st, p, c);
+  if (p.dv > 64) {
+    static DeviceOnce once;
+    int rc = opt_in(chunk_local_kernel<MODE, 2>, (int)sizeof(LocalSmem), once);
+    if (rc) return rc;
+    launch_pdl(chunk_local_kernel<MODE, 2>, dim3(n_chunks, p.H, cdiv(p.dk, 64) * cdiv(p.dv, 128)), dim3(256),
+               sizeof(LocalSmem), st, p, c);
+  } else {
+    static DeviceOnce once;
+    int rc = opt_in(chunk_local_kernel<MODE, 1>, (int)sizeof(LocalSmem), once);
+    if (rc) return rc;
+    launch_pdl(chunk_local_kernel<MODE, 1>, dim3(n_chunks, p.H, cdiv(p.dk, 64)), dim3(128), sizeof(LocalSmem), st, p, c);
+  }
+  LLB_LAUNCH_CHECK();
+  launch_pdl(chunk_scan_kernel<MODE>, dim3(cdiv(p.dk * p.dv / 4, 256), p.H, B), dim3(256), 0, st, p, c);
   LLB_LAUNCH_CHECK();
   const int vt = cdiv(p.dv, 64);
   if (vt == 1) return launch_output<MODE, 1>(p, c, n_chunks, st);
@@ -836,13 +885,15 @@ LLB_EXPORT int llb_recurrent_scan(int kind, int dt, const void* q, const void* k
 }
 
 // bf16 prompts.  tok0, len [n_chunks], cu_chunk [B + 1]; decay: fp32 scratch [T, H * dk] (GLA) or [3, T, H] (mLSTM);
-// m_prev [n_chunks, H], n_prev [n_chunks, H, dk] (mLSTM); s_hi, s_lo: bf16 scratch [n_chunks, H, dk, dv].
+// total: fp32 scratch [n_chunks, H * dk] (GLA) or [n_chunks, H]; m_prev [n_chunks, H], n_prev and n_loc [n_chunks, H, dk] (mLSTM); s_loc: fp32, s_hi, s_lo: bf16 scratch
+// [n_chunks, H, dk, dv].
 LLB_EXPORT int llb_recurrent_chunks(int kind, const void* q, const void* k, const void* v, const void* g, int64_t ld,
                                     const void* a1, const void* a2, const float* a2b, int rank, float inv_tau,
                                     const float* zi, const float* zf, int64_t ldz, float cap, float* state,
                                     int64_t state_row, const float* w, int w_stride, float eps, void* out, int64_t out_ld,
                                     float out_scale, const int* req, const int* first_pos, const int* tok0, const int* len,
-                                    const int* cu_chunk, float* decay, float* m_prev, float* n_prev, void* s_hi, void* s_lo,
+                                    const int* cu_chunk, float* decay, float* total, float* m_prev, float* n_prev, float* n_loc, float* s_loc,
+                                    void* s_hi, void* s_lo,
                                     int T, int n_chunks, int B, int H, int dk, int dv, int dim, int vdim,
                                     cudaStream_t st) {
   if (B <= 0 || n_chunks <= 0) return LLB_OK;
@@ -851,7 +902,7 @@ LLB_EXPORT int llb_recurrent_chunks(int kind, const void* q, const void* k, cons
   if (!sizes_ok(p, B) || dk > 256 || dv > 512 || (kind == GLA && rank > 128)) return LLB_ERR_UNSUPPORTED;
   if ((ld % 8) || (out_ld % 2) || (((uintptr_t)q | (uintptr_t)k | (uintptr_t)v) & 15) || (((uintptr_t)g | (uintptr_t)out) & 3))
     return LLB_ERR_BAD_ARG;
-  const Chunks c{tok0, len, cu_chunk, decay, m_prev, n_prev, (bf16*)s_hi, (bf16*)s_lo, T};
+  const Chunks c{tok0, len, cu_chunk, decay, total, m_prev, n_prev, s_loc, n_loc, (bf16*)s_hi, (bf16*)s_lo, T};
   if (kind == GLA) return launch_chunks<GLA>(p, c, B, n_chunks, st);
   if (kind == MLSTM) return launch_chunks<MLSTM>(p, c, B, n_chunks, st);
   return LLB_ERR_UNSUPPORTED;

@@ -233,15 +233,18 @@ class DecayedState:
             return out
         n, dev = plan.count, q.device
         decay = torch.empty(T * self.H * (self.dk if kind == 0 else 3), dtype=torch.float32, device=dev)
-        m_prev = n_prev = None
+        total = torch.empty(n * self.H * (self.dk if kind == 0 else 1), dtype=torch.float32, device=dev)
+        m_prev, norms = None, (None, None)
         if kind == 1:
             m_prev = torch.empty(n * self.H, dtype=torch.float32, device=dev)
-            n_prev = torch.empty(n * self.H * self.dk, dtype=torch.float32, device=dev)
+            norms = torch.empty((2, n * self.H * self.dk), dtype=torch.float32, device=dev)
+        local = torch.empty(n * self.H * self.dk * self.dv, dtype=torch.float32, device=dev)
         planes = torch.empty((2, n * self.H * self.dk * self.dv), dtype=torch.bfloat16, device=dev)
         check(kernels().llb_recurrent_chunks(c_int(kind), *common, ptr(first), ptr(plan.tok0), ptr(plan.len),
-                                             ptr(plan.cu_chunk), ptr(decay), ptr(m_prev), ptr(n_prev), ptr(planes[0]),
-                                             ptr(planes[1]), c_int(T), c_int(n), *sizes), "recurrent_chunks")
-        _count(3)
+                                             ptr(plan.cu_chunk), ptr(decay), ptr(total), ptr(m_prev), ptr(norms[0]),
+                                             ptr(norms[1]), ptr(local), ptr(planes[0]), ptr(planes[1]), c_int(T), c_int(n), *sizes),
+              "recurrent_chunks")
+        _count(4)
         return out
 
     def _torch(self, q, k, v, g, state, st, a1, zi, zf, out):

@@ -117,15 +117,10 @@ def replayer(path, tgt, pool=512, **kw):
 
 
 def close(got, want, tgt, what=""):
-    """Both [n, vocab]: root-mean-square error over the vocabulary against the logits' own.  In bf16 a token whose router
-    scores are close may go to another expert: a few positions may be far off."""
+    """Both [n, vocab]: root-mean-square error over the vocabulary against the logits' own."""
     want = want.double()
     err = (torch.as_tensor(got).double() - want).pow(2).mean(-1).sqrt() / want.pow(2).mean().sqrt()
-    if tgt[1] == "bfloat16":
-        mid, most = (5e-2, 0.25) if len(err) >= 20 else (0.15, 0.5)
-        assert err.median() < mid and err.quantile(0.9) < most, (what, err.median(), err.quantile(0.9))
-    else:
-        assert err.max() < 5e-5, (what, err.argmax(), err.max())
+    assert err.max() < (6e-2 if tgt[1] == "bfloat16" else 5e-5), (what, err.argmax(), err.max(), err.median())
 
 
 def tokens(n, seed, vocab=VOCAB):
@@ -144,9 +139,18 @@ def run_portions(rep, name, toks, portions):
 
 
 @pytest.fixture(scope="module")
-def mixed_model(tmp_path_factory):
-    t = weights(MIXED, 1, RANKS)
-    return write(tmp_path_factory.mktemp("libulorn"), MIXED, t), t
+def models(tmp_path_factory):
+    """number format -> (folder, configuration, weights).  In bf16 every token uses all experts: with fewer, a token whose
+    router scores are close goes to another expert after rounding, which says nothing about the rest of the layer."""
+    out = {}
+    for dt in ("float32", "bfloat16"):
+        cfg = json.loads(json.dumps(MIXED))
+        for l in cfg["layers"]:
+            if dt == "bfloat16" and l["mlp"]:
+                l["mlp"]["router"]["top"] = l["mlp"]["router"]["experts"]
+        t = weights(cfg, 1, RANKS)
+        out[dt] = write(tmp_path_factory.mktemp("libulorn"), cfg, t), cfg, t
+    return out
 
 
 # ------------------------------------------------------------------------------------------------ mechanisms alone (CPU)
@@ -266,10 +270,10 @@ def test_add_rms_operator():
 
 # ------------------------------------------------------------------------------------------------ the engine
 @target
-def test_stream_after_every_layer(mixed_model, tgt):
-    path, t = mixed_model
+def test_stream_after_every_layer(models, tgt):
+    path, cfg, t = models[tgt[1]]
     toks, want, got = tokens(60, 7), [], []
-    plain.forward(t, MIXED, toks, streams=want)
+    plain.forward(t, cfg, toks, streams=want)
     rep = replayer(path, tgt)
     rep.llm.model.stream_tap = lambda i, x: got.append(x[:, : MIXED["width"]].double().cpu())
     rep.step([("a", toks, [])])
@@ -279,10 +283,10 @@ def test_stream_after_every_layer(mixed_model, tgt):
 
 
 @target
-def test_prompt_decode_and_portions(mixed_model, tgt):
-    path, t = mixed_model
+def test_prompt_decode_and_portions(models, tgt):
+    path, cfg, t = models[tgt[1]]
     toks = tokens(139, 2)
-    want = plain.forward(t, MIXED, toks)
+    want = plain.forward(t, cfg, toks)
     rep = replayer(path, tgt)
     for portions in ([139], [1], [2], [9, 10], [37, 36, 1], [64], [65, 63, 1], [100, 3, 1]):
         close(run_portions(rep, f"p{portions}", toks, portions), want, tgt, portions)
@@ -290,23 +294,23 @@ def test_prompt_decode_and_portions(mixed_model, tgt):
 
 
 @target
-def test_first_tokens(mixed_model, tgt):
-    path, t = mixed_model
+def test_first_tokens(models, tgt):
+    path, cfg, t = models[tgt[1]]
     rep = replayer(path, tgt)
     for n in (1, 2, 3, 5):
         toks = tokens(n, 40 + n)
-        close(run_portions(rep, f"w{n}", toks, [n]), plain.forward(t, MIXED, toks), tgt)
-        close(run_portions(rep, f"s{n}", toks, [1]), plain.forward(t, MIXED, toks), tgt)
+        close(run_portions(rep, f"w{n}", toks, [n]), plain.forward(t, cfg, toks), tgt)
+        close(run_portions(rep, f"s{n}", toks, [1]), plain.forward(t, cfg, toks), tgt)
 
 
 @target
-def test_unequal_batches_and_reused_slots(mixed_model, tgt):
+def test_unequal_batches_and_reused_slots(models, tgt):
     """Four live requests in one step, portions beside single tokens, in a pool they fill: requests end and their cache
     and state slots are used again by others, and requests rest for some steps."""
-    path, t = mixed_model
+    path, cfg, t = models[tgt[1]]
     lens = {"a": 90, "b": 33, "c": 150, "d": 7, "e": 70, "f": 41, "g": 128}
     toks = {k: tokens(n, 60 + i) for i, (k, n) in enumerate(lens.items())}
-    want = {k: plain.forward(t, MIXED, v) for k, v in toks.items()}
+    want = {k: plain.forward(t, cfg, v) for k, v in toks.items()}
     rep = replayer(path, tgt, pool=320)
     g = torch.Generator().manual_seed(5)
     at, waiting, live, seen = {k: 0 for k in lens}, list(lens), [], {k: [] for k in lens}
@@ -419,10 +423,10 @@ def test_state_remembers_far_tokens(tmp_path, tgt, kind):
 
 
 @target
-def test_long_decoding_and_greedy_generation(mixed_model, tgt):
+def test_long_decoding_and_greedy_generation(models, tgt):
     """Greedy generation through the engine's own scheduler: every produced token is the arg-max of the plain restatement up
     to rounding, far beyond the windows; a second run starts from snapshots of the recurrent state."""
-    path, t = mixed_model
+    path, cfg, t = models[tgt[1]]
     llm = LLM(model_dir=path, data_type=tgt[1], max_total_token_num=2000, running_max_req_size=4, max_req_total_len=400,
               chunked_prefill_size=48, batch_max_tokens=96, state_snapshot_slots=24, linear_att_hash_page_size=32,
               pstate=pstate(tgt))
@@ -432,13 +436,10 @@ def test_long_decoding_and_greedy_generation(mixed_model, tgt):
     for p, o, o2 in zip(prompts, outs, again):
         assert len(o["token_ids"]) == 120
         for out in (o, o2):
-            lg = plain.forward(t, MIXED, p + out["token_ids"])[len(p) - 1:-1]
+            lg = plain.forward(t, cfg, p + out["token_ids"])[len(p) - 1:-1]
             chosen = lg.gather(1, torch.tensor(out["token_ids"])[:, None])[:, 0]
             gap = lg.max(-1)[0] - chosen
-            if tgt[1] == "bfloat16":
-                assert (gap > 0.2).float().mean() < 0.1
-            else:
-                assert gap.max() < 1e-3
+            assert gap.max() < (0.1 * lg.std() if tgt[1] == "bfloat16" else 1e-3)
     assert again[2]["prompt_cache_len"] > 0 and llm.backend.state_cache.stats["hits"] > 0
     llm.close()
 
@@ -465,8 +466,8 @@ def test_recurrent_layers_only(tmp_path):
     assert pages.shape == (1, 3, 0)
 
 
-def test_pages_carry_every_layer(mixed_model):
-    mm = replayer(mixed_model[0], ("cpu", "float32")).llm.model.mem_manager
+def test_pages_carry_every_layer(models):
+    mm = replayer(models["float32"][0], ("cpu", "float32")).llm.model.mem_manager
     for i, buf in enumerate(mm.kv_layers):
         buf.normal_(generator=torch.Generator().manual_seed(i))
     src, dst = torch.tensor([3, 9], dtype=torch.int32), torch.tensor([20, 1], dtype=torch.int32)
@@ -534,10 +535,10 @@ def test_wrong_checkpoints_are_refused(tmp_path):
     _bad(tmp_path, "no quantised form", kv_type="int8kv")
 
 
-def test_trace_run_program(tmp_path, mixed_model):
+def test_trace_run_program(tmp_path, models):
     import numpy as np
 
-    path, t = mixed_model
+    path, _, t = models["float32"]
     a, b = tokens(70, 1), tokens(9, 2)
     lines = [{"step": 0, "entries": [{"id": "a", "tokens": a[:50], "want": [0, 49]}], "end": []},
              {"step": 1, "entries": [{"id": "b", "tokens": b[:8], "want": []}, {"id": "a", "tokens": a[50:51], "want": []}],
