@@ -181,46 +181,61 @@ struct Chunks {
   int T;
 };
 
-__global__ void __launch_bounds__(256) gla_prep_kernel(const Mix p, const Chunks c) {
+// Two threads per key channel, one for either half of the chunk's tokens.
+__global__ void __launch_bounds__(512) gla_prep_kernel(const Mix p, const Chunks c) {
   pdl_wait();
-  extern __shared__ float a1s[];  // [C][rank padded to 16]
+  constexpr int HC = C / 2;
+  extern __shared__ float a1s[];  // [C][rank]
+  __shared__ float first[256];    // the first half's sums
   const int ch = blockIdx.x, h = blockIdx.y;
   const int t0 = c.tok0[ch], len = c.len[ch];
-  const int rp = (p.rank + 15) & ~15;
-  for (int i = threadIdx.x; i < C * rp; i += blockDim.x) {
-    const int t = i / rp, r = i - t * rp;
-    a1s[i] = (t < len && r < p.rank) ? ldf((const bf16*)p.a1 + (int64_t)(t0 + t) * p.ld + r) : 0.f;
+  const int rank = p.rank, per = rank >> 3;
+  for (int i = threadIdx.x; i < C * per; i += blockDim.x) {
+    const int t = i / per, r = (i - t * per) * 8;
+    float f[8] = {};
+    if (t < len) unpack8(*reinterpret_cast<const bf16x8*>((const bf16*)p.a1 + (int64_t)(t0 + t) * p.ld + r), f);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) a1s[t * rank + r + e] = f[e];
   }
   __syncthreads();
-  for (int d = threadIdx.x; d < p.dk; d += blockDim.x) {
-    float z[C];
+  const int half = blockDim.x >> 1;
+  const int d = threadIdx.x % half, hf = threadIdx.x / half;
+  const bool live = d < p.dk;
+  float z[HC];
+  if (live) {
     const float bias = p.a2b[h * p.dk + d];
 #pragma unroll
-    for (int t = 0; t < C; ++t) z[t] = bias;
-    const bf16* a2 = (const bf16*)p.a2 + (int64_t)(h * p.dk + d) * p.rank;
-    for (int r0 = 0; r0 < rp; r0 += 16) {
-      float a[16];
+    for (int t = 0; t < HC; ++t) z[t] = bias;
+    const bf16* a2 = (const bf16*)p.a2 + (int64_t)(h * p.dk + d) * rank;
+    for (int r0 = 0; r0 < rank; r0 += 8) {
+      float a[8];
+      unpack8(*reinterpret_cast<const bf16x8*>(a2 + r0), a);
 #pragma unroll
-      for (int r = 0; r < 16; ++r) a[r] = r0 + r < p.rank ? ldf(a2 + r0 + r) : 0.f;
-#pragma unroll
-      for (int t = 0; t < C; ++t) {
-        const float4* x = reinterpret_cast<const float4*>(a1s + t * rp + r0);
-#pragma unroll
-        for (int r = 0; r < 4; ++r) {
-          const float4 y = x[r];
-          z[t] = fmaf(a[4 * r], y.x, fmaf(a[4 * r + 1], y.y, fmaf(a[4 * r + 2], y.z, fmaf(a[4 * r + 3], y.w, z[t]))));
-        }
+      for (int t = 0; t < HC; ++t) {
+        const float4* x = reinterpret_cast<const float4*>(a1s + (hf * HC + t) * rank + r0);
+        const float4 u = x[0], v = x[1];
+        z[t] = fmaf(a[0], u.x, fmaf(a[1], u.y, fmaf(a[2], u.z, fmaf(a[3], u.w, z[t]))));
+        z[t] = fmaf(a[4], v.x, fmaf(a[5], v.y, fmaf(a[6], v.z, fmaf(a[7], v.w, z[t]))));
       }
     }
-    float* dst = c.decay + (int64_t)t0 * p.H * p.dk + h * p.dk + d;
     float sum = 0.f;
 #pragma unroll
-    for (int t = 0; t < C; ++t) {
-      // log1p through log: the argument is in (1, 2], the absolute error stays below 1e-7
-      sum += (fminf(z[t], 0.f) - __logf(1.f + __expf(-fabsf(z[t])))) * p.inv_tau;
-      if (t < len) dst[(int64_t)t * p.H * p.dk] = sum;
-      if (t == len - 1) c.total[((int64_t)ch * p.H + h) * p.dk + d] = __expf(sum);
+    for (int t = 0; t < HC; ++t) {
+      sum += (fminf(z[t], 0.f) - log1pf(__expf(-fabsf(z[t])))) * p.inv_tau;
+      z[t] = sum;
     }
+    if (hf == 0) first[d] = sum;
+  }
+  __syncthreads();
+  if (!live) return;
+  const float before = hf == 0 ? 0.f : first[d];
+  float* dst = c.decay + (int64_t)t0 * p.H * p.dk + h * p.dk + d;
+#pragma unroll
+  for (int t = 0; t < HC; ++t) {
+    const int tt = hf * HC + t;
+    const float v = before + z[t];
+    if (tt < len) dst[(int64_t)tt * p.H * p.dk] = v;
+    if (tt == len - 1) c.total[((int64_t)ch * p.H + h) * p.dk + d] = __expf(v);
   }
 }
 
@@ -542,7 +557,13 @@ __global__ void __launch_bounds__(256) chunk_output_kernel(const Mix p, const Ch
     const int r = tid >> 2;
     const float* n = c.n_prev + ((int64_t)ch * p.H + h) * dk;
     float x = 0.f;
-    for (int d = tid & 3; d < dk; d += 4) x = fmaf(__bfloat162float(qh[r * L.qp + d]), n[d], x);
+    for (int d = (tid & 3) * 8; d < dk; d += 32) {
+      float qf[8];
+      unpack8(*reinterpret_cast<const bf16x8*>(qh + r * L.qp + d), qf);
+      const float4 n0 = *reinterpret_cast<const float4*>(n + d), n1 = *reinterpret_cast<const float4*>(n + d + 4);
+      x = fmaf(qf[0], n0.x, fmaf(qf[1], n0.y, fmaf(qf[2], n0.z, fmaf(qf[3], n0.w, x))));
+      x = fmaf(qf[4], n1.x, fmaf(qf[5], n1.y, fmaf(qf[6], n1.z, fmaf(qf[7], n1.w, x))));
+    }
     x += __shfl_xor_sync(0xffffffffu, x, 1);
     x += __shfl_xor_sync(0xffffffffu, x, 2);
     if ((tid & 3) == 0) s_nq[r] = x;
@@ -817,9 +838,8 @@ int launch_output(const Mix& p, const Chunks& c, int n_chunks, cudaStream_t st) 
 template <int MODE>
 int launch_chunks(const Mix& p, const Chunks& c, int B, int n_chunks, cudaStream_t st) {
   if (MODE == GLA) {
-    const int rp = (p.rank + 15) & ~15;
-    launch_pdl(gla_prep_kernel, dim3(n_chunks, p.H), dim3(p.dk >= 256 ? 256 : cdiv(p.dk, 32) * 32),
-               (size_t)C * rp * sizeof(float), st, p, c);
+    launch_pdl(gla_prep_kernel, dim3(n_chunks, p.H), dim3(2 * cdiv(p.dk, 32) * 32), (size_t)C * p.rank * sizeof(float), st,
+               p, c);
   } else {
     launch_pdl(mlstm_prep_kernel, dim3(p.H, B), dim3(512), 0, st, p, c);
   }
@@ -899,7 +919,8 @@ LLB_EXPORT int llb_recurrent_chunks(int kind, const void* q, const void* k, cons
   if (B <= 0 || n_chunks <= 0) return LLB_OK;
   const Mix p{q,  k,  v,   g,     a1,   a2,        a2b,  zi,     zf,        w, out, state, ld,  ldz, out_ld,
               state_row, req, nullptr, first_pos, H,   dk,   dv, dim, vdim, rank, w_stride, inv_tau, cap, eps, out_scale};
-  if (!sizes_ok(p, B) || dk > 256 || dv > 512 || (kind == GLA && rank > 128)) return LLB_ERR_UNSUPPORTED;
+  if (!sizes_ok(p, B) || dk > 256 || dv > 512 || (kind == GLA && (rank > 128 || rank % 8 || ((uintptr_t)a1 & 15) || ((uintptr_t)a2 & 15))))
+    return LLB_ERR_UNSUPPORTED;
   if ((ld % 8) || (out_ld % 2) || (((uintptr_t)q | (uintptr_t)k | (uintptr_t)v) & 15) || (((uintptr_t)g | (uintptr_t)out) & 3))
     return LLB_ERR_BAD_ARG;
   const Chunks c{tok0, len, cu_chunk, decay, total, m_prev, n_prev, s_loc, n_loc, (bf16*)s_hi, (bf16*)s_lo, T};

@@ -197,7 +197,7 @@ class DecayedState:
 
     @staticmethod
     def chunked_sizes(dk: int, dv: int, rank: int) -> bool:
-        return dk <= 256 and dv <= 512 and rank <= 128
+        return dk <= 256 and dv <= 512 and rank <= 128 and rank % 8 == 0
 
     def __call__(self, q, k, v, g, state, st, a1=None, zi=None, zf=None, out=None, plan=None, token_by_token=False):
         """q, k [T, H * dk], v, g [T, H * dv] (columns of one matrix, or with its row pitch); a1 [T, rank] likewise; zi, zf
