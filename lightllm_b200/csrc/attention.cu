@@ -37,8 +37,9 @@ constexpr float kLn2 = 0.6931471805599453f;
 // ---------------------------------------------------------------------------------------
 // decode
 // ---------------------------------------------------------------------------------------
-// DK, DV: key and value size; pool row [Hkv * DK | Hkv * DV].  window: only the last `window` positions are seen (0: all).
-// SPLIT_P: the weights enter P . V as the sum of two bf16 values (high and low part).  gate (or null): head h of request b
+// DK, DV: key and value size; pool row [Hkv * DK | Hkv * DV].  SPLIT_P (the windowed form): the weights enter P . V as the sum
+// of two bf16 values (high and low part), and `rule` says which positions are seen and which biases the scores get: the kept
+// first positions and the window lie back to back in the key index that is cut into tiles and splits.  gate (or null): head h of request b
 // is multiplied by out_scale * sigmoid(gate[b, h]) when the result is final.
 struct HeadGate {
   const bf16* gate;
@@ -55,7 +56,7 @@ gqa_decode_kernel(const bf16* __restrict__ q, int64_t q_stride, const bf16* __re
                   const int* __restrict__ req_to_token, int64_t r2t_stride, const int* __restrict__ b_req_idx,
                   const int* __restrict__ b_seq_len, bf16* __restrict__ out, int64_t out_stride,
                   float* __restrict__ part_o, float* __restrict__ part_lse, int Hq, int Hkv, int num_splits,
-                  float scale_log2, int window, const HeadGate gate) {
+                  float scale_log2, const KeyRule rule, const HeadGate gate) {
   pdl_wait();
   constexpr int CH = DK / 8, CHV = DV / 8;             // 16-byte chunks per row
   constexpr int TILE_BYTES = 16 * DK * 2;              // 16 tokens' keys
@@ -78,11 +79,14 @@ gqa_decode_kernel(const bf16* __restrict__ q, int64_t q_stride, const bf16* __re
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int g = lane >> 2, tig = lane & 3;
 
-  const int lo = window > 0 ? max(0, L - window) : 0;
-  const int tiles_total = (L - lo + 15) >> 4;
+  const int lo = SPLIT_P && rule.window > 0 ? max(0, L - rule.window) : 0;
+  const int kept = SPLIT_P ? min(rule.keep, lo) : 0;
+  const int skip = lo - kept;  // key index n >= kept is position n + skip
+  const int tiles_total = (L - skip + 15) >> 4;
   const int tiles_per_split = (tiles_total + num_splits - 1) / num_splits;
-  const int s0 = lo + split * tiles_per_split * 16;
-  const int e0 = min(L, s0 + tiles_per_split * 16);
+  const int s0 = split * tiles_per_split * 16;
+  const int e0 = min(L - skip, s0 + tiles_per_split * 16);
+  auto position = [&](int n) { return !SPLIT_P || n < kept ? n : n + skip; };
 
   if (s0 >= e0) {  // empty split: tell the merge kernel to ignore it
     if (num_splits > 1) {
@@ -123,7 +127,7 @@ gqa_decode_kernel(const bf16* __restrict__ q, int64_t q_stride, const bf16* __re
     int slot = -1;
     if (i < my_count) {
       const int p0 = s0 + (warp + 4 * i) * 16;
-      if (lane < 16 && p0 + lane < e0) slot = LLB_CHECK_SLOT(req_to_token[r2t_base + p0 + lane]);
+      if (lane < 16 && p0 + lane < e0) slot = LLB_CHECK_SLOT(req_to_token[r2t_base + position(p0 + lane)]);
     }
     return slot;
   };
@@ -164,6 +168,11 @@ gqa_decode_kernel(const bf16* __restrict__ q, int64_t q_stride, const bf16* __re
   for (int i = 0; i < DV / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
   float m_run[2] = {-INFINITY, -INFINITY};
   float l_run[2] = {0.f, 0.f};
+  const float *rel0 = nullptr, *rel1 = nullptr;  // biases of the heads of my two rows
+  if (SPLIT_P && rule.rel != nullptr) {
+    rel0 = rule.rel + (int64_t)(head0 + min(g, nrows - 1)) * (rule.far + 1);
+    rel1 = rule.rel + (int64_t)(head0 + min(g + 8, nrows - 1)) * (rule.far + 1);
+  }
 
 #pragma unroll
   for (int i = 0; i < STAGES - 1; ++i) issue(i);
@@ -189,14 +198,28 @@ gqa_decode_kernel(const bf16* __restrict__ q, int64_t q_stride, const bf16* __re
         mma_bf16_16816(s[1], qa[ks][0], qa[ks][1], qa[ks][2], qa[ks][3], b2, b3);
       }
     }
-    // scale + tail mask
+    // scale, bias + tail mask
     float mx[2] = {-INFINITY, -INFINITY};
+    float add[2][4];
+    if (SPLIT_P) {
+#pragma unroll
+      for (int j = 0; j < 2; ++j) add[j][0] = add[j][1] = add[j][2] = add[j][3] = 0.f;
+      if (rel0 != nullptr) {
+#pragma unroll
+        for (int j = 0; j < 2; ++j)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const int dist = L - 1 - position(min(p0 + j * 8 + tig * 2 + (e & 1), e0 - 1));
+            add[j][e] = (e < 2 ? rel0 : rel1)[min(dist, rule.far)] * kLog2e;
+          }
+      }
+    }
 #pragma unroll
     for (int j = 0; j < 2; ++j) {
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         int pos = p0 + j * 8 + tig * 2 + (e & 1);
-        float v = pos < e0 ? s[j][e] * scale_log2 : -INFINITY;
+        float v = pos < e0 ? (SPLIT_P ? fmaf(s[j][e], scale_log2, add[j][e]) : s[j][e] * scale_log2) : -INFINITY;
         s[j][e] = v;
         mx[e >> 1] = fmaxf(mx[e >> 1], v);
       }
@@ -544,7 +567,7 @@ LLB_EXPORT int llb_gqa_decode_num_splits(int B, int Hq, int Hkv, int max_seq_len
 template <int DK, int DV, bool SPLIT_P>
 static int launch_decode(const void* q, int64_t q_stride, const void* kv_layer, const int* req_to_token, int64_t r2t_stride,
                          const int* b_req_idx, const int* b_seq_len, void* out, int64_t out_stride, float* part_o,
-                         float* part_lse, int B, int Hq, int Hkv, int num_splits, float sm_scale, int window,
+                         float* part_lse, int B, int Hq, int Hkv, int num_splits, float sm_scale, const KeyRule& rule,
                          const HeadGate& gate, cudaStream_t st) {
   constexpr int STAGES = decode_stages<DK, DV>();
   const int G = Hq / Hkv;
@@ -557,7 +580,7 @@ static int launch_decode(const void* q, int64_t q_stride, const void* kv_layer, 
   }
   launch_pdl(gqa_decode_kernel<DK, DV, STAGES, SPLIT_P>, grid, dim3(128), decode_smem_bytes<DK, DV>(), st, (const bf16*)q,
              q_stride, (const bf16*)kv_layer, req_to_token, r2t_stride, b_req_idx, b_seq_len, (bf16*)out, out_stride, part_o,
-             part_lse, Hq, Hkv, num_splits, sm_scale * kLog2e, window, gate);
+             part_lse, Hq, Hkv, num_splits, sm_scale * kLog2e, rule, gate);
   LLB_LAUNCH_CHECK();
   if (num_splits > 1) {
     launch_pdl(decode_merge_kernel<DV>, dim3(B * Hq), dim3(DV), 0, st, (const float*)part_o, (const float*)part_lse,
@@ -577,30 +600,34 @@ LLB_EXPORT int llb_gqa_decode(const void* q, int64_t q_stride, const void* kv_la
   if (Hkv <= 0 || Hq % Hkv != 0 || num_splits < 1) return LLB_ERR_BAD_ARG;
   if (num_splits > 1 && (part_o == nullptr || part_lse == nullptr)) return LLB_ERR_BAD_ARG;
   const HeadGate none{nullptr, 0, 1.f};
+  const KeyRule all{0, 0, nullptr, 0};
   if (D == 128)
     return launch_decode<128, 128, false>(q, q_stride, kv_layer, req_to_token, r2t_stride, b_req_idx, b_seq_len, out,
-                                          out_stride, part_o, part_lse, B, Hq, Hkv, num_splits, sm_scale, 0, none, st);
+                                          out_stride, part_o, part_lse, B, Hq, Hkv, num_splits, sm_scale, all, none, st);
   if (D == 64)
     return launch_decode<64, 64, false>(q, q_stride, kv_layer, req_to_token, r2t_stride, b_req_idx, b_seq_len, out,
-                                        out_stride, part_o, part_lse, B, Hq, Hkv, num_splits, sm_scale, 0, none, st);
+                                        out_stride, part_o, part_lse, B, Hq, Hkv, num_splits, sm_scale, all, none, st);
   return LLB_ERR_UNSUPPORTED;
 }
 
 // The windowed form: key size dk and value size dv (64, 128, 192 or 256), pool rows [Hkv * dk | Hkv * dv], window (0: none),
-// gate [B, >= Hq] (or null): head h of the output times out_scale * sigmoid(gate).  part_o: fp32 [B, Hq, num_splits, dv].
+// the first `keep` positions always seen, biases by distance rel [Hq, far + 1] (or null), gate [B, >= Hq] (or null): head h of the output times out_scale * sigmoid(gate).  part_o: fp32 [B, Hq, num_splits, dv].
 LLB_EXPORT int llb_window_gqa_decode(const void* q, int64_t q_stride, const void* kv_layer, const int* req_to_token,
                                      int64_t r2t_stride, const int* b_req_idx, const int* b_seq_len, void* out,
                                      int64_t out_stride, float* part_o, float* part_lse, int B, int Hq, int Hkv, int dk,
-                                     int dv, int num_splits, float sm_scale, int window, const void* gate,
-                                     int64_t gate_stride, float out_scale, cudaStream_t st) {
+                                     int dv, int num_splits, float sm_scale, int window, int keep, const float* rel,
+                                     int far, const void* gate, int64_t gate_stride, float out_scale, cudaStream_t st) {
   if (B <= 0) return LLB_OK;
-  if (Hkv <= 0 || Hq % Hkv != 0 || num_splits < 1 || window < 0 || (q_stride % 8) || ((uintptr_t)q & 15)) return LLB_ERR_BAD_ARG;
+  if (Hkv <= 0 || Hq % Hkv != 0 || num_splits < 1 || window < 0 || keep < 0 || (rel != nullptr && far < 0) ||
+      (q_stride % 8) || ((uintptr_t)q & 15))
+    return LLB_ERR_BAD_ARG;
   if (num_splits > 1 && (part_o == nullptr || part_lse == nullptr)) return LLB_ERR_BAD_ARG;
   const HeadGate g{(const bf16*)gate, gate_stride, out_scale};
+  const KeyRule rule{window, keep, rel, far};
 #define LLB_WINDOW_DECODE(DK, DV)                                                                                        \
   if (dk == DK && dv == DV)                                                                                              \
     return launch_decode<DK, DV, true>(q, q_stride, kv_layer, req_to_token, r2t_stride, b_req_idx, b_seq_len, out,       \
-                                       out_stride, part_o, part_lse, B, Hq, Hkv, num_splits, sm_scale, window, g, st);
+                                       out_stride, part_o, part_lse, B, Hq, Hkv, num_splits, sm_scale, rule, g, st);
 #define LLB_WINDOW_DECODE_V(DK)                                                                                          \
   LLB_WINDOW_DECODE(DK, 64) LLB_WINDOW_DECODE(DK, 128) LLB_WINDOW_DECODE(DK, 192) LLB_WINDOW_DECODE(DK, 256)
   LLB_WINDOW_DECODE_V(64)

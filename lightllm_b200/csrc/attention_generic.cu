@@ -1,6 +1,6 @@
 // Paged causal attention for the layer shapes the tensor-core kernels do not cover: any head size up to
 // 256 (Gemma 256, Phi-3 96, StableLM 80 ...; up to 512 in the form with its own value size, in bf16 or fp32),
-// sliding windows, ALiBi slopes, logit soft-capping, attention sinks and a sigmoid output gate per head.  One CTA per (query token, query head); its four warps stride over the keys, each
+// sliding windows (with kept first positions), ALiBi slopes, tables of biases by distance, logit soft-capping, attention sinks and a sigmoid output gate per head.  One CTA per (query token, query head); its four warps stride over the keys, each
 // keeps an online-softmax state with the head vector spread over the lanes, and the states are merged
 // in shared memory.  Prefill and decode use the same kernel: a query is described by its position and
 // the request row it belongs to.
@@ -29,7 +29,7 @@ __global__ void __launch_bounds__(GEN_WARPS * 32)
 attn_generic_kernel(const E* __restrict__ q, int64_t q_stride, const E* __restrict__ kv,
                     const int* __restrict__ req_to_token, int64_t r2t_stride, const int* __restrict__ b_req_idx,
                     const int* __restrict__ pos, const int* __restrict__ batch_of, E* __restrict__ out,
-                    int64_t out_stride, int Hq, int Hkv, int D, int DV, float sm_scale, int window, float softcap,
+                    int64_t out_stride, int Hq, int Hkv, int D, int DV, float sm_scale, const KeyRule rule, float softcap,
                     const float* __restrict__ alibi, const float* __restrict__ sinks, const E* __restrict__ gate,
                     int64_t gate_stride, float out_scale) {
   const int t = blockIdx.x, h = blockIdx.y;
@@ -48,9 +48,12 @@ attn_generic_kernel(const E* __restrict__ q, int64_t q_stride, const E* __restri
     acc[e] = 0.f;
   }
   float m = -INFINITY, l = 0.f;
-  const int j0 = (window > 0 && qpos - window + 1 > 0) ? qpos - window + 1 : 0;
+  const int j0 = (rule.window > 0 && qpos - rule.window + 1 > 0) ? qpos - rule.window + 1 : 0;
+  const int kept = min(rule.keep, j0), n = kept + qpos + 1 - j0;  // kept first positions, then the window
   const float slope = alibi ? alibi[h] : 0.f;
-  for (int j = j0 + warp; j <= qpos; j += GEN_WARPS) {
+  const float* rel = rule.rel ? rule.rel + (int64_t)h * (rule.far + 1) : nullptr;
+  for (int i = warp; i < n; i += GEN_WARPS) {
+    const int j = i < kept ? i : j0 + i - kept;
     const E* kr = kv + (int64_t)slots[j] * row + (int64_t)kvh * D;
     float s = 0.f;
 #pragma unroll
@@ -61,6 +64,7 @@ attn_generic_kernel(const E* __restrict__ q, int64_t q_stride, const E* __restri
     s = warp_sum(s);
     if (softcap > 0.f) s = softcap * tanhf(s / softcap);
     s += slope * (float)(j - qpos);
+    if (rel) s += rel[min(qpos - j, rule.far)];
     const float mn = fmaxf(m, s);
     const float corr = exp_for(m - mn, q), p = exp_for(s - mn, q);
     l = l * corr + p;
@@ -116,23 +120,27 @@ LLB_EXPORT int llb_attn_generic(const void* q, int64_t q_stride, const void* kv_
   dim3 grid(T, Hq);
   attn_generic_kernel<bf16, GEN_MAX_EPL><<<grid, GEN_WARPS * 32, 0, st>>>(
       (const bf16*)q, q_stride, (const bf16*)kv_layer, req_to_token, r2t_stride, b_req_idx, pos, batch_of, (bf16*)out,
-      out_stride, Hq, Hkv, D, D, sm_scale, window, softcap, alibi_slopes, sinks, nullptr, 0, 1.f);
+      out_stride, Hq, Hkv, D, D, sm_scale, KeyRule{window, 0, nullptr, 0}, softcap, alibi_slopes, sinks, nullptr, 0, 1.f);
   LLB_LAUNCH_CHECK();
   return LLB_OK;
 }
 
-// The form with a value size of its own, an output gate per head, and fp32 (dt 0) beside bf16 (dt 1).
+// The form with a value size of its own, kept first positions, biases by distance (see KeyRule), an output gate per head, and
+// fp32 (dt 0) beside bf16 (dt 1).
 LLB_EXPORT int llb_attn_generic_kv(const void* q, int dt, int64_t q_stride, const void* kv_layer, const int* req_to_token,
                                    int64_t r2t_stride, const int* b_req_idx, const int* pos, const int* batch_of,
                                    void* out, int64_t out_stride, int T, int Hq, int Hkv, int D, int DV, float sm_scale,
-                                   int window, const void* gate, int64_t gate_stride, float out_scale, cudaStream_t st) {
+                                   int window, int keep, const float* rel, int far, const void* gate,
+                                   int64_t gate_stride, float out_scale, cudaStream_t st) {
   if (T <= 0) return LLB_OK;
+  if (window < 0 || keep < 0 || (rel != nullptr && far < 0)) return LLB_ERR_BAD_ARG;
+  const KeyRule rule{window, keep, rel, far};
   if (D <= 0 || DV <= 0 || D > 512 || DV > 512 || Hkv <= 0 || Hq % Hkv != 0 || Hq > 65535) return LLB_ERR_UNSUPPORTED;
   const dim3 grid(T, Hq);
 #define LLB_GENERIC(E, EPL)                                                                                           \
   attn_generic_kernel<E, EPL><<<grid, GEN_WARPS * 32, 0, st>>>(                                                       \
       (const E*)q, q_stride, (const E*)kv_layer, req_to_token, r2t_stride, b_req_idx, pos, batch_of, (E*)out,         \
-      out_stride, Hq, Hkv, D, DV, sm_scale, window, 0.f, nullptr, nullptr, (const E*)gate, gate_stride, out_scale)
+      out_stride, Hq, Hkv, D, DV, sm_scale, rule, 0.f, nullptr, nullptr, (const E*)gate, gate_stride, out_scale)
   if (D <= 128 && DV <= 128) {
     if (dt == 0)
       LLB_GENERIC(float, 4);
@@ -200,9 +208,10 @@ LLB_EXPORT int llb_rope_kv_scatter_generic(void* qkv, void* kv_layer, const floa
   return LLB_OK;
 }
 
-// Per-head RMS norm of q and k over the first `dim` of their D elements, rotary positions on the first rot_dim, and the
-// cache write, for layers whose value size DV differs from the key size D.  qkv row: [Hq * D | Hkv * D | Hkv * DV]; q is
-// rewritten in place, K and V go to kv_layer[slot].  Sizes are multiples of 8; a group of 2^k lanes works on one head, a lane
+// Per-head RMS norm of q and k over the first `dim` of their D elements (a null weight is all ones), rotary positions on the
+// first rot_dim, and the cache write, for layers whose value size DV differs from the key size D.  A norm without a weight
+// commutes with the rotation.  qkv row: [Hq * D | Hkv * D | Hkv * DV]; q is rewritten in place, K and V go to kv_layer[slot].
+// Hkv = 0: queries only (a layer that reads another layer's cache).  Sizes are multiples of 8; a group of 2^k lanes works on one head, a lane
 // on 8 elements of it (NIT times, 8 * lanes apart); rotation partners meet in shared memory.
 __device__ __forceinline__ void load8(const bf16* p, float* f) { unpack8(*reinterpret_cast<const bf16x8*>(p), f); }
 __device__ __forceinline__ void load8(const float* p, float* f) {
@@ -236,7 +245,7 @@ qk_norm_rope_scatter_kernel(E* __restrict__ qkv, int64_t qkv_stride, E* __restri
   float* sh = srow + grp * rot_dim;
   const bool qk = live && head < Hq + Hkv;
   E* x = row + (int64_t)head * D;
-  E* kv_row = kv_layer + (int64_t)slot[t] * Hkv * (D + DV);
+  E* kv_row = Hkv > 0 ? kv_layer + (int64_t)slot[t] * Hkv * (D + DV) : nullptr;
   if (live && !qk) {  // V
     const int g = head - Hq - Hkv;
     const uint4* src = reinterpret_cast<const uint4*>(row + (int64_t)(Hq + Hkv) * D + (int64_t)g * DV);
@@ -264,9 +273,9 @@ qk_norm_rope_scatter_kernel(E* __restrict__ qkv, int64_t qkv_stride, E* __restri
       const int d = (gl + n * lanes) * 8;
       if (d >= D) continue;
       float wv[8];
-      load8(w + d, wv);
+      if (w != nullptr) load8(w + d, wv);
 #pragma unroll
-      for (int i = 0; i < 8; ++i) f[n][i] *= inv * wv[i];
+      for (int i = 0; i < 8; ++i) f[n][i] *= w != nullptr ? inv * wv[i] : inv;
       if (d < rot_dim) {
 #pragma unroll
         for (int i = 0; i < 8; ++i)
@@ -296,14 +305,14 @@ qk_norm_rope_scatter_kernel(E* __restrict__ qkv, int64_t qkv_stride, E* __restri
   }
 }
 
-// qw, kw: fp32 [D], zero beyond dim.  dt: 0 = fp32, 1 = bf16.
+// qw, kw: fp32 [D], zero beyond dim, or null.  dt: 0 = fp32, 1 = bf16.
 LLB_EXPORT int llb_qk_norm_rope_scatter(void* qkv, int dt, int64_t qkv_stride, void* kv_layer, const float* cos_t,
                                         const float* sin_t, const int* pos, const int* slot, const float* qw,
                                         const float* kw, float eps, int T, int Hq, int Hkv, int D, int dim, int DV,
                                         int rot_dim, cudaStream_t st) {
   if (T <= 0) return LLB_OK;
   if (D <= 0 || (D % 8) || DV <= 0 || (DV % 8) || D > 512 || dim <= 0 || dim > D || (rot_dim & 1) || rot_dim > dim ||
-      (qkv_stride % 8) || Hkv <= 0)
+      (qkv_stride % 8) || Hq < 0 || Hkv < 0)
     return LLB_ERR_UNSUPPORTED;
   int lg = 2;
   while (lg < 5 && (8 << lg) < D) ++lg;

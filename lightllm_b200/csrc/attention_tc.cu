@@ -1,6 +1,7 @@
 // Prefill attention on the 5th-generation tensor cores (tcgen05 + tensor memory), causal, varlen, aware of an already cached
 // prefix, K/V read through the token-granular slot table of the KV pool.  Head size 128, and a windowed form with key sizes
-// up to 256, any multiple of 64 as value size, and a sigmoid gate per head on the output.
+// up to 256, any multiple of 64 as value size, kept first positions, biases by distance, and a sigmoid gate per head on the
+// output.
 //
 // One CTA computes 128 query rows of one (request, query head).  Per 128-key tile (64 keys for key sizes above 128):
 //   S  = Q . K^T            tcgen05.mma into one of two tensor-memory buffers
@@ -65,14 +66,15 @@ __device__ __forceinline__ uint32_t pack2(float a, float b) {
 }
 
 // DK, DV: key size and the value columns of one CTA (a wider value head is shared out over CTAs: v_blocks per head).
-// window: a query sees its own position and the window - 1 before it (0: all before it).  SPLIT_P: the weights enter P . V
-// as the sum of two bf16 tiles.  gate (or null): head h of row t is multiplied by out_scale * sigmoid(gate[t, h]).
-template <int DK, int DV, int BN, bool SPLIT_P>
+// rule.window: a query sees its own position and the window - 1 before it (0: all before it).  SPLIT_P: the weights enter P . V
+// as the sum of two bf16 tiles.  EXT: positions below rule.keep are seen at any distance (the tiles that hold them come ahead of
+// the window's), and scores get the biases of rule.rel; rule.window is the window in either form.  gate (or null): head h of row t is multiplied by out_scale * sigmoid(gate[t, h]).
+template <int DK, int DV, int BN, bool SPLIT_P, bool EXT>
 __global__ void __launch_bounds__(THREADS, 1)
 gqa_prefill_tc_kernel(const bf16* __restrict__ q, int64_t q_stride, const bf16* __restrict__ kv_layer,
                       const int* __restrict__ req_to_token, int64_t r2t_stride, const int* __restrict__ b_req_idx,
                       const int* __restrict__ cu_q, const int* __restrict__ b_ready_len, bf16* __restrict__ out,
-                      int64_t out_stride, int Hq, int Hkv, float scale_log2, int v_blocks, int window,
+                      int64_t out_stride, int Hq, int Hkv, float scale_log2, int v_blocks, const KeyRule rule,
                       const bf16* __restrict__ gate, int64_t gate_stride, float out_scale) {
   using L = PrefillLayout<DK, DV, BN, SPLIT_P>;
   constexpr int HK = BN / 2;   // keys of a score tile per softmax thread
@@ -101,8 +103,14 @@ gqa_prefill_tc_kernel(const bf16* __restrict__ q, int64_t q_stride, const bf16* 
   const int req = LLB_CHECK_REQ(b_req_idx[b]);
   const int rows_valid = min(BM, q_len - q0);
   const int kv_end = ready + q0 + rows_valid;  // exclusive bound on the keys any row of this tile may see
+  const int window = rule.window;
   const int kv0 = window > 0 ? max(0, ready + q0 - window + 1) : 0;
-  const int n_tiles = (kv_end - kv0 + BN - 1) / BN;
+  const int kept = EXT ? min(rule.keep, kv0) : 0;      // kept positions ahead of the window
+  const int kept_tiles = EXT ? (kept + BN - 1) / BN : 0;
+  const int n_tiles = kept_tiles + (kv_end - kv0 + BN - 1) / BN;
+  // first position of tile j, and the exclusive bound on the positions it holds
+  auto tile_pos = [&](int j) { return EXT && j < kept_tiles ? j * BN : kv0 + (j - kept_tiles) * BN; };
+  auto tile_bound = [&](int j) { return EXT && j < kept_tiles ? kept : kv_end; };
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int64_t r2t_base = (int64_t)req * r2t_stride;
   int* status = &g_attn_tc_status;
@@ -159,12 +167,12 @@ gqa_prefill_tc_kernel(const bf16* __restrict__ q, int64_t q_stride, const bf16* 
     const bf16* v_src = kv_layer + (int64_t)Hkv * DK + ((int64_t)kvh * v_blocks + vb) * DV;
     for (int j = stage; j < n_tiles; j += 2) {
       const uint32_t par = (((uint32_t)j >> 1) & 1u) ^ 1u;
-      const int kt = kv0 + j * BN;
+      const int kt = tile_pos(j), bound = tile_bound(j);
       int slots[BN / 32];
 #pragma unroll
       for (int u = 0; u < BN / 32; ++u) {
         const int pos = kt + u * 32 + lane;
-        slots[u] = pos < kv_end ? LLB_CHECK_SLOT(req_to_token[r2t_base + pos]) : -1;
+        slots[u] = pos < bound ? LLB_CHECK_SLOT(req_to_token[r2t_base + pos]) : -1;
       }
       mbar_wait(k_empty(stage), par, abort_flag, status, 41);
 #pragma unroll
@@ -279,16 +287,33 @@ gqa_prefill_tc_kernel(const bf16* __restrict__ q, int64_t q_stride, const bf16* 
     for (int i = 0; i < OC; ++i) o[i] = 0.f;
     float m_run = -INFINITY, l_run = 0.f;
     for (int j = 0; j < n_tiles; ++j) {
-      const int kt = kv0 + j * BN + half * HK;
+      const int kt = tile_pos(j) + half * HK;
       mbar_wait(s_full(j & 1), ((uint32_t)j >> 1) & 1u, abort_flag, status, 45);
       tc_fence_after();
       uint32_t sr[HK];
 #pragma unroll
       for (int c = 0; c < HK; c += 32) tmem_ld_32x32(t_s + (j & 1) * BN + c, sr + c);
       tmem_wait_ld();
-      const int lim = min(prow, kv_end - 1) - kt;  // my columns lo..lim are visible to this row
+      const int lim = min(prow, tile_bound(j) - 1) - kt;  // my columns lo..lim (and those below `first`) are visible to this row
       const int lo = window > 0 ? prow - window + 1 - kt : 0;
-      const bool all_visible = lim >= HK - 1 && lo <= 0;  // whole tile (every tile but those at the diagonal and the edges)
+      const int first = EXT ? rule.keep - kt : 0;
+      auto seen = [&](int c) { return c <= lim && (c >= lo || (EXT && c < first)); };
+      // whole tile (every tile but those at the diagonal and the edges)
+      const bool all_visible = lim >= HK - 1 && (lo <= 0 || (EXT && first >= HK));
+      const float to_log2 = EXT ? 1.f : scale_log2;
+      if (EXT) {  // scores in log2 units, with the bias of their distance
+        const float* rel = rule.rel != nullptr ? rule.rel + (int64_t)h * (rule.far + 1) : nullptr;
+        const int dist = prow - kt;  // of my first column; the last one is HK - 1 nearer
+        if (rel == nullptr || dist - (HK - 1) >= rule.far) {
+          const float b = rel != nullptr ? rel[rule.far] * kLog2e : 0.f;
+#pragma unroll
+          for (int e = 0; e < HK; ++e) sr[e] = __float_as_uint(fmaf(__uint_as_float(sr[e]), scale_log2, b));
+        } else {
+#pragma unroll
+          for (int e = 0; e < HK; ++e)
+            sr[e] = __float_as_uint(fmaf(__uint_as_float(sr[e]), scale_log2, rel[max(0, min(dist - e, rule.far))] * kLog2e));
+        }
+      }
       float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
       if (all_visible) {
 #pragma unroll
@@ -296,14 +321,14 @@ gqa_prefill_tc_kernel(const bf16* __restrict__ q, int64_t q_stride, const bf16* 
       } else {
 #pragma unroll
         for (int e = 0; e < HK; ++e)
-          if (e >= lo && e <= lim) mx4[e & 3] = fmaxf(mx4[e & 3], __uint_as_float(sr[e]));
+          if (seen(e)) mx4[e & 3] = fmaxf(mx4[e & 3], __uint_as_float(sr[e]));
       }
       float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
       float* x = xch + (j & 1) * 256;
       x[half * 128 + erow] = mx;
       asm volatile("bar.sync 1, 256;" ::: "memory");
       mx = fmaxf(mx, x[(half ^ 1) * 128 + erow]);
-      const float m_new = fmaxf(m_run, mx * scale_log2);
+      const float m_new = fmaxf(m_run, mx * to_log2);
       const float m_use = m_new == -INFINITY ? 0.f : m_new;
       const float alpha = ex2_fast(m_run - m_use);
       m_run = m_new;
@@ -324,8 +349,8 @@ gqa_prefill_tc_kernel(const bf16* __restrict__ q, int64_t q_stride, const bf16* 
 #pragma unroll
         for (int e = 0; e < 8; ++e) {
           const int c = g * 8 + e;
-          const float pe = ex2_fast(fmaf(__uint_as_float(sr[c]), scale_log2, -m_use));
-          pv[e] = (all_visible || (c >= lo && c <= lim)) ? pe : 0.f;
+          const float pe = ex2_fast(fmaf(__uint_as_float(sr[c]), to_log2, -m_use));
+          pv[e] = (all_visible || seen(c)) ? pe : 0.f;
           rs4[e & 3] += pv[e];
         }
         const uint32_t off = tile_off<BLOCK_BYTES>(erow, half * (HK / 8) + g);
@@ -396,24 +421,24 @@ gqa_prefill_tc_kernel(const bf16* __restrict__ q, int64_t q_stride, const bf16* 
   }
 }
 
-template <int DK, int DV, int BN, bool SPLIT_P>
+template <int DK, int DV, int BN, bool SPLIT_P, bool EXT>
 int launch_tc(const bf16* q, int64_t q_stride, const bf16* kv_layer, const int* req_to_token, int64_t r2t_stride,
               const int* b_req_idx, const int* cu_q, const int* b_ready_len, bf16* out, int64_t out_stride, int B,
-              int max_q_len, int Hq, int Hkv, float sm_scale, int v_blocks, int window, const bf16* gate,
+              int max_q_len, int Hq, int Hkv, float sm_scale, int v_blocks, const KeyRule& rule, const bf16* gate,
               int64_t gate_stride, float out_scale, cudaStream_t st) {
   using L = PrefillLayout<DK, DV, BN, SPLIT_P>;
   static_assert(L::BYTES <= 227 * 1024, "shared memory");
   static DeviceOnce configured;
   if (!configured.done()) {
-    cudaError_t e = cudaFuncSetAttribute(gqa_prefill_tc_kernel<DK, DV, BN, SPLIT_P>,
+    cudaError_t e = cudaFuncSetAttribute(gqa_prefill_tc_kernel<DK, DV, BN, SPLIT_P, EXT>,
                                          cudaFuncAttributeMaxDynamicSharedMemorySize, L::BYTES);
     if (e != cudaSuccess) return (int)e;
     configured.set();
   }
   const dim3 grid((max_q_len + BM - 1) / BM, Hq * v_blocks, B);
-  gqa_prefill_tc_kernel<DK, DV, BN, SPLIT_P><<<grid, THREADS, L::BYTES, st>>>(
+  gqa_prefill_tc_kernel<DK, DV, BN, SPLIT_P, EXT><<<grid, THREADS, L::BYTES, st>>>(
       q, q_stride, kv_layer, req_to_token, r2t_stride, b_req_idx, cu_q, b_ready_len, out, out_stride, Hq, Hkv,
-      sm_scale * kLog2e, v_blocks, window, gate, gate_stride, out_scale);
+      sm_scale * kLog2e, v_blocks, rule, gate, gate_stride, out_scale);
   LLB_LAUNCH_CHECK();
   return LLB_OK;
 }
@@ -434,28 +459,31 @@ LLB_EXPORT int llb_gqa_prefill_tc(const void* q, int64_t q_stride, const void* k
   if (B <= 0 || max_q_len <= 0) return LLB_OK;
   if (Hkv <= 0 || Hq % Hkv != 0 || (q_stride % 8) || (out_stride % 8) || ((uintptr_t)q & 15) || ((uintptr_t)out & 15))
     return LLB_ERR_BAD_ARG;
-  return launch_tc<128, 128, 128, false>((const bf16*)q, q_stride, (const bf16*)kv_layer, req_to_token, r2t_stride, b_req_idx,
-                                         cu_q, b_ready_len, (bf16*)out, out_stride, B, max_q_len, Hq, Hkv, sm_scale, 1, 0,
+  return launch_tc<128, 128, 128, false, false>((const bf16*)q, q_stride, (const bf16*)kv_layer, req_to_token, r2t_stride, b_req_idx,
+                                         cu_q, b_ready_len, (bf16*)out, out_stride, B, max_q_len, Hq, Hkv, sm_scale, 1, KeyRule{0, 0, nullptr, 0},
                                          nullptr, 0, 1.f, st);
 }
 
-// Key size dk (64, 128, 192, 256), value size dv (a multiple of 64), window (0: none): pool rows [Hkv * dk | Hkv * dv], q
+// Key size dk (64, 128, 192, 256), value size dv (a multiple of 64), window (0: none), first `keep` positions always seen,
+// biases by distance rel [Hq, far + 1] (or null): pool rows [Hkv * dk | Hkv * dv], q
 // [T, >= Hq * dk], out [T, >= Hq * dv].  gate [T, >= Hq] (or null): head h of the output times out_scale * sigmoid(gate).
 LLB_EXPORT int llb_window_gqa_prefill_tc(const void* q, int64_t q_stride, const void* kv_layer, const int* req_to_token,
                                          int64_t r2t_stride, const int* b_req_idx, const int* cu_q, const int* b_ready_len,
                                          void* out, int64_t out_stride, int B, int max_q_len, int Hq, int Hkv, int dk,
-                                         int dv, float sm_scale, int window, const void* gate, int64_t gate_stride,
-                                         float out_scale, cudaStream_t st) {
+                                         int dv, float sm_scale, int window, int keep, const float* rel, int far,
+                                         const void* gate, int64_t gate_stride, float out_scale, cudaStream_t st) {
   if (B <= 0 || max_q_len <= 0) return LLB_OK;
   if (Hkv <= 0 || Hq % Hkv != 0 || (q_stride % 8) || (out_stride % 8) || ((uintptr_t)q & 15) || ((uintptr_t)out & 15) ||
-      window < 0 || dv <= 0)
+      window < 0 || keep < 0 || (rel != nullptr && far < 0) || dv <= 0)
     return LLB_ERR_BAD_ARG;
+  const KeyRule rule{window, keep, rel, far};
+  const bool ext = (window > 0 && keep > 0) || rel != nullptr;
   if ((dv % 64) || (dk != 64 && dk != 128 && dk != 192 && dk != 256) || Hq * (dv / 64) > 65535 || B > 65535)
     return LLB_ERR_UNSUPPORTED;
 #define LLB_WINDOW_TC(DK, DV, BN)                                                                                         \
-  return launch_tc<DK, DV, BN, true>((const bf16*)q, q_stride, (const bf16*)kv_layer, req_to_token, r2t_stride, b_req_idx, \
-                                     cu_q, b_ready_len, (bf16*)out, out_stride, B, max_q_len, Hq, Hkv, sm_scale, dv / DV,  \
-                                     window, (const bf16*)gate, gate_stride, out_scale, st)
+  return (ext ? launch_tc<DK, DV, BN, true, true> : launch_tc<DK, DV, BN, true, false>)(                                  \
+      (const bf16*)q, q_stride, (const bf16*)kv_layer, req_to_token, r2t_stride, b_req_idx, cu_q, b_ready_len, (bf16*)out, \
+      out_stride, B, max_q_len, Hq, Hkv, sm_scale, dv / DV, rule, (const bf16*)gate, gate_stride, out_scale, st)
   if (dv % 128 == 0) {
     if (dk == 64) LLB_WINDOW_TC(64, 128, 128);
     if (dk == 128) LLB_WINDOW_TC(128, 128, 128);

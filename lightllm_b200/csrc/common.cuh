@@ -187,6 +187,14 @@ __device__ __forceinline__ float tanh_fast(float x) {
   return fabsf(x) < 0.25f ? small : big;
 }
 
+// Which keys a causal query sees and what its scores get added: position p sees j <= p with p - j < window (window 0: all) or
+// j < keep; key j's score of head h gets rel[h, min(p - j, far)] (natural units; rel [heads, far + 1] fp32, or null).
+struct KeyRule {
+  int window, keep;
+  const float* rel;
+  int far;
+};
+
 // Block-wide sum; `red` is a shared array of >= 33 floats. All threads get the result.
 __device__ __forceinline__ float block_sum(float v, float* red) {
   int lane = threadIdx.x & 31, w = threadIdx.x >> 5, nw = (blockDim.x + 31) >> 5;

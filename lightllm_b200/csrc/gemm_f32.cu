@@ -31,6 +31,7 @@ struct F32Params {
   float alpha;
   DytPair d;
   float act_alpha, act_limit;  // F_GATED_CLAMP
+  float softcap;               // F_F32: > 0 stores softcap * tanh(value / softcap)
 };
 
 constexpr int TM = 64, TN = 64, TK = 16;
@@ -120,7 +121,10 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const F32Params p) {
           v = fmaxf(v, 0.f);
           v *= v;
         }
-        if (EPI == F_F32) v *= p.alpha;
+        if (EPI == F_F32) {
+          v *= p.alpha;
+          if (p.softcap > 0.f) v = p.softcap * tanhf(v / p.softcap);
+        }
         if (EPI == F_DYT) {
           const float x = p.d.x[off] + tanhf(p.d.alpha1 * v) * p.d.w1[col] + p.d.b1[col];
           p.d.x[off] = x;
@@ -148,7 +152,7 @@ LLB_EXPORT int llb_gemm_f32(const float* A, int64_t lda, int64_t a_batch, const 
                             float* C, int64_t ldc, int64_t c_batch, const float* residual, const float* bias, float* x,
                             const float* w1, const float* b1, float alpha1, const float* w2, const float* b2,
                             float alpha2, const int* mblock_expert, int M, int N, int K, int batch, int epi,
-                            float alpha, float act_alpha, float act_limit, cudaStream_t st) {
+                            float alpha, float act_alpha, float act_limit, float softcap, cudaStream_t st) {
   if (M <= 0 || N <= 0 || batch <= 0) return LLB_OK;
   if (K <= 0 || cdiv(M, TM) > 65535 || batch > 65535) return LLB_ERR_UNSUPPORTED;
   if (gated_epi(epi) && (N % 64)) return LLB_ERR_UNSUPPORTED;
@@ -175,6 +179,7 @@ LLB_EXPORT int llb_gemm_f32(const float* A, int64_t lda, int64_t a_batch, const 
   p.alpha = alpha;
   p.act_alpha = act_alpha;
   p.act_limit = act_limit;
+  p.softcap = softcap;
   p.d = DytPair{x, w1, b1, w2, b2, alpha1, alpha2};
   switch (epi) {
     case F_STORE: return launch<F_STORE>(p, batch, st);

@@ -77,6 +77,7 @@ struct GemmParams {
   uint32_t* push_cnt[8];
   int push_world, push_rank, push_max_mb;
   float out_scale;  // EPI_F32: factor on the stored value
+  float softcap;    // EPI_F32: > 0 stores softcap * tanh(value / softcap)
   DytFuse dyt;      // EPI_DYT
   float act_alpha, act_limit;  // EPI_GATED_CLAMP
 };
@@ -116,6 +117,13 @@ __device__ __forceinline__ float gated_f(const GemmParams& p, float g, float u) 
     return __fdividef(g, 1.f + __expf(-p.act_alpha * g)) * (u + 1.f);
   }
   return (EPI == EPI_GATED_SILU ? silu_f(g) : gelu_tanh_f(g)) * u;
+}
+__device__ __forceinline__ float f32_out(const GemmParams& p, float v) {
+  v *= p.out_scale;
+  return p.softcap > 0.f ? p.softcap * tanh_fast(__fdividef(v, p.softcap)) : v;
+}
+__device__ __forceinline__ float4 f32_out4(const GemmParams& p, float4 v) {
+  return make_float4(f32_out(p, v.x), f32_out(p, v.y), f32_out(p, v.z), f32_out(p, v.w));
 }
 __device__ __forceinline__ float relu2_f(float v) {
   v = fmaxf(v, 0.f);
@@ -252,14 +260,13 @@ __device__ __forceinline__ void epi_direct32(const GemmParams& p, const uint32_t
           v.z += __bfloat162float(p.bias[col0 + j + 2]);
           v.w += __bfloat162float(p.bias[col0 + j + 3]);
         }
-        v = make_float4(v.x * p.out_scale, v.y * p.out_scale, v.z * p.out_scale, v.w * p.out_scale);
-        *reinterpret_cast<float4*>(crow + j) = v;
+        *reinterpret_cast<float4*>(crow + j) = f32_out4(p, v);
       }
     } else {
 #pragma unroll
       for (int j = 0; j < 32; ++j)
         if (j < ncols)
-          crow[j] = (__uint_as_float(r[j]) + (p.bias ? __bfloat162float(p.bias[col0 + j]) : 0.f)) * p.out_scale;
+          crow[j] = f32_out(p, __uint_as_float(r[j]) + (p.bias ? __bfloat162float(p.bias[col0 + j]) : 0.f));
     }
   } else {
     bf16* crow = (bf16*)p.C + (int64_t)row * p.ldc + col0;
@@ -448,8 +455,7 @@ __device__ __forceinline__ void epilogue_store(const GemmParams& p, uint32_t t_r
             v.z += __bfloat162float(p.bias[col0 + j + 2]);
             v.w += __bfloat162float(p.bias[col0 + j + 3]);
           }
-          v = make_float4(v.x * p.out_scale, v.y * p.out_scale, v.z * p.out_scale, v.w * p.out_scale);
-          *reinterpret_cast<float4*>(my + j * 4) = v;
+          *reinterpret_cast<float4*>(my + j * 4) = f32_out4(p, v);
         }
         __syncwarp();
         epi_flush<4>(p, stage, lane, row_base, col0, false);
@@ -1279,8 +1285,7 @@ gemm_bf16_skinny_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_co
           acc.w += __bfloat162float(p.bias[gcol + 3]);
         }
         if (EPI == EPI_F32) {
-          *reinterpret_cast<float4*>((float*)p.C + (int64_t)grow * p.ldc + gcol) =
-              make_float4(acc.x * p.out_scale, acc.y * p.out_scale, acc.z * p.out_scale, acc.w * p.out_scale);
+          *reinterpret_cast<float4*>((float*)p.C + (int64_t)grow * p.ldc + gcol) = f32_out4(p, acc);
         } else if (EPI == EPI_DYT) {
           const int64_t off = (int64_t)grow * p.ldc + gcol;
           float4 x = *reinterpret_cast<const float4*>(p.dyt.x + off);
@@ -2055,7 +2060,7 @@ void apply_push(GemmParams& p) {
 struct GemmFuse {
   float out_scale = 1.f;
   DytFuse dyt = {nullptr, nullptr, nullptr, nullptr, nullptr, 1.f, 1.f};
-  float act_alpha = 1.f, act_limit = INFINITY;
+  float act_alpha = 1.f, act_limit = INFINITY, softcap = 0.f;
 };
 
 bool g_pair_auto = true;  // measured faster than one-CTA tiles for M >= 1024, K <= 8192 on B200
@@ -2144,6 +2149,7 @@ static int gemm_bf16(const void* A, int64_t lda, const void* W, int64_t ldw, voi
     memset(&p, 0, sizeof(p));
     apply_push(p);
     p.out_scale = fuse.out_scale;
+    p.softcap = fuse.softcap;
     p.dyt = fuse.dyt;
     p.act_alpha = fuse.act_alpha;
     p.act_limit = fuse.act_limit;
@@ -2184,6 +2190,7 @@ static int gemm_bf16(const void* A, int64_t lda, const void* W, int64_t ldw, voi
     memset(&p, 0, sizeof(p));
     apply_push(p);
     p.out_scale = fuse.out_scale;
+    p.softcap = fuse.softcap;
     p.dyt = fuse.dyt;
     p.act_alpha = fuse.act_alpha;
     p.act_limit = fuse.act_limit;
@@ -2240,6 +2247,7 @@ static int gemm_bf16(const void* A, int64_t lda, const void* W, int64_t ldw, voi
     p.w_tiled_kb = w_tiled ? K / 64 : 0;
     apply_push(p);
     p.out_scale = fuse.out_scale;
+    p.softcap = fuse.softcap;
     p.dyt = fuse.dyt;
     p.act_alpha = fuse.act_alpha;
     p.act_limit = fuse.act_limit;
@@ -2275,6 +2283,7 @@ static int gemm_bf16(const void* A, int64_t lda, const void* W, int64_t ldw, voi
   p.w_swz = w_swz ? (const bf16*)W : nullptr;
   apply_push(p);
   p.out_scale = fuse.out_scale;
+  p.softcap = fuse.softcap;
   p.dyt = fuse.dyt;
   p.act_alpha = fuse.act_alpha;
   p.act_limit = fuse.act_limit;
@@ -2316,15 +2325,18 @@ LLB_EXPORT int llb_gemm_bf16(const void* A, int64_t lda, const void* W, int64_t 
                    sk_counters, sk_counters_len, status, GemmFuse{}, st);
 }
 
-// The epilogues with parameters: out_scale multiplies fp32 output (epi 3); for epi 6 (bf16 C, same pitch for x)
+// The epilogues with parameters: out_scale multiplies fp32 output (epi 3), softcap > 0 then takes it to softcap *
+// tanh(v / softcap); for epi 6 (bf16 C, same pitch for x)
 //   x += tanh(alpha1 * acc) * w1 + b1;  C = tanh(alpha2 * x) * w2 + b2        x fp32 [M, ldc], vectors fp32 [N]
 // for epi 7 with g, u the gate and up columns:
 //   g = min(g, act_limit); u = clamp(u, -act_limit, act_limit); C = (u + 1) * g * sigmoid(act_alpha * g)
 LLB_EXPORT int llb_gemm_bf16_fused(const void* A, int64_t lda, const void* W, int64_t ldw, void* C, int64_t ldc,
                                    const void* bias, int M, int N, int K, int epi, int bn, float out_scale, float* x,
                                    const float* w1, const float* b1, float alpha1, const float* w2, const float* b2,
-                                   float alpha2, float act_alpha, float act_limit, int* status, cudaStream_t st) {
+                                   float alpha2, float act_alpha, float act_limit, float softcap, int* status,
+                                   cudaStream_t st) {
   GemmFuse fuse;
+  fuse.softcap = softcap;
   fuse.act_alpha = act_alpha;
   fuse.act_limit = act_limit;
   fuse.out_scale = out_scale;

@@ -1,15 +1,18 @@
-// Latent attention without a rotary part, over a paged pool of latents, with an optional sliding window.
+// Latent attention over a paged pool of latents, with an optional rotary part and an optional sliding window.
 //
-// Pool row of a token: the RMS-normalised latent c (`rank` values, zero-padded to the row pitch), one "head" shared by
-// all query heads.  The query of a head is taken into the latent space with the key up-projection (q_lat = q . W_uk),
-// scores are q_lat . c, the value read is the same c, and the value up-projection follows the attention.
+// Pool row of a token: [the RMS-normalised latent c, zero-padded to `rank` values | rotated key part], `keys` values in all,
+// one "head" shared by all query heads.  The query of a head is taken into the latent space with the key up-projection and
+// followed by its own rotated part (q_lat = [q . W_uk | q_rot]), scores are q_lat . row, the value read is c, and the value
+// up-projection follows the attention.
 // A query sees its own position and the window - 1 positions before it (window 0: all of them).  Scores, weights and
 // their sums are fp32.
 //
-//   latent_norm_scatter    RMSNorm of new latents, written to their pool slots
-//   latent_gather          latents of a range of positions of every request, back to back (for the expanded prefill form)
-//   latent_attn_generic    any rank <= 1024, fp32 or bf16; one CTA per (query token, head), warps stride over the keys
-//   latent_attn_mma        bf16, rank <= 512: one CTA per (query token, 16 heads, share of the keys).  The 16 query rows
+//   latent_prepare         RMSNorm of new latents and rotation of their key parts, written to their pool slots; RMSNorm of the
+//                          queries' own latents
+//   rope_heads             rotation of a range of columns of every query head, in place
+//   latent_gather          rows of a range of positions of every request, back to back (for the expanded prefill form)
+//   latent_attn_generic    up to 1024 values per row, fp32 or bf16; one CTA per (query token, head), warps stride over the keys
+//   latent_attn_mma        bf16, up to 576 values per row, 512 of them latent: one CTA per (query token, 16 heads, share of the keys).  The 16 query rows
 //                          live in registers as MMA fragments; 64-key tiles of the pool are gathered through the slot
 //                          table into a three-stage shared-memory ring and used for both products.  The weights enter
 //                          P . c as a sum of two bf16 values (high and low part), so that they keep fp32-like
@@ -29,23 +32,128 @@ __device__ __forceinline__ float to_f(bf16 v) { return __bfloat162float(v); }
 __device__ __forceinline__ void from_f(float* p, float v) { *p = v; }
 __device__ __forceinline__ void from_f(bf16* p, float v) { *p = __float2bfloat16(v); }
 
-// One warp per token.
+__device__ __forceinline__ void ld8(const float* p, float* f) {
+  const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
+  f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w;
+  f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
+}
+__device__ __forceinline__ void ld8(const bf16* p, float* f) { unpack8(*reinterpret_cast<const bf16x8*>(p), f); }
+__device__ __forceinline__ void st8(float* p, const float* f) {
+  reinterpret_cast<float4*>(p)[0] = make_float4(f[0], f[1], f[2], f[3]);
+  reinterpret_cast<float4*>(p)[1] = make_float4(f[4], f[5], f[6], f[7]);
+}
+__device__ __forceinline__ void st8(bf16* p, const float* f) { *reinterpret_cast<bf16x8*>(p) = pack8(f); }
+
+// A warp writes RMSNorm(s[0 .. rank)) * w to d[0 .. cols), zero beyond rank; cols is a multiple of 8.
 template <typename T>
-__global__ void __launch_bounds__(128)
-latent_norm_scatter_kernel(const T* __restrict__ src, int64_t src_stride, T* __restrict__ pool, int row_elems,
-                           const float* __restrict__ w, const int* __restrict__ slot, int Tn, int rank, float eps) {
-  const int t = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-  if (t >= Tn) return;
-  const T* s = src + (int64_t)t * src_stride;
-  T* d = pool + (int64_t)LLB_CHECK_SLOT(slot[t]) * row_elems;
+__device__ __forceinline__ void norm_row(const T* s, T* d, const float* w, int rank, int cols, float eps, int lane) {
   float ss = 0.f;
-  for (int i = lane; i < rank; i += 32) {
-    const float v = to_f(s[i]);
-    ss += v * v;
+  for (int c = lane * 8; c < rank; c += 256) {
+    float f[8];
+    ld8(s + c, f);
+#pragma unroll
+    for (int i = 0; i < 8; ++i)
+      if (c + i < rank) ss = fmaf(f[i], f[i], ss);
   }
-  ss = warp_sum(ss);
-  const float r = 1.f / sqrtf(ss / (float)rank + eps);
-  for (int i = lane; i < row_elems; i += 32) from_f(d + i, i < rank ? to_f(s[i]) * r * w[i] : 0.f);
+  const float r = 1.f / sqrtf(warp_sum(ss) / (float)rank + eps);
+  for (int c = lane * 8; c < cols; c += 256) {
+    float f[8] = {}, wv[8];
+    if (c < rank) ld8(s + c, f);
+    if (c + 8 <= rank) {
+      ld8(w + c, wv);
+    } else {
+#pragma unroll
+      for (int i = 0; i < 8; ++i) wv[i] = c + i < rank ? w[c + i] : 0.f;
+    }
+#pragma unroll
+    for (int i = 0; i < 8; ++i) f[i] = c + i < rank ? f[i] * r * wv[i] : 0.f;
+    st8(d + c, f);
+  }
+}
+
+// Rotation of the pairs of `dims` columns: neighbours (2 i, 2 i + 1), or halves (i, i + dims / 2).  Tables [positions, dims / 2].
+struct Rotation {
+  const float *cos_t, *sin_t;
+  const int* pos;
+  int dims, neighbours;
+};
+template <typename T>
+__device__ __forceinline__ void rotate_pair(const Rotation& r, const T* s, T* d, int p, int i) {
+  const int half = r.dims >> 1, a = r.neighbours ? 2 * i : i, b = r.neighbours ? 2 * i + 1 : i + half;
+  const float c = r.cos_t[(int64_t)p * half + i], n = r.sin_t[(int64_t)p * half + i];
+  const float u = to_f(s[a]), v = to_f(s[b]);
+  from_f(d + a, u * c - v * n);
+  from_f(d + b, v * c + u * n);
+}
+
+template <typename T>
+struct PrepareArgs {
+  const T* src;  // [T, [latent, padded to cols | rotated part]]
+  int64_t src_stride;
+  T* pool;
+  int row_elems, rank, cols;
+  const float* w;
+  const int* slot;
+  Rotation rot;
+  const T* q_src;  // [T, q_cols] latents of the queries (null: none)
+  int64_t q_stride;
+  T* q_out;
+  int q_rank, q_cols;
+  const float* q_w;
+  int Tn;
+  float eps;
+};
+
+// One warp per token and latent.
+template <typename T>
+__global__ void __launch_bounds__(128) latent_prepare_kernel(const PrepareArgs<T> a) {
+  pdl_wait();
+  const int item = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (item >= a.Tn) {
+    const int t = item - a.Tn;
+    if (a.q_src != nullptr && t < a.Tn)
+      norm_row(a.q_src + (int64_t)t * a.q_stride, a.q_out + (int64_t)t * a.q_cols, a.q_w, a.q_rank, a.q_cols, a.eps, lane);
+    return;
+  }
+  const int t = item;
+  const T* s = a.src + (int64_t)t * a.src_stride;
+  T* d = a.pool + (int64_t)LLB_CHECK_SLOT(a.slot[t]) * a.row_elems;
+  norm_row(s, d, a.w, a.rank, a.cols, a.eps, lane);
+  if (a.rot.dims > 0) {
+    const int p = a.rot.pos[t];
+    for (int i = lane; i < (a.rot.dims >> 1); i += 32) rotate_pair(a.rot, s + a.cols, d + a.cols, p, i);
+  }
+  for (int i = a.cols + a.rot.dims + lane; i < a.row_elems; i += 32) from_f(d + i, 0.f);
+}
+
+// x [T, heads]: columns off .. off + dims of every head (pitch elements apart) rotated in place.  VEC: neighbours, four pairs per
+// thread.
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(256)
+rope_heads_kernel(T* __restrict__ x, int64_t stride, const Rotation r, int64_t items, int H, int pitch, int off) {
+  pdl_wait();
+  const int per = VEC ? r.dims >> 3 : r.dims >> 1;  // threads per head
+  const int64_t id = (int64_t)blockIdx.x * 256 + threadIdx.x;
+  if (id >= items) return;
+  const int i = (int)(id % per);
+  const int64_t th = id / per;
+  const int h = (int)(th % H);
+  const int64_t t = th / H;
+  T* p = x + t * stride + (int64_t)h * pitch + off;
+  if (VEC) {
+    const int64_t at = (int64_t)r.pos[t] * (r.dims >> 1) + i * 4;
+    float f[8], o[8];
+    ld8(p + i * 8, f);
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      const float c = r.cos_t[at + k], n = r.sin_t[at + k];
+      o[2 * k] = f[2 * k] * c - f[2 * k + 1] * n;
+      o[2 * k + 1] = f[2 * k + 1] * c + f[2 * k] * n;
+    }
+    st8(p + i * 8, o);
+  } else {
+    rotate_pair(r, p, p, r.pos[t], i);
+  }
 }
 
 // out row cu_kv[b] + i = latent of position kv_start[b] + i of request b.  One warp per row, 16-byte pieces.
@@ -75,7 +183,7 @@ __global__ void __launch_bounds__(GW * 32)
 latent_attn_generic_kernel(const T* __restrict__ q_lat, const T* __restrict__ pool, int row_elems,
                            const int* __restrict__ req_to_token, int64_t r2t_stride, const int* __restrict__ b_req_idx,
                            const int* __restrict__ pos, const int* __restrict__ batch_of, T* __restrict__ out, int H,
-                           int rank, float scale, int window) {
+                           int keys, int rank, float scale, int window) {
   extern __shared__ float sm[];  // [GW][rank] partial outputs, then [GW] maxima, [GW] sums
   const int t = blockIdx.x, h = blockIdx.y;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -86,7 +194,7 @@ latent_attn_generic_kernel(const T* __restrict__ q_lat, const T* __restrict__ po
 #pragma unroll
   for (int e = 0; e < EPL; ++e) {
     const int d = lane + e * 32;
-    q[e] = d < rank ? to_f(q_lat[((int64_t)t * H + h) * rank + d]) * scale : 0.f;
+    q[e] = d < keys ? to_f(q_lat[((int64_t)t * H + h) * keys + d]) * scale : 0.f;
     acc[e] = 0.f;
   }
   float m = -INFINITY, l = 0.f;
@@ -98,7 +206,7 @@ latent_attn_generic_kernel(const T* __restrict__ q_lat, const T* __restrict__ po
 #pragma unroll
     for (int e = 0; e < EPL; ++e) {
       const int d = lane + e * 32;
-      cv[e] = d < rank ? to_f(c[d]) : 0.f;
+      cv[e] = d < keys ? to_f(c[d]) : 0.f;
       s += q[e] * cv[e];
     }
     s = warp_sum(s);
@@ -141,17 +249,17 @@ latent_attn_generic_kernel(const T* __restrict__ q_lat, const T* __restrict__ po
 
 template <typename T>
 int launch_generic(const void* q_lat, const void* pool, int row_elems, const int* r2t, int64_t r2t_stride,
-                   const int* b_req_idx, const int* pos, const int* batch_of, void* out, int T_n, int H, int rank,
-                   float scale, int window, cudaStream_t st) {
+                   const int* b_req_idx, const int* pos, const int* batch_of, void* out, int T_n, int H, int keys,
+                   int rank, float scale, int window, cudaStream_t st) {
   const dim3 grid(T_n, H);
   const size_t smem = (size_t)(GW * rank + 2 * GW) * sizeof(float);
 #define LLB_GENERIC(EPL)                                                                                              \
   latent_attn_generic_kernel<T, EPL><<<grid, GW * 32, smem, st>>>((const T*)q_lat, (const T*)pool, row_elems, r2t,    \
                                                                   r2t_stride, b_req_idx, pos, batch_of, (T*)out, H,   \
-                                                                  rank, scale, window)
-  if (rank <= 128)
+                                                                  keys, rank, scale, window)
+  if (keys <= 128)
     LLB_GENERIC(4);
-  else if (rank <= 512)
+  else if (keys <= 512)
     LLB_GENERIC(16);
   else
     LLB_GENERIC(32);
@@ -176,19 +284,20 @@ __device__ __forceinline__ uint32_t tile_off(int row, int ch) {
   return (uint32_t)(row * (LAT * 2) + ((ch ^ (row & 7)) << 4));
 }
 
-// LAT: rank rounded up to 128, 256, 384 or 512 (tile columns beyond the row pitch are zero-filled).
+// LAT: columns of a tile, at least `keys` (tile columns beyond the row pitch are zero-filled); LATV: columns read as values, at
+// least `rank`.
 // Partial results (splits > 1): part_o [split][token][head][rank] unnormalised, part_ml [split][token][head] (max, sum).
-template <int LAT>
+template <int LAT, int LATV>
 __global__ void __launch_bounds__(256, 1)
 latent_attn_mma_kernel(const bf16* __restrict__ q_lat, const bf16* __restrict__ pool, int row_elems,
                        const int* __restrict__ req_to_token, int64_t r2t_stride, const int* __restrict__ b_req_idx,
                        const int* __restrict__ pos, const int* __restrict__ batch_of, bf16* __restrict__ out,
-                       float* __restrict__ part_o, float2* __restrict__ part_ml, int Tn, int H, int rank,
+                       float* __restrict__ part_o, float2* __restrict__ part_ml, int Tn, int H, int keys, int rank,
                        float scale_log2, int window) {
   extern __shared__ __align__(128) uint8_t smem[];
   constexpr int CH = LAT / 8;            // 16-byte chunks per tile row
   constexpr int KSTEPS = LAT / 16;
-  constexpr int N2 = LAT / 128;          // pairs of 8-column output blocks per warp
+  constexpr int N2 = LATV / 128;         // pairs of 8-column output blocks per warp
   const uint32_t kv_base = smem_u32(smem);
   float* s_sm = reinterpret_cast<float*>(smem + STAGES * KT * LAT * 2);
   int* slot_sm = reinterpret_cast<int*>(s_sm + 2 * 16 * S_PITCH);
@@ -236,16 +345,16 @@ latent_attn_mma_kernel(const bf16* __restrict__ q_lat, const bf16* __restrict__ 
   // query rows as MMA fragments
   uint32_t qf[KSTEPS][4];
   {
-    const bf16* q0 = q_lat + ((int64_t)t * H + head0 + g) * rank;
-    const bf16* q1 = q0 + (int64_t)8 * rank;
+    const bf16* q0 = q_lat + ((int64_t)t * H + head0 + g) * keys;
+    const bf16* q1 = q0 + (int64_t)8 * keys;
     const bool ok0 = head0 + g < H, ok1 = head0 + g + 8 < H;
 #pragma unroll
     for (int ks = 0; ks < KSTEPS; ++ks) {
       const int d = ks * 16 + tig * 2;
-      qf[ks][0] = ok0 && d < rank ? *reinterpret_cast<const uint32_t*>(q0 + d) : 0u;
-      qf[ks][1] = ok1 && d < rank ? *reinterpret_cast<const uint32_t*>(q1 + d) : 0u;
-      qf[ks][2] = ok0 && d + 8 < rank ? *reinterpret_cast<const uint32_t*>(q0 + d + 8) : 0u;
-      qf[ks][3] = ok1 && d + 8 < rank ? *reinterpret_cast<const uint32_t*>(q1 + d + 8) : 0u;
+      qf[ks][0] = ok0 && d < keys ? *reinterpret_cast<const uint32_t*>(q0 + d) : 0u;
+      qf[ks][1] = ok1 && d < keys ? *reinterpret_cast<const uint32_t*>(q1 + d) : 0u;
+      qf[ks][2] = ok0 && d + 8 < keys ? *reinterpret_cast<const uint32_t*>(q0 + d + 8) : 0u;
+      qf[ks][3] = ok1 && d + 8 < keys ? *reinterpret_cast<const uint32_t*>(q1 + d + 8) : 0u;
     }
   }
   // scores of this warp's 8 keys of tile i over the whole latent, scaled and masked: columns (warp * 8 + tig * 2, + 1) of
@@ -354,7 +463,7 @@ latent_attn_mma_kernel(const bf16* __restrict__ q_lat, const bf16* __restrict__ 
 #pragma unroll
       for (int n = 0; n < N2; ++n) {
         uint32_t b0, b1, b2, b3;
-        ldmatrix_x4_trans(b0, b1, b2, b3, kb + tile_off<LAT>(tok, warp * (LAT / 64) + n * 2 + (lane >> 4)));
+        ldmatrix_x4_trans(b0, b1, b2, b3, kb + tile_off<LAT>(tok, warp * (LATV / 64) + n * 2 + (lane >> 4)));
         mma_bf16_16816(o[2 * n], ah[0], ah[1], ah[2], ah[3], b0, b1);
         mma_bf16_16816(o[2 * n + 1], ah[0], ah[1], ah[2], ah[3], b2, b3);
         mma_bf16_16816(o[2 * n], al[0], al[1], al[2], al[3], b0, b1);
@@ -372,7 +481,7 @@ latent_attn_mma_kernel(const bf16* __restrict__ q_lat, const bf16* __restrict__ 
     const int h = head0 + g + 8 * r;
     if (h >= H) continue;
     const int64_t row = (int64_t)t * H + h;
-    const int col0 = warp * (LAT / 8) + tig * 2;
+    const int col0 = warp * (LATV / 8) + tig * 2;
     if (splits == 1) {
       const float inv = 1.f / l_run[r];
 #pragma unroll
@@ -431,40 +540,80 @@ struct MmaArgs {
   float* part_o;
   float2* part_ml;
   int64_t r2t_stride;
-  int row_elems, T, H, rank, window, splits;
+  int row_elems, T, H, keys, rank, window, splits;
   float scale_log2;
 };
 
-template <int LAT>
+template <int LAT, int LATV>
 int launch_mma(const MmaArgs& a, cudaStream_t st) {
   static DeviceOnce configured;
   if (!configured.done()) {
-    cudaError_t e = cudaFuncSetAttribute(latent_attn_mma_kernel<LAT>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    cudaError_t e = cudaFuncSetAttribute(latent_attn_mma_kernel<LAT, LATV>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                          mma_smem<LAT>());
     if (e != cudaSuccess) return (int)e;
     configured.set();
   }
   const dim3 grid(a.T, (a.H + 15) / 16, a.splits);
-  latent_attn_mma_kernel<LAT><<<grid, 256, mma_smem<LAT>(), st>>>(
+  latent_attn_mma_kernel<LAT, LATV><<<grid, 256, mma_smem<LAT>(), st>>>(
       a.q_lat, a.pool, a.row_elems, a.r2t, a.r2t_stride, a.b_req_idx, a.pos, a.batch_of, a.out, a.part_o, a.part_ml, a.T,
-      a.H, a.rank, a.scale_log2, a.window);
+      a.H, a.keys, a.rank, a.scale_log2, a.window);
   LLB_LAUNCH_CHECK();
   return LLB_OK;
 }
 
 }  // namespace
 
-// dtype: 0 = fp32, 1 = bf16.  `rank` values per latent; the pool row has row_elems >= rank elements.
-LLB_EXPORT int llb_latent_norm_scatter(const void* src, int dtype, int64_t src_stride, void* pool, int row_elems,
-                                       const float* w, const int* slot, int T, int rank, float eps, cudaStream_t st) {
+// dtype: 0 = fp32, 1 = bf16.  src row: [latent, `rank` values in `cols` columns | rot_dims values to rotate]; the pool row gets
+// [RMSNorm(latent) * w, zero to cols | rotated part, zero to row_elems].  q_src (or null): rows of q_rank values in q_cols columns,
+// normalised into q_out [T, q_cols].  Columns and pitches are multiples of 8.
+LLB_EXPORT int llb_latent_prepare(const void* src, int dtype, int64_t src_stride, void* pool, int row_elems, const float* w,
+                                  const int* slot, int T, int rank, int cols, const float* cos_t, const float* sin_t,
+                                  const int* pos, int rot_dims, int neighbours, const void* q_src, int64_t q_stride,
+                                  void* q_out, int q_rank, int q_cols, const float* q_w, float eps, cudaStream_t st) {
   if (T <= 0) return LLB_OK;
-  if (rank <= 0 || rank > row_elems) return LLB_ERR_BAD_ARG;
+  if (rank <= 0 || rank > cols || cols + rot_dims > row_elems || (cols % 8) || (row_elems % 8) || (src_stride % 8) ||
+      rot_dims < 0 || (rot_dims & 1) || ((uintptr_t)src & 15) || ((uintptr_t)pool & 15) || ((uintptr_t)w & 15) ||
+      (rot_dims > 0 && (cos_t == nullptr || sin_t == nullptr || pos == nullptr)))
+    return LLB_ERR_BAD_ARG;
+  if (q_src != nullptr && (q_rank <= 0 || q_rank > q_cols || (q_cols % 8) || (q_stride % 8) || q_out == nullptr ||
+                           q_w == nullptr || (((uintptr_t)q_src | (uintptr_t)q_out | (uintptr_t)q_w) & 15)))
+    return LLB_ERR_BAD_ARG;
+  const Rotation rot{cos_t, sin_t, pos, rot_dims, neighbours};
+  const dim3 grid(cdiv(q_src != nullptr ? 2 * T : T, 4));
+#define LLB_PREPARE(E)                                                                                                     \
+  launch_pdl(latent_prepare_kernel<E>, grid, dim3(128), 0, st,                                                             \
+             PrepareArgs<E>{(const E*)src, src_stride, (E*)pool, row_elems, rank, cols, w, slot, rot, (const E*)q_src,     \
+                            q_stride, (E*)q_out, q_rank, q_cols, q_w, T, eps})
   if (dtype == 0)
-    latent_norm_scatter_kernel<float><<<cdiv(T, 4), 128, 0, st>>>((const float*)src, src_stride, (float*)pool, row_elems,
-                                                                  w, slot, T, rank, eps);
+    LLB_PREPARE(float);
   else
-    latent_norm_scatter_kernel<bf16><<<cdiv(T, 4), 128, 0, st>>>((const bf16*)src, src_stride, (bf16*)pool, row_elems, w,
-                                                                 slot, T, rank, eps);
+    LLB_PREPARE(bf16);
+#undef LLB_PREPARE
+  LLB_LAUNCH_CHECK();
+  return LLB_OK;
+}
+
+// x [T, H heads, `pitch` elements apart] (row pitch `stride`): columns off .. off + dims of every head rotated in place.
+LLB_EXPORT int llb_rope_heads(void* x, int dtype, int64_t stride, const float* cos_t, const float* sin_t, const int* pos, int T,
+                              int H, int pitch, int off, int dims, int neighbours, cudaStream_t st) {
+  if (T <= 0 || dims <= 0) return LLB_OK;
+  if (H <= 0 || off < 0 || off + dims > pitch || (dims & 1)) return LLB_ERR_BAD_ARG;
+  const Rotation rot{cos_t, sin_t, pos, dims, neighbours};
+  const bool vec = neighbours && dims % 8 == 0 && off % 8 == 0 && pitch % 8 == 0 && stride % 8 == 0 && ((uintptr_t)x & 15) == 0;
+  const int64_t items = (int64_t)T * H * (vec ? dims / 8 : dims / 2);
+  const dim3 grid((unsigned)cdiv64(items, 256));
+#define LLB_ROPE(E, V) launch_pdl(rope_heads_kernel<E, V>, grid, dim3(256), 0, st, (E*)x, stride, rot, items, H, pitch, off)
+  if (dtype == 0) {
+    if (vec)
+      LLB_ROPE(float, true);
+    else
+      LLB_ROPE(float, false);
+  } else if (vec) {
+    LLB_ROPE(bf16, true);
+  } else {
+    LLB_ROPE(bf16, false);
+  }
+#undef LLB_ROPE
   LLB_LAUNCH_CHECK();
   return LLB_OK;
 }
@@ -481,41 +630,51 @@ LLB_EXPORT int llb_latent_gather(const void* pool, int row_bytes, const int* req
   return LLB_OK;
 }
 
-// q_lat, out: [T, H, row_elems] contiguous, of which `rank` = row_elems columns are used (padding columns are zero).
+// q_lat [T, H, keys], out [T, H, rank], contiguous (padding columns of q_lat are zero); the pool row has row_elems >= keys values.
 // pos: position of every query token; batch_of: its request (null: token i belongs to request i).
 LLB_EXPORT int llb_latent_attn_generic(const void* q_lat, int dtype, const void* pool, int row_elems,
                                        const int* req_to_token, int64_t r2t_stride, const int* b_req_idx, const int* pos,
-                                       const int* batch_of, void* out, int T, int H, int rank, float scale, int window,
-                                       cudaStream_t st) {
+                                       const int* batch_of, void* out, int T, int H, int keys, int rank, float scale,
+                                       int window, cudaStream_t st) {
   if (T <= 0) return LLB_OK;
-  if (rank <= 0 || rank > 1024 || rank > row_elems || H <= 0 || H > 65535) return LLB_ERR_UNSUPPORTED;
+  if (rank <= 0 || rank > keys || keys > 1024 || keys > row_elems || H <= 0 || H > 65535) return LLB_ERR_UNSUPPORTED;
   return dtype == 0 ? launch_generic<float>(q_lat, pool, row_elems, req_to_token, r2t_stride, b_req_idx, pos, batch_of,
-                                            out, T, H, rank, scale, window, st)
+                                            out, T, H, keys, rank, scale, window, st)
                     : launch_generic<bf16>(q_lat, pool, row_elems, req_to_token, r2t_stride, b_req_idx, pos, batch_of,
-                                           out, T, H, rank, scale, window, st);
+                                           out, T, H, keys, rank, scale, window, st);
 }
 
-// bf16; rank a multiple of 8, at most 512.  splits > 1: part_o [splits * T * H * rank] and part_ml [splits * T * H * 2]
+// bf16; keys and rank multiples of 8, at most 576 and 512.  splits > 1: part_o [splits * T * H * rank] and part_ml [splits * T * H * 2]
 // floats of scratch.
 LLB_EXPORT int llb_latent_attn_mma(const void* q_lat, const void* pool, int row_elems, const int* req_to_token,
                                    int64_t r2t_stride, const int* b_req_idx, const int* pos, const int* batch_of,
-                                   void* out, float* part_o, float* part_ml, int T, int H, int rank, int splits,
-                                   float scale, int window, cudaStream_t st) {
+                                   void* out, float* part_o, float* part_ml, int T, int H, int keys, int rank,
+                                   int splits, float scale, int window, cudaStream_t st) {
   if (T <= 0) return LLB_OK;
-  if (rank <= 0 || rank > 512 || (rank % 8) || (row_elems % 8) || rank > row_elems || H <= 0) return LLB_ERR_UNSUPPORTED;
+  if (rank <= 0 || rank > 512 || rank > keys || keys > 576 || (rank % 8) || (keys % 8) || (row_elems % 8) ||
+      keys > row_elems || H <= 0)
+    return LLB_ERR_UNSUPPORTED;
   if (splits < 1 || splits > 256 || (splits > 1 && (part_o == nullptr || part_ml == nullptr))) return LLB_ERR_BAD_ARG;
   if (((uintptr_t)q_lat & 15) || ((uintptr_t)pool & 15) || ((uintptr_t)out & 3)) return LLB_ERR_BAD_ARG;
   MmaArgs a{(const bf16*)q_lat, (const bf16*)pool, (bf16*)out, req_to_token, b_req_idx, pos, batch_of, part_o,
-            (float2*)part_ml, r2t_stride, row_elems, T, H, rank, window, splits, scale * kLog2e};
+            (float2*)part_ml, r2t_stride, row_elems, T, H, keys, rank, window, splits, scale * kLog2e};
   int rc;
-  if (rank <= 128)
-    rc = launch_mma<128>(a, st);
-  else if (rank <= 256)
-    rc = launch_mma<256>(a, st);
-  else if (rank <= 384)
-    rc = launch_mma<384>(a, st);
+  if (rank <= 128 && keys <= 128)
+    rc = launch_mma<128, 128>(a, st);
+  else if (rank <= 128 && keys <= 192)
+    rc = launch_mma<192, 128>(a, st);
+  else if (rank <= 256 && keys <= 256)
+    rc = launch_mma<256, 256>(a, st);
+  else if (rank <= 256 && keys <= 320)
+    rc = launch_mma<320, 256>(a, st);
+  else if (rank <= 384 && keys <= 384)
+    rc = launch_mma<384, 384>(a, st);
+  else if (rank <= 384 && keys <= 448)
+    rc = launch_mma<448, 384>(a, st);
+  else if (keys <= 512)
+    rc = launch_mma<512, 512>(a, st);
   else
-    rc = launch_mma<512>(a, st);
+    rc = launch_mma<576, 512>(a, st);
   if (rc || splits == 1) return rc;
   latent_attn_merge_kernel<<<cdiv(T * H, 8), 256, 0, st>>>(part_o, (const float2*)part_ml, (bf16*)out, T * H, rank, splits);
   LLB_LAUNCH_CHECK();

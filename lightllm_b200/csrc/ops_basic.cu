@@ -364,6 +364,47 @@ __global__ void __launch_bounds__(256) copy_rows_kernel(uint4* __restrict__ dst,
     for (int v = threadIdx.x; v < row_vec; v += blockDim.x) dp[v] = sp[v];
   }
 }
+// x[t] *= sigmoid(gate[t]), rows of N elements (a multiple of 8) with their own pitches
+template <typename E>
+__global__ void __launch_bounds__(256) sigmoid_mul_kernel(E* __restrict__ x, int64_t x_stride, const E* __restrict__ gate,
+                                                          int64_t gate_stride, int64_t items, int n_vec) {
+  pdl_wait();
+  const int64_t id = (int64_t)blockIdx.x * 256 + threadIdx.x;
+  if (id >= items) return;
+  const int64_t t = id / n_vec;
+  const int c = (int)(id - t * n_vec) * 8;
+  E* xp = x + t * x_stride + c;
+  const E* gp = gate + t * gate_stride + c;
+  if constexpr (sizeof(E) == 2) {
+    float f[8], g[8];
+    unpack8(*reinterpret_cast<const bf16x8*>(xp), f);
+    unpack8(*reinterpret_cast<const bf16x8*>(gp), g);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) f[i] = __fdividef(f[i], 1.f + __expf(-g[i]));
+    *reinterpret_cast<bf16x8*>(xp) = pack8(f);
+  } else {
+#pragma unroll
+    for (int i = 0; i < 8; ++i) xp[i] /= 1.f + expf(-gp[i]);
+  }
+}
+
+// dt: 0 = fp32, 1 = bf16
+LLB_EXPORT int llb_sigmoid_mul(void* x, int dt, int64_t x_stride, const void* gate, int64_t gate_stride, int T, int N,
+                               cudaStream_t st) {
+  if (T <= 0 || N <= 0) return LLB_OK;
+  if ((N % 8) || (x_stride % 8) || (gate_stride % 8) || ((uintptr_t)x & 15) || ((uintptr_t)gate & 15)) return LLB_ERR_BAD_ARG;
+  const int64_t items = (int64_t)T * (N / 8);
+  const dim3 grid((unsigned)cdiv64(items, 256));
+  if (dt == 0)
+    launch_pdl(sigmoid_mul_kernel<float>, grid, dim3(256), 0, st, (float*)x, x_stride, (const float*)gate, gate_stride, items,
+               N / 8);
+  else
+    launch_pdl(sigmoid_mul_kernel<bf16>, grid, dim3(256), 0, st, (bf16*)x, x_stride, (const bf16*)gate, gate_stride, items,
+               N / 8);
+  LLB_LAUNCH_CHECK();
+  return LLB_OK;
+}
+
 LLB_EXPORT int llb_copy_rows(void* dst, const void* src, const int* dst_idx, const int* src_idx, int n_rows,
                              int64_t row_bytes, int64_t dst_row_stride_bytes, int64_t src_row_stride_bytes,
                              cudaStream_t st) {

@@ -1,8 +1,9 @@
-// RMS norms around an fp32 residual stream whose sublayers read the stream itself and are normalised on the way out:
+// RMS norms around an fp32 residual stream: sublayers that read the stream itself and are normalised on the way out (w), and
+// sublayers that read a norm of the stream (w_next) and are added as they are (no w):
 //
 //   embedding_pair    x[t] = table[id] + table2[(prev * mul_prev + id * mul_cur) mod buckets]   (second table optional; a
-//                     sequence's first token takes row `buckets`);  h[t] = x[t]
-//   add_rms           x += rms(y) * w;  h = x, or rms(x) * w_next when a next norm is given
+//                     sequence's first token takes row `buckets`);  h[t] = x[t], or rms(x[t]) * w_next
+//   add_rms           x += rms(y) * w, or x += y;  h = x, or rms(x) * w_next when a next norm is given
 //   moe_combine_rms   y[t] = sum_k weight[t,k] * expert_out[row of (t,k)] + shared[t], then add_rms; or, when a tensor-
 //                     parallel reduction follows, y[t] is written out in fp32
 //
@@ -39,8 +40,10 @@ template <typename TH>
 __global__ void __launch_bounds__(256) embedding_pair_kernel(const int64_t* __restrict__ ids, const TH* __restrict__ table,
                                                              const TH* __restrict__ table2, const Bigram g,
                                                              float* __restrict__ x, TH* __restrict__ h, int64_t vocab,
-                                                             int W) {
+                                                             int W, const float* __restrict__ w_next, int width,
+                                                             float eps) {
   pdl_wait();
+  __shared__ float red[33];
   const int t = blockIdx.x;
   const int64_t id = ids[t];
   const TH* r1 = table + (id >= 0 && id < vocab ? id : 0) * W;
@@ -63,6 +66,7 @@ __global__ void __launch_bounds__(256) embedding_pair_kernel(const int64_t* __re
     r2 = table2 + row * W;
     if (threadIdx.x == 0) g.slot_token[LLB_CHECK_SLOT(g.mem_index[t])] = (int)id;
   }
+  float ss = 0.f;
   for (int v = threadIdx.x * 8; v < W; v += blockDim.x * 8) {
     float a[8];
     ld8(r1 + v, a);
@@ -73,6 +77,18 @@ __global__ void __launch_bounds__(256) embedding_pair_kernel(const int64_t* __re
       for (int i = 0; i < 8; ++i) a[i] += b[i];
     }
     st8(x + (int64_t)t * W + v, a);
+    if (w_next == nullptr) st8(h + (int64_t)t * W + v, a);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) ss = fmaf(a[i], a[i], ss);
+  }
+  if (w_next == nullptr) return;
+  const float inv = rsqrtf(block_sum(ss, red) / (float)width + eps);
+  for (int v = threadIdx.x * 8; v < W; v += blockDim.x * 8) {  // a thread reads back what it wrote
+    float a[8], wv[8];
+    ld8(x + (int64_t)t * W + v, a);
+    ld8(w_next + v, wv);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) a[i] *= inv * wv[i];
     st8(h + (int64_t)t * W + v, a);
   }
 }
@@ -124,14 +140,19 @@ __global__ void __launch_bounds__(256) add_rms_kernel(const TY* __restrict__ y, 
     for (int i = 0; i < 8; ++i) ss = fmaf(yv[j][i], yv[j][i], ss);
   }
   if (x == nullptr) return;
-  const float inv = rsqrtf(block_sum(ss, red) / (float)width + eps);
+  const float inv = w != nullptr ? rsqrtf(block_sum(ss, red) / (float)width + eps) : 1.f;
   float sx = 0.f;
 #pragma unroll
   for (int j = 0; j < VPT; ++j) {
     const int v = threadIdx.x + j * blockDim.x;
     if (v >= nv) continue;
     float wv[8];
-    ld8(w + v * 8, wv);
+    if (w != nullptr) {
+      ld8(w + v * 8, wv);
+    } else {
+#pragma unroll
+      for (int i = 0; i < 8; ++i) wv[i] = 1.f;
+    }
 #pragma unroll
     for (int i = 0; i < 8; ++i) {
       xv[j][i] += yv[j][i] * inv * wv[i];
@@ -183,7 +204,7 @@ int dispatch_add(const void* y, int y_dt, const Combine& c, const void* shared, 
                  const float* w, const float* w_next, int T, int width, int W, float eps, cudaStream_t st) {
   if (T <= 0) return LLB_OK;
   if (W <= 0 || (W % 8) || width <= 0 || width > W) return LLB_ERR_BAD_ARG;
-  if (x == nullptr ? y_out == nullptr : (h == nullptr || w == nullptr)) return LLB_ERR_BAD_ARG;
+  if (x == nullptr ? y_out == nullptr : h == nullptr) return LLB_ERR_BAD_ARG;
   if (y_dt == 0)
     return h_dt == 0 ? launch_add<float, float, COMBINE>(y, c, shared, x, h, y_out, w, w_next, T, width, W, eps, st)
                      : launch_add<float, bf16, COMBINE>(y, c, shared, x, h, y_out, w, w_next, T, width, W, eps, st);
@@ -194,28 +215,29 @@ int dispatch_add(const void* y, int y_dt, const Combine& c, const void* shared, 
 }  // namespace
 
 // Number formats: 0 = fp32, 1 = bf16.  table [vocab, W], table2 [buckets + 1, W] or null; batch_of null: row t belongs to
-// request t (decode).  slot_token [pool slots] receives the token id of every new token at mem_index[t].
+// request t (decode).  slot_token [pool slots] receives the token id of every new token at mem_index[t].  w_next (or null):
+// fp32 [W], zero beyond `width`.
 LLB_EXPORT int llb_embedding_pair(const int64_t* ids, const void* table, int dt, int64_t vocab, const void* table2,
                                   int64_t buckets, int64_t mul_prev, int64_t mul_cur, int* slot_token,
                                   const int* mem_index, const int* pos, const int* batch_of, const int* b_req_idx,
                                   const int* req_to_token, int64_t r2t_stride, float* x, void* h, int T, int W,
-                                  cudaStream_t st) {
+                                  const float* w_next, int width, float eps, cudaStream_t st) {
   if (T <= 0) return LLB_OK;
-  if (W <= 0 || (W % 8)) return LLB_ERR_BAD_ARG;
+  if (W <= 0 || (W % 8) || width <= 0 || width > W) return LLB_ERR_BAD_ARG;
   if (table2 != nullptr && (buckets <= 0 || slot_token == nullptr)) return LLB_ERR_BAD_ARG;
   const Bigram g{buckets, mul_prev, mul_cur, slot_token, mem_index, pos, batch_of, b_req_idx, req_to_token, r2t_stride};
   const int threads = W / 8 >= 256 ? 256 : cdiv(W / 8, 32) * 32;
   if (dt == 0)
     launch_pdl(embedding_pair_kernel<float>, dim3(T), dim3(threads), 0, st, ids, (const float*)table, (const float*)table2, g,
-               x, (float*)h, vocab, W);
+               x, (float*)h, vocab, W, w_next, width, eps);
   else
     launch_pdl(embedding_pair_kernel<bf16>, dim3(T), dim3(threads), 0, st, ids, (const bf16*)table, (const bf16*)table2, g, x,
-               (bf16*)h, vocab, W);
+               (bf16*)h, vocab, W, w_next, width, eps);
   LLB_LAUNCH_CHECK();
   return LLB_OK;
 }
 
-// y [T, W] (y_dt), x fp32 [T, W] in place, h [T, W] (h_dt), w and w_next (or null) fp32 [W].
+// y [T, W] (y_dt), x fp32 [T, W] in place, h [T, W] (h_dt), w and w_next (either may be null) fp32 [W].
 LLB_EXPORT int llb_add_rms(const void* y, int y_dt, float* x, void* h, int h_dt, const float* w, const float* w_next, int T,
                            int width, int W, float eps, cudaStream_t st) {
   return dispatch_add<false>(y, y_dt, Combine{nullptr, nullptr, 0}, nullptr, x, h, h_dt, nullptr, w, w_next, T, width, W, eps,

@@ -1,14 +1,15 @@
 // Prompt attention through a sliding window on the 5th-generation tensor cores, over keys and values that were formed
 // for this pass (latent attention in its expanded form): causal, varlen, aware of cached positions before the new ones.
-// Key sizes and value sizes are 64 or 128 and may differ; every query head has its own keys and values.
+// Key sizes up to 256 and value sizes up to 128, multiples of 64; every query head has its own keys and values.  An optional gate
+// [T, H * DV] multiplies the result element by element with its sigmoid.
 //
 //   kv [rows, H * DK | H * DV]: request b's keys are rows cu_kv[b] .., position kv_start[b] first
 //   a query sees its own position and the window - 1 before it  (window 0: all before it)
 //
-// One CTA computes 128 query rows of one (request, head), as in attention_tc.cu: per 128-key tile S = Q . K^T into one of
+// One CTA computes 128 query rows of one (request, head), as in attention_tc.cu: per tile of 128 keys (64 for key sizes above 128) S = Q . K^T into one of
 // two tensor-memory buffers, softmax by eight warps (two threads per query row), P . V into a third buffer that the
 // softmax threads add to their fp32 rows.  What differs:
-//   * the tiles are rows of a dense matrix, so one thread fetches them with TMA (64 columns x 128 rows per box, 128-byte
+//   * the tiles are rows of a dense matrix, so one thread fetches them with TMA (64 columns x BN rows per box, 128-byte
 //     swizzle); only the tiles the window reaches are visited
 //   * the weights enter P . V as the sum of two bf16 tiles (high and low part): they keep fp32-like precision
 #include "sm100_ptx.cuh"
@@ -18,19 +19,20 @@ using namespace llb::sm100;
 
 namespace {
 
-constexpr int BM = 128, BN = 128;
+constexpr int BM = 128;
 constexpr int BLOCK_BYTES = 128 * 128;  // 128 rows x 64 bf16
 constexpr int THREADS = 10 * 32;        // warp 0: TMA, warp 1: MMA, warps 2..9: softmax
 constexpr float kLog2e = 1.4426950408889634f;
 constexpr uint64_t kIssueWaitNs = 2000000000ull;
-constexpr int P_BYTES = 2 * BLOCK_BYTES;
 
 __device__ int g_window_tc_status = 0;
 
-template <int DK, int DV>
+template <int DK, int DV, int BN>
 struct Layout {
-  static constexpr int K_BYTES = DK / 64 * BLOCK_BYTES, V_BYTES = DV / 64 * BLOCK_BYTES;
-  static constexpr int OFF_Q = 0, OFF_PH = K_BYTES, OFF_PL = OFF_PH + P_BYTES, OFF_KV = OFF_PL + P_BYTES;
+  static constexpr int KV_BLOCK = BN * 128;  // BN rows x 64 bf16
+  static constexpr int Q_BYTES = DK / 64 * BLOCK_BYTES, P_BYTES = BN / 64 * BLOCK_BYTES;
+  static constexpr int K_BYTES = DK / 64 * KV_BLOCK, V_BYTES = DV / 64 * KV_BLOCK;
+  static constexpr int OFF_Q = 0, OFF_PH = Q_BYTES, OFF_PL = OFF_PH + P_BYTES, OFF_KV = OFF_PL + P_BYTES;
   static constexpr int STAGE = K_BYTES + V_BYTES;
   static constexpr int OFF_BAR = OFF_KV + 2 * STAGE;
   static constexpr int OFF_XCH = OFF_BAR + 256;  // float [2 tile parities][2 halves][128 rows]
@@ -52,14 +54,17 @@ struct Params {
   const int *cu_q, *cu_kv, *kv_start, *b_ready_len;
   bf16* out;
   int64_t out_stride;
+  const bf16* gate;  // [T, >= H * DV] or null
+  int64_t gate_stride;
   int H, window;
   float scale_log2;
 };
 
-template <int DK, int DV>
+template <int DK, int DV, int BN>
 __global__ void __launch_bounds__(THREADS, 1)
 window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmKV, const Params p) {
-  using L = Layout<DK, DV>;
+  using L = Layout<DK, DV, BN>;
+  constexpr int HK = BN / 2;  // keys of a score tile per softmax thread
   extern __shared__ __align__(1024) uint8_t smem[];
   const uint32_t smem_base = smem_u32(smem);
   const uint32_t bar_base = smem_base + L::OFF_BAR;
@@ -118,7 +123,7 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
     if (lane == 0) {
       tma_prefetch_desc(&tmQ);
       tma_prefetch_desc(&tmKV);
-      mbar_expect_tx(q_full, L::K_BYTES);
+      mbar_expect_tx(q_full, L::Q_BYTES);
 #pragma unroll
       for (int c = 0; c < DK / 64; ++c)
         tma_load_2d(smem_base + L::OFF_Q + c * BLOCK_BYTES, &tmQ, q_full, h * DK + c * 64, q_begin + q0);
@@ -130,12 +135,12 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
         mbar_expect_tx(k_full(stage), L::K_BYTES);
 #pragma unroll
         for (int c = 0; c < DK / 64; ++c)
-          tma_load_2d(k_dst + c * BLOCK_BYTES, &tmKV, k_full(stage), h * DK + c * 64, row0 + j * BN);
+          tma_load_2d(k_dst + c * L::KV_BLOCK, &tmKV, k_full(stage), h * DK + c * 64, row0 + j * BN);
         if (!mbar_wait(v_empty(stage), par, abort_flag, status, 62)) break;
         mbar_expect_tx(v_full(stage), L::V_BYTES);
 #pragma unroll
         for (int c = 0; c < DV / 64; ++c)
-          tma_load_2d(v_dst + c * BLOCK_BYTES, &tmKV, v_full(stage), p.H * DK + h * DV + c * 64, row0 + j * BN);
+          tma_load_2d(v_dst + c * L::KV_BLOCK, &tmKV, v_full(stage), p.H * DK + h * DV + c * 64, row0 + j * BN);
       }
     }
     __syncwarp();
@@ -155,9 +160,9 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
           const uint32_t k_addr = smem_base + L::OFF_KV + (s_next & 1) * L::STAGE;
 #pragma unroll
           for (int ks = 0; ks < DK / 16; ++ks) {
-            const uint32_t off = (ks >> 2) * BLOCK_BYTES + (ks & 3) * 32;
-            umma_bf16(tmem_base + (s_next & 1) * BN, umma_smem_desc_sw128(smem_base + L::OFF_Q + off),
-                      umma_smem_desc_sw128(k_addr + off), IDESC_S, ks != 0);
+            umma_bf16(tmem_base + (s_next & 1) * BN,
+                      umma_smem_desc_sw128(smem_base + L::OFF_Q + (ks >> 2) * BLOCK_BYTES + (ks & 3) * 32),
+                      umma_smem_desc_sw128(k_addr + (ks >> 2) * L::KV_BLOCK + (ks & 3) * 32), IDESC_S, ks != 0);
           }
           umma_commit(s_full(s_next & 1));
           umma_commit(k_empty(s_next & 1));
@@ -179,7 +184,7 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
               for (int ks = 0; ks < BN / 16; ++ks) {  // 16 keys per instruction
                 const uint32_t a_off = (ks >> 2) * BLOCK_BYTES + (ks & 3) * 32;
                 umma_bf16(tmem_base + 2 * BN + hb * 64, umma_smem_desc_sw128(p_addr + a_off),
-                          umma_smem_desc_sw128_mn(v_addr + hb * BLOCK_BYTES + ks * 2048), IDESC_PV, (part | ks) != 0);
+                          umma_smem_desc_sw128_mn(v_addr + hb * L::KV_BLOCK + ks * 2048), IDESC_PV, (part | ks) != 0);
               }
             }
           }
@@ -205,38 +210,38 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
     }
     __syncwarp();
   } else {
-    // ---- softmax + output accumulation.  Two threads per query row: `half` 0 owns keys 0..63 of every score tile and
-    // the first half of the value columns, half 1 the rest; they exchange the row maximum ----
+    // ---- softmax + output accumulation.  Two threads per query row: `half` 0 owns the first half of the keys of every score
+    // tile and of the value columns, half 1 the rest; they exchange the row maximum ----
     constexpr int OC = DV / 2;  // value columns per thread
     const int lane_grp = warp & 3;
     const int half = (warp - 2) >> 2;
     const int erow = lane_grp * 32 + lane;
     const int prow = ready + q0 + erow;  // absolute position of this row's token
     const uint32_t t_lane = tmem_base + ((uint32_t)(lane_grp * 32) << 16);
-    const uint32_t t_s = t_lane + half * 64, t_o = t_lane + 2 * BN + half * OC;
+    const uint32_t t_s = t_lane + half * HK, t_o = t_lane + 2 * BN + half * OC;
     float o[OC];
 #pragma unroll
     for (int i = 0; i < OC; ++i) o[i] = 0.f;
     float m_run = -INFINITY, l_run = 0.f;
     for (int j = 0; j < n_tiles; ++j) {
-      const int kt = kv0 + j * BN + half * 64;  // position of my first key
+      const int kt = kv0 + j * BN + half * HK;  // position of my first key
       mbar_wait(s_full(j & 1), ((uint32_t)j >> 1) & 1u, abort_flag, status, 65);
       tc_fence_after();
-      uint32_t sr[64];
-      tmem_ld_32x32(t_s + (j & 1) * BN, sr);
-      tmem_ld_32x32(t_s + (j & 1) * BN + 32, sr + 32);
+      uint32_t sr[HK];
+#pragma unroll
+      for (int c = 0; c < HK; c += 32) tmem_ld_32x32(t_s + (j & 1) * BN + c, sr + c);
       tmem_wait_ld();
       // my columns lo..hi are visible to this row
       const int hi = min(prow, kv_end - 1) - kt;
       const int lo = p.window > 0 ? prow - p.window + 1 - kt : 0;
-      const bool all_visible = hi >= 63 && lo <= 0;
+      const bool all_visible = hi >= HK - 1 && lo <= 0;
       float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
       if (all_visible) {
 #pragma unroll
-        for (int e = 0; e < 64; ++e) mx4[e & 3] = fmaxf(mx4[e & 3], __uint_as_float(sr[e]));
+        for (int e = 0; e < HK; ++e) mx4[e & 3] = fmaxf(mx4[e & 3], __uint_as_float(sr[e]));
       } else {
 #pragma unroll
-        for (int e = 0; e < 64; ++e)
+        for (int e = 0; e < HK; ++e)
           if (e >= lo && e <= hi) mx4[e & 3] = fmaxf(mx4[e & 3], __uint_as_float(sr[e]));
       }
       float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
@@ -260,7 +265,7 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
       }
       float rs4[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
-      for (int g = 0; g < 8; ++g) {
+      for (int g = 0; g < HK / 8; ++g) {
         uint32_t ph[4], pl[4];
 #pragma unroll
         for (int e = 0; e < 8; e += 2) {
@@ -276,7 +281,7 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
           pl[e / 2] = pack_bf16x2(pv[0] - __uint_as_float(ph[e / 2] << 16),
                                   pv[1] - __uint_as_float(ph[e / 2] & 0xffff0000u));
         }
-        const uint32_t off = tile_off(erow, half * 8 + g);
+        const uint32_t off = tile_off(erow, half * (HK / 8) + g);
         *reinterpret_cast<uint4*>(smem + L::OFF_PH + off) = make_uint4(ph[0], ph[1], ph[2], ph[3]);
         *reinterpret_cast<uint4*>(smem + L::OFF_PL + off) = make_uint4(pl[0], pl[1], pl[2], pl[3]);
       }
@@ -320,9 +325,20 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
     for (int i = 0; i < SEGS; ++i) {
       const int id = i * 32 + lane, r = id / SEGS, seg = id % SEGS;
       const int lr = lane_grp * 32 + r;
-      if (lr < rows_valid)
-        *reinterpret_cast<uint4*>(p.out + (int64_t)(q_begin + q0 + lr) * p.out_stride + (int64_t)h * DV + half * OC +
-                                  seg * 8) = *reinterpret_cast<const uint4*>(stg + r * PITCH + seg * 16);
+      if (lr < rows_valid) {
+        const int64_t row = q_begin + q0 + lr;
+        const int col = h * DV + half * OC + seg * 8;
+        bf16x8 v = *reinterpret_cast<const bf16x8*>(stg + r * PITCH + seg * 16);
+        if (p.gate != nullptr) {
+          float f[8], g[8];
+          unpack8(v, f);
+          unpack8(*reinterpret_cast<const bf16x8*>(p.gate + row * p.gate_stride + col), g);
+#pragma unroll
+          for (int e = 0; e < 8; ++e) f[e] = __fdividef(f[e], 1.f + __expf(-g[e]));
+          v = pack8(f);
+        }
+        *reinterpret_cast<bf16x8*>(p.out + row * p.out_stride + col) = v;
+      }
     }
     tc_fence_before();
   }
@@ -335,20 +351,20 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
   }
 }
 
-template <int DK, int DV>
+template <int DK, int DV, int BN>
 int launch(const CUtensorMap& tq, const CUtensorMap& tkv, const Params& p, int B, int max_q_len, cudaStream_t st) {
-  using L = Layout<DK, DV>;
+  using L = Layout<DK, DV, BN>;
   static_assert(L::BYTES <= 227 * 1024, "shared memory");
   static_assert(8 * 32 * (DV + 16) <= L::OFF_KV, "output staging fits the Q / P buffers");
   static DeviceOnce configured;
   if (!configured.done()) {
-    cudaError_t e = cudaFuncSetAttribute(window_prefill_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    cudaError_t e = cudaFuncSetAttribute(window_prefill_kernel<DK, DV, BN>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                          L::BYTES);
     if (e != cudaSuccess) return (int)e;
     configured.set();
   }
   const dim3 grid((max_q_len + BM - 1) / BM, p.H, B);
-  window_prefill_kernel<DK, DV><<<grid, THREADS, L::BYTES, st>>>(tq, tkv, p);
+  window_prefill_kernel<DK, DV, BN><<<grid, THREADS, L::BYTES, st>>>(tq, tkv, p);
   LLB_LAUNCH_CHECK();
   return LLB_OK;
 }
@@ -362,21 +378,33 @@ LLB_EXPORT int llb_window_tc_status() {
   return v;
 }
 
-// q [T, >= H * DK] bf16 (row pitch q_stride), kv [kv_rows, H * (DK + DV)] (pitch kv_stride), out [T, H * DV].
+// q [T, >= H * DK] bf16 (row pitch q_stride), kv [kv_rows, H * (DK + DV)] (pitch kv_stride), out [T, H * DV]; gate
+// [T, >= H * DV] or null: out *= sigmoid(gate).
 LLB_EXPORT int llb_window_prefill_tc(const void* q, int64_t q_stride, const void* kv, int64_t kv_stride, int kv_rows,
                                      const int* cu_q, const int* cu_kv, const int* kv_start, const int* b_ready_len,
                                      void* out, int64_t out_stride, int B, int T, int max_q_len, int H, int dk, int dv,
-                                     float sm_scale, int window, cudaStream_t st) {
+                                     float sm_scale, int window, const void* gate, int64_t gate_stride,
+                                     cudaStream_t st) {
   if (B <= 0 || max_q_len <= 0 || T <= 0) return LLB_OK;
   if (H <= 0 || H > 65535 || B > 65535 || kv_rows <= 0 || window < 0) return LLB_ERR_BAD_ARG;
-  if ((dk != 64 && dk != 128) || (dv != 64 && dv != 128)) return LLB_ERR_UNSUPPORTED;
+  if ((dk != 64 && dk != 128 && dk != 192 && dk != 256) || (dv != 64 && dv != 128)) return LLB_ERR_UNSUPPORTED;
+  if (gate != nullptr && ((gate_stride % 8) || ((uintptr_t)gate & 15))) return LLB_ERR_BAD_ARG;
+  const int bn = dk > 128 ? 64 : 128;
   if ((out_stride % 8) || ((uintptr_t)out & 15)) return LLB_ERR_BAD_ARG;
   CUtensorMap tq, tkv;
   int rc = make_tmap_2d(&tq, q, 2, (uint64_t)T, (uint64_t)H * dk, (uint64_t)q_stride, BM, 64);
   if (rc) return rc;
-  rc = make_tmap_2d(&tkv, kv, 2, (uint64_t)kv_rows, (uint64_t)H * (dk + dv), (uint64_t)kv_stride, BN, 64);
+  rc = make_tmap_2d(&tkv, kv, 2, (uint64_t)kv_rows, (uint64_t)H * (dk + dv), (uint64_t)kv_stride, bn, 64);
   if (rc) return rc;
-  const Params p{cu_q, cu_kv, kv_start, b_ready_len, (bf16*)out, out_stride, H, window, sm_scale * kLog2e};
-  if (dk == 64) return dv == 64 ? launch<64, 64>(tq, tkv, p, B, max_q_len, st) : launch<64, 128>(tq, tkv, p, B, max_q_len, st);
-  return dv == 64 ? launch<128, 64>(tq, tkv, p, B, max_q_len, st) : launch<128, 128>(tq, tkv, p, B, max_q_len, st);
+  const Params p{cu_q, cu_kv, kv_start, b_ready_len, (bf16*)out, out_stride, (const bf16*)gate, gate_stride, H, window,
+                 sm_scale * kLog2e};
+#define LLB_WINDOW(DK, BN)                                                                                        \
+  if (dk == DK)                                                                                                   \
+    return dv == 64 ? launch<DK, 64, BN>(tq, tkv, p, B, max_q_len, st) : launch<DK, 128, BN>(tq, tkv, p, B, max_q_len, st);
+  LLB_WINDOW(64, 128)
+  LLB_WINDOW(128, 128)
+  LLB_WINDOW(192, 64)
+  LLB_WINDOW(256, 64)
+#undef LLB_WINDOW
+  return LLB_ERR_UNSUPPORTED;
 }

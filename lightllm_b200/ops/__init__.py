@@ -222,12 +222,13 @@ def _tuned_bn(M: int, N: int, K: int, epi: str) -> int:
 
 
 def gemm(a, w, epi: str = "store", residual=None, bias=None, out=None, bn: int = 0, stream_k: int = 0,
-         out_scale: float = 1.0, x=None, dyt=None, clamp=None):
+         out_scale: float = 1.0, x=None, dyt=None, clamp=None, softcap: float = 0.0):
     """C = A . W^T on the tcgen05 tensor cores.  a [M, K], w [N, K] (checkpoint layout).  fp32 operands run on the
     CUDA cores in fp32 (`csrc/gemm_f32.cu`).
 
     epi: "store" | "residual" (C += residual) | "gated_silu"/"gated_gelu" (w rows interleaved with
-    `reference.interleave_gate_up`, C is [M, N/2]) | "f32" (fp32 output, e.g. logits, times `out_scale`) |
+    `reference.interleave_gate_up`, C is [M, N/2]) | "f32" (fp32 output, e.g. logits, times
+    `out_scale`; with softcap > 0 then softcap * tanh(. / softcap)) |
     "relu2" (square of relu) | "dyt": with the fp32 residual stream x [M, N] and dyt = (post, next) `DytNorm`s,
     x += post(A . W^T) in place and C = next(x) | "gated_clamp": interleaved as the other gated forms, with
     clamp = (alpha, limit): g = min(g, limit), u = clamp(u, -limit, limit), C = (u + 1) g sigmoid(alpha g).
@@ -242,16 +243,16 @@ def gemm(a, w, epi: str = "store", residual=None, bias=None, out=None, bn: int =
 
         return int8.gemm_int8(a, w, epi, residual, bias, out)
     if not _is_cuda(a):
-        res = ref.gemm(a, w, epi, residual, bias, out_scale=out_scale, x=x, dyt=dyt, clamp=clamp)
+        res = ref.gemm(a, w, epi, residual, bias, out_scale=out_scale, x=x, dyt=dyt, clamp=clamp, softcap=softcap)
         if out is not None:
             out.copy_(res)
             return out
         return res
     if a.dtype == torch.float32:
-        return gemm_f32(a, w, epi, residual, bias, out, out_scale, x, dyt, clamp=clamp)
+        return gemm_f32(a, w, epi, residual, bias, out, out_scale, x, dyt, clamp=clamp, softcap=softcap)
     _req_bf16(a, w, residual, bias)
-    if epi in ("dyt", "gated_clamp") or out_scale != 1.0:
-        return _gemm_fused(a, w, epi, bias, out, bn, out_scale, x, dyt, clamp)
+    if epi in ("dyt", "gated_clamp") or out_scale != 1.0 or softcap > 0:
+        return _gemm_fused(a, w, epi, bias, out, bn, out_scale, x, dyt, clamp, softcap)
     if _GEMM_DEBUG_TORCH:  # debugging aid only (LLB_GEMM_DEBUG_TORCH=1): bypasses the tcgen05 kernel
         res = ref.gemm(a, w, epi, residual, bias)
         if out is not None:
@@ -294,7 +295,7 @@ def _clamp_args(clamp):
     return f32(alpha), f32(limit)
 
 
-def _gemm_fused(a, w, epi, bias, out, bn, out_scale, x, dyt, clamp=None):
+def _gemm_fused(a, w, epi, bias, out, bn, out_scale, x, dyt, clamp=None, softcap=0.0):
     M, K = a.shape
     N = w.shape[0]
     assert w.shape[1] == K and w.stride(1) == 1 and a.stride(1) == 1
@@ -307,14 +308,14 @@ def _gemm_fused(a, w, epi, bias, out, bn, out_scale, x, dyt, clamp=None):
     check(kernels().llb_gemm_bf16_fused(ptr(a), i64(a.stride(0)), ptr(w), i64(w.stride(0)), ptr(out),
                                         i64(out.stride(0)), ptr(bias), c_int(M), c_int(N), c_int(K),
                                         c_int(EPI_CODES[epi]), c_int(bn), f32(out_scale), ptr(x), *_dyt_args(post),
-                                        *_dyt_args(nxt), *_clamp_args(clamp), ptr(gemm_status(a.device)), stream()),
-          "gemm_bf16_fused")
+                                        *_dyt_args(nxt), *_clamp_args(clamp), f32(softcap), ptr(gemm_status(a.device)),
+                                        stream()), "gemm_bf16_fused")
     _count()
     return out
 
 
 def gemm_f32(a, w, epi="store", residual=None, bias=None, out=None, out_scale=1.0, x=None, dyt=None,
-             mblock_expert=None, clamp=None):
+             mblock_expert=None, clamp=None, softcap=0.0):
     """fp32 GEMM, same epilogues as `gemm`.  a [M, K] and w [N, K]; or a [M, batch, K] and w [batch, N, K] (per-head
     products, out [M, batch, N]); or grouped with w [E, N, K] and the expert of every 128-row block."""
     grouped = mblock_expert is not None
@@ -336,8 +337,8 @@ def gemm_f32(a, w, epi="store", residual=None, bias=None, out=None, out_scale=1.
                                  i64(w.stride(-2)), i64(w.stride(0) if batched else 0), ptr(out), i64(out.stride(0)),
                                  i64(out.stride(1) if batched else 0), ptr(residual), ptr(bias), ptr(x),
                                  *_dyt_args(post), *_dyt_args(nxt), ptr(mblock_expert), c_int(M), c_int(N), c_int(K),
-                                 c_int(batch), c_int(EPI_CODES[epi]), f32(out_scale), *_clamp_args(clamp), stream()),
-          "gemm_f32")
+                                 c_int(batch), c_int(EPI_CODES[epi]), f32(out_scale), *_clamp_args(clamp), f32(softcap),
+                                 stream()), "gemm_f32")
     _count()
     return out
 
@@ -689,31 +690,32 @@ class BigramTable:
         self.slot_token = None
 
 
-def embedding_pair(ids, table, bigram, req_to_token, b_req_idx, pos, batch_of, mem_index):
-    """(x, h): x = the table's rows (+ the bigram table's) as the fp32 residual stream, h = x in the table's format.
-    batch_of None: row t is the one token of request t."""
+def embedding_pair(ids, table, bigram, req_to_token, b_req_idx, pos, batch_of, mem_index, norm=None):
+    """(x, h): x = the table's rows (+ the bigram table's) as the fp32 residual stream, h = x in the table's format, or
+    rms(x) * w of the first `width` columns with norm = (w, width, eps).  batch_of None: row t is the one token of request t."""
     if not _is_cuda(table):
         x = table[ids].float()
         if bigram is not None:
             x = x + ref.bigram_rows(ids, bigram, req_to_token, b_req_idx, pos, batch_of, mem_index).float()
-        return x, x.to(table.dtype)
+        return x, (x if norm is None else ref.rms_over(x, *norm[1:]) * norm[0]).to(table.dtype)
     T, W = ids.shape[0], table.shape[1]
     x = torch.empty((T, W), dtype=torch.float32, device=table.device)
     h = torch.empty((T, W), dtype=table.dtype, device=table.device)
     assert ids.dtype == torch.int64 and ids.is_contiguous() and table.is_contiguous()
     g = bigram
+    nw, width, eps = norm if norm is not None else (None, W, 1.0)
     check(kernels().llb_embedding_pair(ptr(ids), ptr(table), c_int(DTYPE_CODES[table.dtype]), i64(table.shape[0]),
                                        ptr(g.table if g else None), i64(g.buckets if g else 1),
                                        i64(g.mul_prev if g else 0), i64(g.mul_cur if g else 0),
                                        ptr(g.slot_token if g else None), ptr(mem_index), ptr(pos), ptr(batch_of),
                                        ptr(b_req_idx), ptr(req_to_token), i64(req_to_token.stride(0)), ptr(x), ptr(h),
-                                       c_int(T), c_int(W), stream()), "embedding_pair")
+                                       c_int(T), c_int(W), ptr(nw), c_int(width), f32(eps), stream()), "embedding_pair")
     _count()
     return x, h
 
 
 def add_rms_(x, y, w, width: int, eps: float, dtype, next_w=None):
-    """x += rms(y) * w in place (fp32 stream, the mean taken over the first `width` columns); returns x, or
+    """x += rms(y) * w in place (fp32 stream, the mean taken over the first `width` columns; w None: x += y); returns x, or
     rms(x) * next_w, in `dtype`."""
     if not _is_cuda(x):
         return ref.add_rms_(x, y, w, width, eps, dtype, next_w)
@@ -728,10 +730,11 @@ def add_rms_(x, y, w, width: int, eps: float, dtype, next_w=None):
 
 def qk_norm_rope_scatter_(qkv, kv_layer, cos, sin, pos, slot, q_w, k_w, eps, Hq, Hkv, D, dim, DV, rot_dim):
     """Rows [Hq * D | Hkv * D | Hkv * DV] of qkv: RMS norm of every q and k head over its first `dim` elements (weights
-    q_w, k_w fp32 [D]), rotation of the first rot_dim, q in place, K and V to kv_layer[slot] ([slots, Hkv * (D + DV)])."""
+    q_w, k_w fp32 [D], None: ones), rotation of the first rot_dim, q in place, K and V to kv_layer[slot] ([slots, Hkv * (D + DV)]).
+    Hkv = 0: queries only.  Without weights, norm and rotation may be read in either order."""
     if not _is_cuda(qkv):
         return ref.qk_norm_rope_scatter_(qkv, kv_layer, cos, sin, pos, slot, q_w, k_w, eps, Hq, Hkv, D, dim, DV, rot_dim)
-    assert qkv.stride(1) == 1 and kv_layer.is_contiguous() and qkv.dtype == kv_layer.dtype
+    assert qkv.stride(1) == 1 and (Hkv == 0 or kv_layer.is_contiguous() and qkv.dtype == kv_layer.dtype)
     check(kernels().llb_qk_norm_rope_scatter(ptr(qkv), c_int(DTYPE_CODES[qkv.dtype]), i64(qkv.stride(0)), ptr(kv_layer),
                                              ptr(cos), ptr(sin), ptr(pos), ptr(slot), ptr(q_w), ptr(k_w), f32(eps),
                                              c_int(qkv.shape[0]), c_int(Hq), c_int(Hkv), c_int(D), c_int(dim), c_int(DV),
@@ -740,23 +743,70 @@ def qk_norm_rope_scatter_(qkv, kv_layer, cos, sin, pos, slot, q_w, k_w, eps, Hq,
     return qkv
 
 
+def rope_heads_(x, cos, sin, pos, H, pitch, off, dims, neighbours=True):
+    """Rotary positions on columns off .. off + dims of every head of x [T, >= H * pitch] (heads `pitch` apart), in place: pairs
+    of neighbours (2 i, 2 i + 1), or of halves (i, i + dims / 2).  cos, sin [positions, dims / 2] fp32."""
+    if dims == 0:
+        return x
+    if not _is_cuda(x):
+        v = x[:, : H * pitch].reshape(-1, H, pitch)
+        v[..., off:off + dims] = ref.rotate_pairs(v[..., off:off + dims].float(), cos, sin, pos, neighbours).to(x.dtype)
+        x[:, : H * pitch] = v.reshape(-1, H * pitch)
+        return x
+    assert x.stride(1) == 1 and pos.dtype == torch.int32 and cos.shape[-1] == dims // 2
+    check(kernels().llb_rope_heads(ptr(x), c_int(DTYPE_CODES[x.dtype]), i64(x.stride(0)), ptr(cos), ptr(sin), ptr(pos),
+                                   c_int(x.shape[0]), c_int(H), c_int(pitch), c_int(off), c_int(dims),
+                                   c_int(1 if neighbours else 0), stream()), "rope_heads")
+    _count()
+    return x
+
+
+def sigmoid_mul_(x, gate):
+    """x *= sigmoid(gate) element by element, both [T, N] with rows of any pitch."""
+    if not _is_cuda(x):
+        return x.copy_(x.float() * torch.sigmoid(gate.float()))
+    assert x.stride(1) == 1 and gate.stride(1) == 1 and x.shape == gate.shape and x.dtype == gate.dtype
+    check(kernels().llb_sigmoid_mul(ptr(x), c_int(DTYPE_CODES[x.dtype]), i64(x.stride(0)), ptr(gate), i64(gate.stride(0)),
+                                    c_int(x.shape[0]), c_int(x.shape[1]), stream()), "sigmoid_mul")
+    _count()
+    return x
+
+
 _WINDOW_SIZES = (64, 128, 192, 256)   # head sizes of the tensor-core kernels
 
 
-def window_attention(q, kv_layer, req_to_token, st, Hq, Hkv, D, DV, sm_scale, window, gate=None, out_scale=1.0, out=None):
+class DistanceBias:
+    """Learned bias per head and bucket of the distance n between query and key.  With B rows in the table: bucket n for
+    n < B / 2, beyond that B / 2 buckets spaced by logarithm up to the distance `far`, the last one for all from there on.
+    Kept as `rel` [heads, far + 1] fp32: the bias of every distance up to `far`."""
+
+    def __init__(self, table: torch.Tensor, far: int):
+        B, half = table.shape[0], table.shape[0] // 2
+        assert half >= 1 and far > half, "distance bias: the far distance lies beyond half of the buckets"
+        step = math.log(far / half)
+        rows = [n if n < half else min(B - 1, half + math.floor(math.log(n / half) / step * (B - half)))
+                for n in range(far + 1)]
+        self.far = int(far)
+        self.rel = table.float()[torch.tensor(rows, device=table.device)].t().contiguous()
+
+
+def window_attention(q, kv_layer, req_to_token, st, Hq, Hkv, D, DV, sm_scale, window, gate=None, out_scale=1.0, out=None,
+                     keep=0, bias=None):
     """Causal paged attention with key size D and value size DV through a sliding window (0: none) for the pass `st`
-    (InferState).  q [T, >= Hq * D]; gate [T, Hq] (or None): head h is multiplied by sigmoid(gate[:, h]); all heads by
-    out_scale.  Returns out [T, Hq * DV]."""
+    (InferState); the first `keep` positions are seen through any window.  q [T, >= Hq * D]; bias (`DistanceBias` or None) is
+    added to the scaled scores; gate [T, Hq] (or None): head h is multiplied by sigmoid(gate[:, h]); all heads by out_scale.
+    Returns out [T, Hq * DV]."""
     T = q.shape[0]
     if out is None:
         out = torch.empty((T, Hq * DV), dtype=q.dtype, device=q.device)
     if not _is_cuda(q):
         return ref.window_attention(q, kv_layer, req_to_token, st.b_req_idx, st.seq_pos,
                                     st.batch_of_token if st.is_prefill else None, Hq, Hkv, D, DV, sm_scale, window, gate,
-                                    out_scale, out)
+                                    out_scale, out, keep, bias)
     assert q.stride(1) == 1 and kv_layer.is_contiguous() and out.stride(1) == 1
     gs = 0 if gate is None else gate.stride(0)
-    tail = (f32(sm_scale), c_int(window), ptr(gate), i64(gs), f32(out_scale), stream())
+    rel, far = (bias.rel, bias.far) if bias is not None else (None, 0)
+    tail = (f32(sm_scale), c_int(window), c_int(keep), ptr(rel), c_int(far), ptr(gate), i64(gs), f32(out_scale), stream())
     if q.dtype == torch.bfloat16 and D in _WINDOW_SIZES and DV % 64 == 0:
         common = (ptr(q), i64(q.stride(0)), ptr(kv_layer), ptr(req_to_token), i64(req_to_token.stride(0)),
                   ptr(st.b_req_idx))
@@ -768,7 +818,7 @@ def window_attention(q, kv_layer, req_to_token, st, Hq, Hkv, D, DV, sm_scale, wi
             _count()
             return out
         if DV in _WINDOW_SIZES:
-            keys = min(window, st.max_kv_len) if window > 0 else st.max_kv_len
+            keys = min(window + keep, st.max_kv_len) if window > 0 else st.max_kv_len
             n = gqa_decode_num_splits(T, Hq, Hkv, max(keys, 1))
             po = pl = None
             if n > 1:

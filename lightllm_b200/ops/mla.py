@@ -89,41 +89,76 @@ def gemm_batched(a, w, out=None):
 
 
 # ---------------------------------------------------------------------------------------------------------------------
-# Latent attention without a rotary part: any latent size, optional sliding window, bf16 or fp32.  The pool row is the
-# latent itself, zero-padded to the row pitch.  A query sees its own position and the window - 1 before it (window 0:
+# Latent attention with any latent size, optional rotary part, optional sliding window, bf16 or fp32.  The pool row is
+# [latent, zero-padded to `rank` columns | rotated key part], zero-padded to the row pitch.  A query sees its own position and the window - 1 before it (window 0:
 # all before it).
 #   absorbed form   scores and values in the latent space, straight from the pool (decode, short portions)
 #   expanded form   keys and values of every head are formed for the positions a prompt pass can see, then attention
 #                   per head (fewer operations per key for long prompts)
 # ---------------------------------------------------------------------------------------------------------------------
-def latent_norm_scatter_(kv_a, kv_layer, norm_w, slot, rank: int, eps: float):
-    """kv_layer[slot[t]] = RMSNorm(kv_a[t, :rank]) * norm_w (fp32), padding columns zero."""
-    row = kv_layer.shape[-1]
+class LatentRope:
+    """Rotation of the key part behind a latent: tables [positions, dims / 2] fp32, pairs of neighbours or of halves."""
+
+    def __init__(self, cos, sin, dims: int, neighbours: bool = True):
+        self.cos, self.sin, self.dims, self.neighbours = cos, sin, int(dims), neighbours
+
+
+def latent_prepare_(kv_a, kv_layer, norm_w, slot, rank: int, cols: int, eps: float, rope=None, pos=None, q_a=None, q_w=None,
+                    q_rank: int = 0):
+    """kv_layer[slot[t]] = [RMSNorm(kv_a[t, :rank]) * norm_w (fp32), zero to `cols` columns | kv_a[t, cols : cols + rope.dims]
+    rotated to position pos[t]], padding columns zero.  q_a [T, q_cols]: latents of the queries, q_rank values; returns their
+    RMSNorm * q_w, zero-padded [T, q_cols] (else None)."""
+    row, dims = kv_layer.shape[-1], rope.dims if rope is not None else 0
+    T = kv_a.shape[0]
     if not kv_a.is_cuda:
-        v = kv_a[:, :rank].float()
-        v = v * torch.rsqrt(v.pow(2).mean(-1, keepdim=True) + eps) * norm_w
-        flat = kv_layer.view(-1, row)
-        flat[slot.long()] = torch.nn.functional.pad(v, (0, row - rank)).to(kv_layer.dtype)
-        return
+        from . import reference as ref
+
+        def norm(v, n, w, width):
+            v = ref.rms_over(v[:, :n].float(), n, eps) * w[:n]
+            return torch.nn.functional.pad(v, (0, width - n))
+
+        out = torch.zeros(T, row)
+        out[:, :cols] = norm(kv_a, rank, norm_w, cols)
+        if dims:
+            out[:, cols:cols + dims] = ref.rotate_pairs(kv_a[:, cols:cols + dims].float(), rope.cos, rope.sin, pos,
+                                                        rope.neighbours)
+        kv_layer.view(-1, row)[slot.long()] = out.to(kv_layer.dtype)
+        return None if q_a is None else norm(q_a, q_rank, q_w, q_a.shape[1]).to(q_a.dtype)
     assert kv_a.stride(1) == 1 and kv_a.dtype == kv_layer.dtype and kv_layer.is_contiguous()
     assert norm_w.dtype == torch.float32 and slot.dtype == torch.int32
-    check(kernels().llb_latent_norm_scatter(ptr(kv_a), c_int(DTYPE_CODES[kv_a.dtype]), i64(kv_a.stride(0)), ptr(kv_layer),
-                                            c_int(row), ptr(norm_w), ptr(slot), c_int(kv_a.shape[0]), c_int(rank),
-                                            f32(eps), stream()), "latent_norm_scatter")
+    q_out = None
+    if q_a is not None:
+        assert q_a.stride(1) == 1 and q_a.dtype == kv_a.dtype and q_w.dtype == torch.float32
+        q_out = torch.empty(q_a.shape, dtype=q_a.dtype, device=q_a.device)
+    r = rope if dims else None
+    check(kernels().llb_latent_prepare(ptr(kv_a), c_int(DTYPE_CODES[kv_a.dtype]), i64(kv_a.stride(0)), ptr(kv_layer),
+                                       c_int(row), ptr(norm_w), ptr(slot), c_int(T), c_int(rank), c_int(cols),
+                                       ptr(r.cos if r else None), ptr(r.sin if r else None), ptr(pos), c_int(dims),
+                                       c_int(1 if r is None or r.neighbours else 0), ptr(q_a),
+                                       i64(q_a.stride(0) if q_a is not None else 0), ptr(q_out), c_int(q_rank),
+                                       c_int(q_a.shape[1] if q_a is not None else 0), ptr(q_w), f32(eps), stream()),
+          "latent_prepare")
     _count()
+    return q_out
 
 
-def ref_latent_attention(q_lat, kv_layer, req_to_token, b_req_idx, pos, batch_of, scale, window: int = 0):
-    T, H, rank = q_lat.shape
+def latent_norm_scatter_(kv_a, kv_layer, norm_w, slot, rank: int, eps: float):
+    """`latent_prepare_` of rows that are a latent alone."""
+    latent_prepare_(kv_a, kv_layer, norm_w, slot, rank, kv_layer.shape[-1], eps)
+
+
+def ref_latent_attention(q_lat, kv_layer, req_to_token, b_req_idx, pos, batch_of, scale, window: int = 0, rank: int = 0):
+    T, H, keys = q_lat.shape
+    rank = rank or keys
     flat = kv_layer.view(-1, kv_layer.shape[-1])
-    out = torch.empty_like(q_lat)
+    out = torch.empty((T, H, rank), dtype=q_lat.dtype, device=q_lat.device)
     for t in range(T):
         b = int(batch_of[t]) if batch_of is not None else t
         p = int(pos[t])
         j0 = max(0, p - window + 1) if window else 0
-        c = flat[req_to_token[int(b_req_idx[b]), j0:p + 1].long(), :rank].float()
+        c = flat[req_to_token[int(b_req_idx[b]), j0:p + 1].long(), :keys].float()
         w = torch.softmax(q_lat[t].float() @ c.t() * scale, dim=-1)
-        out[t] = (w @ c).to(out.dtype)
+        out[t] = (w @ c[:, :rank]).to(out.dtype)
     return out
 
 
@@ -141,22 +176,24 @@ def latent_num_splits(T: int, H: int, max_keys: int, sms: int = 148) -> int:
 
 
 def latent_attention(q_lat, kv_layer, req_to_token, b_req_idx, pos, batch_of, scale, window: int = 0, max_keys: int = 0,
-                     num_splits: int = 0, generic: bool = False):
-    """Absorbed form.  q_lat [T, H, rank] (padding columns zero), pos / batch_of: position and request of every query
-    token (batch_of None: token i belongs to request i).  Returns [T, H, rank].
+                     num_splits: int = 0, generic: bool = False, rank: int = 0):
+    """Absorbed form.  q_lat [T, H, keys] (padding columns zero), of whose columns the first `rank` are latent (0: all);
+    pos / batch_of: position and request of every query token (batch_of None: token i belongs to request i).  Returns
+    [T, H, rank].
     `max_keys`: the most keys a query may see.  `generic`: the kernel without tensor cores (always used for fp32 and for
-    a rank above 512)."""
+    rows above 576 values, 512 of them latent)."""
     if not q_lat.is_cuda:
-        return ref_latent_attention(q_lat, kv_layer, req_to_token, b_req_idx, pos, batch_of, scale, window)
-    T, H, rank = q_lat.shape
+        return ref_latent_attention(q_lat, kv_layer, req_to_token, b_req_idx, pos, batch_of, scale, window, rank)
+    T, H, keys = q_lat.shape
+    rank = rank or keys
     row = kv_layer.shape[-1]
     assert q_lat.is_contiguous() and kv_layer.is_contiguous() and q_lat.dtype == kv_layer.dtype
     assert pos.dtype == torch.int32 and b_req_idx.dtype == torch.int32
-    out = torch.empty_like(q_lat)
-    if generic or q_lat.dtype != torch.bfloat16 or rank > 512 or rank % 8:
+    out = torch.empty((T, H, rank), dtype=q_lat.dtype, device=q_lat.device)
+    if generic or q_lat.dtype != torch.bfloat16 or rank > 512 or keys > 576 or rank % 8 or keys % 8:
         check(kernels().llb_latent_attn_generic(ptr(q_lat), c_int(DTYPE_CODES[q_lat.dtype]), ptr(kv_layer), c_int(row),
                                                 ptr(req_to_token), i64(req_to_token.stride(0)), ptr(b_req_idx), ptr(pos),
-                                                ptr(batch_of), ptr(out), c_int(T), c_int(H), c_int(rank), f32(scale),
+                                                ptr(batch_of), ptr(out), c_int(T), c_int(H), c_int(keys), c_int(rank), f32(scale),
                                                 c_int(window), stream()), "latent_attn_generic")
         _count()
         return out
@@ -168,8 +205,8 @@ def latent_attention(q_lat, kv_layer, req_to_token, b_req_idx, pos, batch_of, sc
         pl = torch.empty(n * 2, dtype=torch.float32, device=q_lat.device)
     check(kernels().llb_latent_attn_mma(ptr(q_lat), ptr(kv_layer), c_int(row), ptr(req_to_token),
                                         i64(req_to_token.stride(0)), ptr(b_req_idx), ptr(pos), ptr(batch_of), ptr(out),
-                                        ptr(po), ptr(pl), c_int(T), c_int(H), c_int(rank), c_int(splits), f32(scale),
-                                        c_int(window), stream()), "latent_attn_mma")
+                                        ptr(po), ptr(pl), c_int(T), c_int(H), c_int(keys), c_int(rank), c_int(splits),
+                                        f32(scale), c_int(window), stream()), "latent_attn_mma")
     _count(2 if splits > 1 else 1)
     return out
 
@@ -200,9 +237,10 @@ def latent_gather(kv_layer, req_to_token, b_req_idx, kr: KeyRange):
     return out
 
 
-def window_prefill(q, kv, H: int, dk: int, dv: int, cu_q, b_ready_len, kr: KeyRange, max_q_len: int, scale):
-    """Expanded form on the tcgen05 tensor cores: q [T, >= H * dk] (row stride free), kv [rows, H * dk | H * dv], head
-    sizes 64 or 128.  Returns [T, H * dv]."""
+def window_prefill(q, kv, H: int, dk: int, dv: int, cu_q, b_ready_len, kr: KeyRange, max_q_len: int, scale, gate=None):
+    """Expanded form on the tcgen05 tensor cores: q [T, >= H * dk] (row stride free), kv [rows, H * dk | H * dv], key sizes
+    up to 256 and value sizes up to 128, multiples of 64; gate [T, H * dv] or None: the result times sigmoid(gate).  Returns
+    [T, H * dv]."""
     assert q.dtype == torch.bfloat16 and kv.dtype == torch.bfloat16 and q.stride(1) == 1 and kv.is_contiguous()
     assert kv.shape == (kr.rows, H * (dk + dv)) and cu_q.dtype == torch.int32
     T, B = q.shape[0], cu_q.shape[0] - 1
@@ -210,6 +248,7 @@ def window_prefill(q, kv, H: int, dk: int, dv: int, cu_q, b_ready_len, kr: KeyRa
     check(kernels().llb_window_prefill_tc(ptr(q), i64(q.stride(0)), ptr(kv), i64(kv.stride(0)), c_int(kr.rows), ptr(cu_q),
                                           ptr(kr.cu_kv), ptr(kr.kv_start), ptr(b_ready_len), ptr(out),
                                           i64(out.stride(0)), c_int(B), c_int(T), c_int(max_q_len), c_int(H), c_int(dk),
-                                          c_int(dv), f32(scale), c_int(kr.window), stream()), "window_prefill_tc")
+                                          c_int(dv), f32(scale), c_int(kr.window), ptr(gate),
+                                          i64(gate.stride(0) if gate is not None else 0), stream()), "window_prefill_tc")
     _count()
     return out

@@ -327,8 +327,8 @@ def uniform_experts_dyt_(h, lay, w13, w2, act, shared, gate_w, x, post, nxt, e0:
 
 def routed_experts_rms_(h, ids, weights, w13, w2, clamp, shared, x, w, width, eps, next_w=None, e0: int = 0):
     """Routed experts with the clamped gate plus a shared expert's output `shared` [T, H] (or None), inside an output norm:
-    x += rms(sum) * w in place, returns x (or rms(x) * next_w) in h's format (`ops.add_rms_`).  x None: returns the fp32 sum
-    instead (a tensor-parallel reduction follows)."""
+    x += rms(sum) * w in place (w None: x += sum), returns x (or rms(x) * next_w) in h's format (`ops.add_rms_`).  x None:
+    returns the fp32 sum instead (a tensor-parallel reduction follows)."""
     from . import add_rms_
 
     if not h.is_cuda:

@@ -69,7 +69,7 @@ def dyt(x, norm):
 
 
 def gemm(a, w, epi="store", residual=None, bias=None, out_dtype=None, out_scale=1.0, x=None, dyt=None,
-         clamp=None):
+         clamp=None, softcap=0.0):
     """C = A . W^T with the epilogues of the tcgen05 GEMM. `w` is [N, K]."""
     acc = a.float() @ w.float().t()
     if bias is not None:
@@ -79,7 +79,8 @@ def gemm(a, w, epi="store", residual=None, bias=None, out_dtype=None, out_scale=
     if epi == "residual":
         return (acc + residual.float()).to(out_dtype or a.dtype)
     if epi == "f32":
-        return acc * out_scale if out_scale != 1.0 else acc
+        acc = acc * out_scale if out_scale != 1.0 else acc
+        return softcap * torch.tanh(acc / softcap) if softcap > 0 else acc
     if epi == "relu2":
         return torch.relu(acc).square().to(out_dtype or a.dtype)
     if epi == "dyt":
@@ -425,13 +426,13 @@ def bigram_rows(ids, bigram, req_to_token, b_req_idx, pos, batch_of, mem_index):
     return bigram.table[rows]
 
 
-def _rms_over(v, width, eps):
+def rms_over(v, width, eps):
     return v * torch.rsqrt(v.square().sum(-1, keepdim=True) / width + eps)
 
 
 def add_rms_(x, y, w, width, eps, dtype, next_w=None):
-    x.add_(_rms_over(y.float(), width, eps) * w)
-    return (x if next_w is None else _rms_over(x, width, eps) * next_w).to(dtype)
+    x.add_(y.float() if w is None else rms_over(y.float(), width, eps) * w)
+    return (x if next_w is None else rms_over(x, width, eps) * next_w).to(dtype)
 
 
 def qk_norm_rope_scatter_(qkv, kv_layer, cos, sin, pos, slot, q_w, k_w, eps, Hq, Hkv, D, dim, DV, rot_dim):
@@ -440,28 +441,43 @@ def qk_norm_rope_scatter_(qkv, kv_layer, cos, sin, pos, slot, q_w, k_w, eps, Hq,
     c, s = cos[pos.long()].unsqueeze(1), sin[pos.long()].unsqueeze(1)
 
     def turn(x, w):
-        x = _rms_over(x.float(), dim, eps) * w
+        x = rms_over(x.float(), dim, eps)
+        x = x if w is None else x * w
         u, v = x[..., :half], x[..., half:2 * half]
         return torch.cat([u * c - v * s, v * c + u * s, x[..., 2 * half:]], -1).reshape(T, -1).to(qkv.dtype)
 
     q = turn(qkv[:, :nq].reshape(T, Hq, D), q_w)
-    kv_layer[slot.long(), :nk] = turn(qkv[:, nq:nq + nk].reshape(T, Hkv, D), k_w)
-    kv_layer[slot.long(), nk:] = qkv[:, nq + nk:nq + nk + Hkv * DV]
+    if Hkv:
+        kv_layer[slot.long(), :nk] = turn(qkv[:, nq:nq + nk].reshape(T, Hkv, D), k_w)
+        kv_layer[slot.long(), nk:] = qkv[:, nq + nk:nq + nk + Hkv * DV]
     qkv[:, :nq] = q
     return qkv
 
 
+def rotate_pairs(x, cos, sin, pos, neighbours):
+    """x [T, ..., dims] fp32, rotated by the angles of its row's position."""
+    T, n = x.shape[0], x.shape[-1] // 2
+    c, s = (t[pos.long()].view(T, *[1] * (x.dim() - 2), n) for t in (cos, sin))
+    u, v = (x[..., 0::2], x[..., 1::2]) if neighbours else (x[..., :n], x[..., n:])
+    a, b = u * c - v * s, v * c + u * s
+    return torch.stack([a, b], -1).flatten(-2) if neighbours else torch.cat([a, b], -1)
+
+
 def window_attention(q, kv_layer, req_to_token, b_req_idx, pos, batch_of, Hq, Hkv, D, DV, sm_scale, window, gate, out_scale,
-                     out):
+                     out, keep=0, bias=None):
     G = Hq // Hkv
     for t in range(q.shape[0]):
         b = int(batch_of[t]) if batch_of is not None else t
         p = int(pos[t])
         j0 = max(0, p - window + 1) if window > 0 else 0
-        rows = kv_layer[req_to_token[int(b_req_idx[b]), j0:p + 1].long()].float()
+        j = torch.cat([torch.arange(min(keep, j0)), torch.arange(j0, p + 1)])
+        rows = kv_layer[req_to_token[int(b_req_idx[b]), j].long()].float()
         k = rows[:, : Hkv * D].view(-1, Hkv, D).repeat_interleave(G, dim=1)
         v = rows[:, Hkv * D:].reshape(-1, Hkv, DV).repeat_interleave(G, dim=1)
-        pr = torch.softmax(torch.einsum("hd,lhd->hl", q[t, : Hq * D].view(Hq, D).float(), k) * sm_scale, dim=-1)
+        sc = torch.einsum("hd,lhd->hl", q[t, : Hq * D].view(Hq, D).float(), k) * sm_scale
+        if bias is not None:
+            sc = sc + bias.rel[:, (p - j).clamp_max(bias.far)]
+        pr = torch.softmax(sc, dim=-1)
         o = torch.einsum("hl,lhd->hd", pr, v) * out_scale
         if gate is not None:
             o = o * torch.sigmoid(gate[t].float())[:, None]
