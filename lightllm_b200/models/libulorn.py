@@ -25,19 +25,18 @@ from typing import Dict
 import torch
 
 from .. import ops
-from ..common.infer_state import InferState, ShardedLogits
-from ..common.mem_manager import LayeredKVMemoryManager
+from ..common.infer_state import InferState
 from ..common.recurrent_state import RecurrentStateMixin, RecurrentStates
 from ..ops import moe as moe_ops
 from ..ops import reference as ref
 from ..ops.linear_attn import ChunkPlan, DecayedState
-from .base import LayerWeights, TransformerLM
+from .base import LayerWeights
 from .registry import register_config, register_model
+from .stream_lm import ACT_ALPHA, StreamLM
 from .weights import get_shaped, kv_head_range, tp_range
 from .weights import pad_zeros as _pad
 from .weights import round_up as _up
 
-ACT_ALPHA = 1.702          # slope of the experts' gate
 RANDOM_DECAY_RANK = 16     # low-rank size of the decay projection for random weights (checkpoints bring their own)
 
 
@@ -111,10 +110,8 @@ class LayerSpec:
 
 
 @register_model("libulorn")
-class LibulornLM(RecurrentStateMixin, TransformerLM):
+class LibulornLM(RecurrentStateMixin, StreamLM):
     model_type = "libulorn"
-    supports_float32 = True
-    stream_tap = None          # fn(layer, stream): sees the residual stream after every layer (tests)
     native_units = ("attention", "attention_generic", "attention_tc", "gemm_f32", "gemm_tcgen05", "moe", "ops_basic",
                     "recurrent", "rms_stream", "sampling")
 
@@ -135,13 +132,7 @@ class LibulornLM(RecurrentStateMixin, TransformerLM):
         self.head_dim = max([max(a.dp, a.vp) for a in left] or [64])
         self.rot_dim = 0
         self.inter = None
-        self.ep = bool(self.extra.get("enable_ep_moe", False))
-        if self.quant_cfg.any_fp8:
-            raise ValueError("libulorn: weights run in bf16 or fp32 only (--quant_type none)")
-        if self.ep and self.ps.dp_size > 1:
-            raise ValueError("libulorn: expert parallelism works inside a tensor-parallel group, not with --dp > 1")
-        if self.extra.get("enable_return_routed_experts") and len({s.top for s in self.specs if s.moe}) > 1:
-            raise ValueError("libulorn: returned routed experts need the same number of experts in every layer")
+        self._check_options()
 
     # ------------------------------------------------------------------ weights
     def weight_shapes(self) -> Dict[str, tuple]:
@@ -190,42 +181,19 @@ class LibulornLM(RecurrentStateMixin, TransformerLM):
 
         return {n: fill(1.0 if "norm" in n else 0.0) for n, shape in self.weight_shapes().items() if len(shape) == 1}
 
-    def _heads(self, src, name, heads, size, padded, h0, h1):
-        """Rows of heads h0 .. h1 of a per-head projection, every head padded to `padded` rows: [n * padded, hidden_p]."""
-        w = get_shaped(src, name, heads * size, self.hidden).view(heads, size, self.hidden)[h0:h1]
-        return _pad(w, h1 - h0, padded, self.hidden_p).reshape(-1, self.hidden_p)
-
-    def _narrow(self, w, rows):
-        """Rows of a narrow projection, padded to a multiple of 8 rows."""
-        return _pad(w, _up(rows, 8), self.hidden_p)
-
-    def _vec(self, t, *sizes):
-        return self._dev(_pad(t.float(), *sizes), torch.float32)
-
     def _load_norm(self, src, name):
         return self._vec(get_shaped(src, name, self.hidden), self.hidden_p)
 
-    def _load_gated(self, src, p, ff, i0, i1):
-        """(gate | up interleaved [2I, width], down [width, I]) of the columns i0 .. i1 of a feed-forward, padded."""
-        W, P, I = self.hidden, self.hidden_p, _up(i1 - i0, 64)
-        g, u = (_pad(get_shaped(src, p + n, ff, W)[i0:i1], I, P) for n in ("gate", "up"))
-        return ref.interleave_gate_up(g, u), _pad(get_shaped(src, p + "down", W, ff)[:, i0:i1], P, I)
-
     def _load_weights(self, src):
-        tp, r = self.tp.size, self.tp.rank
         W, P = self.hidden, self.hidden_p
-        self.embed_w = self._dev(_pad(get_shaped(src, "embed", self.vocab, W), self.vocab, P))
-        self.embed_range = (0, self.vocab)
+        self._load_embed_and_head(src)
         self.bigram = None
         if self.bigram_cfg:
             b = self.bigram_cfg
             n = b["buckets"] + 1
             self.bigram = ops.BigramTable(self._dev(_pad(get_shaped(src, "bigram", n, W), n, P)), b["buckets"],
                                           b["mul_prev"], b["mul_cur"])
-        v0, v1 = tp_range(self.vocab, r, tp)
-        self.lm_head_w = self._dev(_pad(get_shaped(src, "head", self.vocab, W)[v0:v1], _up(v1 - v0, 8), P))
         self.final_norm = self._load_norm(src, "final.norm")
-        self.final_norm_w = None
         self.layers = []
         for i, l in enumerate(self.specs[: self.num_layers]):
             lw = LayerWeights()
@@ -260,8 +228,7 @@ class LibulornLM(RecurrentStateMixin, TransformerLM):
         add("gate", self._narrow(get_shaped(src, p + "g", a.heads, self.hidden)[h0:h1], h1 - h0))
         lw.q_norm = self._vec(get_shaped(src, p + "q.norm", a.dim), a.dp)
         lw.k_norm = self._vec(get_shaped(src, p + "k.norm", a.dim), a.dp)
-        o = get_shaped(src, p + "o", self.hidden, a.heads * a.vdim).view(self.hidden, a.heads, a.vdim)[:, h0:h1]
-        outs.append(_pad(o, self.hidden_p, a.hq, a.vp).reshape(self.hidden_p, -1))
+        outs.append(self._out_heads(src, p + "o", a.heads, a.vdim, a.vp, h0, h1))
 
     def _load_recurrent(self, lw, src, p, s: RecurrentSpec, add, outs, out_scale):
         h0, h1 = tp_range(s.heads, self.tp.rank, self.tp.size)
@@ -285,20 +252,13 @@ class LibulornLM(RecurrentStateMixin, TransformerLM):
             w = get_shaped(src, p + "norm", s.heads * s.vdim).view(s.heads, s.vdim)[h0:h1]
             kw.update(cap=s.cap, weight=self._vec(w, s.h, s.vp).view(-1))
         lw.rec = DecayedState(s.kind, s.h, s.dp, s.vp, s.dim, s.vdim, **kw)
-        o = get_shaped(src, p + "o", self.hidden, s.heads * s.vdim).view(self.hidden, s.heads, s.vdim)[:, h0:h1]
-        outs.append(_pad(o, self.hidden_p, s.h, s.vp).reshape(self.hidden_p, -1))
+        outs.append(self._out_heads(src, p + "o", s.heads, s.vdim, s.vp, h0, h1))
 
     def _load_moe(self, lw, src, p, l: LayerSpec):
         """Router, experts stacked as in `models/moe.py`, shared expert."""
         tp, r = self.tp.size, self.tp.rank
         lw.router_w = self._dev(self._narrow(get_shaped(src, p + "router", l.experts, self.hidden), l.experts))
-        if self.ep and tp > 1:
-            (lw.e0, e1), (i0, i1) = tp_range(l.experts, r, tp), (0, l.ff)
-        else:
-            (lw.e0, e1), (i0, i1) = (0, l.experts), tp_range(l.ff, r, tp)
-        mats = [self._load_gated(src, f"{p}e{e}.", l.ff, i0, i1) for e in range(lw.e0, e1)]
-        lw.w13 = self._dev(torch.stack([a for a, _ in mats]))
-        lw.w2 = self._dev(torch.stack([b for _, b in mats]))
+        self._load_experts(lw, src, p, l.experts, l.ff)
         if l.shared_ff:
             a, b = self._load_gated(src, p + "shared.", l.shared_ff, *tp_range(l.shared_ff, r, tp))
             lw.shared_gate_up_w, lw.shared_down_w = self._dev(a), self._dev(b)
@@ -324,12 +284,7 @@ class LibulornLM(RecurrentStateMixin, TransformerLM):
         return [s.left.kv_row for s in self.specs[: self.num_layers] if s.left is not None]
 
     def kv_bytes_per_token(self):
-        return LayeredKVMemoryManager.bytes_per_token(self.dtype, self._kv_rows()) + 4     # + its token id
-
-    def _make_mem_manager(self, size):
-        if self.extra.get("kv_type") not in (None, "none", "None"):
-            raise ValueError("--llm_kv_type: the layers' caches have no quantised form here")
-        return LayeredKVMemoryManager(size, self.dtype, self._kv_rows(), self.device)
+        return super().kv_bytes_per_token() + 4     # + its token id
 
     def _init_mem(self, max_total_token_num, mem_fraction):
         # the requests' recurrent states come out of the same budget: allocate them first
@@ -346,13 +301,6 @@ class LibulornLM(RecurrentStateMixin, TransformerLM):
             self.bigram.slot_token = torch.zeros(self.mem_manager.size + 1, dtype=torch.int32, device=self.device)
 
     # ------------------------------------------------------------------ forward
-    def _make_decode_state(self, B, b_req_idx, b_seq_len, mem_index, max_kv_len, num_splits=None):
-        return InferState(is_prefill=False, batch_size=B, num_tokens=B, max_kv_len=max_kv_len, max_q_len=1,
-                          b_req_idx=b_req_idx, b_seq_len=b_seq_len, mem_index=mem_index)
-
-    def _graph_decode_splits(self, bucket):
-        return 1        # per layer, from its window (ops.window_attention)
-
     def _embed(self, ids, st):
         x, st.extra["stream_h"] = ops.embedding_pair(ids, self.embed_w, self.bigram, self.req_manager.req_to_token_indexs,
                                                      st.b_req_idx, st.seq_pos,
@@ -375,14 +323,6 @@ class LibulornLM(RecurrentStateMixin, TransformerLM):
                 self.stream_tap(i, x)
         st.extra["normed"] = True
         return h
-
-    def _reduced(self, a, w):
-        """a . w^T, summed over the tensor-parallel ranks."""
-        if self.tp.size == 1:
-            return ops.gemm(a, w)
-        y = ops.gemm(a, w, epi="f32")
-        self.tp.all_reduce_(y)
-        return y
 
     def _mixer(self, i, lw, h, st: InferState):
         """The mixer's heads, gated, side by side (input of the output projection)."""
@@ -425,11 +365,3 @@ class LibulornLM(RecurrentStateMixin, TransformerLM):
             return out
         self.tp.all_reduce_(out)
         return ops.add_rms_(x, out, lw.norm2, self.hidden, self.eps, self.dtype, after)
-
-    def _lm_head(self, h, normed: bool = True):
-        assert normed, "the layer stack returns normalised rows"
-        v = self.vocab // self.tp.size
-        logits = ops.gemm(h, self.lm_head_w, epi="f32")[:, :v]
-        if self.tp.size == 1:
-            return logits
-        return ShardedLogits(logits.contiguous(), self.tp, self.tp.rank * v, self.vocab)

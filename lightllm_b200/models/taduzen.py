@@ -29,8 +29,10 @@ from ..common.mem_manager import MLAMemoryManager
 from ..ops import mla as mla_ops
 from ..ops import moe as moe_ops
 from ..ops import reference as ref
-from .base import LayerWeights, TransformerLM
+from .base import LayerWeights
+from .latent import LatentHeads
 from .registry import register_config, register_model
+from .stream_lm import StreamLM
 from .weights import get_shaped, tp_range
 from .weights import pad_zeros as _pad
 from .weights import round_up as _up
@@ -64,6 +66,7 @@ class LayerSpec:
         self.dp, self.vp, self.rp = _up(self.dim, 64), _up(self.vdim, 64), _up(self.rank, 16)
         f = c.get("mlp")
         self.kind = f["kind"] if f else None
+        self.moe = self.kind == "moe"
         if self.kind not in (None, "dense", "moe"):
             raise ValueError(f"unknown feed-forward {self.kind!r}")
         if self.kind == "dense":
@@ -75,10 +78,8 @@ class LayerSpec:
 
 
 @register_model("taduzen")
-class TaduzenLM(TransformerLM):
+class TaduzenLM(StreamLM):
     model_type = "taduzen"
-    supports_float32 = True
-    stream_tap = None          # fn(layer, stream): sees the residual stream after every layer (tests)
     native_units = ("dyt", "gemm_f32", "gemm_tcgen05", "latent_attn", "moe", "ops_basic", "sampling",
                     "window_prefill_tc")
 
@@ -102,14 +103,7 @@ class TaduzenLM(TransformerLM):
         self.head_dim = self.kv_row
         self.rot_dim = 0
         self.inter = None
-        self.ep = bool(self.extra.get("enable_ep_moe", False))
-        if self.quant_cfg.any_fp8:
-            raise ValueError("taduzen: weights run in bf16 or fp32 only (--quant_type none)")
-        if self.ep and self.ps.dp_size > 1:
-            raise ValueError("taduzen: expert parallelism works inside a tensor-parallel group, not with --dp > 1")
-        tops = {s.top for s in self.specs if s.kind == "moe"}
-        if self.extra.get("enable_return_routed_experts") and len(tops) > 1:
-            raise ValueError("taduzen: returned routed experts need the same number of experts in every layer")
+        self._check_options()
 
     # ------------------------------------------------------------------ weights
     def weight_shapes(self) -> Dict[str, tuple]:
@@ -177,21 +171,11 @@ class TaduzenLM(TransformerLM):
                            _pad(get_shaped(src, name + ".b", W).float(), P).to(self.device),
                            float(get_shaped(src, name + ".alpha").float()))
 
-    def _load_gated(self, src, p, ff, i0, i1):
-        """(gate | up interleaved [2I, width], down [width, I]) of the columns i0 .. i1 of a feed-forward, padded."""
-        W, P, I = self.hidden, self.hidden_p, _up(i1 - i0, 64)
-        g, u = (_pad(get_shaped(src, p + n, ff, W)[i0:i1], I, P) for n in ("gate", "up"))
-        return ref.interleave_gate_up(g, u), _pad(get_shaped(src, p + "down", W, ff)[:, i0:i1], P, I)
-
     def _load_weights(self, src):
         tp, r = self.tp.size, self.tp.rank
         W, P = self.hidden, self.hidden_p
-        self.embed_w = self._dev(_pad(get_shaped(src, "embed", self.vocab, W), self.vocab, P))
-        self.embed_range = (0, self.vocab)
-        v0, v1 = tp_range(self.vocab, r, tp)
-        self.lm_head_w = self._dev(_pad(get_shaped(src, "head", self.vocab, W)[v0:v1], _up(v1 - v0, 8), P))
+        self._load_embed_and_head(src)
         self.final_norm = self._load_norm(src, "final.norm")
-        self.final_norm_w = None
         self.layers, tables = [], []
         for i, l in enumerate(self.specs[: self.num_layers]):
             lw = LayerWeights()
@@ -215,32 +199,21 @@ class TaduzenLM(TransformerLM):
     def _load_mixer(self, lw, src, m, l: LayerSpec):
         W, P = self.hidden, self.hidden_p
         h0, h1 = tp_range(l.heads, self.tp.rank, self.tp.size)
-        n = lw.heads = h1 - h0
-        q = get_shaped(src, m + "q", l.heads * l.dim, W).view(l.heads, l.dim, W)[h0:h1]
+        lw.heads = h1 - h0
+        q = self._heads(src, m + "q", l.heads, l.dim, l.dp, h0, h1)
         dkv = get_shaped(src, m + "dkv", l.rank, W)
-        lw.qkv_w = self._dev(torch.cat([_pad(q, n, l.dp, P).view(n * l.dp, P), _pad(dkv, l.rp, P)]))
+        lw.qkv_w = self._dev(torch.cat([q, _pad(dkv, l.rp, P)]))
         lw.kv_norm = self._dev(get_shaped(src, m + "dkv.norm", l.rank), torch.float32)
-        uk = _pad(get_shaped(src, m + "uk", l.heads * l.dim, l.rank).view(l.heads, l.dim, l.rank)[h0:h1], n, l.dp, l.rp)
-        uv = _pad(get_shaped(src, m + "uv", l.heads * l.vdim, l.rank).view(l.heads, l.vdim, l.rank)[h0:h1], n, l.vp, l.rp)
-        lw.w_uk_t = self._dev(uk.transpose(1, 2))                                     # [heads, rank, dim]: q -> q_lat
-        lw.w_ukv = self._dev(torch.cat([uk.reshape(n * l.dp, l.rp), uv.reshape(n * l.vp, l.rp)]))  # latent -> k | v
-        lw.w_uv = lw.w_ukv[n * l.dp:].view(n, l.vp, l.rp)                             # o_lat -> o
-        o = get_shaped(src, m + "o", W, l.heads * l.vdim).view(W, l.heads, l.vdim)[:, h0:h1]
-        lw.o_w = self._dev(_pad(o, P, n, l.vp).view(P, n * l.vp))
+        uk = get_shaped(src, m + "uk", l.heads * l.dim, l.rank).view(l.heads, l.dim, l.rank)[h0:h1]
+        uv = get_shaped(src, m + "uv", l.heads * l.vdim, l.rank).view(l.heads, l.vdim, l.rank)[h0:h1]
+        lw.latent = LatentHeads(h1 - h0, l.dim, 0, l.vdim, l.rank, l.scale, l.window)
+        lw.latent.load(lw, self._dev, uk, uv)
+        lw.o_w = self._dev(self._out_heads(src, m + "o", l.heads, l.vdim, l.vp, h0, h1))
 
     def _load_moe(self, lw, src, p, l: LayerSpec):
         """Experts stacked as in `models/moe.py`; returns the routing entry (table, first expert, experts) of this rank."""
         tp, r = self.tp.size, self.tp.rank
-        if self.ep and tp > 1:
-            e0, e1 = tp_range(l.experts, r, tp)
-            i0, i1 = 0, l.ff
-        else:
-            e0, e1 = 0, l.experts
-            i0, i1 = tp_range(l.ff, r, tp)
-        mats = [self._load_gated(src, f"{p}e{e}.", l.ff, i0, i1) for e in range(e0, e1)]
-        lw.w13 = self._dev(torch.stack([a for a, _ in mats]))
-        lw.w2 = self._dev(torch.stack([b for _, b in mats]))
-        lw.e0 = e0
+        e0, e1 = self._load_experts(lw, src, p, l.experts, l.ff)
         if l.shared_ff:
             s0, s1 = tp_range(l.shared_ff, r, tp)
             a, b = self._load_gated(src, p + "shared.", l.shared_ff, s0, s1)
@@ -265,13 +238,6 @@ class TaduzenLM(TransformerLM):
         return MLAMemoryManager(size, self.dtype, self.kv_row, 0, self.num_layers, self.device)
 
     # ------------------------------------------------------------------ forward
-    def _make_decode_state(self, B, b_req_idx, b_seq_len, mem_index, max_kv_len, num_splits=None):
-        return InferState(is_prefill=False, batch_size=B, num_tokens=B, max_kv_len=max_kv_len, max_q_len=1,
-                          b_req_idx=b_req_idx, b_seq_len=b_seq_len, mem_index=mem_index)
-
-    def _graph_decode_splits(self, bucket):
-        return 1        # per layer, from its window (ops.mla.latent_attention)
-
     def _embed(self, ids, st):
         x, st.extra["first_normed"] = ops.embedding_dyt(ids, self.embed_w, self.layers[0].norm1)
         if self.routing is not None:
@@ -322,41 +288,12 @@ class TaduzenLM(TransformerLM):
         return out if one else self._reduce_dyt(out, x, lw.norm2b, after)
 
     def _attention_block(self, i, lw, h, st: InferState):
-        l, n = lw.spec, lw.heads
-        T = h.shape[0]
-        qc = ops.gemm(h, lw.qkv_w)                               # [T, heads * dim | latent]
-        q = qc[:, : n * l.dp]
-        kv_layer = self._kv_layer(i)
-        mla_ops.latent_norm_scatter_(qc[:, n * l.dp:], kv_layer, lw.kv_norm, st.mem_index, l.rank, self.eps)
-        r2t = self.req_manager.req_to_token_indexs
-        kr = self._expanded_range(lw, st) if st.is_prefill else None
-        if kr is not None:
-            c = mla_ops.latent_gather(kv_layer, r2t, st.b_req_idx, kr)
-            kv = ops.gemm(c[:, : l.rp], lw.w_ukv)                # [rows, heads * dim | heads * vdim]
-            return mla_ops.window_prefill(q, kv, n, l.dp, l.vp, st.cu_q, st.b_ready_cache_len, kr, st.max_q_len, l.scale)
-        q_lat = mla_ops.gemm_batched(q.view(T, n, l.dp), lw.w_uk_t)
-        o_lat = mla_ops.latent_attention(q_lat, kv_layer, r2t, st.b_req_idx, st.seq_pos,
-                                         st.batch_of_token if st.is_prefill else None, l.scale, l.window,
-                                         min(l.window or st.max_kv_len, st.max_kv_len))
-        return mla_ops.gemm_batched(o_lat, lw.w_uv).reshape(T, n * l.vp)
-
-    def _expanded_range(self, lw, st: InferState):
-        """The positions to expand keys and values for when this prompt pass runs the expanded form, else None."""
         l = lw.spec
-        if self.device.type != "cuda" or self.dtype != torch.bfloat16 or l.dp > 128 or l.vp > 128:
-            return None
-        cache = st.extra.setdefault("key_ranges", {})
-        if l.window not in cache:
-            q_len, ready = st.extra["q_len_cpu"].to(torch.int64), st.extra["ready_cpu"].to(torch.int64)
-            seq = ready + q_len
-            pairs = int((q_len * (seq.clamp_max(l.window) if l.window else seq)).sum())
-            cache[l.window] = (mla_ops.KeyRange(ready, q_len, l.window, self.device), pairs)
-        kr, pairs = cache[l.window]
-        # multiply-adds per head; the absorbed kernel works on 16-row tiles of heads with mma.sync at about a quarter
-        # of the tcgen05 rate
-        expanded = kr.rows * l.rp * (l.dp + l.vp) + pairs * (l.dp + 2 * l.vp)
-        absorbed = st.num_tokens * l.rp * (l.dp + l.vp) + 4 * pairs * 3 * l.rp * (_up(lw.heads, 16) / lw.heads)
-        return kr if expanded < absorbed else None
+        qc = ops.gemm(h, lw.qkv_w)                               # [T, heads * dim | latent]
+        q = qc[:, : lw.heads * l.dp]
+        kv_layer = self._kv_layer(i)
+        mla_ops.latent_norm_scatter_(qc[:, lw.heads * l.dp:], kv_layer, lw.kv_norm, st.mem_index, l.rank, self.eps)
+        return lw.latent.attend(lw, q, kv_layer, self.req_manager.req_to_token_indexs, st)
 
     def _lm_head(self, h, normed: bool = True):
         assert normed, "the layer stack returns normalised rows"
