@@ -13,3 +13,4 @@ from . import deepseek_v32  # noqa: F401
 from . import gemma4  # noqa: F401
 from . import taduzen  # noqa: F401
 from . import libulorn  # noqa: F401
+from . import katarax  # noqa: F401
