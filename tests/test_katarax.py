@@ -126,10 +126,14 @@ def replayer(path, tgt, pool=512, **kw):
 
 
 def close(got, want, tgt, what=""):
-    """Both [n, vocab]: root-mean-square error over the vocabulary against the logits' own."""
+    """Both [n, vocab]: root-mean-square error over the vocabulary against the logits' own.  Eight layers of bf16 rounding alone
+    (the plain operators on the CPU) have a median of 1.2e-2 and take single positions to 3.4e-2."""
     want = want.double()
     err = (torch.as_tensor(got).double() - want).pow(2).mean(-1).sqrt() / want.pow(2).mean().sqrt()
-    assert err.max() < (3e-2 if tgt[1] == "bfloat16" else 2e-5), (what, err.argmax(), err.max())
+    if tgt[1] == "bfloat16":
+        assert err.max() < 5e-2 and (len(err) < 20 or err.median() < 2e-2), (what, err.argmax(), err.max(), err.median())
+    else:
+        assert err.max() < 2e-5, (what, err.argmax(), err.max())
 
 
 def tokens(n, seed, vocab=VOCAB):
