@@ -1,8 +1,8 @@
 """Prefill and decode throughput of a model design beside the framework's closest model at equal sizes, and the kernels
 of both with their roofline fractions.  Taduzen: DeepSeek-V2 (latent attention, routed and shared experts); Libulorn:
-Qwen3-Next (`design_libulorn.py`).
+Qwen3-Next (`design_libulorn.py`); Katarax: DeepSeek-V3 and Qwen3-MoE (`design_katarax.py`).
 
-    python bench.py --design taduzen|libulorn [--design-size small|base|wide] [--design-kernels]
+    python bench.py --design taduzen|libulorn|katarax [--design-size small|base|wide] [--design-kernels]
 
 Random weights, random tokens, bf16.  Whole passes through the models' own forward (decode as CUDA graph), timed with CUDA
 events after three warm-up passes; a pass reads far more weight bytes than L2 holds.  Kernels: median of 10 samples with L2
@@ -90,21 +90,25 @@ DECODE = [(16, 4096), (64, 4096), (256, 1024)]              # requests, context
 
 
 def _design(name):
-    """(sizes, configuration, closest model's name and configuration, kernels)"""
+    """(sizes, configuration, {closest model: its configuration}, kernels)"""
     if name == "taduzen":
         from .design_kernels import kernels
 
-        return SIZES, taduzen_config, "deepseek_v2", deepseek_config, kernels
+        return SIZES, taduzen_config, {"deepseek_v2": deepseek_config}, kernels
+    if name == "katarax":
+        from . import design_katarax as d
+
+        return d.SIZES, d.config, d.CLOSEST, d.kernels
     from . import design_libulorn as d
 
-    return d.SIZES, d.config, "qwen3_next", d.closest_config, d.kernels
+    return d.SIZES, d.config, {"qwen3_next": d.closest_config}, d.kernels
 
 
 def passes(design: str, size: str, steps: int):
-    sizes, config, closest, closest_config, _ = _design(design)
+    sizes, config, closest, _ = _design(design)
     z = sizes[size]
     res = {}
-    for name, cfg in ((design, config(z)), (closest, closest_config(z))):
+    for name, cfg in ((design, config(z)), *((n, make(z)) for n, make in closest.items())):
         tokens = max(max(b * (r + n) for b, r, n in PREFILL), max(b * (c + 1) for b, c in DECODE)) + 64
         model = _model(cfg, tokens, 8192, 256)
         for b, ready, new in PREFILL:
@@ -119,11 +123,12 @@ def passes(design: str, size: str, steps: int):
     for (name, what), (ms, n) in res.items():
         if name != design:
             continue
-        other = res[closest, what][0]
-        print(json.dumps({"design": design, "size": size, "pass": what, "ms": round(ms, 3),
-                          "tokens_per_s": round(n / ms * 1e3), f"{closest}_ms": round(other, 3),
-                          f"{closest}_tokens_per_s": round(n / other * 1e3), "speedup": round(other / ms, 2),
-                          "layers": LAYERS, "dtype": "bf16", "data": "synthetic"}), flush=True)
+        line = {"design": design, "size": size, "pass": what, "ms": round(ms, 3), "tokens_per_s": round(n / ms * 1e3)}
+        for c in closest:
+            other = res[c, what][0]
+            line.update({f"{c}_ms": round(other, 3), f"{c}_tokens_per_s": round(n / other * 1e3),
+                         "speedup" if len(closest) == 1 else f"speedup_{c}": round(other / ms, 2)})
+        print(json.dumps(dict(line, layers=LAYERS, dtype="bf16", data="synthetic")), flush=True)
 
 
 def run(args):
