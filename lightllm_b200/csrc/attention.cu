@@ -169,9 +169,12 @@ gqa_decode_kernel(const bf16* __restrict__ q, int64_t q_stride, const bf16* __re
   float m_run[2] = {-INFINITY, -INFINITY};
   float l_run[2] = {0.f, 0.f};
   const float *rel0 = nullptr, *rel1 = nullptr;  // biases of the heads of my two rows
+  float far_bias[2] = {0.f, 0.f};
   if (SPLIT_P && rule.rel != nullptr) {
-    rel0 = rule.rel + (int64_t)(head0 + min(g, nrows - 1)) * (rule.far + 1);
-    rel1 = rule.rel + (int64_t)(head0 + min(g + 8, nrows - 1)) * (rule.far + 1);
+    rel0 = rule.rel + (head0 + min(g, nrows - 1)) * rule.rel_stride;
+    rel1 = rule.rel + (head0 + min(g + 8, nrows - 1)) * rule.rel_stride;
+    far_bias[0] = rel0[rule.far] * kLog2e;
+    far_bias[1] = rel1[rule.far] * kLog2e;
   }
 
 #pragma unroll
@@ -203,8 +206,10 @@ gqa_decode_kernel(const bf16* __restrict__ q, int64_t q_stride, const bf16* __re
     float add[2][4];
     if (SPLIT_P) {
 #pragma unroll
-      for (int j = 0; j < 2; ++j) add[j][0] = add[j][1] = add[j][2] = add[j][3] = 0.f;
-      if (rel0 != nullptr) {
+      for (int j = 0; j < 2; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) add[j][e] = far_bias[e >> 1];
+      if (rel0 != nullptr && L - 1 - position(min(p0 + 15, e0 - 1)) < rule.far) {  // some key of the tile is nearer
 #pragma unroll
         for (int j = 0; j < 2; ++j)
 #pragma unroll
@@ -600,7 +605,7 @@ LLB_EXPORT int llb_gqa_decode(const void* q, int64_t q_stride, const void* kv_la
   if (Hkv <= 0 || Hq % Hkv != 0 || num_splits < 1) return LLB_ERR_BAD_ARG;
   if (num_splits > 1 && (part_o == nullptr || part_lse == nullptr)) return LLB_ERR_BAD_ARG;
   const HeadGate none{nullptr, 0, 1.f};
-  const KeyRule all{0, 0, nullptr, 0};
+  const KeyRule all{0, 0, nullptr, 0, 0};
   if (D == 128)
     return launch_decode<128, 128, false>(q, q_stride, kv_layer, req_to_token, r2t_stride, b_req_idx, b_seq_len, out,
                                           out_stride, part_o, part_lse, B, Hq, Hkv, num_splits, sm_scale, all, none, st);
@@ -611,19 +616,19 @@ LLB_EXPORT int llb_gqa_decode(const void* q, int64_t q_stride, const void* kv_la
 }
 
 // The windowed form: key size dk and value size dv (64, 128, 192 or 256), pool rows [Hkv * dk | Hkv * dv], window (0: none),
-// the first `keep` positions always seen, biases by distance rel [Hq, far + 1] (or null), gate [B, >= Hq] (or null): head h of the output times out_scale * sigmoid(gate).  part_o: fp32 [B, Hq, num_splits, dv].
+// the first `keep` positions always seen, biases by distance rel [Hq, far + 1] (or null; see KeyRule), gate [B, >= Hq] (or null): head h of the output times out_scale * sigmoid(gate).  part_o: fp32 [B, Hq, num_splits, dv].
 LLB_EXPORT int llb_window_gqa_decode(const void* q, int64_t q_stride, const void* kv_layer, const int* req_to_token,
                                      int64_t r2t_stride, const int* b_req_idx, const int* b_seq_len, void* out,
                                      int64_t out_stride, float* part_o, float* part_lse, int B, int Hq, int Hkv, int dk,
                                      int dv, int num_splits, float sm_scale, int window, int keep, const float* rel,
-                                     int far, const void* gate, int64_t gate_stride, float out_scale, cudaStream_t st) {
+                                     int far, int64_t rel_stride, const void* gate, int64_t gate_stride, float out_scale, cudaStream_t st) {
   if (B <= 0) return LLB_OK;
   if (Hkv <= 0 || Hq % Hkv != 0 || num_splits < 1 || window < 0 || keep < 0 || (rel != nullptr && far < 0) ||
       (q_stride % 8) || ((uintptr_t)q & 15))
     return LLB_ERR_BAD_ARG;
   if (num_splits > 1 && (part_o == nullptr || part_lse == nullptr)) return LLB_ERR_BAD_ARG;
   const HeadGate g{(const bf16*)gate, gate_stride, out_scale};
-  const KeyRule rule{window, keep, rel, far};
+  const KeyRule rule{window, keep, rel, far, rel_stride};
 #define LLB_WINDOW_DECODE(DK, DV)                                                                                        \
   if (dk == DK && dv == DV)                                                                                              \
     return launch_decode<DK, DV, true>(q, q_stride, kv_layer, req_to_token, r2t_stride, b_req_idx, b_seq_len, out,       \

@@ -51,7 +51,7 @@ attn_generic_kernel(const E* __restrict__ q, int64_t q_stride, const E* __restri
   const int j0 = (rule.window > 0 && qpos - rule.window + 1 > 0) ? qpos - rule.window + 1 : 0;
   const int kept = min(rule.keep, j0), n = kept + qpos + 1 - j0;  // kept first positions, then the window
   const float slope = alibi ? alibi[h] : 0.f;
-  const float* rel = rule.rel ? rule.rel + (int64_t)h * (rule.far + 1) : nullptr;
+  const float* rel = rule.rel ? rule.rel + h * rule.rel_stride : nullptr;
   for (int i = warp; i < n; i += GEN_WARPS) {
     const int j = i < kept ? i : j0 + i - kept;
     const E* kr = kv + (int64_t)slots[j] * row + (int64_t)kvh * D;
@@ -120,7 +120,7 @@ LLB_EXPORT int llb_attn_generic(const void* q, int64_t q_stride, const void* kv_
   dim3 grid(T, Hq);
   attn_generic_kernel<bf16, GEN_MAX_EPL><<<grid, GEN_WARPS * 32, 0, st>>>(
       (const bf16*)q, q_stride, (const bf16*)kv_layer, req_to_token, r2t_stride, b_req_idx, pos, batch_of, (bf16*)out,
-      out_stride, Hq, Hkv, D, D, sm_scale, KeyRule{window, 0, nullptr, 0}, softcap, alibi_slopes, sinks, nullptr, 0, 1.f);
+      out_stride, Hq, Hkv, D, D, sm_scale, KeyRule{window, 0, nullptr, 0, 0}, softcap, alibi_slopes, sinks, nullptr, 0, 1.f);
   LLB_LAUNCH_CHECK();
   return LLB_OK;
 }
@@ -130,11 +130,11 @@ LLB_EXPORT int llb_attn_generic(const void* q, int64_t q_stride, const void* kv_
 LLB_EXPORT int llb_attn_generic_kv(const void* q, int dt, int64_t q_stride, const void* kv_layer, const int* req_to_token,
                                    int64_t r2t_stride, const int* b_req_idx, const int* pos, const int* batch_of,
                                    void* out, int64_t out_stride, int T, int Hq, int Hkv, int D, int DV, float sm_scale,
-                                   int window, int keep, const float* rel, int far, const void* gate,
-                                   int64_t gate_stride, float out_scale, cudaStream_t st) {
+                                   int window, int keep, const float* rel, int far, int64_t rel_stride,
+                                   const void* gate, int64_t gate_stride, float out_scale, cudaStream_t st) {
   if (T <= 0) return LLB_OK;
   if (window < 0 || keep < 0 || (rel != nullptr && far < 0)) return LLB_ERR_BAD_ARG;
-  const KeyRule rule{window, keep, rel, far};
+  const KeyRule rule{window, keep, rel, far, rel_stride};
   if (D <= 0 || DV <= 0 || D > 512 || DV > 512 || Hkv <= 0 || Hq % Hkv != 0 || Hq > 65535) return LLB_ERR_UNSUPPORTED;
   const dim3 grid(T, Hq);
 #define LLB_GENERIC(E, EPL)                                                                                           \
@@ -225,7 +225,8 @@ __device__ __forceinline__ void store8(float* p, const float* f) {
   reinterpret_cast<float4*>(p)[1] = make_float4(f[4], f[5], f[6], f[7]);
 }
 
-template <typename E, int NIT>
+// FAST (NIT = 1, rot_dim a multiple of 16): a lane's 8 elements lie in one half, their partners in one other lane.
+template <typename E, int NIT, bool FAST>
 __global__ void __launch_bounds__(256)
 qk_norm_rope_scatter_kernel(E* __restrict__ qkv, int64_t qkv_stride, E* __restrict__ kv_layer,
                             const float* __restrict__ cos_t, const float* __restrict__ sin_t, const int* __restrict__ pos,
@@ -252,7 +253,7 @@ qk_norm_rope_scatter_kernel(E* __restrict__ qkv, int64_t qkv_stride, E* __restri
     uint4* dst = reinterpret_cast<uint4*>(kv_row + (int64_t)Hkv * D + (int64_t)g * DV);
     for (int v = gl; v < DV * (int)sizeof(E) / 16; v += lanes) dst[v] = src[v];
   }
-  float f[NIT][8];
+  float f[NIT][8] = {};
   float ss = 0.f;
   if (qk) {
 #pragma unroll
@@ -276,17 +277,36 @@ qk_norm_rope_scatter_kernel(E* __restrict__ qkv, int64_t qkv_stride, E* __restri
       if (w != nullptr) load8(w + d, wv);
 #pragma unroll
       for (int i = 0; i < 8; ++i) f[n][i] *= w != nullptr ? inv * wv[i] : inv;
-      if (d < rot_dim) {
+      if (!FAST && d < rot_dim) {
 #pragma unroll
         for (int i = 0; i < 8; ++i)
           if (d + i < rot_dim) sh[d + i] = f[n][i];
       }
     }
   }
+  E* dst = head < Hq ? x : kv_row + (int64_t)(head - Hq) * D;
+  if (FAST) {
+    const int d = gl * 8, step = half >> 3;
+    const bool turns = d < rot_dim, upper = d >= half;
+    float o[8];
+    const int lane = threadIdx.x & 31, src = turns ? (upper ? lane - step : lane + step) : lane;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) o[i] = __shfl_sync(0xffffffffu, f[0][i], src);
+    if (!qk || d >= D) return;
+    if (turns) {
+      const int64_t at = (int64_t)pos[t] * half + (upper ? d - half : d);
+      float c[8], s[8];
+      load8(cos_t + at, c);
+      load8(sin_t + at, s);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) f[0][i] = f[0][i] * c[i] + (upper ? o[i] : -o[i]) * s[i];
+    }
+    store8(dst + d, f[0]);
+    return;
+  }
   __syncwarp();
   if (!qk) return;
   const float *cr = cos_t + (int64_t)pos[t] * half, *sr = sin_t + (int64_t)pos[t] * half;
-  E* dst = head < Hq ? x : kv_row + (int64_t)(head - Hq) * D;
 #pragma unroll
   for (int n = 0; n < NIT; ++n) {
     const int d = (gl + n * lanes) * 8;
@@ -321,18 +341,23 @@ LLB_EXPORT int llb_qk_norm_rope_scatter(void* qkv, int dt, int64_t qkv_stride, v
   const size_t smem = (size_t)groups * rot_dim * sizeof(float);
   if (smem > 48 * 1024 || items > 0x7fffff00) return LLB_ERR_UNSUPPORTED;
   const dim3 grid((unsigned)cdiv64(items, groups));
-#define LLB_QK(E, NIT)                                                                                                    \
-  launch_pdl(qk_norm_rope_scatter_kernel<E, NIT>, grid, dim3(256), smem, st, (E*)qkv, qkv_stride, (E*)kv_layer, cos_t,  \
-             sin_t, pos, slot, qw, kw, eps, (unsigned)items, Hq, Hkv, D, dim, DV, rot_dim, lg)
-  if (D <= 256) {
+#define LLB_QK(E, NIT, FAST)                                                                                              \
+  launch_pdl(qk_norm_rope_scatter_kernel<E, NIT, FAST>, grid, dim3(256), FAST ? 0 : smem, st, (E*)qkv, qkv_stride,        \
+             (E*)kv_layer, cos_t, sin_t, pos, slot, qw, kw, eps, (unsigned)items, Hq, Hkv, D, dim, DV, rot_dim, lg)
+  if (D <= 256 && rot_dim > 0 && rot_dim % 16 == 0) {
     if (dt == 0)
-      LLB_QK(float, 1);
+      LLB_QK(float, 1, true);
     else
-      LLB_QK(bf16, 1);
+      LLB_QK(bf16, 1, true);
+  } else if (D <= 256) {
+    if (dt == 0)
+      LLB_QK(float, 1, false);
+    else
+      LLB_QK(bf16, 1, false);
   } else if (dt == 0) {
-    LLB_QK(float, 2);
+    LLB_QK(float, 2, false);
   } else {
-    LLB_QK(bf16, 2);
+    LLB_QK(bf16, 2, false);
   }
 #undef LLB_QK
   LLB_LAUNCH_CHECK();

@@ -286,6 +286,8 @@ gqa_prefill_tc_kernel(const bf16* __restrict__ q, int64_t q_stride, const bf16* 
 #pragma unroll
     for (int i = 0; i < OC; ++i) o[i] = 0.f;
     float m_run = -INFINITY, l_run = 0.f;
+    const float* rel = EXT && rule.rel != nullptr ? rule.rel + h * rule.rel_stride : nullptr;
+    const float far_bias = EXT && rel != nullptr ? rel[rule.far] * kLog2e : 0.f;
     for (int j = 0; j < n_tiles; ++j) {
       const int kt = tile_pos(j) + half * HK;
       mbar_wait(s_full(j & 1), ((uint32_t)j >> 1) & 1u, abort_flag, status, 45);
@@ -300,18 +302,16 @@ gqa_prefill_tc_kernel(const bf16* __restrict__ q, int64_t q_stride, const bf16* 
       auto seen = [&](int c) { return c <= lim && (c >= lo || (EXT && c < first)); };
       // whole tile (every tile but those at the diagonal and the edges)
       const bool all_visible = lim >= HK - 1 && (lo <= 0 || (EXT && first >= HK));
-      const float to_log2 = EXT ? 1.f : scale_log2;
-      if (EXT) {  // scores in log2 units, with the bias of their distance
-        const float* rel = rule.rel != nullptr ? rule.rel + (int64_t)h * (rule.far + 1) : nullptr;
+      float to_log2 = scale_log2, shift = 0.f;  // score in log2 units = sr * to_log2 + shift
+      if (EXT && rel != nullptr) {
         const int dist = prow - kt;  // of my first column; the last one is HK - 1 nearer
-        if (rel == nullptr || dist - (HK - 1) >= rule.far) {
-          const float b = rel != nullptr ? rel[rule.far] * kLog2e : 0.f;
+        if (dist - (HK - 1) >= rule.far) {
+          shift = far_bias;
+        } else {  // columns of a negative distance are not seen, whatever they are added
+          const float* at = rel + max(dist, 0);
+          to_log2 = 1.f;
 #pragma unroll
-          for (int e = 0; e < HK; ++e) sr[e] = __float_as_uint(fmaf(__uint_as_float(sr[e]), scale_log2, b));
-        } else {
-#pragma unroll
-          for (int e = 0; e < HK; ++e)
-            sr[e] = __float_as_uint(fmaf(__uint_as_float(sr[e]), scale_log2, rel[max(0, min(dist - e, rule.far))] * kLog2e));
+          for (int e = 0; e < HK; ++e) sr[e] = __float_as_uint(fmaf(__uint_as_float(sr[e]), scale_log2, at[-e] * kLog2e));
         }
       }
       float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
@@ -324,11 +324,12 @@ gqa_prefill_tc_kernel(const bf16* __restrict__ q, int64_t q_stride, const bf16* 
           if (seen(e)) mx4[e & 3] = fmaxf(mx4[e & 3], __uint_as_float(sr[e]));
       }
       float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
+      if (EXT) mx = fmaf(mx, to_log2, shift);
       float* x = xch + (j & 1) * 256;
       x[half * 128 + erow] = mx;
       asm volatile("bar.sync 1, 256;" ::: "memory");
       mx = fmaxf(mx, x[(half ^ 1) * 128 + erow]);
-      const float m_new = fmaxf(m_run, mx * to_log2);
+      const float m_new = fmaxf(m_run, EXT ? mx : mx * to_log2);
       const float m_use = m_new == -INFINITY ? 0.f : m_new;
       const float alpha = ex2_fast(m_run - m_use);
       m_run = m_new;
@@ -349,7 +350,7 @@ gqa_prefill_tc_kernel(const bf16* __restrict__ q, int64_t q_stride, const bf16* 
 #pragma unroll
         for (int e = 0; e < 8; ++e) {
           const int c = g * 8 + e;
-          const float pe = ex2_fast(fmaf(__uint_as_float(sr[c]), to_log2, -m_use));
+          const float pe = ex2_fast(fmaf(__uint_as_float(sr[c]), to_log2, EXT ? shift - m_use : -m_use));
           pv[e] = (all_visible || seen(c)) ? pe : 0.f;
           rs4[e & 3] += pv[e];
         }
@@ -460,23 +461,23 @@ LLB_EXPORT int llb_gqa_prefill_tc(const void* q, int64_t q_stride, const void* k
   if (Hkv <= 0 || Hq % Hkv != 0 || (q_stride % 8) || (out_stride % 8) || ((uintptr_t)q & 15) || ((uintptr_t)out & 15))
     return LLB_ERR_BAD_ARG;
   return launch_tc<128, 128, 128, false, false>((const bf16*)q, q_stride, (const bf16*)kv_layer, req_to_token, r2t_stride, b_req_idx,
-                                         cu_q, b_ready_len, (bf16*)out, out_stride, B, max_q_len, Hq, Hkv, sm_scale, 1, KeyRule{0, 0, nullptr, 0},
+                                         cu_q, b_ready_len, (bf16*)out, out_stride, B, max_q_len, Hq, Hkv, sm_scale, 1, KeyRule{0, 0, nullptr, 0, 0},
                                          nullptr, 0, 1.f, st);
 }
 
 // Key size dk (64, 128, 192, 256), value size dv (a multiple of 64), window (0: none), first `keep` positions always seen,
-// biases by distance rel [Hq, far + 1] (or null): pool rows [Hkv * dk | Hkv * dv], q
+// biases by distance rel [Hq, far + 1] (or null; see KeyRule): pool rows [Hkv * dk | Hkv * dv], q
 // [T, >= Hq * dk], out [T, >= Hq * dv].  gate [T, >= Hq] (or null): head h of the output times out_scale * sigmoid(gate).
 LLB_EXPORT int llb_window_gqa_prefill_tc(const void* q, int64_t q_stride, const void* kv_layer, const int* req_to_token,
                                          int64_t r2t_stride, const int* b_req_idx, const int* cu_q, const int* b_ready_len,
                                          void* out, int64_t out_stride, int B, int max_q_len, int Hq, int Hkv, int dk,
                                          int dv, float sm_scale, int window, int keep, const float* rel, int far,
-                                         const void* gate, int64_t gate_stride, float out_scale, cudaStream_t st) {
+                                         int64_t rel_stride, const void* gate, int64_t gate_stride, float out_scale, cudaStream_t st) {
   if (B <= 0 || max_q_len <= 0) return LLB_OK;
   if (Hkv <= 0 || Hq % Hkv != 0 || (q_stride % 8) || (out_stride % 8) || ((uintptr_t)q & 15) || ((uintptr_t)out & 15) ||
       window < 0 || keep < 0 || (rel != nullptr && far < 0) || dv <= 0)
     return LLB_ERR_BAD_ARG;
-  const KeyRule rule{window, keep, rel, far};
+  const KeyRule rule{window, keep, rel, far, rel_stride};
   const bool ext = (window > 0 && keep > 0) || rel != nullptr;
   if ((dv % 64) || (dk != 64 && dk != 128 && dk != 192 && dk != 256) || Hq * (dv / 64) > 65535 || B > 65535)
     return LLB_ERR_UNSUPPORTED;

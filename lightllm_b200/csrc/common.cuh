@@ -188,11 +188,14 @@ __device__ __forceinline__ float tanh_fast(float x) {
 }
 
 // Which keys a causal query sees and what its scores get added: position p sees j <= p with p - j < window (window 0: all) or
-// j < keep; key j's score of head h gets rel[h, min(p - j, far)] (natural units; rel [heads, far + 1] fp32, or null).
+// j < keep; key j's score of head h gets rel[h, min(p - j, far)] (natural units; fp32, heads rel_stride apart, or null).  Every
+// head's entries may also be read kRelPad places before 0 and after `far` (those beyond `far` repeat it).
+constexpr int kRelPad = 64;
 struct KeyRule {
   int window, keep;
   const float* rel;
   int far;
+  int64_t rel_stride;
 };
 
 // Block-wide sum; `red` is a shared array of >= 33 floats. All threads get the result.

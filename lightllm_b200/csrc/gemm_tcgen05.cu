@@ -120,7 +120,8 @@ __device__ __forceinline__ float gated_f(const GemmParams& p, float g, float u) 
 }
 __device__ __forceinline__ float f32_out(const GemmParams& p, float v) {
   v *= p.out_scale;
-  return p.softcap > 0.f ? p.softcap * tanh_fast(__fdividef(v, p.softcap)) : v;
+  // c tanh(v / c) = c - 2 c / (1 + e^(2 v / c)): an absolute error of a few 1e-7 c, like the rounding of values of that size
+  return p.softcap > 0.f ? p.softcap - __fdividef(2.f * p.softcap, 1.f + __expf(v * __fdividef(2.f, p.softcap))) : v;
 }
 __device__ __forceinline__ float4 f32_out4(const GemmParams& p, float4 v) {
   return make_float4(f32_out(p, v.x), f32_out(p, v.y), f32_out(p, v.z), f32_out(p, v.w));

@@ -778,7 +778,10 @@ _WINDOW_SIZES = (64, 128, 192, 256)   # head sizes of the tensor-core kernels
 class DistanceBias:
     """Learned bias per head and bucket of the distance n between query and key.  With B rows in the table: bucket n for
     n < B / 2, beyond that B / 2 buckets spaced by logarithm up to the distance `far`, the last one for all from there on.
-    Kept as `rel` [heads, far + 1] fp32: the bias of every distance up to `far`."""
+    Kept as `rel` [heads, far + 1] fp32: the bias of every distance up to `far`, rows that may be read PAD places further on
+    either side."""
+
+    PAD = 64
 
     def __init__(self, table: torch.Tensor, far: int):
         B, half = table.shape[0], table.shape[0] // 2
@@ -786,8 +789,9 @@ class DistanceBias:
         step = math.log(far / half)
         rows = [n if n < half else min(B - 1, half + math.floor(math.log(n / half) / step * (B - half)))
                 for n in range(far + 1)]
+        rows = [rows[0]] * self.PAD + rows + [rows[-1]] * self.PAD
         self.far = int(far)
-        self.rel = table.float()[torch.tensor(rows, device=table.device)].t().contiguous()
+        self.rel = table.float()[torch.tensor(rows, device=table.device)].t().contiguous()[:, self.PAD:self.PAD + far + 1]
 
 
 def window_attention(q, kv_layer, req_to_token, st, Hq, Hkv, D, DV, sm_scale, window, gate=None, out_scale=1.0, out=None,
@@ -805,8 +809,9 @@ def window_attention(q, kv_layer, req_to_token, st, Hq, Hkv, D, DV, sm_scale, wi
                                     out_scale, out, keep, bias)
     assert q.stride(1) == 1 and kv_layer.is_contiguous() and out.stride(1) == 1
     gs = 0 if gate is None else gate.stride(0)
-    rel, far = (bias.rel, bias.far) if bias is not None else (None, 0)
-    tail = (f32(sm_scale), c_int(window), c_int(keep), ptr(rel), c_int(far), ptr(gate), i64(gs), f32(out_scale), stream())
+    rel, far, stride = (bias.rel, bias.far, bias.rel.stride(0)) if bias is not None else (None, 0, 0)
+    tail = (f32(sm_scale), c_int(window), c_int(keep), ptr(rel), c_int(far), i64(stride), ptr(gate), i64(gs), f32(out_scale),
+            stream())
     if q.dtype == torch.bfloat16 and D in _WINDOW_SIZES and DV % 64 == 0:
         common = (ptr(q), i64(q.stride(0)), ptr(kv_layer), ptr(req_to_token), i64(req_to_token.stride(0)),
                   ptr(st.b_req_idx))
