@@ -309,20 +309,20 @@ gqa_prefill_tc_kernel(const bf16* __restrict__ q, int64_t q_stride, const bf16* 
           shift = far_bias;
         } else {  // columns of a negative distance are not seen, whatever they are added
           const float* at = rel + max(dist, 0);
-          to_log2 = 1.f;
+          to_log2 = kLog2e;
+          const float scale = scale_log2 * (1.f / kLog2e);
 #pragma unroll
-          for (int e = 0; e < HK; ++e) sr[e] = __float_as_uint(fmaf(__uint_as_float(sr[e]), scale_log2, at[-e] * kLog2e));
+          for (int e = 0; e < HK; ++e) sr[e] = __float_as_uint(fmaf(__uint_as_float(sr[e]), scale, at[-e]));
         }
       }
       float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
-      if (all_visible) {
-#pragma unroll
-        for (int e = 0; e < HK; ++e) mx4[e & 3] = fmaxf(mx4[e & 3], __uint_as_float(sr[e]));
-      } else {
+      if (!all_visible) {  // scores that are not seen: -inf, whose weight comes out as 0
 #pragma unroll
         for (int e = 0; e < HK; ++e)
-          if (seen(e)) mx4[e & 3] = fmaxf(mx4[e & 3], __uint_as_float(sr[e]));
+          if (!seen(e)) sr[e] = 0xff800000u;
       }
+#pragma unroll
+      for (int e = 0; e < HK; ++e) mx4[e & 3] = fmaxf(mx4[e & 3], __uint_as_float(sr[e]));
       float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
       if (EXT) mx = fmaf(mx, to_log2, shift);
       float* x = xch + (j & 1) * 256;
@@ -350,8 +350,7 @@ gqa_prefill_tc_kernel(const bf16* __restrict__ q, int64_t q_stride, const bf16* 
 #pragma unroll
         for (int e = 0; e < 8; ++e) {
           const int c = g * 8 + e;
-          const float pe = ex2_fast(fmaf(__uint_as_float(sr[c]), to_log2, EXT ? shift - m_use : -m_use));
-          pv[e] = (all_visible || seen(c)) ? pe : 0.f;
+          pv[e] = ex2_fast(fmaf(__uint_as_float(sr[c]), to_log2, EXT ? shift - m_use : -m_use));
           rs4[e & 3] += pv[e];
         }
         const uint32_t off = tile_off<BLOCK_BYTES>(erow, half * (HK / 8) + g);
@@ -458,7 +457,7 @@ LLB_EXPORT int llb_gqa_prefill_tc(const void* q, int64_t q_stride, const void* k
                                   void* out, int64_t out_stride, int B, int max_q_len, int Hq, int Hkv, float sm_scale,
                                   cudaStream_t st) {
   if (B <= 0 || max_q_len <= 0) return LLB_OK;
-  if (Hkv <= 0 || Hq % Hkv != 0 || (q_stride % 8) || (out_stride % 8) || ((uintptr_t)q & 15) || ((uintptr_t)out & 15))
+  if (!(sm_scale > 0.f) || Hkv <= 0 || Hq % Hkv != 0 || (q_stride % 8) || (out_stride % 8) || ((uintptr_t)q & 15) || ((uintptr_t)out & 15))
     return LLB_ERR_BAD_ARG;
   return launch_tc<128, 128, 128, false, false>((const bf16*)q, q_stride, (const bf16*)kv_layer, req_to_token, r2t_stride, b_req_idx,
                                          cu_q, b_ready_len, (bf16*)out, out_stride, B, max_q_len, Hq, Hkv, sm_scale, 1, KeyRule{0, 0, nullptr, 0, 0},
@@ -474,7 +473,7 @@ LLB_EXPORT int llb_window_gqa_prefill_tc(const void* q, int64_t q_stride, const 
                                          int dv, float sm_scale, int window, int keep, const float* rel, int far,
                                          int64_t rel_stride, const void* gate, int64_t gate_stride, float out_scale, cudaStream_t st) {
   if (B <= 0 || max_q_len <= 0) return LLB_OK;
-  if (Hkv <= 0 || Hq % Hkv != 0 || (q_stride % 8) || (out_stride % 8) || ((uintptr_t)q & 15) || ((uintptr_t)out & 15) ||
+  if (!(sm_scale > 0.f) || Hkv <= 0 || Hq % Hkv != 0 || (q_stride % 8) || (out_stride % 8) || ((uintptr_t)q & 15) || ((uintptr_t)out & 15) ||
       window < 0 || keep < 0 || (rel != nullptr && far < 0) || dv <= 0)
     return LLB_ERR_BAD_ARG;
   const KeyRule rule{window, keep, rel, far, rel_stride};

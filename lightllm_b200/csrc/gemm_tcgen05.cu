@@ -118,13 +118,17 @@ __device__ __forceinline__ float gated_f(const GemmParams& p, float g, float u) 
   }
   return (EPI == EPI_GATED_SILU ? silu_f(g) : gelu_tanh_f(g)) * u;
 }
-__device__ __forceinline__ float f32_out(const GemmParams& p, float v) {
-  v *= p.out_scale;
-  // c tanh(v / c) = c - 2 c / (1 + e^(2 v / c)): an absolute error of a few 1e-7 c, like the rounding of values of that size
-  return p.softcap > 0.f ? p.softcap - __fdividef(2.f * p.softcap, 1.f + __expf(v * __fdividef(2.f, p.softcap))) : v;
-}
-__device__ __forceinline__ float4 f32_out4(const GemmParams& p, float4 v) {
-  return make_float4(f32_out(p, v.x), f32_out(p, v.y), f32_out(p, v.z), f32_out(p, v.w));
+// EPI_F32: n values, finished in place (one branch for all of them).
+//   c tanh(v / c) = c - 2 c / (1 + e^(2 v / c)): an absolute error of a few 1e-7 c, like the rounding of values of that size
+template <int N>
+__device__ __forceinline__ void f32_finish(const GemmParams& p, float* v) {
+#pragma unroll
+  for (int j = 0; j < N; ++j) v[j] *= p.out_scale;
+  if (p.softcap > 0.f) {
+    const float c = p.softcap, k = __fdividef(2.f, c);
+#pragma unroll
+    for (int j = 0; j < N; ++j) v[j] = c - __fdividef(2.f * c, 1.f + __expf(v[j] * k));
+  }
 }
 __device__ __forceinline__ float relu2_f(float v) {
   v = fmaxf(v, 0.f);
@@ -250,24 +254,18 @@ __device__ __forceinline__ void epi_direct32(const GemmParams& p, const uint32_t
     }
   } else if (EPI == EPI_F32) {
     float* crow = (float*)p.C + (int64_t)row * p.ldc + col0;
+    float v[32];
+#pragma unroll
+    for (int j = 0; j < 32; ++j)
+      v[j] = __uint_as_float(r[j]) + (p.bias && j < ncols ? __bfloat162float(p.bias[col0 + j]) : 0.f);
+    f32_finish<32>(p, v);
     if (ncols == 32) {
 #pragma unroll
-      for (int j = 0; j < 32; j += 4) {
-        float4 v = make_float4(__uint_as_float(r[j]), __uint_as_float(r[j + 1]), __uint_as_float(r[j + 2]),
-                               __uint_as_float(r[j + 3]));
-        if (p.bias) {
-          v.x += __bfloat162float(p.bias[col0 + j]);
-          v.y += __bfloat162float(p.bias[col0 + j + 1]);
-          v.z += __bfloat162float(p.bias[col0 + j + 2]);
-          v.w += __bfloat162float(p.bias[col0 + j + 3]);
-        }
-        *reinterpret_cast<float4*>(crow + j) = f32_out4(p, v);
-      }
+      for (int j = 0; j < 32; j += 4) *reinterpret_cast<float4*>(crow + j) = make_float4(v[j], v[j + 1], v[j + 2], v[j + 3]);
     } else {
 #pragma unroll
       for (int j = 0; j < 32; ++j)
-        if (j < ncols)
-          crow[j] = f32_out(p, __uint_as_float(r[j]) + (p.bias ? __bfloat162float(p.bias[col0 + j]) : 0.f));
+        if (j < ncols) crow[j] = v[j];
     }
   } else {
     bf16* crow = (bf16*)p.C + (int64_t)row * p.ldc + col0;
@@ -446,18 +444,12 @@ __device__ __forceinline__ void epilogue_store(const GemmParams& p, uint32_t t_r
       if (has_add) add_partials(r, c);
       const int col0 = col_tile0 + c;
       if (stage != nullptr && col0 + 32 <= p.N) {
+        float v[32];
 #pragma unroll
-        for (int j = 0; j < 32; j += 4) {
-          float4 v = make_float4(__uint_as_float(r[j]), __uint_as_float(r[j + 1]), __uint_as_float(r[j + 2]),
-                                 __uint_as_float(r[j + 3]));
-          if (p.bias) {
-            v.x += __bfloat162float(p.bias[col0 + j]);
-            v.y += __bfloat162float(p.bias[col0 + j + 1]);
-            v.z += __bfloat162float(p.bias[col0 + j + 2]);
-            v.w += __bfloat162float(p.bias[col0 + j + 3]);
-          }
-          *reinterpret_cast<float4*>(my + j * 4) = f32_out4(p, v);
-        }
+        for (int j = 0; j < 32; ++j) v[j] = __uint_as_float(r[j]) + (p.bias ? __bfloat162float(p.bias[col0 + j]) : 0.f);
+        f32_finish<32>(p, v);
+#pragma unroll
+        for (int j = 0; j < 32; j += 4) *reinterpret_cast<float4*>(my + j * 4) = make_float4(v[j], v[j + 1], v[j + 2], v[j + 3]);
         __syncwarp();
         epi_flush<4>(p, stage, lane, row_base, col0, false);
         __syncwarp();
@@ -1286,7 +1278,9 @@ gemm_bf16_skinny_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_co
           acc.w += __bfloat162float(p.bias[gcol + 3]);
         }
         if (EPI == EPI_F32) {
-          *reinterpret_cast<float4*>((float*)p.C + (int64_t)grow * p.ldc + gcol) = f32_out4(p, acc);
+          float v[4] = {acc.x, acc.y, acc.z, acc.w};
+          f32_finish<4>(p, v);
+          *reinterpret_cast<float4*>((float*)p.C + (int64_t)grow * p.ldc + gcol) = make_float4(v[0], v[1], v[2], v[3]);
         } else if (EPI == EPI_DYT) {
           const int64_t off = (int64_t)grow * p.ldc + gcol;
           float4 x = *reinterpret_cast<const float4*>(p.dyt.x + off);

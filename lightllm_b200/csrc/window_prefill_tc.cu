@@ -236,14 +236,13 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
       const int lo = p.window > 0 ? prow - p.window + 1 - kt : 0;
       const bool all_visible = hi >= HK - 1 && lo <= 0;
       float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
-      if (all_visible) {
-#pragma unroll
-        for (int e = 0; e < HK; ++e) mx4[e & 3] = fmaxf(mx4[e & 3], __uint_as_float(sr[e]));
-      } else {
+      if (!all_visible) {  // scores that are not seen: -inf, whose weight comes out as 0
 #pragma unroll
         for (int e = 0; e < HK; ++e)
-          if (e >= lo && e <= hi) mx4[e & 3] = fmaxf(mx4[e & 3], __uint_as_float(sr[e]));
+          if (e < lo || e > hi) sr[e] = 0xff800000u;
       }
+#pragma unroll
+      for (int e = 0; e < HK; ++e) mx4[e & 3] = fmaxf(mx4[e & 3], __uint_as_float(sr[e]));
       float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
       float* x = xch + (j & 1) * 256;
       x[half * 128 + erow] = mx;
@@ -273,8 +272,7 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
 #pragma unroll
           for (int u = 0; u < 2; ++u) {
             const int c = g * 8 + e + u;
-            const float pe = ex2_fast(fmaf(__uint_as_float(sr[c]), p.scale_log2, -m_use));
-            pv[u] = (all_visible || (c >= lo && c <= hi)) ? pe : 0.f;
+            pv[u] = ex2_fast(fmaf(__uint_as_float(sr[c]), p.scale_log2, -m_use));
             rs4[(e + u) & 3] += pv[u];
           }
           ph[e / 2] = pack_bf16x2(pv[0], pv[1]);
@@ -386,7 +384,7 @@ LLB_EXPORT int llb_window_prefill_tc(const void* q, int64_t q_stride, const void
                                      float sm_scale, int window, const void* gate, int64_t gate_stride,
                                      cudaStream_t st) {
   if (B <= 0 || max_q_len <= 0 || T <= 0) return LLB_OK;
-  if (H <= 0 || H > 65535 || B > 65535 || kv_rows <= 0 || window < 0) return LLB_ERR_BAD_ARG;
+  if (!(sm_scale > 0.f) || H <= 0 || H > 65535 || B > 65535 || kv_rows <= 0 || window < 0) return LLB_ERR_BAD_ARG;
   if ((dk != 64 && dk != 128 && dk != 192 && dk != 256) || (dv != 64 && dv != 128)) return LLB_ERR_UNSUPPORTED;
   if (gate != nullptr && ((gate_stride % 8) || ((uintptr_t)gate & 15))) return LLB_ERR_BAD_ARG;
   const int bn = dk > 128 ? 64 : 128;

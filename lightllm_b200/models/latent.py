@@ -54,7 +54,7 @@ class LatentHeads:
 
     def _expanded_range(self, q, st: InferState):
         """The positions to expand keys and values for when this prompt pass runs the expanded form, else None."""
-        if not q.is_cuda or q.dtype != torch.bfloat16 or self.dp > 256 or self.vp > 128:
+        if not q.is_cuda or q.dtype != torch.bfloat16 or self.dp > 256 or self.vp > 128 or self.scale <= 0:
             return None
         cache = st.extra.setdefault("key_ranges", {})
         if self.window not in cache:

@@ -772,6 +772,12 @@ def sigmoid_mul_(x, gate):
     return x
 
 
+def window_decode_splits(T: int, Hq: int, Hkv: int, keys: int) -> int:
+    """Shares the keys of a decode step are cut into: about two CTAs per SM (more measured slower), at least 256 keys each."""
+    ctas = T * Hkv * -(-(Hq // Hkv) // 16)
+    return max(1, min(296 // ctas, -(-keys // 256), 64))
+
+
 _WINDOW_SIZES = (64, 128, 192, 256)   # head sizes of the tensor-core kernels
 
 
@@ -812,7 +818,7 @@ def window_attention(q, kv_layer, req_to_token, st, Hq, Hkv, D, DV, sm_scale, wi
     rel, far, stride = (bias.rel, bias.far, bias.rel.stride(0)) if bias is not None else (None, 0, 0)
     tail = (f32(sm_scale), c_int(window), c_int(keep), ptr(rel), c_int(far), i64(stride), ptr(gate), i64(gs), f32(out_scale),
             stream())
-    if q.dtype == torch.bfloat16 and D in _WINDOW_SIZES and DV % 64 == 0:
+    if q.dtype == torch.bfloat16 and D in _WINDOW_SIZES and DV % 64 == 0 and sm_scale > 0:
         common = (ptr(q), i64(q.stride(0)), ptr(kv_layer), ptr(req_to_token), i64(req_to_token.stride(0)),
                   ptr(st.b_req_idx))
         if st.is_prefill:
@@ -824,7 +830,7 @@ def window_attention(q, kv_layer, req_to_token, st, Hq, Hkv, D, DV, sm_scale, wi
             return out
         if DV in _WINDOW_SIZES:
             keys = min(window + keep, st.max_kv_len) if window > 0 else st.max_kv_len
-            n = gqa_decode_num_splits(T, Hq, Hkv, max(keys, 1))
+            n = window_decode_splits(T, Hq, Hkv, keys)
             po = pl = None
             if n > 1:
                 po = torch.empty(T * Hq * n * DV, dtype=torch.float32, device=q.device)
