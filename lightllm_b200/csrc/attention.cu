@@ -39,16 +39,13 @@ constexpr float kLn2 = 0.6931471805599453f;
 // ---------------------------------------------------------------------------------------
 // DK, DV: key and value size; pool row [Hkv * DK | Hkv * DV].  SPLIT_P (the windowed form): the weights enter P . V as the sum
 // of two bf16 values (high and low part), and `rule` says which positions are seen and which biases the scores get: the kept
-// first positions and the window lie back to back in the key index that is cut into tiles and splits.  gate (or null): head h of request b
-// is multiplied by out_scale * sigmoid(gate[b, h]) when the result is final.
-struct HeadGate {
-  const bf16* gate;
-  int64_t stride;
-  float scale;
-  __device__ __forceinline__ float factor(int b, int h) const {
-    return gate == nullptr ? scale : scale / (1.f + __expf(-__bfloat162float(gate[b * stride + h])));
-  }
-};
+// first positions and the window (or chunk) lie back to back in the key index that is cut into tiles and splits.  gate: factor on
+// the output (OutGate, bf16) when the result is final.
+template <int DV>
+__device__ __forceinline__ float gate_factor(const OutGate& g, int b, int h, int d) {
+  const bf16* p = reinterpret_cast<const bf16*>(g.gate);
+  return p == nullptr ? g.scale : g.scale / (1.f + __expf(-__bfloat162float(p[b * g.stride + (g.elem ? h * DV + d : h)])));
+}
 
 template <int DK, int DV, int STAGES, bool SPLIT_P>
 __global__ void __launch_bounds__(128)
@@ -56,7 +53,7 @@ gqa_decode_kernel(const bf16* __restrict__ q, int64_t q_stride, const bf16* __re
                   const int* __restrict__ req_to_token, int64_t r2t_stride, const int* __restrict__ b_req_idx,
                   const int* __restrict__ b_seq_len, bf16* __restrict__ out, int64_t out_stride,
                   float* __restrict__ part_o, float* __restrict__ part_lse, int Hq, int Hkv, int num_splits,
-                  float scale_log2, const KeyRule rule, const HeadGate gate) {
+                  float scale_log2, const KeyRule rule, const OutGate gate) {
   pdl_wait();
   constexpr int CH = DK / 8, CHV = DV / 8;             // 16-byte chunks per row
   constexpr int TILE_BYTES = 16 * DK * 2;              // 16 tokens' keys
@@ -79,7 +76,7 @@ gqa_decode_kernel(const bf16* __restrict__ q, int64_t q_stride, const bf16* __re
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int g = lane >> 2, tig = lane & 3;
 
-  const int lo = SPLIT_P && rule.window > 0 ? max(0, L - rule.window) : 0;
+  const int lo = SPLIT_P ? rule.first_seen(L - 1) : 0;
   const int kept = SPLIT_P ? min(rule.keep, lo) : 0;
   const int skip = lo - kept;  // key index n >= kept is position n + skip
   const int tiles_total = (L - skip + 15) >> 4;
@@ -170,6 +167,7 @@ gqa_decode_kernel(const bf16* __restrict__ q, int64_t q_stride, const bf16* __re
   float l_run[2] = {0.f, 0.f};
   const float *rel0 = nullptr, *rel1 = nullptr;  // biases of the heads of my two rows
   float far_bias[2] = {0.f, 0.f};
+  const float cap_log2 = SPLIT_P ? rule.cap * kLog2e : 0.f, cap_in = cap_log2 > 0.f ? scale_log2 / cap_log2 : 0.f;
   if (SPLIT_P && rule.rel != nullptr) {
     rel0 = rule.rel + (head0 + min(g, nrows - 1)) * rule.rel_stride;
     rel1 = rule.rel + (head0 + min(g + 8, nrows - 1)) * rule.rel_stride;
@@ -224,7 +222,12 @@ gqa_decode_kernel(const bf16* __restrict__ q, int64_t q_stride, const bf16* __re
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         int pos = p0 + j * 8 + tig * 2 + (e & 1);
-        float v = pos < e0 ? (SPLIT_P ? fmaf(s[j][e], scale_log2, add[j][e]) : s[j][e] * scale_log2) : -INFINITY;
+        float v = s[j][e] * scale_log2;
+        if (SPLIT_P) {
+          if (rule.cap > 0.f) v = cap_log2 * tanh_fast(s[j][e] * cap_in);
+          v += add[j][e];
+        }
+        if (pos >= e0) v = -INFINITY;
         s[j][e] = v;
         mx[e >> 1] = fmaxf(mx[e >> 1], v);
       }
@@ -325,7 +328,7 @@ gqa_decode_kernel(const bf16* __restrict__ q, int64_t q_stride, const bf16* __re
     float val = den > 0.f ? num / den : 0.f;
     int head = head0 + r;
     if (num_splits == 1) {
-      out[(int64_t)b * out_stride + (int64_t)head * DV + d] = __float2bfloat16(val * gate.factor(b, head));
+      out[(int64_t)b * out_stride + (int64_t)head * DV + d] = __float2bfloat16(val * gate_factor<DV>(gate, b, head, d));
     } else {
       int64_t pi = ((int64_t)b * Hq + head) * num_splits + split;
       part_o[pi * DV + d] = val;
@@ -337,7 +340,7 @@ gqa_decode_kernel(const bf16* __restrict__ q, int64_t q_stride, const bf16* __re
 template <int D>
 __global__ void __launch_bounds__(D)
 decode_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_lse, bf16* __restrict__ out,
-                    int64_t out_stride, int Hq, int num_splits, const HeadGate gate) {
+                    int64_t out_stride, int Hq, int num_splits, const OutGate gate) {
   pdl_wait();
   const int bh = blockIdx.x;
   const int b = bh / Hq, h = bh % Hq;
@@ -354,7 +357,7 @@ decode_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ 
       den += w;
     }
   }
-  out[(int64_t)b * out_stride + (int64_t)h * D + d] = __float2bfloat16(den > 0.f ? num / den * gate.factor(b, h) : 0.f);
+  out[(int64_t)b * out_stride + (int64_t)h * D + d] = __float2bfloat16(den > 0.f ? num / den * gate_factor<D>(gate, b, h, d) : 0.f);
 }
 
 // ---------------------------------------------------------------------------------------
@@ -573,7 +576,7 @@ template <int DK, int DV, bool SPLIT_P>
 static int launch_decode(const void* q, int64_t q_stride, const void* kv_layer, const int* req_to_token, int64_t r2t_stride,
                          const int* b_req_idx, const int* b_seq_len, void* out, int64_t out_stride, float* part_o,
                          float* part_lse, int B, int Hq, int Hkv, int num_splits, float sm_scale, const KeyRule& rule,
-                         const HeadGate& gate, cudaStream_t st) {
+                         const OutGate& gate, cudaStream_t st) {
   constexpr int STAGES = decode_stages<DK, DV>();
   const int G = Hq / Hkv;
   const dim3 grid(num_splits, Hkv * ((G + 15) / 16), B);
@@ -604,8 +607,8 @@ LLB_EXPORT int llb_gqa_decode(const void* q, int64_t q_stride, const void* kv_la
   if (B <= 0) return LLB_OK;
   if (Hkv <= 0 || Hq % Hkv != 0 || num_splits < 1) return LLB_ERR_BAD_ARG;
   if (num_splits > 1 && (part_o == nullptr || part_lse == nullptr)) return LLB_ERR_BAD_ARG;
-  const HeadGate none{nullptr, 0, 1.f};
-  const KeyRule all{0, 0, nullptr, 0, 0};
+  const OutGate none{nullptr, 0, 1.f, 0};
+  const KeyRule all{};
   if (D == 128)
     return launch_decode<128, 128, false>(q, q_stride, kv_layer, req_to_token, r2t_stride, b_req_idx, b_seq_len, out,
                                           out_stride, part_o, part_lse, B, Hq, Hkv, num_splits, sm_scale, all, none, st);
@@ -615,20 +618,24 @@ LLB_EXPORT int llb_gqa_decode(const void* q, int64_t q_stride, const void* kv_la
   return LLB_ERR_UNSUPPORTED;
 }
 
-// The windowed form: key size dk and value size dv (64, 128, 192 or 256), pool rows [Hkv * dk | Hkv * dv], window (0: none),
-// the first `keep` positions always seen, biases by distance rel [Hq, far + 1] (or null; see KeyRule), gate [B, >= Hq] (or null): head h of the output times out_scale * sigmoid(gate).  part_o: fp32 [B, Hq, num_splits, dv].
+// The windowed form: key size dk and value size dv (64, 128, 192 or 256), pool rows [Hkv * dk | Hkv * dv], window or chunk (0: none),
+// the first `keep` positions always seen, biases by distance rel [Hq, far + 1] (or null), cap on the scores (0: none; see KeyRule),
+// gate [B, >= Hq], with gate_elem [B, >= Hq * dv], or null: the output times out_scale * sigmoid(gate).  part_o: fp32
+// [B, Hq, num_splits, dv].
 LLB_EXPORT int llb_window_gqa_decode(const void* q, int64_t q_stride, const void* kv_layer, const int* req_to_token,
                                      int64_t r2t_stride, const int* b_req_idx, const int* b_seq_len, void* out,
                                      int64_t out_stride, float* part_o, float* part_lse, int B, int Hq, int Hkv, int dk,
                                      int dv, int num_splits, float sm_scale, int window, int keep, const float* rel,
-                                     int far, int64_t rel_stride, const void* gate, int64_t gate_stride, float out_scale, cudaStream_t st) {
+                                     int far, int64_t rel_stride, int chunk, float cap, const void* gate,
+                                     int64_t gate_stride, int gate_elem, float out_scale, cudaStream_t st) {
   if (B <= 0) return LLB_OK;
   if (Hkv <= 0 || Hq % Hkv != 0 || num_splits < 1 || window < 0 || keep < 0 || (rel != nullptr && far < 0) ||
+      chunk < 0 || (chunk > 0 && window > 0) || !(cap >= 0.f) ||
       (q_stride % 8) || ((uintptr_t)q & 15))
     return LLB_ERR_BAD_ARG;
   if (num_splits > 1 && (part_o == nullptr || part_lse == nullptr)) return LLB_ERR_BAD_ARG;
-  const HeadGate g{(const bf16*)gate, gate_stride, out_scale};
-  const KeyRule rule{window, keep, rel, far, rel_stride};
+  const OutGate g{gate, gate_stride, out_scale, gate_elem};
+  const KeyRule rule{window, keep, rel, far, rel_stride, chunk, cap};
 #define LLB_WINDOW_DECODE(DK, DV)                                                                                        \
   if (dk == DK && dv == DV)                                                                                              \
     return launch_decode<DK, DV, true>(q, q_stride, kv_layer, req_to_token, r2t_stride, b_req_idx, b_seq_len, out,       \

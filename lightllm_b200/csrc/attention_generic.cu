@@ -1,6 +1,6 @@
 // Paged causal attention for the layer shapes the tensor-core kernels do not cover: any head size up to
 // 256 (Gemma 256, Phi-3 96, StableLM 80 ...; up to 512 in the form with its own value size, in bf16 or fp32),
-// sliding windows (with kept first positions), ALiBi slopes, tables of biases by distance, logit soft-capping, attention sinks and a sigmoid output gate per head.  One CTA per (query token, query head); its four warps stride over the keys, each
+// sliding windows (with kept first positions), chunks of positions, ALiBi slopes, tables of biases by distance, logit soft-capping, attention sinks and a sigmoid output gate (per head or per element).  One CTA per (query token, query head); its four warps stride over the keys, each
 // keeps an online-softmax state with the head vector spread over the lanes, and the states are merged
 // in shared memory.  Prefill and decode use the same kernel: a query is described by its position and
 // the request row it belongs to.
@@ -22,16 +22,14 @@ __device__ __forceinline__ float exp_for(float v, const float*) { return expf(v)
 __device__ __forceinline__ float exp_for(float v, const bf16*) { return __expf(v); }
 }  // namespace
 
-// EPL: elements per lane (sizes up to 32 * EPL).  gate [T, >= Hq] (row pitch gate_stride) or null: head h of the output
-// is multiplied by out_scale * sigmoid(gate[t, h]).
+// EPL: elements per lane (sizes up to 32 * EPL).  gate: factor on the output (OutGate, format E).
 template <typename E, int EPL>
 __global__ void __launch_bounds__(GEN_WARPS * 32)
 attn_generic_kernel(const E* __restrict__ q, int64_t q_stride, const E* __restrict__ kv,
                     const int* __restrict__ req_to_token, int64_t r2t_stride, const int* __restrict__ b_req_idx,
                     const int* __restrict__ pos, const int* __restrict__ batch_of, E* __restrict__ out,
-                    int64_t out_stride, int Hq, int Hkv, int D, int DV, float sm_scale, const KeyRule rule, float softcap,
-                    const float* __restrict__ alibi, const float* __restrict__ sinks, const E* __restrict__ gate,
-                    int64_t gate_stride, float out_scale) {
+                    int64_t out_stride, int Hq, int Hkv, int D, int DV, float sm_scale, const KeyRule rule,
+                    const float* __restrict__ alibi, const float* __restrict__ sinks, const OutGate gate) {
   const int t = blockIdx.x, h = blockIdx.y;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int b = batch_of ? batch_of[t] : t;
@@ -48,7 +46,7 @@ attn_generic_kernel(const E* __restrict__ q, int64_t q_stride, const E* __restri
     acc[e] = 0.f;
   }
   float m = -INFINITY, l = 0.f;
-  const int j0 = (rule.window > 0 && qpos - rule.window + 1 > 0) ? qpos - rule.window + 1 : 0;
+  const int j0 = rule.first_seen(qpos);
   const int kept = min(rule.keep, j0), n = kept + qpos + 1 - j0;  // kept first positions, then the window
   const float slope = alibi ? alibi[h] : 0.f;
   const float* rel = rule.rel ? rule.rel + h * rule.rel_stride : nullptr;
@@ -62,7 +60,7 @@ attn_generic_kernel(const E* __restrict__ q, int64_t q_stride, const E* __restri
       if (d < D) s += qv[e] * to_f(kr[d]);
     }
     s = warp_sum(s);
-    if (softcap > 0.f) s = softcap * tanhf(s / softcap);
+    if (rule.cap > 0.f) s = rule.cap * tanhf(s / rule.cap);
     s += slope * (float)(j - qpos);
     if (rel) s += rel[min(qpos - j, rule.far)];
     const float mn = fmaxf(m, s);
@@ -101,12 +99,16 @@ attn_generic_kernel(const E* __restrict__ q, int64_t q_stride, const E* __restri
 #pragma unroll
       for (int e = 0; e < EPL; ++e) o[e] += s_acc[w][lane + e * 32] * c;
     }
-    float inv = L > 0.f ? out_scale / L : 0.f;
-    if (gate != nullptr) inv /= 1.f + exp_for(-to_f(gate[(int64_t)t * gate_stride + h]), q);
+    float inv = L > 0.f ? gate.scale / L : 0.f;
+    const E* gt = gate.gate != nullptr ? (const E*)gate.gate + (int64_t)t * gate.stride : nullptr;
+    if (gt != nullptr && !gate.elem) inv /= 1.f + exp_for(-to_f(gt[h]), q);
 #pragma unroll
     for (int e = 0; e < EPL; ++e) {
       int d = lane + e * 32;
-      if (d < DV) from_f(o[e] * inv, &out[(int64_t)t * out_stride + (int64_t)h * DV + d]);
+      if (d >= DV) continue;
+      float r = o[e] * inv;
+      if (gt != nullptr && gate.elem) r /= 1.f + exp_for(-to_f(gt[h * DV + d]), q);
+      from_f(r, &out[(int64_t)t * out_stride + (int64_t)h * DV + d]);
     }
   }
 }
@@ -120,27 +122,31 @@ LLB_EXPORT int llb_attn_generic(const void* q, int64_t q_stride, const void* kv_
   dim3 grid(T, Hq);
   attn_generic_kernel<bf16, GEN_MAX_EPL><<<grid, GEN_WARPS * 32, 0, st>>>(
       (const bf16*)q, q_stride, (const bf16*)kv_layer, req_to_token, r2t_stride, b_req_idx, pos, batch_of, (bf16*)out,
-      out_stride, Hq, Hkv, D, D, sm_scale, KeyRule{window, 0, nullptr, 0, 0}, softcap, alibi_slopes, sinks, nullptr, 0, 1.f);
+      out_stride, Hq, Hkv, D, D, sm_scale, KeyRule{window, 0, nullptr, 0, 0, 0, softcap}, alibi_slopes, sinks,
+      OutGate{nullptr, 0, 1.f, 0});
   LLB_LAUNCH_CHECK();
   return LLB_OK;
 }
 
-// The form with a value size of its own, kept first positions, biases by distance (see KeyRule), an output gate per head, and
-// fp32 (dt 0) beside bf16 (dt 1).
+// The form with a value size of its own, chunks, kept first positions, biases by distance, capped scores (see KeyRule), an output
+// gate per head or (gate_elem) per element, and fp32 (dt 0) beside bf16 (dt 1).
 LLB_EXPORT int llb_attn_generic_kv(const void* q, int dt, int64_t q_stride, const void* kv_layer, const int* req_to_token,
                                    int64_t r2t_stride, const int* b_req_idx, const int* pos, const int* batch_of,
                                    void* out, int64_t out_stride, int T, int Hq, int Hkv, int D, int DV, float sm_scale,
-                                   int window, int keep, const float* rel, int far, int64_t rel_stride,
-                                   const void* gate, int64_t gate_stride, float out_scale, cudaStream_t st) {
+                                   int window, int keep, const float* rel, int far, int64_t rel_stride, int chunk,
+                                   float cap, const void* gate, int64_t gate_stride, int gate_elem, float out_scale,
+                                   cudaStream_t st) {
   if (T <= 0) return LLB_OK;
-  if (window < 0 || keep < 0 || (rel != nullptr && far < 0)) return LLB_ERR_BAD_ARG;
-  const KeyRule rule{window, keep, rel, far, rel_stride};
+  if (window < 0 || keep < 0 || (rel != nullptr && far < 0) || chunk < 0 || (chunk > 0 && window > 0) || !(cap >= 0.f))
+    return LLB_ERR_BAD_ARG;
+  const KeyRule rule{window, keep, rel, far, rel_stride, chunk, cap};
+  const OutGate og{gate, gate_stride, out_scale, gate_elem};
   if (D <= 0 || DV <= 0 || D > 512 || DV > 512 || Hkv <= 0 || Hq % Hkv != 0 || Hq > 65535) return LLB_ERR_UNSUPPORTED;
   const dim3 grid(T, Hq);
 #define LLB_GENERIC(E, EPL)                                                                                           \
   attn_generic_kernel<E, EPL><<<grid, GEN_WARPS * 32, 0, st>>>(                                                       \
       (const E*)q, q_stride, (const E*)kv_layer, req_to_token, r2t_stride, b_req_idx, pos, batch_of, (E*)out,         \
-      out_stride, Hq, Hkv, D, DV, sm_scale, rule, 0.f, nullptr, nullptr, (const E*)gate, gate_stride, out_scale)
+      out_stride, Hq, Hkv, D, DV, sm_scale, rule, nullptr, nullptr, og)
   if (D <= 128 && DV <= 128) {
     if (dt == 0)
       LLB_GENERIC(float, 4);
@@ -208,8 +214,8 @@ LLB_EXPORT int llb_rope_kv_scatter_generic(void* qkv, void* kv_layer, const floa
   return LLB_OK;
 }
 
-// Per-head RMS norm of q and k over the first `dim` of their D elements (a null weight is all ones), rotary positions on the
-// first rot_dim, and the cache write, for layers whose value size DV differs from the key size D.  A norm without a weight
+// Per-head RMS norm of q and k over the first `dim` of their D elements (a null weight is all ones; norm 0: none), a factor per
+// query head (q_scale fp32 [Hq] or null), rotary positions on the first rot_dim, and the cache write, for layers whose value size DV differs from the key size D.  A norm without a weight
 // commutes with the rotation.  qkv row: [Hq * D | Hkv * D | Hkv * DV]; q is rewritten in place, K and V go to kv_layer[slot].
 // Hkv = 0: queries only (a layer that reads another layer's cache).  Sizes are multiples of 8; a group of 2^k lanes works on one head, a lane
 // on 8 elements of it (NIT times, 8 * lanes apart); rotation partners meet in shared memory.
@@ -231,7 +237,7 @@ __global__ void __launch_bounds__(256)
 qk_norm_rope_scatter_kernel(E* __restrict__ qkv, int64_t qkv_stride, E* __restrict__ kv_layer,
                             const float* __restrict__ cos_t, const float* __restrict__ sin_t, const int* __restrict__ pos,
                             const int* __restrict__ slot, const float* __restrict__ qw, const float* __restrict__ kw,
-                            float eps, unsigned items, int Hq, int Hkv, int D, int dim, int DV, int rot_dim, int lanes_log2) {
+                            float eps, int norm, const float* __restrict__ q_scale, unsigned items, int Hq, int Hkv, int D, int dim, int DV, int rot_dim, int lanes_log2) {
   pdl_wait();
   extern __shared__ float srow[];  // [groups][rot_dim]
   const int lanes = 1 << lanes_log2;
@@ -266,7 +272,8 @@ qk_norm_rope_scatter_kernel(E* __restrict__ qkv, int64_t qkv_stride, E* __restri
     }
   }
   for (int o = lanes >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-  const float inv = rsqrtf(ss / (float)dim + eps);
+  float inv = norm ? rsqrtf(ss / (float)dim + eps) : 1.f;
+  if (q_scale != nullptr && head < Hq) inv *= q_scale[head];
   const float* w = head < Hq ? qw : kw;
   if (qk) {
 #pragma unroll
@@ -325,14 +332,14 @@ qk_norm_rope_scatter_kernel(E* __restrict__ qkv, int64_t qkv_stride, E* __restri
   }
 }
 
-// qw, kw: fp32 [D], zero beyond dim, or null.  dt: 0 = fp32, 1 = bf16.
+// qw, kw: fp32 [D], zero beyond dim, or null.  norm 0: no norm (qw, kw null).  q_scale: fp32 [Hq] or null.  dt: 0 = fp32, 1 = bf16.
 LLB_EXPORT int llb_qk_norm_rope_scatter(void* qkv, int dt, int64_t qkv_stride, void* kv_layer, const float* cos_t,
                                         const float* sin_t, const int* pos, const int* slot, const float* qw,
-                                        const float* kw, float eps, int T, int Hq, int Hkv, int D, int dim, int DV,
+                                        const float* kw, float eps, int norm, const float* q_scale, int T, int Hq, int Hkv, int D, int dim, int DV,
                                         int rot_dim, cudaStream_t st) {
   if (T <= 0) return LLB_OK;
   if (D <= 0 || (D % 8) || DV <= 0 || (DV % 8) || D > 512 || dim <= 0 || dim > D || (rot_dim & 1) || rot_dim > dim ||
-      (qkv_stride % 8) || Hq < 0 || Hkv < 0)
+      (qkv_stride % 8) || Hq < 0 || Hkv < 0 || (!norm && (qw != nullptr || kw != nullptr)))
     return LLB_ERR_UNSUPPORTED;
   int lg = 2;
   while (lg < 5 && (8 << lg) < D) ++lg;
@@ -343,7 +350,7 @@ LLB_EXPORT int llb_qk_norm_rope_scatter(void* qkv, int dt, int64_t qkv_stride, v
   const dim3 grid((unsigned)cdiv64(items, groups));
 #define LLB_QK(E, NIT, FAST)                                                                                              \
   launch_pdl(qk_norm_rope_scatter_kernel<E, NIT, FAST>, grid, dim3(256), FAST ? 0 : smem, st, (E*)qkv, qkv_stride,        \
-             (E*)kv_layer, cos_t, sin_t, pos, slot, qw, kw, eps, (unsigned)items, Hq, Hkv, D, dim, DV, rot_dim, lg)
+             (E*)kv_layer, cos_t, sin_t, pos, slot, qw, kw, eps, norm, q_scale, (unsigned)items, Hq, Hkv, D, dim, DV, rot_dim, lg)
   if (D <= 256 && rot_dim > 0 && rot_dim % 16 == 0) {
     if (dt == 0)
       LLB_QK(float, 1, true);

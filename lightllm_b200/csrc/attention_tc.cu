@@ -1,7 +1,7 @@
 // Prefill attention on the 5th-generation tensor cores (tcgen05 + tensor memory), causal, varlen, aware of an already cached
 // prefix, K/V read through the token-granular slot table of the KV pool.  Head size 128, and a windowed form with key sizes
-// up to 256, any multiple of 64 as value size, kept first positions, biases by distance, and a sigmoid gate per head on the
-// output.
+// up to 256, any multiple of 64 as value size, chunks of positions, kept first positions, biases by distance, soft-capped scores, and
+// a sigmoid gate on the output.
 //
 // One CTA computes 128 query rows of one (request, query head).  Per 128-key tile (64 keys for key sizes above 128):
 //   S  = Q . K^T            tcgen05.mma into one of two tensor-memory buffers
@@ -60,22 +60,47 @@ __device__ __forceinline__ float ex2_fast(float x) {  // 2^x, one MUFU instructi
   return y;
 }
 
+// v[e] (fp32 bits) = top * tanh(v[e] * in).  Where all of a warp's arguments are below 1/4 the Taylor series of tanh_fast, else
+// top - 2 top / (1 + e^2x), whose absolute error (a few 1e-7 top) is that of rounding values of the cap's size.
+template <int N>
+__device__ __forceinline__ void cap_scores(uint32_t* v, float in, float top) {
+  float big = 0.f;
+#pragma unroll
+  for (int e = 0; e < N; ++e) big = fmaxf(big, fabsf(__uint_as_float(v[e])));
+  if (__all_sync(0xffffffffu, big * in < 0.25f)) {
+    // top (x - x^3/3 + 2x^5/15 - 17x^7/315 + 62x^9/2835), in powers of the score itself
+    const float i2 = in * in, k1 = top * in;
+    const float c3 = -1.f / 3.f * i2, c5 = 2.f / 15.f * i2 * i2, c7 = -17.f / 315.f * i2 * i2 * i2,
+                c9 = 62.f / 2835.f * i2 * i2 * i2 * i2;
+#pragma unroll
+    for (int e = 0; e < N; ++e) {
+      const float x = __uint_as_float(v[e]), x2 = x * x;
+      v[e] = __float_as_uint(x * k1 * fmaf(x2, fmaf(x2, fmaf(x2, fmaf(x2, c9, c7), c5), c3), 1.f));
+    }
+  } else {
+    const float to2 = 2.f * kLog2e * in;
+#pragma unroll
+    for (int e = 0; e < N; ++e)
+      v[e] = __float_as_uint(fmaf(-2.f * top, __fdividef(1.f, 1.f + ex2_fast(__uint_as_float(v[e]) * to2)), top));
+  }
+}
+
 __device__ __forceinline__ uint32_t pack2(float a, float b) {
   const bf162 h = __floats2bfloat162_rn(a, b);
   return *reinterpret_cast<const uint32_t*>(&h);
 }
 
 // DK, DV: key size and the value columns of one CTA (a wider value head is shared out over CTAs: v_blocks per head).
-// rule.window: a query sees its own position and the window - 1 before it (0: all before it).  SPLIT_P: the weights enter P . V
-// as the sum of two bf16 tiles.  EXT: positions below rule.keep are seen at any distance (the tiles that hold them come ahead of
-// the window's), and scores get the biases of rule.rel; rule.window is the window in either form.  gate (or null): head h of row t is multiplied by out_scale * sigmoid(gate[t, h]).
+// rule.window, rule.chunk: the positions a query sees (see KeyRule).  SPLIT_P: the weights enter P . V as the sum of two bf16
+// tiles.  EXT: positions below rule.keep are seen at any distance (the tiles that hold them come ahead of the window's), scores
+// are capped (rule.cap) and get the biases of rule.rel.  gate: factor on the output (OutGate, bf16).
 template <int DK, int DV, int BN, bool SPLIT_P, bool EXT>
 __global__ void __launch_bounds__(THREADS, 1)
 gqa_prefill_tc_kernel(const bf16* __restrict__ q, int64_t q_stride, const bf16* __restrict__ kv_layer,
                       const int* __restrict__ req_to_token, int64_t r2t_stride, const int* __restrict__ b_req_idx,
                       const int* __restrict__ cu_q, const int* __restrict__ b_ready_len, bf16* __restrict__ out,
                       int64_t out_stride, int Hq, int Hkv, float scale_log2, int v_blocks, const KeyRule rule,
-                      const bf16* __restrict__ gate, int64_t gate_stride, float out_scale) {
+                      const OutGate gate) {
   using L = PrefillLayout<DK, DV, BN, SPLIT_P>;
   constexpr int HK = BN / 2;   // keys of a score tile per softmax thread
   constexpr int OC = DV / 2;   // value columns per softmax thread
@@ -103,8 +128,7 @@ gqa_prefill_tc_kernel(const bf16* __restrict__ q, int64_t q_stride, const bf16* 
   const int req = LLB_CHECK_REQ(b_req_idx[b]);
   const int rows_valid = min(BM, q_len - q0);
   const int kv_end = ready + q0 + rows_valid;  // exclusive bound on the keys any row of this tile may see
-  const int window = rule.window;
-  const int kv0 = window > 0 ? max(0, ready + q0 - window + 1) : 0;
+  const int kv0 = rule.first_seen(ready + q0);
   const int kept = EXT ? min(rule.keep, kv0) : 0;      // kept positions ahead of the window
   const int kept_tiles = EXT ? (kept + BN - 1) / BN : 0;
   const int n_tiles = kept_tiles + (kv_end - kv0 + BN - 1) / BN;
@@ -279,6 +303,7 @@ gqa_prefill_tc_kernel(const bf16* __restrict__ q, int64_t q_stride, const bf16* 
     const int half = (warp - 2) >> 2;
     const int erow = lane_grp * 32 + lane;
     const int prow = ready + q0 + erow;  // absolute position of this row's token
+    const int row_first = rule.first_seen(prow);
     const uint32_t t_lane = tmem_base + ((uint32_t)(lane_grp * 32) << 16);
     const uint32_t t_s = t_lane + half * HK, t_o = t_lane + 2 * BN + half * OC;
     uint8_t* p_tile = smem_gen + L::OFF_P;
@@ -297,20 +322,24 @@ gqa_prefill_tc_kernel(const bf16* __restrict__ q, int64_t q_stride, const bf16* 
       for (int c = 0; c < HK; c += 32) tmem_ld_32x32(t_s + (j & 1) * BN + c, sr + c);
       tmem_wait_ld();
       const int lim = min(prow, tile_bound(j) - 1) - kt;  // my columns lo..lim (and those below `first`) are visible to this row
-      const int lo = window > 0 ? prow - window + 1 - kt : 0;
+      const int lo = row_first - kt;
       const int first = EXT ? rule.keep - kt : 0;
       auto seen = [&](int c) { return c <= lim && (c >= lo || (EXT && c < first)); };
       // whole tile (every tile but those at the diagonal and the edges)
       const bool all_visible = lim >= HK - 1 && (lo <= 0 || (EXT && first >= HK));
       float to_log2 = scale_log2, shift = 0.f;  // score in log2 units = sr * to_log2 + shift
+      if (EXT && rule.cap > 0.f) {
+        cap_scores<HK>(sr, scale_log2 * (1.f / kLog2e) / rule.cap, rule.cap * kLog2e);
+        to_log2 = 1.f;
+      }
       if (EXT && rel != nullptr) {
         const int dist = prow - kt;  // of my first column; the last one is HK - 1 nearer
         if (dist - (HK - 1) >= rule.far) {
           shift = far_bias;
         } else {  // columns of a negative distance are not seen, whatever they are added
           const float* at = rel + max(dist, 0);
+          const float scale = to_log2 * (1.f / kLog2e);
           to_log2 = kLog2e;
-          const float scale = scale_log2 * (1.f / kLog2e);
 #pragma unroll
           for (int e = 0; e < HK; ++e) sr[e] = __float_as_uint(fmaf(__uint_as_float(sr[e]), scale, at[-e]));
         }
@@ -379,9 +408,10 @@ gqa_prefill_tc_kernel(const bf16* __restrict__ q, int64_t q_stride, const bf16* 
     x[half * 128 + erow] = l_run;
     asm volatile("bar.sync 1, 256;" ::: "memory");
     const float l_tot = l_run + x[(half ^ 1) * 128 + erow];
-    float inv = l_tot > 0.f ? out_scale / l_tot : 0.f;
-    if (gate != nullptr && erow < rows_valid)
-      inv = __fdividef(inv, 1.f + __expf(-__bfloat162float(gate[(int64_t)(q_begin + q0 + erow) * gate_stride + h])));
+    float inv = l_tot > 0.f ? gate.scale / l_tot : 0.f;
+    const bf16* gt = reinterpret_cast<const bf16*>(gate.gate);
+    if (gt != nullptr && !gate.elem && erow < rows_valid)
+      inv = __fdividef(inv, 1.f + __expf(-__bfloat162float(gt[(int64_t)(q_begin + q0 + erow) * gate.stride + h])));
     // output: every warp parks its 32 rows x OC columns in its own part of the (now idle) Q / P buffers and
     // writes whole lines
     constexpr int PITCH = OC * 2 + 16, SEGS = OC / 8;
@@ -406,9 +436,19 @@ gqa_prefill_tc_kernel(const bf16* __restrict__ q, int64_t q_stride, const bf16* 
     for (int i = 0; i < SEGS; ++i) {
       const int id = i * 32 + lane, r = id / SEGS, seg = id % SEGS;
       const int lr = lane_grp * 32 + r;
-      if (lr < rows_valid)
-        *reinterpret_cast<uint4*>(out + (int64_t)(q_begin + q0 + lr) * out_stride + ((int64_t)h * v_blocks + vb) * DV +
-                                  half * OC + seg * 8) = *reinterpret_cast<const uint4*>(stg + r * PITCH + seg * 16);
+      if (lr < rows_valid) {
+        const int64_t row = q_begin + q0 + lr, col = ((int64_t)h * v_blocks + vb) * DV + half * OC + seg * 8;
+        bf16x8 v = *reinterpret_cast<const bf16x8*>(stg + r * PITCH + seg * 16);
+        if (gt != nullptr && gate.elem) {
+          float f[8], gv[8];
+          unpack8(v, f);
+          unpack8(*reinterpret_cast<const bf16x8*>(gt + row * gate.stride + col), gv);
+#pragma unroll
+          for (int e = 0; e < 8; ++e) f[e] = __fdividef(f[e], 1.f + __expf(-gv[e]));
+          v = pack8(f);
+        }
+        *reinterpret_cast<bf16x8*>(out + row * out_stride + col) = v;
+      }
     }
     tc_fence_before();
   }
@@ -424,8 +464,8 @@ gqa_prefill_tc_kernel(const bf16* __restrict__ q, int64_t q_stride, const bf16* 
 template <int DK, int DV, int BN, bool SPLIT_P, bool EXT>
 int launch_tc(const bf16* q, int64_t q_stride, const bf16* kv_layer, const int* req_to_token, int64_t r2t_stride,
               const int* b_req_idx, const int* cu_q, const int* b_ready_len, bf16* out, int64_t out_stride, int B,
-              int max_q_len, int Hq, int Hkv, float sm_scale, int v_blocks, const KeyRule& rule, const bf16* gate,
-              int64_t gate_stride, float out_scale, cudaStream_t st) {
+              int max_q_len, int Hq, int Hkv, float sm_scale, int v_blocks, const KeyRule& rule, const OutGate& gate,
+              cudaStream_t st) {
   using L = PrefillLayout<DK, DV, BN, SPLIT_P>;
   static_assert(L::BYTES <= 227 * 1024, "shared memory");
   static DeviceOnce configured;
@@ -438,7 +478,7 @@ int launch_tc(const bf16* q, int64_t q_stride, const bf16* kv_layer, const int* 
   const dim3 grid((max_q_len + BM - 1) / BM, Hq * v_blocks, B);
   gqa_prefill_tc_kernel<DK, DV, BN, SPLIT_P, EXT><<<grid, THREADS, L::BYTES, st>>>(
       q, q_stride, kv_layer, req_to_token, r2t_stride, b_req_idx, cu_q, b_ready_len, out, out_stride, Hq, Hkv,
-      sm_scale * kLog2e, v_blocks, rule, gate, gate_stride, out_scale);
+      sm_scale * kLog2e, v_blocks, rule, gate);
   LLB_LAUNCH_CHECK();
   return LLB_OK;
 }
@@ -460,30 +500,34 @@ LLB_EXPORT int llb_gqa_prefill_tc(const void* q, int64_t q_stride, const void* k
   if (!(sm_scale > 0.f) || Hkv <= 0 || Hq % Hkv != 0 || (q_stride % 8) || (out_stride % 8) || ((uintptr_t)q & 15) || ((uintptr_t)out & 15))
     return LLB_ERR_BAD_ARG;
   return launch_tc<128, 128, 128, false, false>((const bf16*)q, q_stride, (const bf16*)kv_layer, req_to_token, r2t_stride, b_req_idx,
-                                         cu_q, b_ready_len, (bf16*)out, out_stride, B, max_q_len, Hq, Hkv, sm_scale, 1, KeyRule{0, 0, nullptr, 0, 0},
-                                         nullptr, 0, 1.f, st);
+                                         cu_q, b_ready_len, (bf16*)out, out_stride, B, max_q_len, Hq, Hkv, sm_scale, 1, KeyRule{},
+                                         OutGate{nullptr, 0, 1.f, 0}, st);
 }
 
-// Key size dk (64, 128, 192, 256), value size dv (a multiple of 64), window (0: none), first `keep` positions always seen,
-// biases by distance rel [Hq, far + 1] (or null; see KeyRule): pool rows [Hkv * dk | Hkv * dv], q
-// [T, >= Hq * dk], out [T, >= Hq * dv].  gate [T, >= Hq] (or null): head h of the output times out_scale * sigmoid(gate).
+// Key size dk (64, 128, 192, 256), value size dv (a multiple of 64), window or chunk (0: none), first `keep` positions always seen,
+// biases by distance rel [Hq, far + 1] (or null), cap on the scores (0: none; see KeyRule): pool rows [Hkv * dk | Hkv * dv], q
+// [T, >= Hq * dk], out [T, >= Hq * dv].  gate [T, >= Hq], with gate_elem [T, >= Hq * dv], or null: the output times
+// out_scale * sigmoid(gate).
 LLB_EXPORT int llb_window_gqa_prefill_tc(const void* q, int64_t q_stride, const void* kv_layer, const int* req_to_token,
                                          int64_t r2t_stride, const int* b_req_idx, const int* cu_q, const int* b_ready_len,
                                          void* out, int64_t out_stride, int B, int max_q_len, int Hq, int Hkv, int dk,
                                          int dv, float sm_scale, int window, int keep, const float* rel, int far,
-                                         int64_t rel_stride, const void* gate, int64_t gate_stride, float out_scale, cudaStream_t st) {
+                                         int64_t rel_stride, int chunk, float cap, const void* gate, int64_t gate_stride,
+                                         int gate_elem, float out_scale, cudaStream_t st) {
   if (B <= 0 || max_q_len <= 0) return LLB_OK;
   if (!(sm_scale > 0.f) || Hkv <= 0 || Hq % Hkv != 0 || (q_stride % 8) || (out_stride % 8) || ((uintptr_t)q & 15) || ((uintptr_t)out & 15) ||
-      window < 0 || keep < 0 || (rel != nullptr && far < 0) || dv <= 0)
+      window < 0 || keep < 0 || (rel != nullptr && far < 0) || dv <= 0 || chunk < 0 || (chunk > 0 && window > 0) || !(cap >= 0.f) ||
+      (gate_elem && ((gate_stride % 8) || ((uintptr_t)gate & 15))))
     return LLB_ERR_BAD_ARG;
-  const KeyRule rule{window, keep, rel, far, rel_stride};
-  const bool ext = (window > 0 && keep > 0) || rel != nullptr;
+  const KeyRule rule{window, keep, rel, far, rel_stride, chunk, cap};
+  const OutGate og{gate, gate_stride, out_scale, gate_elem};
+  const bool ext = ((window > 0 || chunk > 0) && keep > 0) || rel != nullptr || cap > 0.f;
   if ((dv % 64) || (dk != 64 && dk != 128 && dk != 192 && dk != 256) || Hq * (dv / 64) > 65535 || B > 65535)
     return LLB_ERR_UNSUPPORTED;
 #define LLB_WINDOW_TC(DK, DV, BN)                                                                                         \
   return (ext ? launch_tc<DK, DV, BN, true, true> : launch_tc<DK, DV, BN, true, false>)(                                  \
       (const bf16*)q, q_stride, (const bf16*)kv_layer, req_to_token, r2t_stride, b_req_idx, cu_q, b_ready_len, (bf16*)out, \
-      out_stride, B, max_q_len, Hq, Hkv, sm_scale, dv / DV, rule, (const bf16*)gate, gate_stride, out_scale, st)
+      out_stride, B, max_q_len, Hq, Hkv, sm_scale, dv / DV, rule, og, st)
   if (dv % 128 == 0) {
     if (dk == 64) LLB_WINDOW_TC(64, 128, 128);
     if (dk == 128) LLB_WINDOW_TC(128, 128, 128);

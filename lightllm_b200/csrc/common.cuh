@@ -187,15 +187,31 @@ __device__ __forceinline__ float tanh_fast(float x) {
   return fabsf(x) < 0.25f ? small : big;
 }
 
-// Which keys a causal query sees and what its scores get added: position p sees j <= p with p - j < window (window 0: all) or
-// j < keep; key j's score of head h gets rel[h, min(p - j, far)] (natural units; fp32, heads rel_stride apart, or null).  Every
-// head's entries may also be read kRelPad places before 0 and after `far` (those beyond `far` repeat it).
+// Which keys a causal query sees and what becomes of its scores: position p sees j <= p with p - j < window (window 0: all), or in
+// the same chunk of positions counted from 0 (chunk > 0, without a window), or j < keep.  A score s (scaled) becomes
+// cap tanh(s / cap) when cap > 0, then key j's score of head h gets rel[h, min(p - j, far)] added (natural units; fp32, heads
+// rel_stride apart, or null).  Every head's entries may also be read kRelPad places before 0 and after `far` (those beyond `far`
+// repeat it).
 constexpr int kRelPad = 64;
 struct KeyRule {
   int window, keep;
   const float* rel;
   int far;
   int64_t rel_stride;
+  int chunk;
+  float cap;
+  // first position that p sees (besides the kept ones)
+  __host__ __device__ __forceinline__ int first_seen(int p) const {
+    if (window > 0) return p - window + 1 > 0 ? p - window + 1 : 0;
+    return chunk > 0 ? p - p % chunk : 0;
+  }
+};
+// Sigmoid gate on attention outputs: one value per row and head, or (elem) one per row and output element, at gate[row * stride].
+struct OutGate {
+  const void* gate;  // or null
+  int64_t stride;
+  float scale;       // factor on every output
+  int elem;
 };
 
 // Block-wide sum; `red` is a shared array of >= 33 floats. All threads get the result.
