@@ -14,3 +14,4 @@ from . import gemma4  # noqa: F401
 from . import taduzen  # noqa: F401
 from . import libulorn  # noqa: F401
 from . import katarax  # noqa: F401
+from . import silupel  # noqa: F401

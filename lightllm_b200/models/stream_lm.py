@@ -99,11 +99,11 @@ class StreamLM(TransformerLM):
     def _graph_decode_splits(self, bucket):
         return 1        # per layer, from its window (ops.window_attention, ops.mla.latent_attention)
 
-    def _reduced(self, a, w):
-        """a . w^T, summed over the tensor-parallel ranks."""
+    def _reduced(self, a, w, bias=None):
+        """a . w^T (+ bias, of one rank), summed over the tensor-parallel ranks."""
         if self.tp.size == 1:
-            return ops.gemm(a, w)
-        y = ops.gemm(a, w, epi="f32")
+            return ops.gemm(a, w, bias=bias)
+        y = ops.gemm(a, w, epi="f32", bias=bias)
         self.tp.all_reduce_(y)
         return y
 

@@ -728,16 +728,53 @@ def add_rms_(x, y, w, width: int, eps: float, dtype, next_w=None):
     return h
 
 
-def qk_norm_rope_scatter_(qkv, kv_layer, cos, sin, pos, slot, q_w, k_w, eps, Hq, Hkv, D, dim, DV, rot_dim):
+class TokenShift:
+    """Shift of a norm's output towards the row of the token before (`norm_shift`): h = n + (n_before - n) * mu, element by element;
+    mu fp32 [W]; state fp32 [slots, W] (any row pitch) keeps the n of every request's last token."""
+
+    def __init__(self, mu, state, st):
+        self.mu, self.state, self.st = mu, state, st
+
+
+def norm_shift(x, y, w, width: int, eps: float, dtype, shift=None, ids=None, centred=True):
+    """(x', h): x' = x + y (fp32 stream; x None: y; ids given: y is a table and row t is y[ids[t]]), h = norm(x') * w in `dtype`, the
+    statistics taken over the first `width` columns (centred: layer norm without a bias, else RMS norm), moved by `shift`
+    (`TokenShift` or None).  x may be changed in place."""
+    if not _is_cuda(y):
+        return ref.norm_shift(x, y, w, width, eps, dtype, shift, ids, centred)
+    T = y.shape[0] if ids is None else ids.shape[0]
+    W = y.shape[1]
+    prompt = shift is not None and shift.st.is_prefill
+    assert y.is_contiguous() and (x is None or x.is_contiguous() and x.dtype == torch.float32 and x.shape == (T, W))
+    assert ids is None or ids.dtype == torch.int64 and ids.is_contiguous()
+    out = x if x is not None and not prompt else torch.empty((T, W), dtype=torch.float32, device=y.device)
+    h = torch.empty((T, W), dtype=dtype, device=y.device)
+    mu = state = req = cu = first = batch = None
+    if shift is not None:
+        st, mu, state = shift.st, shift.mu, shift.state
+        assert state.dtype == torch.float32 and state.stride(1) == 1 and state.shape[1] == W
+        req, first = st.b_req_idx, st.b_ready_cache_len if prompt else st.seq_pos
+        cu, batch = (st.cu_q, st.batch_of_token) if prompt else (None, None)
+    check(kernels().llb_norm_shift(ptr(y), c_int(DTYPE_CODES[y.dtype]), ptr(ids), i64(y.shape[0]), ptr(x), ptr(out), ptr(h),
+                                   c_int(DTYPE_CODES[dtype]), ptr(w), c_int(T), c_int(width), c_int(W), c_int(int(centred)),
+                                   f32(eps), ptr(mu), ptr(state), i64(state.stride(0) if state is not None else 0), ptr(req),
+                                   ptr(cu), ptr(first), ptr(batch), stream()), "norm_shift")
+    _count()
+    return out, h
+
+
+def qk_norm_rope_scatter_(qkv, kv_layer, cos, sin, pos, slot, q_w, k_w, eps, Hq, Hkv, D, dim, DV, rot_dim, norm=True, q_scale=None):
     """Rows [Hq * D | Hkv * D | Hkv * DV] of qkv: RMS norm of every q and k head over its first `dim` elements (weights
     q_w, k_w fp32 [D], None: ones), rotation of the first rot_dim, q in place, K and V to kv_layer[slot] ([slots, Hkv * (D + DV)]).
-    Hkv = 0: queries only.  Without weights, norm and rotation may be read in either order."""
+    Hkv = 0: queries only.  Without weights, norm and rotation may be read in either order.  norm False: no norm.  q_scale (fp32
+    [Hq] or None): a factor per query head."""
     if not _is_cuda(qkv):
-        return ref.qk_norm_rope_scatter_(qkv, kv_layer, cos, sin, pos, slot, q_w, k_w, eps, Hq, Hkv, D, dim, DV, rot_dim)
+        return ref.qk_norm_rope_scatter_(qkv, kv_layer, cos, sin, pos, slot, q_w, k_w, eps, Hq, Hkv, D, dim, DV, rot_dim,
+                                          norm, q_scale)
     assert qkv.stride(1) == 1 and (Hkv == 0 or kv_layer.is_contiguous() and qkv.dtype == kv_layer.dtype)
     check(kernels().llb_qk_norm_rope_scatter(ptr(qkv), c_int(DTYPE_CODES[qkv.dtype]), i64(qkv.stride(0)), ptr(kv_layer),
                                              ptr(cos), ptr(sin), ptr(pos), ptr(slot), ptr(q_w), ptr(k_w), f32(eps),
-                                             c_int(qkv.shape[0]), c_int(Hq), c_int(Hkv), c_int(D), c_int(dim), c_int(DV),
+                                             c_int(int(norm)), ptr(q_scale), c_int(qkv.shape[0]), c_int(Hq), c_int(Hkv), c_int(D), c_int(dim), c_int(DV),
                                              c_int(rot_dim), stream()), "qk_norm_rope_scatter")
     _count()
     return qkv
@@ -801,23 +838,26 @@ class DistanceBias:
 
 
 def window_attention(q, kv_layer, req_to_token, st, Hq, Hkv, D, DV, sm_scale, window, gate=None, out_scale=1.0, out=None,
-                     keep=0, bias=None):
+                     keep=0, bias=None, chunk=0, softcap=0.0):
     """Causal paged attention with key size D and value size DV through a sliding window (0: none) for the pass `st`
-    (InferState); the first `keep` positions are seen through any window.  q [T, >= Hq * D]; bias (`DistanceBias` or None) is
-    added to the scaled scores; gate [T, Hq] (or None): head h is multiplied by sigmoid(gate[:, h]); all heads by out_scale.
-    Returns out [T, Hq * DV]."""
+    (InferState); the first `keep` positions are seen through any window.  chunk > 0, instead of a window: only positions of the
+    query's own chunk (of `chunk` positions, counted from 0).  q [T, >= Hq * D]; softcap > 0: scaled scores s become
+    softcap * tanh(s / softcap); bias (`DistanceBias` or None) is added to them; gate [T, Hq] (or None): head h is multiplied by
+    sigmoid(gate[:, h]), gate [T, Hq * DV]: element by element; all heads by out_scale.  Returns out [T, Hq * DV]."""
+    assert not (window and chunk)
     T = q.shape[0]
     if out is None:
         out = torch.empty((T, Hq * DV), dtype=q.dtype, device=q.device)
     if not _is_cuda(q):
         return ref.window_attention(q, kv_layer, req_to_token, st.b_req_idx, st.seq_pos,
                                     st.batch_of_token if st.is_prefill else None, Hq, Hkv, D, DV, sm_scale, window, gate,
-                                    out_scale, out, keep, bias)
+                                    out_scale, out, keep, bias, chunk, softcap)
     assert q.stride(1) == 1 and kv_layer.is_contiguous() and out.stride(1) == 1
-    gs = 0 if gate is None else gate.stride(0)
+    gs, elem = (0, 0) if gate is None else (gate.stride(0), int(gate.shape[1] != Hq))
+    assert not elem or gate.shape[1] == Hq * DV
     rel, far, stride = (bias.rel, bias.far, bias.rel.stride(0)) if bias is not None else (None, 0, 0)
-    tail = (f32(sm_scale), c_int(window), c_int(keep), ptr(rel), c_int(far), i64(stride), ptr(gate), i64(gs), f32(out_scale),
-            stream())
+    tail = (f32(sm_scale), c_int(window), c_int(keep), ptr(rel), c_int(far), i64(stride), c_int(chunk), f32(softcap), ptr(gate),
+            i64(gs), c_int(elem), f32(out_scale), stream())
     if q.dtype == torch.bfloat16 and D in _WINDOW_SIZES and DV % 64 == 0 and sm_scale > 0:
         common = (ptr(q), i64(q.stride(0)), ptr(kv_layer), ptr(req_to_token), i64(req_to_token.stride(0)),
                   ptr(st.b_req_idx))
@@ -829,7 +869,8 @@ def window_attention(q, kv_layer, req_to_token, st, Hq, Hkv, D, DV, sm_scale, wi
             _count()
             return out
         if DV in _WINDOW_SIZES:
-            keys = min(window + keep, st.max_kv_len) if window > 0 else st.max_kv_len
+            reach = window or chunk
+            keys = min(reach + keep, st.max_kv_len) if reach > 0 else st.max_kv_len
             n = window_decode_splits(T, Hq, Hkv, keys)
             po = pl = None
             if n > 1:

@@ -115,7 +115,7 @@ def kernels():
     return _kernels
 
 
-_DEBUG_UNITS = ("ops_basic", "attention", "attention_tc", "latent_attn", "mla", "moe", "rms_stream")
+_DEBUG_UNITS = ("ops_basic", "attention", "attention_tc", "latent_attn", "mla", "moe", "norm_shift", "rms_stream")
 
 
 def set_debug_bounds(pool_slots: int = 0, req_rows: int = 0, r2t_cols: int = 0, num_experts: int = 0, status=None):

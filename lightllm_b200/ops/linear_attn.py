@@ -155,20 +155,20 @@ CHUNK = 64
 
 
 class ChunkPlan:
-    """The 64-token chunks of a prompt pass: first token row and length of every chunk, chunks of every request."""
+    """The chunks (64 tokens) of a prompt pass: first token row, length and request of every chunk, chunks of every request."""
 
-    def __init__(self, q_len: torch.Tensor, device):
+    def __init__(self, q_len: torch.Tensor, device, size: int = CHUNK):
         q_len = q_len.to(torch.int64)
-        n = (q_len + CHUNK - 1) // CHUNK
+        n = (q_len + size - 1) // size
         zero = torch.zeros(1, dtype=torch.int64)
         cu_q, cu_c = torch.cat([zero, q_len.cumsum(0)]), torch.cat([zero, n.cumsum(0)])
         self.count = int(cu_c[-1])
         b = torch.repeat_interleave(torch.arange(len(q_len)), n)
-        off = (torch.arange(self.count) - cu_c[b]) * CHUNK
-        tok0, length = cu_q[b] + off, (q_len[b] - off).clamp_max(CHUNK)
-        host = torch.cat([tok0, length, cu_c]).to(torch.int32)
+        off = (torch.arange(self.count) - cu_c[b]) * size
+        tok0, length = cu_q[b] + off, (q_len[b] - off).clamp_max(size)
+        host = torch.cat([tok0, length, b, cu_c]).to(torch.int32)
         dev = host.to(device, non_blocking=True)
-        self.tok0, self.len, self.cu_chunk = torch.split(dev, [self.count, self.count, len(q_len) + 1])
+        self.tok0, self.len, self.req, self.cu_chunk = torch.split(dev, [self.count] * 3 + [len(q_len) + 1])
 
 
 class DecayedState:
@@ -286,3 +286,55 @@ class DecayedState:
         gate = torch.sigmoid(gf) * (gf if self.kind == "gla" else 1.0)
         out.copy_((o * gate).view(T, H * dv))
         return out
+
+
+# ---------------------------------------------------------------- elementwise gated states (minGRU)
+SHORT_SCAN = 16       # passes whose portions are at most this long run token by token
+
+
+def scan_plan(q_len: torch.Tensor, device):
+    """Chunks of a prompt pass for `gated_scan`: at most 64 per request, so that composing the earlier ones stays cheap; None when
+    all portions are short."""
+    longest = int(q_len.max())
+    return ChunkPlan(q_len, device, CHUNK * max(1, -(-longest // (64 * CHUNK)))) if longest > SHORT_SCAN else None
+
+
+def gated_scan(z, x, g, state, st, dtype, plan=None):
+    """minGRU over per-request states: S = (1 - sigmoid(z)) S + sigmoid(z) c(x), c(x) = x + 1/2 where x >= 0, else sigmoid(x); returns
+    S * silu(g) [T, n] in `dtype`.  z, x, g [T, n]: columns of one matrix; state fp32 [slots, n] (any row pitch); plan
+    (`scan_plan`): the chunks of a prompt pass, None: token by token."""
+    T, n = z.shape
+    first = st.b_ready_cache_len if st.is_prefill else st.seq_pos
+    if not z.is_cuda:
+        zf, xf, gf = z.float(), x.float(), g.float()
+        keep, add = torch.sigmoid(-zf), torch.sigmoid(zf) * torch.where(xf >= 0, xf + 0.5, torch.sigmoid(xf))
+        ends = st.cu_q.tolist() if st.is_prefill else list(range(T + 1))
+        s = torch.empty(T, n)
+        for b, r in enumerate(st.b_req_idx.tolist()):
+            row = state[r]
+            if first[b] == 0:
+                row.zero_()
+            for t in range(ends[b], ends[b + 1]):
+                row.mul_(keep[t]).add_(add[t])
+                s[t] = row
+        return (s * F.silu(gf)).to(dtype)
+    from . import DTYPE_CODES, _count
+    from ._native import c_int, check, i64, kernels, ptr, stream
+
+    ld = z.stride(0)
+    assert x.stride(0) == ld and g.stride(0) == ld and z.stride(1) == x.stride(1) == g.stride(1) == 1
+    assert z.dtype == x.dtype == g.dtype and state.dtype == torch.float32 and state.stride(1) == 1 and state.shape[1] == n
+    out = torch.empty((T, n), dtype=dtype, device=z.device)
+    common = (ptr(z), ptr(x), ptr(g), c_int(DTYPE_CODES[z.dtype]), i64(ld), ptr(out), c_int(DTYPE_CODES[dtype]), i64(n), ptr(state),
+              i64(state.stride(0)), ptr(st.b_req_idx))
+    if plan is None:
+        check(kernels().llb_gated_scan(*common, ptr(st.cu_q if st.is_prefill else None), ptr(first), c_int(st.batch_size), c_int(n),
+                                       stream()), "gated_scan")
+        _count()
+        return out
+    steps = torch.empty((2 * plan.count + st.batch_size, n), dtype=torch.float32, device=z.device)
+    check(kernels().llb_gated_chunks(*common, ptr(first), ptr(plan.tok0), ptr(plan.len), ptr(plan.cu_chunk), ptr(plan.req),
+                                     ptr(steps), ptr(steps[plan.count:]), ptr(steps[2 * plan.count:]), c_int(plan.count), c_int(n),
+                                     stream()), "gated_chunks")
+    _count(2)
+    return out

@@ -435,18 +435,40 @@ def add_rms_(x, y, w, width, eps, dtype, next_w=None):
     return (x if next_w is None else rms_over(x, width, eps) * next_w).to(dtype)
 
 
-def qk_norm_rope_scatter_(qkv, kv_layer, cos, sin, pos, slot, q_w, k_w, eps, Hq, Hkv, D, dim, DV, rot_dim):
+def norm_shift(x, y, w, width, eps, dtype, shift, ids, centred):
+    x = (y if ids is None else y[ids]).float() if x is None else x.add_(y.float())
+    d = x
+    if centred:
+        d = x - x.sum(-1, keepdim=True) / width
+        d[:, width:] = 0
+    n = rms_over(d, width, eps) * w
+    if shift is None:
+        return x, n.to(dtype)
+    st = shift.st
+    ends = st.cu_q.tolist() if st.is_prefill else list(range(len(x) + 1))
+    first = (st.b_ready_cache_len if st.is_prefill else st.seq_pos).tolist()
+    before = torch.cat([n[:1], n[:-1]])
+    for b, r in enumerate(st.b_req_idx.tolist()):
+        if ends[b] == ends[b + 1]:
+            continue
+        before[ends[b]] = shift.state[r] if first[b] else 0
+        shift.state[r] = n[ends[b + 1] - 1]
+    return x, (n + (before - n) * shift.mu).to(dtype)
+
+
+def qk_norm_rope_scatter_(qkv, kv_layer, cos, sin, pos, slot, q_w, k_w, eps, Hq, Hkv, D, dim, DV, rot_dim, norm=True, q_scale=None):
     T, half = qkv.shape[0], rot_dim // 2
     nq, nk = Hq * D, Hkv * D
     c, s = cos[pos.long()].unsqueeze(1), sin[pos.long()].unsqueeze(1)
 
-    def turn(x, w):
-        x = rms_over(x.float(), dim, eps)
+    def turn(x, w, factor=None):
+        x = rms_over(x.float(), dim, eps) if norm else x.float()
         x = x if w is None else x * w
+        x = x if factor is None else x * factor[:, None]
         u, v = x[..., :half], x[..., half:2 * half]
         return torch.cat([u * c - v * s, v * c + u * s, x[..., 2 * half:]], -1).reshape(T, -1).to(qkv.dtype)
 
-    q = turn(qkv[:, :nq].reshape(T, Hq, D), q_w)
+    q = turn(qkv[:, :nq].reshape(T, Hq, D), q_w, q_scale)
     if Hkv:
         kv_layer[slot.long(), :nk] = turn(qkv[:, nq:nq + nk].reshape(T, Hkv, D), k_w)
         kv_layer[slot.long(), nk:] = qkv[:, nq + nk:nq + nk + Hkv * DV]
@@ -464,22 +486,24 @@ def rotate_pairs(x, cos, sin, pos, neighbours):
 
 
 def window_attention(q, kv_layer, req_to_token, b_req_idx, pos, batch_of, Hq, Hkv, D, DV, sm_scale, window, gate, out_scale,
-                     out, keep=0, bias=None):
+                     out, keep=0, bias=None, chunk=0, softcap=0.0):
     G = Hq // Hkv
     for t in range(q.shape[0]):
         b = int(batch_of[t]) if batch_of is not None else t
         p = int(pos[t])
-        j0 = max(0, p - window + 1) if window > 0 else 0
+        j0 = max(0, p - window + 1) if window > 0 else p - p % chunk if chunk > 0 else 0
         j = torch.cat([torch.arange(min(keep, j0)), torch.arange(j0, p + 1)])
         rows = kv_layer[req_to_token[int(b_req_idx[b]), j].long()].float()
         k = rows[:, : Hkv * D].view(-1, Hkv, D).repeat_interleave(G, dim=1)
         v = rows[:, Hkv * D:].reshape(-1, Hkv, DV).repeat_interleave(G, dim=1)
         sc = torch.einsum("hd,lhd->hl", q[t, : Hq * D].view(Hq, D).float(), k) * sm_scale
+        if softcap > 0:
+            sc = softcap * torch.tanh(sc / softcap)
         if bias is not None:
             sc = sc + bias.rel[:, (p - j).clamp_max(bias.far)]
         pr = torch.softmax(sc, dim=-1)
         o = torch.einsum("hl,lhd->hd", pr, v) * out_scale
         if gate is not None:
-            o = o * torch.sigmoid(gate[t].float())[:, None]
+            o = o * torch.sigmoid(gate[t].float()).view(Hq, -1)
         out[t] = o.reshape(-1).to(out.dtype)
     return out
