@@ -96,7 +96,7 @@ def parse():
     ap.add_argument("--rate", type=float, default=8.0, help="config 3: Poisson arrival rate, requests per second")
     ap.add_argument("--in-range", default="128,4096", help="config 3: uniform prompt length range")
     ap.add_argument("--out-range", default="64,1024", help="config 3: uniform output length range")
-    ap.add_argument("--design", default=None, choices=["taduzen", "libulorn", "katarax"],
+    ap.add_argument("--design", default=None, choices=["taduzen", "libulorn", "katarax", "silupel"],
                     help="instead of the serving workload: prefill and decode passes of this model design beside the "
                          "closest other model at equal sizes")
     ap.add_argument("--design-size", default=None, choices=["small", "base", "wide"], help="one size only (default: all)")

@@ -1,8 +1,9 @@
 """Prefill and decode throughput of a model design beside the framework's closest model at equal sizes, and the kernels
 of both with their roofline fractions.  Taduzen: DeepSeek-V2 (latent attention, routed and shared experts); Libulorn:
-Qwen3-Next (`design_libulorn.py`); Katarax: DeepSeek-V3 and Qwen3-MoE (`design_katarax.py`).
+Qwen3-Next (`design_libulorn.py`); Katarax: DeepSeek-V3 and Qwen3-MoE (`design_katarax.py`); Silupel: Qwen2 and
+DeepSeek-V2 with dense feed-forwards (`design_silupel.py`).
 
-    python bench.py --design taduzen|libulorn|katarax [--design-size small|base|wide] [--design-kernels]
+    python bench.py --design taduzen|libulorn|katarax|silupel [--design-size small|base|wide] [--design-kernels]
 
 Random weights, random tokens, bf16.  Whole passes through the models' own forward (decode as CUDA graph), timed with CUDA
 events after three warm-up passes; a pass reads far more weight bytes than L2 holds.  Kernels: median of 10 samples with L2
@@ -10,6 +11,7 @@ flushed before each.  One JSON object per line.
 """
 from __future__ import annotations
 
+import importlib
 import json
 import os
 
@@ -95,9 +97,8 @@ def _design(name):
         from .design_kernels import kernels
 
         return SIZES, taduzen_config, {"deepseek_v2": deepseek_config}, kernels
-    if name == "katarax":
-        from . import design_katarax as d
-
+    if name in ("katarax", "silupel"):
+        d = importlib.import_module(f".design_{name}", __package__)
         return d.SIZES, d.config, d.CLOSEST, d.kernels
     from . import design_libulorn as d
 

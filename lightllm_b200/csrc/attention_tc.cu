@@ -60,22 +60,28 @@ __device__ __forceinline__ float ex2_fast(float x) {  // 2^x, one MUFU instructi
   return y;
 }
 
-// v[e] (fp32 bits) = top * tanh(v[e] * in).  Where all of a warp's arguments are below 1/4 the Taylor series of tanh_fast, else
-// top - 2 top / (1 + e^2x), whose absolute error (a few 1e-7 top) is that of rounding values of the cap's size.
+// v[e] (fp32 bits) = top * tanh(v[e] * in).  Where all of a warp's arguments x are small, the Taylor series
+// x - x^3/3 + 2x^5/15 (|x| < 1/8), or up to 62x^9/2835 (|x| < 0.35), with a relative error below 3e-7; else top - 2 top / (1 + e^2x),
+// whose absolute error (a few 1e-7 top) is that of rounding values of the cap's size.
 template <int N>
 __device__ __forceinline__ void cap_scores(uint32_t* v, float in, float top) {
   float big = 0.f;
 #pragma unroll
   for (int e = 0; e < N; ++e) big = fmaxf(big, fabsf(__uint_as_float(v[e])));
-  if (__all_sync(0xffffffffu, big * in < 0.25f)) {
-    // top (x - x^3/3 + 2x^5/15 - 17x^7/315 + 62x^9/2835), in powers of the score itself
-    const float i2 = in * in, k1 = top * in;
-    const float c3 = -1.f / 3.f * i2, c5 = 2.f / 15.f * i2 * i2, c7 = -17.f / 315.f * i2 * i2 * i2,
-                c9 = 62.f / 2835.f * i2 * i2 * i2 * i2;
+  const float i2 = in * in, k1 = top * in;  // the series in powers of the score itself
+  const float c3 = k1 * i2 * (-1.f / 3.f), c5 = k1 * i2 * i2 * (2.f / 15.f);
+  if (__all_sync(0xffffffffu, big * in < 0.125f)) {
 #pragma unroll
     for (int e = 0; e < N; ++e) {
       const float x = __uint_as_float(v[e]), x2 = x * x;
-      v[e] = __float_as_uint(x * k1 * fmaf(x2, fmaf(x2, fmaf(x2, fmaf(x2, c9, c7), c5), c3), 1.f));
+      v[e] = __float_as_uint(x * fmaf(x2, fmaf(x2, c5, c3), k1));
+    }
+  } else if (__all_sync(0xffffffffu, big * in < 0.35f)) {
+    const float c7 = k1 * i2 * i2 * i2 * (-17.f / 315.f), c9 = k1 * i2 * i2 * i2 * i2 * (62.f / 2835.f);
+#pragma unroll
+    for (int e = 0; e < N; ++e) {
+      const float x = __uint_as_float(v[e]), x2 = x * x;
+      v[e] = __float_as_uint(x * fmaf(x2, fmaf(x2, fmaf(x2, fmaf(x2, c9, c7), c5), c3), k1));
     }
   } else {
     const float to2 = 2.f * kLog2e * in;

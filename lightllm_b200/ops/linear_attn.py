@@ -290,13 +290,14 @@ class DecayedState:
 
 # ---------------------------------------------------------------- elementwise gated states (minGRU)
 SHORT_SCAN = 16       # passes whose portions are at most this long run token by token
+SCAN_CHUNKS = 128
 
 
 def scan_plan(q_len: torch.Tensor, device):
-    """Chunks of a prompt pass for `gated_scan`: at most 64 per request, so that composing the earlier ones stays cheap; None when
-    all portions are short."""
+    """Chunks of a prompt pass for `gated_scan`: at most SCAN_CHUNKS per request, so that composing the earlier ones stays cheap;
+    None when all portions are short."""
     longest = int(q_len.max())
-    return ChunkPlan(q_len, device, CHUNK * max(1, -(-longest // (64 * CHUNK)))) if longest > SHORT_SCAN else None
+    return ChunkPlan(q_len, device, CHUNK * max(1, -(-longest // (SCAN_CHUNKS * CHUNK)))) if longest > SHORT_SCAN else None
 
 
 def gated_scan(z, x, g, state, st, dtype, plan=None):

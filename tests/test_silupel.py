@@ -253,9 +253,9 @@ def test_scan_plan():
     assert linear_attn.scan_plan(torch.tensor([1, 16, 3]), "cpu") is None
     p = linear_attn.scan_plan(torch.tensor([1, 130]), "cpu")
     assert p.len.tolist() == [1, 64, 64, 2] and p.req.tolist() == [0, 1, 1, 1] and p.cu_chunk.tolist() == [0, 1, 4]
-    for longest, size in ((4096, 64), (4097, 128), (8192, 128), (12000, 192)):
+    for longest, size in ((8192, 64), (8193, 128), (16384, 128), (24000, 192)):
         p = linear_attn.scan_plan(torch.tensor([longest, 70]), "cpu")
-        assert p.len.max() == min(size, longest) and p.count <= 64 + 2
+        assert p.len.max() == min(size, longest) and p.count <= linear_attn.SCAN_CHUNKS + 2
 
 
 def test_rotation_and_frequency_scaling():
