@@ -100,7 +100,7 @@ class LayerSpec:
         self.vp = _up(self.vdim, 64)
         self.rot = m.get("rot") or {"base": 10000.0, "dims": 0}
         if self.type == LATENT:
-            self.rank, self.rot_dim, self.q_rank = m["kv_rank"], m["rot_dim"], m["q_rank"]
+            self.rank, self.rot_dim, self.q_rank = m["kv_rank"], m["rot_dim"], m.get("q_rank")
             self.kv_heads = 1
             if self.rot["dims"] != self.rot_dim:
                 raise ValueError("latent attention: rot.dims must be rot_dim")
@@ -164,10 +164,10 @@ class SilupelLM(RecurrentStateMixin, StreamLM):
                 s.update({m + "z": (l.size, W), m + "z.b": (l.size,), m + "x": (l.size, W), m + "x.b": (l.size,),
                           m + "g": (l.size, W), m + "o": (W, l.size)})
             elif l.type == LATENT:
-                s.update({m + "dq": (l.q_rank, W), m + "dq.norm": (l.q_rank,),
-                          m + "uq": (l.heads * (l.dim + l.rot_dim), l.q_rank), m + "dkv": (l.rank + l.rot_dim, W),
-                          m + "dkv.norm": (l.rank,), m + "uk": (l.heads * l.dim, l.rank), m + "uv": (l.heads * l.vdim, l.rank),
-                          m + "o": (W, l.heads * l.vdim)})
+                qr = l.q_rank or l.rank
+                s.update({m + "dq": (qr, W), m + "dq.norm": (qr,), m + "uq": (l.heads * (l.dim + l.rot_dim), qr),
+                          m + "dkv": (l.rank + l.rot_dim, W), m + "dkv.norm": (l.rank,), m + "uk": (l.heads * l.dim, l.rank),
+                          m + "uv": (l.heads * l.vdim, l.rank), m + "o": (W, l.heads * l.vdim)})
             else:
                 for n, rows in (("q", l.heads * l.dim), ("k", l.kv_heads * l.dim), ("v", l.kv_heads * l.vdim)):
                     s.update({m + n: (rows, W), m + n + ".b": (rows,)})
@@ -234,15 +234,17 @@ class SilupelLM(RecurrentStateMixin, StreamLM):
 
     def _load_latent(self, lw, src, m, l: LayerSpec):
         h0, h1 = tp_range(l.heads, self.tp.rank, self.tp.size)
-        W, per, q16 = self.hidden, l.dim + l.rot_dim, _up(l.q_rank, 16)
+        W, per = self.hidden, l.dim + l.rot_dim
+        qr = l.q_rank or src.shape(m + "dq")[0]
+        q16 = _up(qr, 16)
         lat = lw.latent = LatentHeads(l.hq, l.dim, l.rot_dim, l.vdim, l.rank, l.scale, 0)
         dkv = get_shaped(src, m + "dkv", l.rank + l.rot_dim, W)
-        lw.in_w = self._dev(torch.cat([self._narrow(get_shaped(src, m + "dq", l.q_rank, W), l.q_rank, 16),
+        lw.in_w = self._dev(torch.cat([self._narrow(get_shaped(src, m + "dq", qr, W), qr, 16),
                                        self._narrow(dkv[: l.rank], l.rank, 16), self._narrow(dkv[l.rank:], l.rot_dim, 16)]))
-        lw.q_cols = q16
-        lw.q_norm = self._vec(get_shaped(src, m + "dq.norm", l.q_rank), q16)
+        lw.q_rank, lw.q_cols = qr, q16
+        lw.q_norm = self._vec(get_shaped(src, m + "dq.norm", qr), q16)
         lw.kv_norm = self._vec(get_shaped(src, m + "dkv.norm", l.rank), lat.rp)
-        uq = get_shaped(src, m + "uq", l.heads * per, l.q_rank).view(l.heads, per, l.q_rank)[h0:h1]
+        uq = get_shaped(src, m + "uq", l.heads * per, qr).view(l.heads, per, qr)[h0:h1]
         lw.uq_w = self._dev(_pad(uq, l.hq, l.dp, q16).reshape(l.hq * l.dp, q16))
         uk = get_shaped(src, m + "uk", l.heads * l.dim, l.rank).view(l.heads, l.dim, l.rank)[h0:h1]
         uv = get_shaped(src, m + "uv", l.heads * l.vdim, l.rank).view(l.heads, l.vdim, l.rank)[h0:h1]
@@ -335,7 +337,7 @@ class SilupelLM(RecurrentStateMixin, StreamLM):
         proj = ops.gemm(h, lw.in_w)                              # [T, query latent | latent | rotated part]
         kv_layer = self._kv_layer(run.kv_slot)
         cq = mla_ops.latent_prepare_(proj[:, lw.q_cols:], kv_layer, lw.kv_norm, st.mem_index, l.rank, lat.rp, self.eps, lw.rope,
-                                     st.position_ids, proj[:, : lw.q_cols], lw.q_norm, l.q_rank)
+                                     st.position_ids, proj[:, : lw.q_cols], lw.q_norm, lw.q_rank)
         q = ops.gemm(cq, lw.uq_w)
         ops.rope_heads_(q, lw.rope.cos, lw.rope.sin, st.position_ids, l.hq, l.dp, l.dim, lw.rope.dims, lw.rope.neighbours)
         return lat.attend(lw, q, kv_layer, self.req_manager.req_to_token_indexs, st)

@@ -617,6 +617,14 @@ def test_random_weights_and_sampling(tgt):
     llm.close()
 
 
+def test_query_latent_size_from_the_checkpoint(tmp_path):
+    cfg = config([latent(2, 16, 8, 24, 40, 24, 0.3)])
+    t, toks = weights(cfg, 2), tokens(40, 1)
+    want = plain.forward(t, cfg, toks)
+    del cfg["layers"][0]["mixer"]["q_rank"]
+    close(run_portions(replayer(write(tmp_path, cfg, t), ("cpu", "float32")), "a", toks, [30, 9, 1]), want, ("cpu", "float32"))
+
+
 def test_recurrent_layers_only(tmp_path):
     """Without attention the pool has no rows, only slots."""
     cfg = config([mingru(8, dense(16)), mingru(40, None)], loop=(0, 1, 2))
